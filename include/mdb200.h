@@ -333,6 +333,229 @@ int mdb_lmhead_sample_tp(const void* hidden, int64_t ld_hidden, const void* w, i
 int64_t mdb_lmhead_tp_workspace_bytes(int m, int vocab);
 int mdb_lmhead_tp_slots(int m, int cols);
 
+/* ---- decoders with an fp32 residual: recurrent mixers, latent attention, experts ----
+ *
+ * Activations are MDB_BF16 or MDB_F32 (argument `dtype`); in the fp32 form every product is true fp32.  Argument
+ * blocks are host structs read during the call.  A "portion" is the run of tokens a sequence brings to a step:
+ * rows [cu_q[s], cu_q[s + 1]) of the step, the first of them at position start[s] of the sequence.  state_slot[s]
+ * is the sequence's slot in the state pools (-1: padding entry, skipped); a sequence at position 0 starts from a
+ * zero state whatever the slot holds.  Sizes with the suffix _pad are storage sizes; the surplus holds zeros. */
+enum { MDB_BF16 = 0, MDB_F32 = 1 };
+
+/* Output of a projection, columns [col, ...) of rows of `ld` elements: rows of the activation type (x), or fp32
+ * split-k slices part_stride elements apart (parts) that the consumer sums and rounds. */
+typedef struct {
+  const void* x;
+  const float* parts;
+  int64_t ld, part_stride;
+  int32_t nparts, col;
+} mdb_rows;
+
+enum { MDB_GEMM_PLAIN = 0, MDB_GEMM_HEADS = 1, MDB_GEMM_EXPERTS = 2 };
+enum { MDB_ACT_NONE = 0, MDB_ACT_RELU2 = 1 };
+/* y = act(x W^T).  PLAIN: x [m, k], w [n, k], y [m, n].  HEADS: head h takes columns [h k, (h + 1) k) of x, rows
+ * [h n, (h + 1) n) of w and writes columns [h n, (h + 1) n) of y.  EXPERTS: rows of x and y are laid out by expert
+ * in tiles of 128 (mdb_moe_plan); tile t uses rows [e n, (e + 1) n) of w, e = tile_expert[t], for t < *num_tiles;
+ * m = rows of the buffers; max_rows_per_expert (0: unknown) bounds the rows in use in a tile.  y is of the
+ * activation type, or fp32 with y_f32. */
+typedef struct {
+  int32_t dtype, form, act, y_f32;
+  const void* x;
+  const void* w;
+  void* y;
+  int64_t ldx, ldy;
+  int32_t m, n, k;
+  int32_t heads, experts, max_rows_per_expert;
+  const int32_t* tile_expert;
+  const int32_t* num_tiles;
+} mdb_gemm_args;
+int mdb_gemm(const mdb_gemm_args* args, mdb_stream_t stream);
+
+/* residual [m][width_pad] fp32: with ids, = embed[id] * embed_scale, else += ; plus the rows of up to two
+ * projections, plus sum_k moe_weight[row][k] * moe_rows[moe_slot[row][k]].  y (may be NULL) = residual / sqrt(mean
+ * of its first `width` columns squared + eps) * weight. */
+typedef struct {
+  int32_t dtype, m, width, width_pad;
+  float* residual;
+  const int64_t* ids;
+  const void* embed;
+  int64_t vocab;
+  mdb_rows add[2];
+  const void* moe_rows;
+  int64_t moe_ld;
+  const int32_t* moe_slot;
+  const float* moe_weight;
+  const float* weight;
+  void* y;
+  int64_t ldy;
+  float embed_scale, eps;
+  int32_t moe_top;
+} mdb_residual_norm_args;
+int mdb_residual_norm(const mdb_residual_norm_args* args, mdb_stream_t stream);
+
+/* RMSNorm of column segments of a projection into row `row` of out, or into row slots[row] (-1: skipped). */
+#define MDB_MAX_RMS_SEGMENTS 4
+typedef struct {
+  mdb_rows src;
+  const float* weight;
+  void* out;
+  int64_t ld_out;
+  const int32_t* slots;
+  int64_t num_slots;
+  int32_t n, n_pad;
+  float eps;
+} mdb_rms_segment;
+int mdb_rms_rows(int dtype, const mdb_rms_segment* segments, int nseg, int m, mdb_stream_t stream);
+
+/* y[row][h][c] = o / sqrt(mean over c of o^2 + eps) * weight[h * weight_head_stride + c] * sigmoid(gate) */
+typedef struct {
+  int32_t dtype, m, heads, vdim;
+  const float* o;
+  mdb_rows gate;
+  const float* weight;
+  void* y;
+  int64_t ldy;
+  int32_t weight_head_stride;
+  float eps;
+} mdb_gated_norm_args;
+int mdb_gated_norm(const mdb_gated_norm_args* args, mdb_stream_t stream);
+
+/* Key channels of a recurrent head as the state stores them (a multiple of 32; 0: not supported), and the number of
+ * copies of the mLSTM normaliser and maximum a head keeps. */
+int mdb_scan_dim_pad(int dim);
+int mdb_scan_blocks(int vdim);
+/* 1 when the one-token form of mdb_scan takes this head shape */
+int mdb_scan_fusable(int dim_pad, int vdim);
+
+/* Inputs of the delta scan: causal short convolution over time per channel (weights fp32 [channels][taps], the last
+ * tap is the current token's) and silu of q, k, v; q and k as unit vectors (q times dim^-1/2), k . q, beta =
+ * sigmoid(b).  conv_state [slot][taps - 1][channels] of the activation type, channels ordered q | k | v, holds the
+ * last inputs and is moved on: in the same kernel when shift_state is set (every portion is one token), else by a
+ * second one.  copy_cols columns of `copy` are written to copy_out (materialises split-k slices). */
+typedef struct {
+  int32_t dtype, m, bs, heads, kv_heads, dim, dim_pad, vdim, taps, channels, shift_state, copy_cols;
+  mdb_rows q, k, v, b, copy;
+  void* copy_out;
+  int64_t copy_ld;
+  const float* conv_q;
+  const float* conv_k;
+  const float* conv_v;
+  void* conv_state;
+  int64_t conv_slot_stride, num_slots;
+  const int32_t* row_seq;
+  const int32_t* cu_q;
+  const int32_t* start;
+  const int32_t* state_slot;
+  float* q_out;    /* [m][kv_heads][dim_pad] */
+  float* k_out;
+  float* v_out;    /* [m][heads][vdim] */
+  float* beta_out; /* [m][heads] */
+  float* kq_out;   /* [m][kv_heads] */
+} mdb_delta_prep_args;
+int mdb_delta_prep(const mdb_delta_prep_args* args, mdb_stream_t stream);
+
+/* g [m][heads][dim_pad] = exp(-exp(a_log[h]) * softplus(x + dt_bias)), x [m] rows of heads * dim columns */
+int mdb_channel_decay(const float* x, int64_t ldx, const float* a_log, const float* dt_bias, float* g, int m, int heads,
+                      int dim, int dim_pad, mdb_stream_t stream);
+
+/* Inputs of the mLSTM scan: q times dim^-1/2, k, v as fp32 rows; log_i = cap tanh((i + bias_i) / cap), log_f =
+ * logsigmoid(cap tanh((f + bias_f) / cap)). */
+typedef struct {
+  int32_t dtype, m, heads, dim, dim_pad, vdim;
+  mdb_rows q, k, v, i, f;
+  const float* bias_i;
+  const float* bias_f;
+  float* q_out;
+  float* k_out;
+  float* v_out;
+  float* log_i; /* [m][heads] */
+  float* log_f;
+  float cap;
+} mdb_mlstm_prep_args;
+int mdb_mlstm_prep(const mdb_mlstm_prep_args* args, mdb_stream_t stream);
+
+/* The recurrences over every sequence's portion; state [slot][heads][vdim][dim_pad] fp32 is read and written.
+ * DELTA: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; s0 = beta, s1 = k . q.  MLSTM: m' = max(f + m, i);
+ * S, n <- exp(f + m - m') (.) + exp(i - m') k (v^T, 1); o = S^T q / (max(|n . q|, exp(-m')) + 1e-6); s0 = i, s1 = f;
+ * nstate [slot][heads][mdb_scan_blocks][dim_pad], mstate [slot][heads][mdb_scan_blocks].
+ * out [m][heads][vdim] fp32; with `fused` (every portion is one token) the decay comes from raw_decay + dt_bias and
+ * a_log, and y = the gated norm of o (as mdb_gated_norm) is written instead. */
+enum { MDB_SCAN_DELTA = 0, MDB_SCAN_MLSTM = 1 };
+typedef struct {
+  int32_t mode, dtype, fused, bs, heads, kv_heads, dim, dim_pad, vdim;
+  float eps;
+  const float* q;
+  const float* k;
+  const float* v;
+  const float* g;
+  const float* s0;
+  const float* s1;
+  float* state;
+  int64_t state_slot_stride, num_slots;
+  float* nstate;
+  float* mstate;
+  const int32_t* cu_q;
+  const int32_t* start;
+  const int32_t* state_slot;
+  float* out;
+  mdb_rows raw_decay; /* fp32 */
+  const float* a_log;
+  const float* dt_bias;
+  mdb_rows gate;
+  const float* norm;
+  int64_t norm_head_stride;
+  void* y;
+  int64_t ldy;
+} mdb_scan_args;
+int mdb_scan(const mdb_scan_args* args, mdb_stream_t stream);
+
+/* Group-limited top-k routing of fp32 logits [m][experts]: ids and weights [m][top]; rows with row_slot < 0 (may be
+ * NULL) get ids -1. */
+typedef struct {
+  int32_t m, experts, top, groups, keep;
+  mdb_rows logits; /* fp32 */
+  const int32_t* row_slot;
+  int32_t* ids;
+  float* weights;
+} mdb_moe_route_args;
+int mdb_moe_route(const mdb_moe_route_args* args, mdb_stream_t stream);
+
+/* Lays the (token, k) pairs out by expert in tiles of 128 rows: slot [m][top] (row of the pair, -1: none), row_token
+ * [max_tiles * 128] (-1: padding), tile_expert [max_tiles], num_tiles [1]. */
+typedef struct {
+  int32_t m, top, experts, max_tiles;
+  const int32_t* ids;
+  int32_t* slot;
+  int32_t* row_token;
+  int32_t* tile_expert;
+  int32_t* num_tiles;
+} mdb_moe_plan_args;
+int mdb_moe_plan(const mdb_moe_plan_args* args, mdb_stream_t stream);
+/* Most tiles m rows with `top` experts each can need. */
+int mdb_moe_max_tiles(int m, int top, int experts);
+int mdb_moe_gather(int dtype, const void* x, int64_t ldx, void* out, int width, const int32_t* row_token,
+                   const int32_t* num_tiles, int max_tiles, mdb_stream_t stream);
+
+/* Causal attention over cached latents (cache [pages * 256][width], one row per token, key and value of every head
+ * alike): q, out [m][heads][width]; the row at position p of its sequence sees keys 0 .. p. */
+int64_t mdb_latent_attn_workspace_bytes(int m, int heads, int width, int nsplit);
+int mdb_latent_attn(int dtype, const void* q, const void* cache, void* out, const int32_t* block_table, int table_stride,
+                    const int32_t* row_seq, const int32_t* row_pos, int m, int heads, int width, int num_pages, float scale,
+                    int nsplit, void* workspace, int64_t workspace_bytes, mdb_stream_t stream);
+/* out [total][width] = the latents of positions 0 .. cu[s + 1] - cu[s] - 1 of every sequence, in order. */
+int mdb_gather_latents(int dtype, const void* cache, const int32_t* block_table, int table_stride, int num_pages,
+                       const int32_t* cu, int nseq, int total, void* out, int width, mdb_stream_t stream);
+/* Causal attention over packed rows (bf16, head size 128): the queries of sequence s are its last cu_q[s + 1] -
+ * cu_q[s] tokens, the keys all of them (cu_k). */
+int mdb_attn_causal_varlen(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride,
+                           void* out, int64_t out_stride, const int32_t* cu_q, const int32_t* cu_k, int nseq, int max_q,
+                           int64_t total_q, int64_t total_k, int hq, int hkv, float scale, mdb_stream_t stream);
+
+/* token = argmax of logits / temperature + Gumbel noise (seed, *step_dev, row), or of the logits where the row's
+ * temperature is 0; status_out (may be NULL) receives and clears the device status word. */
+int mdb_pick_token(const float* logits, int64_t ld, int m, int vocab, const float* temperatures, uint32_t seed,
+                   const uint32_t* step_dev, int64_t* out, uint32_t* status_out, mdb_stream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -16,6 +16,47 @@ _i64 = C.c_int64
 _u32 = C.c_uint32
 _f = C.c_float
 
+
+def _struct(name, fields):
+    return type(name, (C.Structure,), {"_fields_": fields})
+
+
+# argument blocks of the fp32-residual decoders, field for field as in include/mdb200.h
+Rows = _struct("Rows", [("x", _p), ("parts", _p), ("ld", _i64), ("part_stride", _i64), ("nparts", _i), ("col", _i)])
+GemmArgs = _struct("GemmArgs", [
+    ("dtype", _i), ("form", _i), ("act", _i), ("y_f32", _i), ("x", _p), ("w", _p), ("y", _p), ("ldx", _i64), ("ldy", _i64),
+    ("m", _i), ("n", _i), ("k", _i), ("heads", _i), ("experts", _i), ("max_rows_per_expert", _i), ("tile_expert", _p),
+    ("num_tiles", _p)])
+ResidualNormArgs = _struct("ResidualNormArgs", [
+    ("dtype", _i), ("m", _i), ("width", _i), ("width_pad", _i), ("residual", _p), ("ids", _p), ("embed", _p), ("vocab", _i64),
+    ("add", Rows * 2), ("moe_rows", _p), ("moe_ld", _i64), ("moe_slot", _p), ("moe_weight", _p), ("weight", _p), ("y", _p),
+    ("ldy", _i64), ("embed_scale", _f), ("eps", _f), ("moe_top", _i)])
+RmsSegment = _struct("RmsSegment", [
+    ("src", Rows), ("weight", _p), ("out", _p), ("ld_out", _i64), ("slots", _p), ("num_slots", _i64), ("n", _i),
+    ("n_pad", _i), ("eps", _f)])
+GatedNormArgs = _struct("GatedNormArgs", [
+    ("dtype", _i), ("m", _i), ("heads", _i), ("vdim", _i), ("o", _p), ("gate", Rows), ("weight", _p), ("y", _p),
+    ("ldy", _i64), ("weight_head_stride", _i), ("eps", _f)])
+DeltaPrepArgs = _struct("DeltaPrepArgs", [(n, _i) for n in (
+    "dtype", "m", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim", "taps", "channels", "shift_state", "copy_cols")] + [
+    ("q", Rows), ("k", Rows), ("v", Rows), ("b", Rows), ("copy", Rows), ("copy_out", _p), ("copy_ld", _i64), ("conv_q", _p),
+    ("conv_k", _p), ("conv_v", _p), ("conv_state", _p), ("conv_slot_stride", _i64), ("num_slots", _i64), ("row_seq", _p),
+    ("cu_q", _p), ("start", _p), ("state_slot", _p), ("q_out", _p), ("k_out", _p), ("v_out", _p), ("beta_out", _p),
+    ("kq_out", _p)])
+MlstmPrepArgs = _struct("MlstmPrepArgs", [(n, _i) for n in ("dtype", "m", "heads", "dim", "dim_pad", "vdim")] + [
+    ("q", Rows), ("k", Rows), ("v", Rows), ("i", Rows), ("f", Rows), ("bias_i", _p), ("bias_f", _p), ("q_out", _p),
+    ("k_out", _p), ("v_out", _p), ("log_i", _p), ("log_f", _p), ("cap", _f)])
+ScanArgs = _struct("ScanArgs", [(n, _i) for n in (
+    "mode", "dtype", "fused", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim")] + [
+    ("eps", _f), ("q", _p), ("k", _p), ("v", _p), ("g", _p), ("s0", _p), ("s1", _p), ("state", _p),
+    ("state_slot_stride", _i64), ("num_slots", _i64), ("nstate", _p), ("mstate", _p), ("cu_q", _p), ("start", _p),
+    ("state_slot", _p), ("out", _p), ("raw_decay", Rows), ("a_log", _p), ("dt_bias", _p), ("gate", Rows), ("norm", _p),
+    ("norm_head_stride", _i64), ("y", _p), ("ldy", _i64)])
+MoeRouteArgs = _struct("MoeRouteArgs", [(n, _i) for n in ("m", "experts", "top", "groups", "keep")] + [
+    ("logits", Rows), ("row_slot", _p), ("ids", _p), ("weights", _p)])
+MoePlanArgs = _struct("MoePlanArgs", [(n, _i) for n in ("m", "top", "experts", "max_tiles")] + [
+    ("ids", _p), ("slot", _p), ("row_token", _p), ("tile_expert", _p), ("num_tiles", _p)])
+
 # name -> (restype, argtypes); mirrors include/mdb200.h one to one
 SIGNATURES = {
     "mdb_strerror": (C.c_char_p, [_i]),
@@ -61,6 +102,26 @@ SIGNATURES = {
     "mdb_add_rmsnorm_tp_rows": (_i, [_p, _p, _p, _p, _f, _p, _p, _i, _i, _p, _i, _u32, _p, _p]),
     "mdb_lmhead_sample_tp": (_i, [_p, _i64, _p, _i, _i, _i, _p, _i, _i, _p, _u32, _u32, _p, _p, _p, _i64, _i, _i, _p,
                                   _p, _i, _u32, _p, _p, _p, _p]),
+    "mdb_gemm": (_i, [C.POINTER(GemmArgs), _p]),
+    "mdb_residual_norm": (_i, [C.POINTER(ResidualNormArgs), _p]),
+    "mdb_rms_rows": (_i, [_i, C.POINTER(RmsSegment), _i, _i, _p]),
+    "mdb_gated_norm": (_i, [C.POINTER(GatedNormArgs), _p]),
+    "mdb_scan_dim_pad": (_i, [_i]),
+    "mdb_scan_blocks": (_i, [_i]),
+    "mdb_scan_fusable": (_i, [_i, _i]),
+    "mdb_delta_prep": (_i, [C.POINTER(DeltaPrepArgs), _p]),
+    "mdb_channel_decay": (_i, [_p, _i64, _p, _p, _p, _i, _i, _i, _i, _p]),
+    "mdb_mlstm_prep": (_i, [C.POINTER(MlstmPrepArgs), _p]),
+    "mdb_scan": (_i, [C.POINTER(ScanArgs), _p]),
+    "mdb_moe_route": (_i, [C.POINTER(MoeRouteArgs), _p]),
+    "mdb_moe_plan": (_i, [C.POINTER(MoePlanArgs), _p]),
+    "mdb_moe_max_tiles": (_i, [_i, _i, _i]),
+    "mdb_moe_gather": (_i, [_i, _p, _i64, _p, _i, _p, _p, _i, _p]),
+    "mdb_latent_attn_workspace_bytes": (_i64, [_i, _i, _i, _i]),
+    "mdb_latent_attn": (_i, [_i, _p, _p, _p, _p, _i, _p, _p, _i, _i, _i, _i, _f, _i, _p, _i64, _p]),
+    "mdb_gather_latents": (_i, [_i, _p, _p, _i, _i, _p, _i, _i, _p, _i, _p]),
+    "mdb_attn_causal_varlen": (_i, [_p, _i64, _p, _i64, _p, _i64, _p, _i64, _p, _p, _i, _i, _i64, _i64, _i, _i, _f, _p]),
+    "mdb_pick_token": (_i, [_p, _i64, _i, _i, _p, _u32, _p, _p, _p, _p]),
 }
 
 _lib = None

@@ -42,7 +42,8 @@ static bool attn_tc_supported(int block, int hq, int hkv, float softmax_scale);
 static int attn_tc_launch(const AttnPagedArgs& a, int bs, cudaStream_t st);
 struct AttnStairArgs;
 static bool attn_stair_tc_supported(int hq, int hkv, int64_t q_stride, int64_t k_stride, int64_t v_stride);
-static int attn_stair_tc_launch(const AttnStairArgs& a, int nseq, int max_seqlen, int64_t total_tokens, cudaStream_t st);
+static int attn_stair_tc_launch(const AttnStairArgs& a, int nseq, int max_seqlen, int64_t total_q, int64_t total_tokens,
+                                cudaStream_t st);
 
 struct AttnStairArgs {
   const bf16* q;
@@ -50,9 +51,11 @@ struct AttnStairArgs {
   const bf16* v;
   bf16* out;
   const int32_t* cu_seqlens;
+  const int32_t* cu_seqlens_q;   // NULL: queries for every key row
   int64_t q_stride, k_stride, v_stride, out_stride;
   int hq, hkv, log2_stairs;
-  float q_scale;  // log2(e) / sqrt(D)
+  float q_scale;     // multiplies q, rounded to bf16: log2(e) / sqrt(D), or 1
+  float scale_log2;  // multiplies the fp32 scores
 };
 
 // Merge the nsplit partials of one (request, head, token) row; one warp per row.
@@ -215,6 +218,7 @@ int mdb_attn_staircase_varlen(const void* q, int64_t q_stride, const void* k, in
   a.v = static_cast<const bf16*>(v);
   a.out = static_cast<bf16*>(out);
   a.cu_seqlens = cu_seqlens;
+  a.cu_seqlens_q = nullptr;
   a.q_stride = q_stride;
   a.k_stride = k_stride;
   a.v_stride = v_stride;
@@ -225,7 +229,39 @@ int mdb_attn_staircase_varlen(const void* q, int64_t q_stride, const void* k, in
   while ((1 << lg) < stairs) ++lg;
   a.log2_stairs = lg;
   a.q_scale = 1.0f / sqrtf(static_cast<float>(kHeadDim)) * 1.44269504f;
-  return attn_stair_tc_launch(a, nseq, max_seqlen, total_tokens, static_cast<cudaStream_t>(stream));
+  a.scale_log2 = 1.0f;
+  return attn_stair_tc_launch(a, nseq, max_seqlen, total_tokens, total_tokens, static_cast<cudaStream_t>(stream));
+}
+
+int mdb_attn_causal_varlen(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride,
+                           void* out, int64_t out_stride, const int32_t* cu_q, const int32_t* cu_k, int nseq, int max_q,
+                           int64_t total_q, int64_t total_k, int hq, int hkv, float scale, mdb_stream_t stream) {
+  MDB_REQUIRE(nseq >= 0 && max_q >= 0 && hq > 0 && hkv > 0 && total_q >= 0 && total_k >= total_q, MDB_ERR_ARG);
+  if (nseq == 0 || max_q == 0 || total_q == 0) return MDB_OK;
+  MDB_REQUIRE(q && k && v && out && cu_q && cu_k && hq % hkv == 0 && scale > 0.f, MDB_ERR_ARG);
+  MDB_REQUIRE(nseq <= 65535 && hq <= 65535, MDB_ERR_UNSUPPORTED);
+  MDB_REQUIRE(q_stride >= static_cast<int64_t>(hq) * kHeadDim && out_stride >= static_cast<int64_t>(hq) * kHeadDim &&
+                  k_stride >= static_cast<int64_t>(hkv) * kHeadDim && v_stride >= static_cast<int64_t>(hkv) * kHeadDim,
+              MDB_ERR_ARG);
+  MDB_REQUIRE(out_stride % 8 == 0 && mdb_aligned16(q) && mdb_aligned16(k) && mdb_aligned16(v) && mdb_aligned16(out), MDB_ERR_ALIGN);
+  MDB_REQUIRE(attn_stair_tc_supported(hq, hkv, q_stride, k_stride, v_stride), MDB_ERR_UNSUPPORTED);
+  AttnStairArgs a;
+  a.q = static_cast<const bf16*>(q);
+  a.k = static_cast<const bf16*>(k);
+  a.v = static_cast<const bf16*>(v);
+  a.out = static_cast<bf16*>(out);
+  a.cu_seqlens = cu_k;
+  a.cu_seqlens_q = cu_q;
+  a.q_stride = q_stride;
+  a.k_stride = k_stride;
+  a.v_stride = v_stride;
+  a.out_stride = out_stride;
+  a.hq = hq;
+  a.hkv = hkv;
+  a.log2_stairs = 0;             // stairs of one token: a row sees the keys up to its own
+  a.q_scale = 1.0f;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  return attn_stair_tc_launch(a, nseq, max_q, total_q, total_k, static_cast<cudaStream_t>(stream));
 }
 
 // ---------------------------------------------------------------------------

@@ -101,10 +101,11 @@ struct AtArgs {
   float* part_ml;           // [bs][nsplit][hq][block][2]  (max in log2 units, sum)
   int table_stride, block, num_pages, nsplit, bs, row_blocks;
   // staircase form
-  const int32_t* cu_seqlens;
+  const int32_t* cu_seqlens;   // rows of the keys
+  const int32_t* cu_seqlens_q; // rows of the queries: the last ones of every sequence (NULL: all of them)
   int64_t out_stride;
   int nseq, max_qtiles, log2_stairs;
-  float q_scale;            // log2(e) / sqrt(D), applied to q and rounded to bf16 as the reference kernel does
+  float q_scale;            // applied to q and rounded to bf16: log2(e) / sqrt(D) as the reference kernel does, or 1
 };
 
 __device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int c0, int c1, int c2, uint32_t bar) {
@@ -176,7 +177,8 @@ struct AtUnit {
   int q_tok0;       // row of the unit's first token in the q tensor
   int req, split, tok0;        // paged: request, key-range part, first token of the block covered
   bool ctx_clamped;            // paged: the context length exceeded what the page table can address
-  int seq_start, m0, T;        // staircase: first packed row of the sequence, first token of the unit, length
+  int seq_start, T;            // staircase: first packed key row of the sequence, its length
+  int q_start, q_off, m0, Tq;  // ... first packed query row, tokens in front of it, first query of the unit, number of queries
 };
 
 template <bool STAIR>
@@ -195,12 +197,16 @@ __device__ __forceinline__ AtUnit at_unit(const AtArgs& a, const uint16_t* order
     w.seq_start = a.cu_seqlens[seq];
     w.T = a.cu_seqlens[seq + 1] - w.seq_start;
     w.m0 = qt * a.tokens_per_unit;
-    if (w.m0 >= w.T) return w;
+    const int32_t* cu_q = a.cu_seqlens_q != nullptr ? a.cu_seqlens_q : a.cu_seqlens;
+    w.q_start = cu_q[seq];
+    w.Tq = cu_q[seq + 1] - w.q_start;
+    w.q_off = w.T - w.Tq;
+    if (w.m0 >= w.Tq) return w;
     w.valid = true;
-    w.q_tok0 = w.seq_start + w.m0;
+    w.q_tok0 = w.q_start + w.m0;
     const int S = 1 << a.log2_stairs;
     const int pad = ((w.T + S - 1) >> a.log2_stairs << a.log2_stairs) - w.T;
-    const int last = min(w.m0 + a.tokens_per_unit, w.T) - 1;
+    const int last = w.q_off + min(w.m0 + a.tokens_per_unit, w.Tq) - 1;
     w.kbeg = 0;
     w.kend = min(w.T, ((((last + pad) >> a.log2_stairs) + 1) << a.log2_stairs) - pad);
     w.ntiles = (w.kend + kAtKeys - 1) / kAtKeys;
@@ -489,12 +495,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
       bf16* out_row;
       int64_t prow = 0;
       if (STAIR) {
-        const int i = w.m0 + tok_local;
-        row_valid = row_valid && i < w.T;
+        const int qi = w.m0 + tok_local, i = w.q_off + qi;
+        row_valid = row_valid && qi < w.Tq;
         const int S = 1 << a.log2_stairs;
         const int pad = ((w.T + S - 1) >> a.log2_stairs << a.log2_stairs) - w.T;
         limit = row_valid ? min(w.T - 1, ((((i + pad) >> a.log2_stairs) + 1) << a.log2_stairs) - 1 - pad) : -1;
-        out_row = a.out + static_cast<int64_t>(w.seq_start + (row_valid ? i : 0)) * a.out_stride + head * kHeadDim;
+        out_row = a.out + static_cast<int64_t>(w.q_start + (row_valid ? qi : 0)) * a.out_stride + head * kHeadDim;
       } else {
         const int tok = w.tok0 + tok_local;
         row_valid = row_valid && tok < a.block;
@@ -837,14 +843,16 @@ static bool attn_stair_tc_supported(int hq, int hkv, int64_t q_stride, int64_t k
   return q_stride % 8 == 0 && k_stride % 8 == 0 && v_stride % 8 == 0;
 }
 
-static int attn_stair_tc_launch(const AttnStairArgs& sa, int nseq, int max_seqlen, int64_t total_tokens, cudaStream_t st) {
+static int attn_stair_tc_launch(const AttnStairArgs& sa, int nseq, int max_seqlen, int64_t total_q, int64_t total_tokens,
+                                cudaStream_t st) {
   AtArgs a = {};
   a.q = sa.q;
   a.out = sa.out;
   a.hq = sa.hq; a.hkv = sa.hkv; a.group = sa.hq / sa.hkv;
-  a.scale_log2 = 1.0f;
+  a.scale_log2 = sa.scale_log2;
   a.q_scale = sa.q_scale;
   a.cu_seqlens = sa.cu_seqlens;
+  a.cu_seqlens_q = sa.cu_seqlens_q;
   a.out_stride = sa.out_stride;
   a.nseq = nseq;
   a.log2_stairs = sa.log2_stairs;
@@ -852,7 +860,7 @@ static int attn_stair_tc_launch(const AttnStairArgs& sa, int nseq, int max_seqle
   a.max_qtiles = (max_seqlen + a.tokens_per_unit - 1) / a.tokens_per_unit;
   a.nsplit = 1;
   CUtensorMap map_q, map_k, map_v;
-  if (!get_q_tensor_map(sa.q, total_tokens, sa.q_stride, sa.hq, a.group, a.tokens_per_unit, &map_q)) return MDB_ERR_CUDA;
+  if (!get_q_tensor_map(sa.q, total_q, sa.q_stride, sa.hq, a.group, a.tokens_per_unit, &map_q)) return MDB_ERR_CUDA;
   if (!get_tensor_map(sa.k, total_tokens, sa.hkv * kHeadDim, sa.k_stride, kAtKeys, &map_k)) return MDB_ERR_CUDA;
   if (!get_tensor_map(sa.v, total_tokens, sa.hkv * kHeadDim, sa.v_stride, kAtKeys, &map_v)) return MDB_ERR_CUDA;
   const int64_t units = static_cast<int64_t>(a.max_qtiles) * nseq * sa.hkv;

@@ -20,7 +20,15 @@
 // 73-82, nanovllm/layers/sdar_attention.py:37-38): a 256-column tile is two
 // heads, and the thread that owns a step row holds a whole head of it.
 // Tiles are ordered so that consecutive CTAs share a weight tile: it is read
-// from HBM once and served from L2 to the others.
+// from HBM once and served from L2 to the others.  The plain form can also
+// square the positive part of its result (relu^2) and store fp32 rows.
+//
+// GROUP form: many products of one shape in one launch, with the plain
+// epilogue.  Either one weight per head (head h multiplies column block h of
+// the activations and writes column block h of the output) or one weight per
+// expert (activation rows laid out by expert in tiles of 128, the expert of a
+// tile and the number of tiles read from device memory; a step of few rows
+// loads only the rows a tile can hold).
 //
 // PAIR form (taken from 2048 rows on): a cluster of two CTAs owns a tile of
 // 256 step rows x 256 weight rows (tcgen05.mma.cta_group::2).  Each CTA stages
@@ -39,7 +47,7 @@
 
 namespace mdb {
 
-enum TcEpilogue { kTcBf16 = 0, kTcSwiglu = 1, kTcLmHead = 2, kTcQkvRope = 3 };
+enum TcEpilogue { kTcBf16 = 0, kTcSwiglu = 1, kTcLmHead = 2, kTcQkvRope = 3, kTcGroup = 4 };
 
 constexpr int kTcBM = 128, kTcBN = 256, kTcBK = 64;
 constexpr int kTcStages = 4;
@@ -93,7 +101,20 @@ struct TcArgs {
   // bf16 form with few tiles: a cluster of ksplit CTAs shares one tile, each CTA a slice of k; the fp32 partial
   // tiles meet in shared memory (0 or 1: off)
   int ksplit;
+  // plain and GROUP epilogues: activation applied to the fp32 accumulator, and fp32 rows instead of bf16 (same ldy)
+  int act;
+  float* y32;
+  // GROUP form
+  int heads;                   // > 0: per-head products; 0: per-expert products
+  int a_rows;                  // activation rows a tile loads (16 .. 128); the rest of the operand tile is not stored
+  const int32_t* tile_expert;  // [tiles_m]
+  const int32_t* num_tiles;    // row tiles in use
 };
+
+__device__ __forceinline__ float tc_act(int act, float v) {
+  if (act == MDB_ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+  return v;
+}
 
 constexpr int kTcParkStride = (kTcBN + 4) * 4;   // bytes per parked fp32 accumulator row: 16-byte pad against bank conflicts
 
@@ -177,7 +198,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
   const uint32_t kr = ks > 1 ? cluster_ctarank() : 0u;
   const int work0 = PAIR ? static_cast<int>(blockIdx.x >> 1) : static_cast<int>(blockIdx.x) / ks;
   const int work_stride = PAIR ? static_cast<int>(gridDim.x >> 1) : static_cast<int>(gridDim.x) / ks;
-  const int tiles = a.tiles_m * a.tiles_n;
+  int tiles = a.tiles_m * a.tiles_n * (EPI == kTcGroup && a.heads > 0 ? a.heads : 1);
   const int kchunks = a.k / kTcBK;
   const int c_begin = static_cast<int>(kr) * kchunks / ks, c_end = (static_cast<int>(kr) + 1) * kchunks / ks;
   int parked_tile = -1;                                          // split-k: the tile whose partial this CTA parked
@@ -209,6 +230,23 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
   else __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = misc[0];
+  if (EPI == kTcGroup && a.heads == 0) {
+    pdl_wait();                            // the tile list comes from a preceding kernel
+    tiles = min(*a.num_tiles, a.tiles_m) * a.tiles_n;
+  }
+  // GROUP: row tile, column tile and group (head or expert) of work item t
+  auto group_tile = [&](int t, int& tn, int& tm, int& g) {
+    if (a.heads > 0) {
+      g = t / (a.tiles_m * a.tiles_n);
+      const int r = t % (a.tiles_m * a.tiles_n);
+      tn = r / a.tiles_m;
+      tm = r % a.tiles_m;
+    } else {
+      tm = t / a.tiles_n;
+      tn = t % a.tiles_n;
+      g = a.tile_expert[tm];
+    }
+  };
   // where an epilogue warp reports that it has drained an accumulator buffer
   const uint32_t acc_empty_target = PAIR ? map_to_cta(bar_acc_empty, 0) : bar_acc_empty;
   auto arrive_acc_empty = [&](int acc_buf) {
@@ -219,7 +257,16 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
   if (warp == kProducerWarp) {
     // the whole warp walks the loop (warp-uniform operands), one elected lane issues each instruction
     const uint32_t full_target = PAIR ? map_to_cta(bar_full, 0) : bar_full;
+    int w_row = 0, x_col = 0;              // GROUP: first weight row and first activation column of the group
+    const uint32_t a_bytes = EPI == kTcGroup ? static_cast<uint32_t>(a.a_rows) * kTcBK * 2 : kTcABytes;
     auto tile_of = [&](int t, int& tn, int& tm) {
+      if (EPI == kTcGroup) {
+        int g;
+        group_tile(t, tn, tm, g);
+        w_row = g * a.n;
+        x_col = a.heads > 0 ? g * a.k : 0;
+        return;
+      }
       tn = a.n_fastest ? t % a.tiles_n : t / a.tiles_m;   // consecutive CTAs share a weight tile, or,
       tm = a.n_fastest ? t / a.tiles_n : t % a.tiles_m;   // when the activations outgrow L2, an activation tile
     };
@@ -235,12 +282,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                                           : tn * kTcBN + static_cast<int>(rank) * 128;
         tma_load_2d_pair_w(bdst, &map_w, c * kTcBK, brow, full);
       } else {
-        mbar_arrive_expect_tx_w(full, kTcABytes + kTcBBytes);
+        mbar_arrive_expect_tx_w(full, a_bytes + kTcBBytes);
         if (EPI == kTcSwiglu) {
           tma_load_2d_w(bdst, &map_w, c * kTcBK, tn * 128, full);                             // 128 gate rows
           tma_load_2d_w(bdst + kTcBBytes / 2, &map_w, c * kTcBK, a.inter + tn * 128, full);   // their up rows
         } else {
-          tma_load_2d_w(bdst, &map_w, c * kTcBK, tn * kTcBN, full);
+          tma_load_2d_w(bdst, &map_w, c * kTcBK, w_row + tn * kTcBN, full);
         }
       }
     };
@@ -248,7 +295,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
       const uint32_t full = full_target + 8 * stage;
       const uint32_t adst = a_tiles + stage * kTcABytes;
       if (PAIR) tma_load_2d_pair_w(adst, &map_x, c * kTcBK, tm * kRowsPerTile + static_cast<int>(rank) * kTcBM, full);
-      else tma_load_2d_w(adst, &map_x, c * kTcBK, tm * kTcBM, full);
+      else tma_load_2d_w(adst, &map_x, x_col + c * kTcBK, tm * kTcBM, full);
     };
     // Weights are written by no kernel of a step: the first ring-full of weight tiles is requested before the
     // dependency wait (the stages are fresh, nothing to wait for), the activation tiles follow after it.
@@ -319,8 +366,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
     uint32_t acc_phase_tile = 0;   // tiles done (LM head: picks the record buffer)
     pdl_wait();   // the output buffer may still be read by the preceding kernel
     for (int t = work0; t < tiles; t += work_stride) {
-      const int tn = a.n_fastest ? t % a.tiles_n : t / a.tiles_m;
-      const int tm = a.n_fastest ? t / a.tiles_n : t % a.tiles_m;
+      int tn = a.n_fastest ? t % a.tiles_n : t / a.tiles_m;
+      int tm = a.n_fastest ? t / a.tiles_n : t % a.tiles_m;
+      int y_col = 0;                       // GROUP, per head: first output column of the head
+      if (EPI == kTcGroup) {
+        int g;
+        group_tile(t, tn, tm, g);
+        if (a.heads > 0) y_col = g * a.n;
+      }
       // q/k-norm + rotation form: this lane's position (-1: none, or outside the table) and the request for the
       // first quarter of the warp's cos | sin rows go out before the accumulator is waited for
       const uint32_t rope_smem = base + bars_off + 256 + warp * 4096;
@@ -385,8 +438,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
         parked_tile = t;
         break;
       }
-      if (EPI == kTcBf16) {
-        bf16* dst = a.y + static_cast<int64_t>(row) * a.ldy + tn * kTcBN;
+      if (EPI == kTcBf16 || EPI == kTcGroup) {
+        bf16* dst = a.y + static_cast<int64_t>(row) * a.ldy + y_col + tn * kTcBN;
         // Tensor-parallel pair: the copy for the peer is staged in shared memory, 32 rows x 64 columns per warp,
         // and leaves as 128-byte row segments (four rows per store instruction): over NVLink the 16-byte pieces
         // a thread holds of its own row would travel one by one.
@@ -401,7 +454,21 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           tmem_ld16(taddr + 32 * c + 16, v1);
           tmem_ld_wait();
           const int col = tn * kTcBN + 32 * c;
-          if (row < a.m) {
+          if (a.act != MDB_ACT_NONE) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) { v0[i] = tc_act(a.act, v0[i]); v1[i] = tc_act(a.act, v1[i]); }
+          }
+          if (a.y32 != nullptr) {
+            if (row < a.m) {
+              float* d32 = a.y32 + static_cast<int64_t>(row) * a.ldy + y_col + col;
+#pragma unroll
+              for (int i = 0; i < 16; i += 4) {
+                if (col + i + 4 <= a.n) *reinterpret_cast<float4*>(d32 + i) = make_float4(v0[i], v0[i + 1], v0[i + 2], v0[i + 3]);
+                if (col + 16 + i + 4 <= a.n)
+                  *reinterpret_cast<float4*>(d32 + 16 + i) = make_float4(v1[i], v1[i + 1], v1[i + 2], v1[i + 3]);
+              }
+            }
+          } else if (row < a.m) {
             if (col + 32 <= a.n) {
               uint4 o[4];
               o[0] = make_uint4(pack_bf16x2(v0[0], v0[1]), pack_bf16x2(v0[2], v0[3]), pack_bf16x2(v0[4], v0[5]), pack_bf16x2(v0[6], v0[7]));
@@ -748,7 +815,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           for (int j = 1; j < 8; ++j)
             if (j < ks) { sum.x += v[j].x; sum.y += v[j].y; sum.z += v[j].z; sum.w += v[j].w; }
           const int grow = tm * kTcBM + r, col = tn * kTcBN + 4 * c4;
-          if (grow < a.m) {
+          sum.x = tc_act(a.act, sum.x); sum.y = tc_act(a.act, sum.y);
+          sum.z = tc_act(a.act, sum.z); sum.w = tc_act(a.act, sum.w);
+          if (grow < a.m && a.y32 != nullptr) {
+            if (col + 4 <= a.n) *reinterpret_cast<float4*>(a.y32 + static_cast<int64_t>(grow) * a.ldy + col) = sum;
+          } else if (grow < a.m) {
             bf16* dst = a.y + static_cast<int64_t>(grow) * a.ldy + col;
             if (col + 4 <= a.n) {
               *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(sum.x, sum.y), pack_bf16x2(sum.z, sum.w));
@@ -795,7 +866,7 @@ static int launch_tc_impl(const bf16* x, int64_t ldx, const bf16* w, int w_rows,
   constexpr int kRowsPerTile = PAIR ? 2 * kTcBM : kTcBM;
   // after the barriers: sampler records (LM head), or 4 KB per epilogue warp: the peer's staged tile (bf16 form),
   // the cos | sin rows and the turned-around stores (q/k-norm + rotation form)
-  constexpr int kTail = (EPI == kTcQkvRope || EPI == kTcBf16) ? tc_epi_warps(EPI) * 4096 : kTcLmRecBytes;
+  constexpr int kTail = (EPI == kTcQkvRope || EPI == kTcBf16 || EPI == kTcGroup) ? tc_epi_warps(EPI) * 4096 : kTcLmRecBytes;
   constexpr int kSmem = 1024 + (PAIR ? kTcPairStages * (kTcABytes + kTcBBytes / 2) : kTcStages * (kTcABytes + kTcBBytes)) +
                         256 + kTail;
   static_assert(kSmem <= 232448, "shared memory of the tile GEMM");
@@ -888,6 +959,37 @@ static int launch_tc_impl(const bf16* x, int64_t ldx, const bf16* w, int w_rows,
   a.grid = 2 * pairs;
   cfg.numAttrs = g_opt_pdl ? 2 : 1;
   return cudaLaunchKernelEx(&cfg, gemm_tc_kernel<EPI, PAIR>, map_x, map_w, a) == cudaSuccess ? MDB_OK : MDB_ERR_CUDA;
+}
+
+// GROUP form: x [rows, x_cols], w [groups * n, k]; a.m = rows (of the buffer, in the per-expert form), a.heads or
+// the tile list, a.a_rows, a.y / a.y32, a.ldy, a.act set by the caller.
+static int launch_tc_group(const bf16* x, int64_t x_cols, int64_t ldx, const bf16* w, int64_t w_rows, TcArgs& a, cudaStream_t st) {
+  static int sm_count = 0;
+  if (sm_count == 0) {
+    int dev = 0;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sm_count, cudaDevAttrMultiProcessorCount, dev);
+    if (sm_count <= 0) sm_count = 148;
+  }
+  constexpr int kSmem = 1024 + kTcStages * (kTcABytes + kTcBBytes) + 256 + tc_epi_warps(kTcGroup) * 4096;
+  a.tiles_m = (a.m + kTcBM - 1) / kTcBM;
+  a.tiles_n = (a.n + kTcBN - 1) / kTcBN;
+  a.ksplit = 1;
+  CUtensorMap map_x, map_w;
+  if (!get_tensor_map(x, a.m, x_cols, ldx, a.a_rows, &map_x)) return MDB_ERR_CUDA;
+  if (!get_tensor_map(w, w_rows, a.k, a.k, kTcBN, &map_w)) return MDB_ERR_CUDA;
+  static PerDeviceOnce attr_once;
+  const int dev = attr_once.slot();
+  if (dev < 0) return MDB_ERR_CUDA;
+  if (!attr_once.done[dev]) {
+    if (cudaFuncSetAttribute(gemm_tc_kernel<kTcGroup, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess)
+      return MDB_ERR_CUDA;
+    attr_once.done[dev] = true;
+  }
+  const int64_t tiles = static_cast<int64_t>(a.tiles_m) * a.tiles_n * (a.heads > 0 ? a.heads : 1);
+  if (tiles > (1 << 30)) return MDB_ERR_UNSUPPORTED;
+  a.grid = tiles < sm_count ? static_cast<int>(tiles) : sm_count;
+  return mdb_launch(gemm_tc_kernel<kTcGroup, false>, dim3(a.grid), dim3(tc_threads(kTcGroup)), kSmem, st, map_x, map_w, a);
 }
 
 // CTA pairs from 2048 rows on (measured: +12 .. 15 % on the bf16-store projections at 4096 and 16384 rows, even at

@@ -8,4 +8,10 @@
 #include "gemm_tc.cu"
 #include "attention_tc.cu"
 #include "api_linear.cu"
+#include "rows32.cu"
+#include "moe.cu"
+#include "gemm_f32.cu"
+#include "api_gemm.cu"
+#include "recurrent.cu"
+#include "latent_attention.cu"
 #include "tp_p2p.cu"

@@ -1,0 +1,355 @@
+// Row kernels of the decoders whose residual stream is kept in fp32: embedding with a scale, residual add (from a
+// projection, from split-k slices, from the outputs of a mixture of experts) fused with the RMSNorm that follows,
+// RMSNorm of column segments of a projection (one of which may go straight into a paged cache), the per-head
+// normalisation and output gate behind a recurrence, and the row gather out of a paged latent cache.
+// Activations are bf16 or fp32 (template parameter), all arithmetic is fp32.
+#include "mdb_common.cuh"
+
+namespace mdb {
+
+template <typename T> __device__ __forceinline__ float act_to_f(T v);
+template <> __device__ __forceinline__ float act_to_f<bf16>(bf16 v) { return __bfloat162float(v); }
+template <> __device__ __forceinline__ float act_to_f<float>(float v) { return v; }
+template <typename T> __device__ __forceinline__ T act_from_f(float v);
+template <> __device__ __forceinline__ bf16 act_from_f<bf16>(float v) { return __float2bfloat16_rn(v); }
+template <> __device__ __forceinline__ float act_from_f<float>(float v) { return v; }
+
+template <typename T> __device__ __forceinline__ float4 act_load4(const T* p);
+template <> __device__ __forceinline__ float4 act_load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 act_load4<bf16>(const bf16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+template <typename T> __device__ __forceinline__ void act_store4(T* p, float4 v);
+template <> __device__ __forceinline__ void act_store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void act_store4<bf16>(bf16* p, float4 v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+
+// A projection's output as its consumer finds it: rows of T, or fp32 split-k slices that the consumer sums in slice
+// order and rounds to T, as the projection itself would have.
+template <typename T>
+__device__ __forceinline__ float rows_at(const mdb_rows& s, int64_t row, int col) {
+  const int64_t off = row * s.ld + s.col + col;
+  if (s.parts != nullptr) {
+    float a = 0.f;
+    for (int p = 0; p < s.nparts; ++p) a += s.parts[p * s.part_stride + off];
+    return act_to_f(act_from_f<T>(a));
+  }
+  return act_to_f(static_cast<const T*>(s.x)[off]);
+}
+template <typename T>
+__device__ __forceinline__ float4 rows_at4(const mdb_rows& s, int64_t row, int col) {
+  const int64_t off = row * s.ld + s.col + col;
+  if (s.parts != nullptr) {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int p0 = 0; p0 < s.nparts; p0 += 8) {
+      float4 v[8];                       // eight slices requested together: one round trip to L2 instead of eight
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (p0 + i < s.nparts) v[i] = *reinterpret_cast<const float4*>(s.parts + (p0 + i) * s.part_stride + off);
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (p0 + i < s.nparts) { a.x += v[i].x; a.y += v[i].y; a.z += v[i].z; a.w += v[i].w; }
+    }
+    a.x = act_to_f(act_from_f<T>(a.x)); a.y = act_to_f(act_from_f<T>(a.y));
+    a.z = act_to_f(act_from_f<T>(a.z)); a.w = act_to_f(act_from_f<T>(a.w));
+    return a;
+  }
+  return act_load4(static_cast<const T*>(s.x) + off);
+}
+__host__ __device__ __forceinline__ bool rows_present(const mdb_rows& s) { return s.x != nullptr || s.parts != nullptr; }
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// Sum over the CTA; `red` holds one float per warp and is free again after the call's last barrier.
+__device__ __forceinline__ float cta_sum(float v, float* red) {
+  v = warp_sum(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+  for (int w = 0; w < static_cast<int>(blockDim.x + 31) / 32; ++w) t += red[w];
+  return t;
+}
+
+constexpr int kRes32Threads = 256;
+
+// One CTA per row.  residual (+= or, with ids, = embed[id] * scale) + up to two projections + the weighted sum of
+// the chosen experts' rows; y = residual / rms * weight.  NV float4 chunks of the row per thread.
+template <typename T, int NV>
+__global__ void __launch_bounds__(kRes32Threads) residual_norm_kernel(const mdb_residual_norm_args a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[kRes32Threads / 32];
+  const int64_t row = blockIdx.x;
+  float* res = a.residual + row * a.width_pad;
+  float4 v[NV];
+  float ss = 0.f;
+  int64_t id = 0;
+  if (a.ids != nullptr) {
+    id = a.ids[row];
+    if (id < 0 || id >= a.vocab) {
+      if (threadIdx.x == 0) report_status(MDB_STATUS_BAD_TOKEN);
+      id = -1;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (threadIdx.x + i * kRes32Threads) * 4;
+    if (c >= a.width_pad) continue;
+    float4 x;
+    if (a.ids != nullptr) {
+      x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (id >= 0) {
+        x = act_load4(static_cast<const T*>(a.embed) + id * a.width_pad + c);
+        x.x *= a.embed_scale; x.y *= a.embed_scale; x.z *= a.embed_scale; x.w *= a.embed_scale;
+      }
+    } else {
+      x = *reinterpret_cast<const float4*>(res + c);
+    }
+#pragma unroll
+    for (int s = 0; s < 2; ++s) {
+      if (!rows_present(a.add[s])) continue;
+      const float4 d = rows_at4<T>(a.add[s], row, c);
+      x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
+    }
+    if (a.moe_rows != nullptr) {
+      float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int k = 0; k < a.moe_top; ++k) {
+        const int slot = a.moe_slot[row * a.moe_top + k];
+        if (slot < 0) continue;
+        const float w = a.moe_weight[row * a.moe_top + k];
+        const float4 e = act_load4(static_cast<const T*>(a.moe_rows) + slot * a.moe_ld + c);
+        d.x = fmaf(w, e.x, d.x); d.y = fmaf(w, e.y, d.y); d.z = fmaf(w, e.z, d.z); d.w = fmaf(w, e.w, d.w);
+      }
+      x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
+    }
+    *reinterpret_cast<float4*>(res + c) = x;
+    v[i] = x;
+    ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;      // columns past width hold zeros
+  }
+  if (a.y == nullptr) return;
+  const float rstd = 1.0f / sqrtf(cta_sum(ss, red) / static_cast<float>(a.width) + a.eps);
+  T* y = static_cast<T*>(a.y) + row * a.ldy;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (threadIdx.x + i * kRes32Threads) * 4;
+    if (c >= a.width_pad) continue;
+    const float4 w = *reinterpret_cast<const float4*>(a.weight + c);
+    act_store4(y + c, make_float4(v[i].x * rstd * w.x, v[i].y * rstd * w.y, v[i].z * rstd * w.z, v[i].w * rstd * w.w));
+  }
+}
+
+// One CTA per (row, segment): RMSNorm of n columns of a projection, zero-padded to n_pad, into row `row` of the
+// output or, with slots, into cache row slots[row].
+struct RmsSegments {
+  mdb_rms_segment s[MDB_MAX_RMS_SEGMENTS];
+};
+constexpr int kRmsRowsThreads = 128;
+template <typename T>
+__global__ void __launch_bounds__(kRmsRowsThreads) rms_rows_kernel(const RmsSegments segs) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[kRmsRowsThreads / 32];
+  const mdb_rms_segment& s = segs.s[blockIdx.y];
+  const int64_t row = blockIdx.x;
+  int64_t out_row = row;
+  if (s.slots != nullptr) {
+    const int slot = s.slots[row];
+    if (slot == -1) return;
+    if (slot < 0 || slot >= s.num_slots) {
+      if (threadIdx.x == 0) report_status(MDB_STATUS_BAD_SLOT);
+      return;
+    }
+    out_row = slot;
+  }
+  float ss = 0.f;
+  for (int c = threadIdx.x * 4; c < s.n_pad; c += kRmsRowsThreads * 4) {
+    const float4 x = rows_at4<T>(s.src, row, c);        // columns n .. n_pad of the projection are zeros
+    ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+  }
+  const float rstd = 1.0f / sqrtf(cta_sum(ss, red) / static_cast<float>(s.n) + s.eps);
+  T* out = static_cast<T*>(s.out) + out_row * s.ld_out;
+  for (int c = threadIdx.x * 4; c < s.n_pad; c += kRmsRowsThreads * 4) {
+    const float4 x = rows_at4<T>(s.src, row, c);
+    const float4 w = *reinterpret_cast<const float4*>(s.weight + c);
+    act_store4(out + c, make_float4(x.x * rstd * w.x, x.y * rstd * w.y, x.z * rstd * w.z, x.w * rstd * w.w));
+  }
+}
+
+// Behind a recurrence: one warp per (row, head).  y = o / rms(o) * weight * sigmoid(gate).
+template <typename T>
+__global__ void __launch_bounds__(128) gated_norm_kernel(const mdb_gated_norm_args a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t item = static_cast<int64_t>(blockIdx.x) * 4 + (threadIdx.x >> 5);
+  if (item >= static_cast<int64_t>(a.m) * a.heads) return;
+  const int64_t row = item / a.heads;
+  const int head = static_cast<int>(item % a.heads), lane = threadIdx.x & 31;
+  const float* o = a.o + (row * a.heads + head) * a.vdim;
+  float ss = 0.f;
+  for (int c = lane; c < a.vdim; c += 32) ss += o[c] * o[c];
+  const float rstd = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(a.vdim) + a.eps);
+  const float* w = a.weight + static_cast<int64_t>(head) * a.weight_head_stride;
+  T* y = static_cast<T*>(a.y) + row * a.ldy + static_cast<int64_t>(head) * a.vdim;
+  for (int c = lane; c < a.vdim; c += 32)
+    y[c] = act_from_f<T>(o[c] * rstd * w[c] * sigmoid_f(rows_at<T>(a.gate, row, head * a.vdim + c)));
+}
+
+// Row r of the output = the latent of token r - cu[seq] of its sequence, read through the page table.
+template <typename T>
+__global__ void __launch_bounds__(64) gather_latents_kernel(const T* cache, const int32_t* table,
+                                                            int table_stride, int num_pages, const int32_t* cu,
+                                                            int nseq, T* out, int width) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x;
+  int lo = 0, hi = nseq;                         // the last sequence that starts at or before this row
+  while (hi - lo > 1) {
+    const int mid = (lo + hi) >> 1;
+    if (cu[mid] <= row) lo = mid; else hi = mid;
+  }
+  const int pos = row - cu[lo];
+  int page = pos / kPage < table_stride ? table[static_cast<int64_t>(lo) * table_stride + pos / kPage] : -1;
+  if (page < 0 || page >= num_pages) {
+    if (threadIdx.x == 0) report_status(MDB_STATUS_BAD_PAGE);
+    page = 0;
+  }
+  const uint4* src = reinterpret_cast<const uint4*>(cache + (static_cast<int64_t>(page) * kPage + pos % kPage) * width);
+  uint4* dst = reinterpret_cast<uint4*>(out + static_cast<int64_t>(row) * width);
+  const int chunks = width * static_cast<int>(sizeof(T)) / 16;
+  for (int c = threadIdx.x; c < chunks; c += 64) dst[c] = src[c];
+}
+
+// Last kernel of a causal step: one CTA per wanted row of fp32 logits.  token = argmax of logit / temperature +
+// Gumbel noise, or of the logit itself where the row asks for the greedy choice (temperature 0); ties go to the
+// lower id.
+constexpr int kPickThreads = 512;
+__global__ void __launch_bounds__(kPickThreads)
+pick_token_kernel(const float* logits, int64_t ld, int vocab, const float* temperatures,
+                  uint32_t seed, const uint32_t* step_dev, int64_t* out,
+                  uint32_t* status_out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  if (status_out != nullptr && blockIdx.x == 0 && threadIdx.x == 0) *status_out = atomicExch(&g_device_status, 0u);
+  __shared__ float sv[kPickThreads / 32];
+  __shared__ int si[kPickThreads / 32];
+  const int row = blockIdx.x;
+  const float temp = temperatures[row];
+  const float inv = temp > 0.f ? 1.0f / temp : 1.0f;
+  const uint32_t key = gumbel_row_key(seed, step_dev != nullptr ? *step_dev : 0u, row);
+  float bv = -INFINITY;
+  int bi = 0x7fffffff;
+  for (int c = threadIdx.x; c < vocab; c += kPickThreads) {
+    float v = logits[row * ld + c] * inv;
+    if (temp > 0.f) v += gumbel_from_key(key, c);
+    if (v > bv) { bv = v; bi = c; }
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+    if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+  }
+  if ((threadIdx.x & 31) == 0) { sv[threadIdx.x >> 5] = bv; si[threadIdx.x >> 5] = bi; }
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    for (int w = 1; w < kPickThreads / 32; ++w)
+      if (sv[w] > bv || (sv[w] == bv && si[w] < bi)) { bv = sv[w]; bi = si[w]; }
+    out[row] = bi == 0x7fffffff ? 0 : bi;
+  }
+}
+
+}  // namespace mdb
+
+using namespace mdb;
+
+namespace {
+bool rows_ok(const mdb_rows& s) {
+  return !rows_present(s) || (s.ld % 4 == 0 && s.col % 4 == 0 && mdb_aligned16(s.x) && mdb_aligned16(s.parts) &&
+                              (s.parts == nullptr || (s.nparts >= 1 && s.part_stride % 4 == 0)));
+}
+
+template <typename T>
+int launch_residual_norm(const mdb_residual_norm_args& a, cudaStream_t st) {
+  const int chunks = (a.width_pad / 4 + kRes32Threads - 1) / kRes32Threads;
+  if (chunks <= 1) return mdb_launch(residual_norm_kernel<T, 1>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  if (chunks <= 2) return mdb_launch(residual_norm_kernel<T, 2>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  if (chunks <= 4) return mdb_launch(residual_norm_kernel<T, 4>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  if (chunks <= 8) return mdb_launch(residual_norm_kernel<T, 8>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  return MDB_ERR_UNSUPPORTED;
+}
+}  // namespace
+
+extern "C" {
+
+int mdb_residual_norm(const mdb_residual_norm_args* args, mdb_stream_t stream) {
+  MDB_REQUIRE(args != nullptr, MDB_ERR_ARG);
+  const mdb_residual_norm_args a = *args;
+  MDB_REQUIRE(a.m >= 0 && a.width > 0 && a.width_pad >= a.width, MDB_ERR_ARG);
+  if (a.m == 0) return MDB_OK;
+  MDB_REQUIRE(a.residual && (a.ids == nullptr || (a.embed && a.vocab > 0)), MDB_ERR_ARG);
+  MDB_REQUIRE(a.y == nullptr || (a.weight && a.ldy >= a.width_pad && a.ldy % 4 == 0), MDB_ERR_ARG);
+  MDB_REQUIRE(a.moe_rows == nullptr || (a.moe_slot && a.moe_weight && a.moe_top > 0 && a.moe_ld % 4 == 0), MDB_ERR_ARG);
+  MDB_REQUIRE(a.width_pad % 4 == 0 && rows_ok(a.add[0]) && rows_ok(a.add[1]) && mdb_aligned16(a.residual) &&
+                  mdb_aligned16(a.embed) && mdb_aligned16(a.weight) && mdb_aligned16(a.y) && mdb_aligned16(a.moe_rows),
+              MDB_ERR_ALIGN);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return a.dtype == MDB_F32 ? launch_residual_norm<float>(a, st) : launch_residual_norm<bf16>(a, st);
+}
+
+int mdb_rms_rows(int dtype, const mdb_rms_segment* segments, int nseg, int m, mdb_stream_t stream) {
+  MDB_REQUIRE(segments && nseg >= 1 && nseg <= MDB_MAX_RMS_SEGMENTS && m >= 0, MDB_ERR_ARG);
+  if (m == 0) return MDB_OK;
+  RmsSegments segs = {};
+  for (int i = 0; i < nseg; ++i) {
+    const mdb_rms_segment& s = segments[i];
+    MDB_REQUIRE(s.n > 0 && s.n_pad >= s.n && s.weight && s.out && s.ld_out >= s.n_pad && rows_present(s.src), MDB_ERR_ARG);
+    MDB_REQUIRE(s.n_pad % 4 == 0 && s.ld_out % 4 == 0 && rows_ok(s.src) && mdb_aligned16(s.weight) && mdb_aligned16(s.out),
+                MDB_ERR_ALIGN);
+    segs.s[i] = s;
+  }
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (dtype == MDB_F32) return mdb_launch(rms_rows_kernel<float>, dim3(m, nseg), dim3(kRmsRowsThreads), 0, st, segs);
+  return mdb_launch(rms_rows_kernel<bf16>, dim3(m, nseg), dim3(kRmsRowsThreads), 0, st, segs);
+}
+
+int mdb_gated_norm(const mdb_gated_norm_args* args, mdb_stream_t stream) {
+  MDB_REQUIRE(args != nullptr, MDB_ERR_ARG);
+  const mdb_gated_norm_args a = *args;
+  MDB_REQUIRE(a.m >= 0 && a.heads > 0 && a.vdim > 0, MDB_ERR_ARG);
+  if (a.m == 0) return MDB_OK;
+  MDB_REQUIRE(a.o && a.weight && a.y && rows_present(a.gate) && a.ldy >= static_cast<int64_t>(a.heads) * a.vdim, MDB_ERR_ARG);
+  const int64_t items = static_cast<int64_t>(a.m) * a.heads;
+  const int grid = static_cast<int>((items + 3) / 4);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (a.dtype == MDB_F32) return mdb_launch(gated_norm_kernel<float>, dim3(grid), dim3(128), 0, st, a);
+  return mdb_launch(gated_norm_kernel<bf16>, dim3(grid), dim3(128), 0, st, a);
+}
+
+int mdb_gather_latents(int dtype, const void* cache, const int32_t* block_table, int table_stride, int num_pages,
+                       const int32_t* cu, int nseq, int total, void* out, int width, mdb_stream_t stream) {
+  MDB_REQUIRE(total >= 0 && nseq >= 0 && width > 0 && num_pages > 0 && table_stride > 0, MDB_ERR_ARG);
+  if (total == 0 || nseq == 0) return MDB_OK;
+  MDB_REQUIRE(cache && block_table && cu && out, MDB_ERR_ARG);
+  MDB_REQUIRE(width % 8 == 0 && mdb_aligned16(cache) && mdb_aligned16(out), MDB_ERR_ALIGN);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (dtype == MDB_F32)
+    return mdb_launch(gather_latents_kernel<float>, dim3(total), dim3(64), 0, st, static_cast<const float*>(cache),
+                      block_table, table_stride, num_pages, cu, nseq, static_cast<float*>(out), width);
+  return mdb_launch(gather_latents_kernel<bf16>, dim3(total), dim3(64), 0, st, static_cast<const bf16*>(cache), block_table,
+                    table_stride, num_pages, cu, nseq, static_cast<bf16*>(out), width);
+}
+
+int mdb_pick_token(const float* logits, int64_t ld, int m, int vocab, const float* temperatures, uint32_t seed,
+                   const uint32_t* step_dev, int64_t* out, uint32_t* status_out, mdb_stream_t stream) {
+  MDB_REQUIRE(m >= 0 && vocab > 0 && ld >= vocab, MDB_ERR_ARG);
+  if (m == 0) return MDB_OK;
+  MDB_REQUIRE(logits && temperatures && out, MDB_ERR_ARG);
+  return mdb_launch(pick_token_kernel, dim3(m), dim3(kPickThreads), 0, static_cast<cudaStream_t>(stream), logits, ld, vocab,
+                    temperatures, seed, step_dev, out, status_out);
+}
+
+}  // extern "C"

@@ -12,6 +12,8 @@ import os
 from dataclasses import dataclass
 from types import SimpleNamespace
 
+from .hybrid_config import HybridConfig
+
 
 @dataclass
 class DecoderConfig:
@@ -56,7 +58,7 @@ class Config:
     num_kvcache_blocks: int = -1
     mask_token_id: int = 151669
     block_size: int = 32
-    decoder_config: DecoderConfig | None = None
+    decoder_config: DecoderConfig | HybridConfig | None = None
     # Not in the reference: a request whose block is complete runs the pass that writes the block's final K/V
     # and, in the same step, the first denoising pass of its next block (one pass per block saved; the tokens
     # are the ones the two separate passes would produce from the same noise).  Off: the reference's schedule.
@@ -67,8 +69,16 @@ class Config:
     # are thrown away and the step asked for runs.  Same tokens either way; the host's work between two steps
     # overlaps with the GPU's.
     launch_ahead: bool = True
+    # Not in the reference: activation type of the designs that also run in true fp32 ("bfloat16" or "float32"); the
+    # block-diffusion decoder is bf16 only.
+    dtype: str = "bfloat16"
+    # Not in the reference: recurrent-state slots of the designs that have recurrent layers (-1: one per request in
+    # flight).
+    num_state_slots: int = -1
 
     def __post_init__(self):
+        if self.dtype not in ("bfloat16", "float32"):
+            raise AssertionError("dtype must be bfloat16 or float32")
         if self.kvcache_block_size % 256 != 0:
             raise AssertionError("kvcache_block_size must be a multiple of 256")
         if not 1 <= self.tensor_parallel_size <= 8:
@@ -79,10 +89,10 @@ class Config:
             path = self.model if self.checkpoint is None else os.path.join(self.model, self.checkpoint)
             with open(os.path.join(path, "config.json")) as f:
                 raw = json.load(f)
-            text = raw.get("language_model_config") or raw.get("text_config") or raw
             self.hf_config = SimpleNamespace(**raw)
             if self.decoder_config is None:
-                self.decoder_config = DecoderConfig.from_namespace(SimpleNamespace(**text))
+                from .registry import read_config
+                self.decoder_config = read_config(raw)
         if self.decoder_config is None:
             self.decoder_config = DecoderConfig()
         self.max_model_len = min(self.max_model_len, self.decoder_config.max_position_embeddings)

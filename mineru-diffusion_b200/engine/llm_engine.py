@@ -2,15 +2,16 @@
 
 The part of the reference's ``LLMEngine`` that drives the hot path
 (``engines/nano_dvlm/nanovllm/engine/llm_engine.py:66-105``): schedule, run,
-post-process, collect finished requests.  Tokenizer, processor and the CLI
-stay with the reference; requests enter here as ``Sequence`` objects.
+post-process, collect finished requests.  Tokenizer and processor stay with the
+reference; requests enter here as ``Sequence`` objects.  The design named by the
+configuration decides which runner and scheduler work together (``registry``).
 """
 from __future__ import annotations
 
 from time import perf_counter
 
+from . import registry
 from .config import Config
-from .scheduler import Scheduler
 from .sequence import Sequence
 
 
@@ -19,9 +20,14 @@ class LLMEngine:
     def __init__(self, config: Config, model_runner):
         self.config = config
         self.model_runner = model_runner      # sets config.num_kvcache_blocks before the scheduler reads it
-        self.scheduler = Scheduler(config)
+        self.scheduler = registry.of_config(getattr(config, "decoder_config", None)).load("scheduler")(config)
         self.num_prefill_steps = 0
         self.num_decode_steps = 0
+
+    @classmethod
+    def from_config(cls, config: Config, **runner_args) -> "LLMEngine":
+        """Engine with the runner of the configuration's design."""
+        return cls(config, registry.of_config(config.decoder_config).load("runner")(config, **runner_args))
 
     def add_sequence(self, seq: Sequence):
         self.scheduler.add(seq)

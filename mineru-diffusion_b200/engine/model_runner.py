@@ -96,6 +96,8 @@ class ModelRunner:
             raise RuntimeError("ModelRunner needs a CUDA device: the decode path has no CPU implementation")
         if config.tensor_parallel_size not in (1, 2):
             raise NotImplementedError("tensor_parallel_size must be 1 or 2 (more GPUs serve as request-parallel replicas)")
+        if getattr(config, "dtype", "bfloat16") != "bfloat16":
+            raise NotImplementedError("the block-diffusion decoder runs in bfloat16 only")
         if noise not in ("gumbel", "none", "explicit"):
             raise ValueError("noise must be 'gumbel', 'none' or 'explicit'")
         self.config = config
@@ -466,6 +468,8 @@ class ModelRunner:
         sp = seqs[0].sampling_params
         if sp.denoising_strategy != "low_confidence_dynamic":
             raise NotImplementedError(f"Denoising strategy {sp.denoising_strategy} not implemented")
+        if getattr(sp, "greedy", False):
+            raise NotImplementedError("the block-diffusion sampler has no greedy form")
         with torch.inference_mode():
             quotas = self._step_quotas(seqs, is_prefill)
             graph_tail = (not is_prefill) and quotas is None and not self.keep_last and self._use_graph(bs)

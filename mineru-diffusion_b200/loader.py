@@ -22,6 +22,8 @@ import torch
 
 from .decoder import DecoderWeights, LayerWeights
 from .engine.config import DecoderConfig
+from .engine.hybrid_config import HybridConfig
+from .hybrid import HybridWeights
 
 _LAYER = re.compile(r"^model\.layers\.(\d+)\.(.+)\.weight$")
 _SKIPPED_PREFIXES = ("vision_model.", "vision_abstractor.", "visual.", "vision_tower.")
@@ -133,6 +135,21 @@ def load_decoder_weights(path: str, cfg: DecoderConfig, device, tp_rank: int = 0
         raise KeyError(f"checkpoint lacks {len(missing)} tensors, first: {missing[:4]}")
     lm_head = top["embed"] if cfg.tie_word_embeddings else top["lm_head"]
     return DecoderWeights(top["embed"], [LayerWeights(**w) for w in lw], top["final_ln"], lm_head)
+
+
+def load_hybrid_weights(path: str, cfg: HybridConfig, device, dtype=torch.bfloat16) -> HybridWeights:
+    """Weights of a ``HybridConfig`` design from every ``*.safetensors`` file of ``path``.  Raises ``KeyError`` for a
+    missing tensor and ``ValueError`` for one of the wrong shape or an unknown name."""
+    from safetensors import safe_open
+    files = sorted(glob(os.path.join(path, "*.safetensors")))
+    if not files:
+        raise FileNotFoundError(f"no *.safetensors file in {path}")
+    tensors = {}
+    for file in files:
+        with safe_open(file, "pt", "cpu") as f:
+            for name in f.keys():
+                tensors[name] = f.get_tensor(name)
+    return HybridWeights.build(cfg, tensors, device, dtype)
 
 
 def has_checkpoint(path: str | None) -> bool:

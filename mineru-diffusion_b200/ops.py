@@ -537,3 +537,257 @@ def lm_head_sample_tp(hidden: torch.Tensor, weight: torch.Tensor, temperatures: 
                                                peer_flags_ptr, wait_flags_ptr, wait_count, tag, epoch.data_ptr(),
                                                x0.data_ptr(), conf.data_ptr(), _stream()), "mdb_lmhead_sample_tp")
     return x0, conf
+
+
+# --------------------------------------------------------------------------
+# Decoders with an fp32 residual: recurrent mixers, latent attention, experts.  Activations are bf16 or fp32 tensors.
+
+_DTYPES = {torch.bfloat16: 0, torch.float32: 1}
+ACT_NONE, ACT_RELU2 = 0, 1
+
+
+class Rows:
+    """A projection's output as its consumer takes it: rows of the activation type, or the fp32 split-k slices of a
+    short step, which the consumer sums and rounds.  ``cols(c)`` is the view that starts at column ``c``."""
+    __slots__ = ("x", "parts", "ld", "col")
+
+    def __init__(self, x: torch.Tensor | None = None, parts: torch.Tensor | None = None, col: int = 0, ld: int | None = None):
+        self.x, self.parts, self.col = x, parts, col
+        self.ld = ld if ld is not None else (x.stride(0) if x is not None else parts.shape[-1])
+
+    def cols(self, c: int) -> "Rows":
+        return Rows(self.x, self.parts, self.col + c, self.ld)
+
+    def c(self) -> _lib.Rows:
+        if self.parts is not None:
+            return _lib.Rows(None, self.parts.data_ptr(), self.ld, self.parts.stride(0), self.parts.shape[0], self.col)
+        return _lib.Rows(self.x.data_ptr(), None, self.ld, 0, 0, self.col)
+
+
+_NO_ROWS = _lib.Rows()
+
+
+def _rows_c(r: Rows | None) -> _lib.Rows:
+    return _NO_ROWS if r is None else r.c()
+
+
+def _act_dtype(t: torch.Tensor, name: str) -> int:
+    if not t.is_cuda:
+        raise RuntimeError(f"{name} must be a CUDA tensor (libmdb200 has no CPU path)")
+    if t.dtype not in _DTYPES:
+        raise TypeError(f"{name} must be bfloat16 or float32, got {t.dtype}")
+    return _DTYPES[t.dtype]
+
+
+def gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: int = ACT_NONE) -> torch.Tensor:
+    """out = act(x w^T); x [m, k] (row stride free), w [n, k]; out of the activation type, or fp32."""
+    m, k = x.shape
+    n = w.shape[0]
+    a = _lib.GemmArgs(_act_dtype(x, "x"), 0, act, int(out.dtype == torch.float32), x.data_ptr(), w.data_ptr(),
+                      out.data_ptr(), _rows(x, "x"), _rows(out, "out"), m, n, k, 0, 0, 0, None, None)
+    _lib.check(_lib.lib().mdb_gemm(a, _stream()), "mdb_gemm")
+    return out
+
+
+def gemm_heads(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """Head h: out[:, h n : (h + 1) n] = x[:, h k : (h + 1) k] w[h]^T; w [heads, n, k]."""
+    heads, n, k = w.shape
+    a = _lib.GemmArgs(_act_dtype(x, "x"), 1, 0, int(out.dtype == torch.float32), x.data_ptr(), w.data_ptr(), out.data_ptr(),
+                      _rows(x, "x"), _rows(out, "out"), x.shape[0], n, k, heads, 0, 0, None, None)
+    _lib.check(_lib.lib().mdb_gemm(a, _stream()), "mdb_gemm (per head)")
+    return out
+
+
+def gemm_experts(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_expert: torch.Tensor, num_tiles: torch.Tensor,
+                 max_rows_per_expert: int = 0, act: int = ACT_NONE) -> torch.Tensor:
+    """Rows of x / out laid out by expert in tiles of 128; w [experts, n, k]."""
+    experts, n, k = w.shape
+    a = _lib.GemmArgs(_act_dtype(x, "x"), 2, act, int(out.dtype == torch.float32), x.data_ptr(), w.data_ptr(),
+                      out.data_ptr(), _rows(x, "x"), _rows(out, "out"), x.shape[0], n, k, 0, experts, max_rows_per_expert,
+                      tile_expert.data_ptr(), num_tiles.data_ptr())
+    _lib.check(_lib.lib().mdb_gemm(a, _stream()), "mdb_gemm (per expert)")
+    return out
+
+
+def residual_norm(residual: torch.Tensor, width: int, eps: float, dtype: torch.dtype, weight: torch.Tensor | None = None,
+                  out: torch.Tensor | None = None, add: tuple = (), ids: torch.Tensor | None = None,
+                  embed: torch.Tensor | None = None, embed_scale: float = 1.0, moe: tuple | None = None) -> None:
+    """Folds projections (``add``), chosen experts' rows (``moe`` = rows, slots [m, top], weights [m, top]) or the scaled
+    embedding (``ids``) into the fp32 residual and writes its RMSNorm to ``out``."""
+    m, wp = residual.shape
+    a = _lib.ResidualNormArgs(dtype=_DTYPES[dtype], m=m, width=width, width_pad=wp, residual=residual.data_ptr(), eps=eps,
+                              weight=_ptr(weight), y=_ptr(out), ldy=0 if out is None else _rows(out, "out"))
+    if ids is not None:
+        _need(ids, torch.int64, "ids")
+        a.ids, a.embed, a.vocab, a.embed_scale = ids.data_ptr(), embed.data_ptr(), embed.shape[0], embed_scale
+    for i, r in enumerate(add):
+        a.add[i] = r.c()
+    if moe is not None:
+        rows, slots, weights = moe
+        a.moe_rows, a.moe_ld, a.moe_slot, a.moe_weight, a.moe_top = (rows.data_ptr(), rows.stride(0), slots.data_ptr(),
+                                                                     weights.data_ptr(), slots.shape[1])
+    _lib.check(_lib.lib().mdb_residual_norm(a, _stream()), "mdb_residual_norm")
+
+
+def rms_segment(src: Rows, n: int, n_pad: int, weight: torch.Tensor, eps: float, out: torch.Tensor,
+                slots: torch.Tensor | None = None) -> _lib.RmsSegment:
+    """Columns [0, n) of ``src``, RMS-normalised and zero-padded to n_pad, into rows of ``out`` ([rows, >= n_pad])."""
+    return _lib.RmsSegment(src.c(), weight.data_ptr(), out.data_ptr(), out.stride(0), _ptr(slots), out.shape[0], n, n_pad, eps)
+
+
+def rms_rows(segments: list, m: int, dtype: torch.dtype) -> None:
+    arr = (_lib.RmsSegment * len(segments))(*segments)
+    _lib.check(_lib.lib().mdb_rms_rows(_DTYPES[dtype], arr, len(segments), m, _stream()), "mdb_rms_rows")
+
+
+def gated_norm(o: torch.Tensor, gate: Rows, weight: torch.Tensor, per_head_weight: bool, eps: float, out: torch.Tensor) -> None:
+    """o [m, heads, vdim] fp32, normalised per head, times weight, times sigmoid(gate), into out [m, heads * vdim]."""
+    m, heads, vdim = o.shape
+    a = _lib.GatedNormArgs(_act_dtype(out, "out"), m, heads, vdim, o.data_ptr(), gate.c(), weight.data_ptr(), out.data_ptr(),
+                           _rows(out, "out"), vdim if per_head_weight else 0, eps)
+    _lib.check(_lib.lib().mdb_gated_norm(a, _stream()), "mdb_gated_norm")
+
+
+def scan_dim_pad(dim: int) -> int:
+    p = int(_lib.lib().mdb_scan_dim_pad(dim))
+    if p == 0:
+        raise ValueError(f"recurrent heads of {dim} key channels are not supported (at most 512)")
+    return p
+
+
+def scan_blocks(vdim: int) -> int:
+    return int(_lib.lib().mdb_scan_blocks(vdim))
+
+
+def scan_fusable(dim_pad: int, vdim: int) -> bool:
+    return bool(_lib.lib().mdb_scan_fusable(dim_pad, vdim))
+
+
+def delta_prep(dtype: torch.dtype, m: int, bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q: Rows, k: Rows, v: Rows,
+               b: Rows, conv: tuple, conv_state: torch.Tensor, portions: tuple, outs: tuple, shift_state: bool,
+               copy: Rows | None = None, copy_out: torch.Tensor | None = None) -> None:
+    """``conv`` = fp32 [channels, taps] weights of q, k, v; ``conv_state`` [slots, taps - 1, channels]; ``portions`` =
+    (row_seq, cu_q, start, state_slot); ``outs`` = fp32 (q, k [m, kv_heads, dim_pad], v [m, heads, vdim], beta [m, heads],
+    k.q [m, kv_heads])."""
+    qo, ko, vo, bo, kqo = outs
+    row_seq, cu_q, start, slot = portions
+    a = _lib.DeltaPrepArgs(
+        dtype=_DTYPES[dtype], m=m, bs=bs, heads=heads, kv_heads=kv_heads, dim=dim, dim_pad=qo.shape[-1], vdim=vdim,
+        taps=conv[0].shape[1], channels=conv_state.shape[-1], shift_state=int(shift_state),
+        copy_cols=0 if copy is None else copy_out.shape[1], q=q.c(), k=k.c(), v=v.c(), b=b.c(), copy=_rows_c(copy),
+        copy_out=_ptr(copy_out), copy_ld=0 if copy_out is None else copy_out.stride(0), conv_q=conv[0].data_ptr(),
+        conv_k=conv[1].data_ptr(), conv_v=conv[2].data_ptr(), conv_state=conv_state.data_ptr() or None,
+        conv_slot_stride=conv_state.stride(0), num_slots=conv_state.shape[0], row_seq=row_seq.data_ptr(),
+        cu_q=cu_q.data_ptr(), start=start.data_ptr(), state_slot=slot.data_ptr(), q_out=qo.data_ptr(), k_out=ko.data_ptr(),
+        v_out=vo.data_ptr(), beta_out=bo.data_ptr(), kq_out=kqo.data_ptr())
+    _lib.check(_lib.lib().mdb_delta_prep(a, _stream()), "mdb_delta_prep")
+
+
+def channel_decay(x: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, out: torch.Tensor, dim: int) -> None:
+    """out [m, heads, dim_pad] = exp(-exp(a_log) softplus(x + dt_bias)); x fp32 [m, >= heads * dim]."""
+    m, heads, dp = out.shape
+    _lib.check(_lib.lib().mdb_channel_decay(x.data_ptr(), _rows(x, "x"), a_log.data_ptr(), dt_bias.data_ptr(),
+                                            out.data_ptr(), m, heads, dim, dp, _stream()), "mdb_channel_decay")
+
+
+def mlstm_prep(dtype: torch.dtype, m: int, heads: int, dim: int, vdim: int, q: Rows, k: Rows, v: Rows, i: Rows, f: Rows,
+               bias_i: torch.Tensor, bias_f: torch.Tensor, cap: float, outs: tuple) -> None:
+    qo, ko, vo, li, lf = outs
+    a = _lib.MlstmPrepArgs(_DTYPES[dtype], m, heads, dim, qo.shape[-1], vdim, q.c(), k.c(), v.c(), i.c(), f.c(),
+                           bias_i.data_ptr(), bias_f.data_ptr(), qo.data_ptr(), ko.data_ptr(), vo.data_ptr(), li.data_ptr(),
+                           lf.data_ptr(), cap)
+    _lib.check(_lib.lib().mdb_mlstm_prep(a, _stream()), "mdb_mlstm_prep")
+
+
+SCAN_DELTA, SCAN_MLSTM = 0, 1
+
+
+def scan(mode: int, dtype: torch.dtype, bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q, k, v, s0, s1, state,
+         portions: tuple, eps: float = 0.0, g=None, nstate=None, mstate=None, out=None, raw_decay: Rows | None = None,
+         a_log=None, dt_bias=None, gate: Rows | None = None, norm=None, per_head_norm: bool = False, y=None) -> None:
+    """The recurrence over every sequence's portion; ``state`` [slots, heads, vdim, dim_pad] fp32.  With ``y`` the fused
+    one-token form runs (decay from ``raw_decay``, gated norm into ``y``), else ``out`` [m, heads, vdim] fp32 is written."""
+    _, cu_q, start, slot = portions
+    a = _lib.ScanArgs(
+        mode=mode, dtype=_DTYPES[dtype], fused=int(y is not None), bs=bs, heads=heads, kv_heads=kv_heads, dim=dim,
+        dim_pad=q.shape[-1], vdim=vdim, eps=eps, q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), g=_ptr(g), s0=s0.data_ptr(),
+        s1=s1.data_ptr(), state=state.data_ptr(), state_slot_stride=state.stride(0), num_slots=state.shape[0],
+        nstate=_ptr(nstate), mstate=_ptr(mstate), cu_q=cu_q.data_ptr(), start=start.data_ptr(), state_slot=slot.data_ptr(),
+        out=_ptr(out), raw_decay=_rows_c(raw_decay), a_log=_ptr(a_log), dt_bias=_ptr(dt_bias), gate=_rows_c(gate),
+        norm=_ptr(norm), norm_head_stride=vdim if per_head_norm else 0, y=_ptr(y), ldy=0 if y is None else _rows(y, "y"))
+    _lib.check(_lib.lib().mdb_scan(a, _stream()), "mdb_scan")
+
+
+def moe_route(logits: Rows, m: int, experts: int, top: int, groups: int, keep: int, ids: torch.Tensor, weights: torch.Tensor,
+              row_slot: torch.Tensor | None = None) -> None:
+    a = _lib.MoeRouteArgs(m, experts, top, groups, keep, logits.c(), _ptr(row_slot), ids.data_ptr(), weights.data_ptr())
+    _lib.check(_lib.lib().mdb_moe_route(a, _stream()), "mdb_moe_route")
+
+
+def moe_max_tiles(m: int, top: int, experts: int) -> int:
+    return int(_lib.lib().mdb_moe_max_tiles(m, top, experts))
+
+
+def moe_plan(ids: torch.Tensor, experts: int, max_tiles: int, slot: torch.Tensor, row_token: torch.Tensor,
+             tile_expert: torch.Tensor, num_tiles: torch.Tensor) -> None:
+    m, top = ids.shape
+    a = _lib.MoePlanArgs(m, top, experts, max_tiles, ids.data_ptr(), slot.data_ptr(), row_token.data_ptr(),
+                         tile_expert.data_ptr(), num_tiles.data_ptr())
+    _lib.check(_lib.lib().mdb_moe_plan(a, _stream()), "mdb_moe_plan")
+
+
+def moe_gather(x: torch.Tensor, out: torch.Tensor, row_token: torch.Tensor, num_tiles: torch.Tensor, max_tiles: int) -> None:
+    _lib.check(_lib.lib().mdb_moe_gather(_act_dtype(x, "x"), x.data_ptr(), _rows(x, "x"), out.data_ptr(), out.shape[1],
+                                         row_token.data_ptr(), num_tiles.data_ptr(), max_tiles, _stream()), "mdb_moe_gather")
+
+
+def latent_attn_workspace_bytes(m: int, heads: int, width: int, nsplit: int) -> int:
+    return int(_lib.lib().mdb_latent_attn_workspace_bytes(m, heads, width, nsplit))
+
+
+def latent_attn(q: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, row_seq: torch.Tensor, row_pos: torch.Tensor,
+                heads: int, scale: float, out: torch.Tensor, nsplit: int = 1, workspace: torch.Tensor | None = None) -> None:
+    """q, out [m, heads * width]; cache [pages * 256, width]; the row at position p sees keys 0 .. p (p = -1: no row)."""
+    m, width = q.shape[0], cache.shape[1]
+    _need(block_table, torch.int32, "block_table")
+    _lib.check(_lib.lib().mdb_latent_attn(
+        _act_dtype(q, "q"), q.data_ptr(), cache.data_ptr(), out.data_ptr(), block_table.data_ptr(), block_table.stride(0),
+        row_seq.data_ptr(), row_pos.data_ptr(), m, heads, width, cache.shape[0] // 256, scale, nsplit, _ptr(workspace),
+        0 if workspace is None else workspace.numel() * workspace.element_size(), _stream()), "mdb_latent_attn")
+
+
+def gather_latents(cache: torch.Tensor, block_table: torch.Tensor, cu: torch.Tensor, nseq: int, out: torch.Tensor) -> None:
+    """out [total, width] = the cached rows of every sequence in order (cu [nseq + 1] row offsets)."""
+    _lib.check(_lib.lib().mdb_gather_latents(_act_dtype(cache, "cache"), cache.data_ptr(), block_table.data_ptr(),
+                                             block_table.stride(0), cache.shape[0] // 256, cu.data_ptr(), nseq, out.shape[0],
+                                             out.data_ptr(), cache.shape[1], _stream()), "mdb_gather_latents")
+
+
+def causal_attn_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_q: torch.Tensor, cu_k: torch.Tensor, nseq: int,
+                       max_q: int, scale: float, out: torch.Tensor) -> None:
+    """Causal attention over packed rows, head size 128: q/out [total_q, hq, 128], k/v [total_k, hkv, 128] (row strides
+    free); the queries of a sequence are its last ones."""
+    for t, nm in ((q, "q"), (k, "k"), (v, "v"), (out, "out")):
+        _need(t, _BF16, nm)
+        if t.shape[-1] != 128 or t.stride(-1) != 1 or t.stride(1) != 128:
+            raise ValueError(f"{nm}: heads of 128 must be densely packed")
+    _lib.check(_lib.lib().mdb_attn_causal_varlen(
+        q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), out.data_ptr(), out.stride(0),
+        cu_q.data_ptr(), cu_k.data_ptr(), nseq, max_q, q.shape[0], k.shape[0], q.shape[1], k.shape[1], scale, _stream()),
+        "mdb_attn_causal_varlen")
+
+
+def pick_token(logits: torch.Tensor, vocab: int, temperatures: torch.Tensor, seed: int, step_dev: torch.Tensor | None,
+               out: torch.Tensor, status_out: torch.Tensor | None = None) -> None:
+    """Token per row of fp32 logits [m, >= vocab]: Gumbel-max at the row's temperature, or arg-max at temperature 0."""
+    _need(logits, torch.float32, "logits")
+    _lib.check(_lib.lib().mdb_pick_token(logits.data_ptr(), _rows(logits, "logits"), logits.shape[0], vocab,
+                                         temperatures.data_ptr(), seed & 0xFFFFFFFF, _ptr(step_dev), out.data_ptr(),
+                                         _ptr(status_out), _stream()), "mdb_pick_token")
+
+
+def copy_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out[i] = table[ids[i]] for rows of either activation type (a byte copy)."""
+    t, o = (table, out) if table.dtype == _BF16 else (table.view(_BF16), out.view(_BF16))
+    gather_rows(t, ids, out=o)
+    return out
