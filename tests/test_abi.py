@@ -74,3 +74,23 @@ def test_ops_refuse_cpu_tensors(built):
         built.ops.linear(x, x)
     with pytest.raises(RuntimeError):
         built.ops.store_kvcache(x.view(4, 1, 64), x.view(4, 1, 64), x, x, torch.zeros(4, dtype=torch.int32))
+
+
+def test_argument_blocks_match_the_header(tmp_path):
+    """Size and field offsets of every struct of the header against its ctypes twin, as the C compiler sees them."""
+    import importlib
+    import subprocess
+    lib = importlib.import_module("mineru-diffusion_b200._lib")
+    names = re.findall(r"\}\s*(mdb_\w+)\s*;", open(HEADER).read())
+    twins = {n: getattr(lib, "".join(p.capitalize() for p in n[len("mdb_"):].split("_"))) for n in names}
+    assert len(twins) >= 10
+    lines = [f'printf("{n} %zu\\n", sizeof({n}));' for n in twins]
+    lines += [f'printf("{n}.{f} %zu\\n", offsetof({n}, {f}));' for n, t in twins.items() for f, _ in t._fields_]
+    src = tmp_path / "sizes.c"
+    src.write_text('#include <stddef.h>\n#include <stdio.h>\n#include "mdb200.h"\nint main(void) {\n' + "\n".join(lines) + "\nreturn 0; }\n")
+    subprocess.run(["gcc", "-I", os.path.dirname(HEADER), "-o", str(tmp_path / "sizes"), str(src)], check=True)
+    out = dict(l.split() for l in subprocess.run([str(tmp_path / "sizes")], capture_output=True, text=True, check=True).stdout.splitlines())
+    for n, t in twins.items():
+        assert int(out[n]) == ctypes.sizeof(t), n
+        for f, _ in t._fields_:
+            assert int(out[f"{n}.{f}"]) == getattr(t, f).offset, f"{n}.{f}"
