@@ -407,10 +407,12 @@ typedef struct {
 } mdb_rms_segment;
 int mdb_rms_rows(int dtype, const mdb_rms_segment* segments, int nseg, int m, mdb_stream_t stream);
 
-/* y[row][h][c] = o / sqrt(mean over c of o^2 + eps) * weight[h * weight_head_stride + c] * sigmoid(gate) */
+/* y[row][h][c] = o' / sqrt(mean over c of o'^2 + eps) * weight[h * weight_head_stride + c] * sigmoid(gate), with
+ * o' = o / den[row][h] (den may be NULL: 1) */
 typedef struct {
   int32_t dtype, m, heads, vdim;
   const float* o;
+  const float* den;
   mdb_rows gate;
   const float* weight;
   void* y;
@@ -421,7 +423,7 @@ typedef struct {
 int mdb_gated_norm(const mdb_gated_norm_args* args, mdb_stream_t stream);
 
 /* Key channels of a recurrent head as the state stores them (a multiple of 32; 0: not supported), and the number of
- * copies of the mLSTM normaliser and maximum a head keeps. */
+ * copies of the mLSTM maximum a head keeps. */
 int mdb_scan_dim_pad(int dim);
 int mdb_scan_blocks(int vdim);
 /* 1 when the one-token form of mdb_scan takes this head shape */
@@ -454,9 +456,23 @@ typedef struct {
 } mdb_delta_prep_args;
 int mdb_delta_prep(const mdb_delta_prep_args* args, mdb_stream_t stream);
 
-/* g [m][heads][dim_pad] = exp(-exp(a_log[h]) * softplus(x + dt_bias)), x [m] rows of heads * dim columns */
-int mdb_channel_decay(const float* x, int64_t ldx, const float* a_log, const float* dt_bias, float* g, int m, int heads,
-                      int dim, int dim_pad, mdb_stream_t stream);
+/* g [m][heads][dim_pad] = exp(-exp(a_log[h]) * softplus(x + dt_bias)), x [m] rows of heads * dim columns; cross
+ * [m][heads][2], written for the odd tokens of every portion: ((g k_prev) . k, (g k_prev) . q) with the outputs of
+ * mdb_delta_prep. */
+typedef struct {
+  int32_t m, heads, kv_heads, dim, dim_pad;
+  const float* x;
+  int64_t ldx;
+  const float* a_log;
+  const float* dt_bias;
+  const float* q;
+  const float* k;
+  float* g;
+  float* cross;
+  const int32_t* row_seq;
+  const int32_t* cu_q;
+} mdb_decay_args;
+int mdb_channel_decay(const mdb_decay_args* args, mdb_stream_t stream);
 
 /* Inputs of the mLSTM scan: q times dim^-1/2, k, v as fp32 rows; log_i = cap tanh((i + bias_i) / cap), log_f =
  * logsigmoid(cap tanh((f + bias_f) / cap)). */
@@ -476,10 +492,10 @@ int mdb_mlstm_prep(const mdb_mlstm_prep_args* args, mdb_stream_t stream);
 
 /* The recurrences over every sequence's portion; state [slot][heads][vdim][dim_pad] fp32 is read and written.
  * DELTA: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; s0 = beta, s1 = k . q.  MLSTM: m' = max(f + m, i);
- * S, n <- exp(f + m - m') (.) + exp(i - m') k (v^T, 1); o = S^T q / (max(|n . q|, exp(-m')) + 1e-6); s0 = i, s1 = f;
- * nstate [slot][heads][mdb_scan_blocks][dim_pad], mstate [slot][heads][mdb_scan_blocks].
+ * S, n <- exp(f + m - m') (.) + exp(i - m') k (v^T, 1); o = S^T q, den [m][heads] = max(|n . q|, exp(-m')) + 1e-6;
+ * s0 = i, s1 = f; its state has one more column per head (vdim + 1), which is n; mstate [slot][heads][mdb_scan_blocks].
  * out [m][heads][vdim] fp32; with `fused` (every portion is one token) the decay comes from raw_decay + dt_bias and
- * a_log, and y = the gated norm of o (as mdb_gated_norm) is written instead. */
+ * a_log, and y = the gated norm of o / den (as mdb_gated_norm) is written instead. */
 enum { MDB_SCAN_DELTA = 0, MDB_SCAN_MLSTM = 1 };
 typedef struct {
   int32_t mode, dtype, fused, bs, heads, kv_heads, dim, dim_pad, vdim;
@@ -492,8 +508,9 @@ typedef struct {
   const float* s1;
   float* state;
   int64_t state_slot_stride, num_slots;
-  float* nstate;
   float* mstate;
+  const float* cross; /* DELTA: of mdb_channel_decay */
+  float* den;         /* MLSTM */
   const int32_t* cu_q;
   const int32_t* start;
   const int32_t* state_slot;

@@ -35,7 +35,7 @@ RmsSegment = _struct("RmsSegment", [
     ("src", Rows), ("weight", _p), ("out", _p), ("ld_out", _i64), ("slots", _p), ("num_slots", _i64), ("n", _i),
     ("n_pad", _i), ("eps", _f)])
 GatedNormArgs = _struct("GatedNormArgs", [
-    ("dtype", _i), ("m", _i), ("heads", _i), ("vdim", _i), ("o", _p), ("gate", Rows), ("weight", _p), ("y", _p),
+    ("dtype", _i), ("m", _i), ("heads", _i), ("vdim", _i), ("o", _p), ("den", _p), ("gate", Rows), ("weight", _p), ("y", _p),
     ("ldy", _i64), ("weight_head_stride", _i), ("eps", _f)])
 DeltaPrepArgs = _struct("DeltaPrepArgs", [(n, _i) for n in (
     "dtype", "m", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim", "taps", "channels", "shift_state", "copy_cols")] + [
@@ -43,13 +43,17 @@ DeltaPrepArgs = _struct("DeltaPrepArgs", [(n, _i) for n in (
     ("conv_k", _p), ("conv_v", _p), ("conv_state", _p), ("conv_slot_stride", _i64), ("num_slots", _i64), ("row_seq", _p),
     ("cu_q", _p), ("start", _p), ("state_slot", _p), ("q_out", _p), ("k_out", _p), ("v_out", _p), ("beta_out", _p),
     ("kq_out", _p)])
+DecayArgs = _struct("DecayArgs", [(n, _i) for n in ("m", "heads", "kv_heads", "dim", "dim_pad")] + [
+    ("x", _p), ("ldx", _i64), ("a_log", _p), ("dt_bias", _p), ("q", _p), ("k", _p), ("g", _p), ("cross", _p), ("row_seq", _p),
+    ("cu_q", _p)])
 MlstmPrepArgs = _struct("MlstmPrepArgs", [(n, _i) for n in ("dtype", "m", "heads", "dim", "dim_pad", "vdim")] + [
     ("q", Rows), ("k", Rows), ("v", Rows), ("i", Rows), ("f", Rows), ("bias_i", _p), ("bias_f", _p), ("q_out", _p),
     ("k_out", _p), ("v_out", _p), ("log_i", _p), ("log_f", _p), ("cap", _f)])
 ScanArgs = _struct("ScanArgs", [(n, _i) for n in (
     "mode", "dtype", "fused", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim")] + [
     ("eps", _f), ("q", _p), ("k", _p), ("v", _p), ("g", _p), ("s0", _p), ("s1", _p), ("state", _p),
-    ("state_slot_stride", _i64), ("num_slots", _i64), ("nstate", _p), ("mstate", _p), ("cu_q", _p), ("start", _p),
+    ("state_slot_stride", _i64), ("num_slots", _i64), ("mstate", _p), ("cross", _p),
+    ("den", _p), ("cu_q", _p), ("start", _p),
     ("state_slot", _p), ("out", _p), ("raw_decay", Rows), ("a_log", _p), ("dt_bias", _p), ("gate", Rows), ("norm", _p),
     ("norm_head_stride", _i64), ("y", _p), ("ldy", _i64)])
 MoeRouteArgs = _struct("MoeRouteArgs", [(n, _i) for n in ("m", "experts", "top", "groups", "keep")] + [
@@ -110,7 +114,7 @@ SIGNATURES = {
     "mdb_scan_blocks": (_i, [_i]),
     "mdb_scan_fusable": (_i, [_i, _i]),
     "mdb_delta_prep": (_i, [C.POINTER(DeltaPrepArgs), _p]),
-    "mdb_channel_decay": (_i, [_p, _i64, _p, _p, _p, _i, _i, _i, _i, _p]),
+    "mdb_channel_decay": (_i, [C.POINTER(DecayArgs), _p]),
     "mdb_mlstm_prep": (_i, [C.POINTER(MlstmPrepArgs), _p]),
     "mdb_scan": (_i, [C.POINTER(ScanArgs), _p]),
     "mdb_moe_route": (_i, [C.POINTER(MoeRouteArgs), _p]),

@@ -5,11 +5,18 @@
 // State layout: [slot][head][value column][key channel padded to a multiple of 32], so a value column is contiguous.
 // The columns of a head are independent of one another (the delta rule's correction of a column only needs that
 // column), so a CTA owns a block of columns: eight lanes share a column, each holding every eighth float4 of it in
-// registers, CPT columns per thread; a token needs one three-step shuffle reduction over the eight lanes.  k, q and
-// the decays of a block of tokens come through a double-buffered shared-memory stage (cp.async).
+// registers, CPT columns per thread.  k, q and the decays of a block of tokens come through a double-buffered
+// shared-memory stage (cp.async).
 //
-// The read-out of the delta rule is rewritten so that both products with the old state share one reduction:
-//   a = (g S)^T k,  b = (g S)^T q,  u = beta (v - a),  o = b + (k . q) u,  S <- g S + k u^T.
+// The read-out of the delta rule is rewritten so that both products with the old state share one reduction,
+//   a = (g S)^T k,  b = (g S)^T q,  u = beta (v - a),  o = b + (k . q) u,  S <- g S + k u^T,
+// and prompts take two tokens per reduction: with S' = g2 g1 S the second token's products are
+//   a2 = S'^T k2 + ((g2 k1) . k2) u1,  b2 = S'^T q2 + ((g2 k1) . q2) u1,  S <- S' + (g2 k1) u1^T + k2 u2^T,
+// the same number of FMAs per token with half the dependent shuffle reductions; the two cross products per token are
+// computed beforehand, with the decays.
+//
+// mLSTM: the normaliser n is one more column of the state (its value is 1 for every token); the division by
+// max(|n . q|, exp(-m)) + 1e-6 happens where the read-out is normalised.
 #include "mdb_common.cuh"
 
 namespace mdb {
@@ -160,6 +167,136 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const mdb_d
   }
 }
 
+// The same work for heads of at most 128 channels and up to four taps, sizes in multiples of four: a lane owns four
+// channels and walks `run` consecutive rows with the last inputs in registers, so every input is read once.
+template <typename T, bool PARTS>
+struct ConvWindow {
+  float4 x[3];         // inputs 3, 2 and 1 tokens ago
+  float4 w[4];         // taps of the four channels: w[j] belongs to the input 3 - j tokens ago
+  __device__ __forceinline__ void load_taps(const float* weights, int col, int taps) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int t = j - (4 - taps);
+      float e[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) e[c] = t >= 0 ? weights[static_cast<int64_t>(col + c) * taps + t] : 0.f;
+      w[j] = make_float4(e[0], e[1], e[2], e[3]);
+    }
+  }
+  __device__ __forceinline__ void refill(const mdb_delta_prep_args& a, const mdb_rows& src, int64_t row, int tloc, int slot, int col,
+                                         int channel) {
+#pragma unroll
+    for (int back = 1; back <= 3; ++back) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (back < a.taps) {
+        if (back <= tloc) v = rows_at4_of<T, PARTS>(src, row - back, col);
+        else if (slot >= 0)
+          v = act_load4(static_cast<const T*>(a.conv_state) + slot * a.conv_slot_stride +
+                        static_cast<int64_t>(a.taps - 1 - (back - tloc)) * a.channels + channel);
+      }
+      x[3 - back] = v;
+    }
+  }
+  __device__ __forceinline__ float4 step(float4 now) {
+    float4 y;
+    y.x = fmaf(w[3].x, now.x, fmaf(w[2].x, x[2].x, fmaf(w[1].x, x[1].x, w[0].x * x[0].x)));
+    y.y = fmaf(w[3].y, now.y, fmaf(w[2].y, x[2].y, fmaf(w[1].y, x[1].y, w[0].y * x[0].y)));
+    y.z = fmaf(w[3].z, now.z, fmaf(w[2].z, x[2].z, fmaf(w[1].z, x[1].z, w[0].z * x[0].z)));
+    y.w = fmaf(w[3].w, now.w, fmaf(w[2].w, x[2].w, fmaf(w[1].w, x[1].w, w[0].w * x[0].w)));
+    x[0] = x[1]; x[1] = x[2]; x[2] = now;
+    y.x = y.x / (1.0f + expf(-y.x)); y.y = y.y / (1.0f + expf(-y.y));
+    y.z = y.z / (1.0f + expf(-y.z)); y.w = y.w / (1.0f + expf(-y.w));
+    return y;
+  }
+  // one-token portions: the last taps - 1 inputs back into the slot
+  __device__ __forceinline__ void save(const mdb_delta_prep_args& a, int slot, int channel) const {
+    T* st = static_cast<T*>(a.conv_state) + slot * a.conv_slot_stride + channel;
+    for (int j = 0; j < a.taps - 1; ++j) {
+      const int i = 3 - (a.taps - 1) + j;          // oldest first
+      act_store4(st + static_cast<int64_t>(j) * a.channels, i == 0 ? x[0] : (i == 1 ? x[1] : x[2]));
+    }
+  }
+};
+__device__ __forceinline__ float dot4(float4 a, float4 b) { return a.x * b.x + a.y * b.y + a.z * b.z + a.w * b.w; }
+__device__ __forceinline__ float4 scale4(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
+
+template <typename T, bool PARTS>
+__global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_rows_kernel(const mdb_delta_prep_args a, const int run) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, c = lane * 4;
+  const int unit = blockIdx.y * kPrepWarps + (threadIdx.x >> 5);
+  const int64_t row0 = static_cast<int64_t>(blockIdx.x) * run, row1 = min(row0 + run, static_cast<int64_t>(a.m));
+  const int vblocks = (a.vdim + 127) / 128;        // a head's values in blocks of 128
+  const bool is_qk = unit < a.kv_heads, is_v = !is_qk && unit < a.kv_heads + a.heads * vblocks;
+  const int kc = a.kv_heads * a.dim;
+  if (is_qk || is_v) {
+    const int vu = unit - a.kv_heads, head = vu / vblocks, vc = (vu % vblocks) * 128 + c;
+    const bool live = is_qk ? c < a.dim : vc < a.vdim;
+    const int col = is_qk ? unit * a.dim + c : head * a.vdim + vc;
+    const mdb_rows& src = is_qk ? a.q : a.v;
+    const int channel = is_qk ? col : 2 * kc + col;
+    ConvWindow<T, PARTS> w0, w1;
+    if (live) {
+      w0.load_taps(is_qk ? a.conv_q : a.conv_v, col, a.taps);
+      if (is_qk) w1.load_taps(a.conv_k, col, a.taps);
+    }
+    int seq = -1, slot = -1;
+    for (int64_t row = row0; row < row1; ++row) {
+      const int s = a.row_seq[row];
+      if (s != seq) {
+        seq = s;
+        slot = a.state_slot[s];
+        if (slot >= a.num_slots) {
+          if (lane == 0) report_status(MDB_STATUS_BAD_SLOT);
+          slot = -1;
+        }
+        if (slot >= 0 && live) {
+          const int from = a.start[s] == 0 ? -1 : slot, tloc = static_cast<int>(row) - a.cu_q[s];
+          w0.refill(a, src, row, tloc, from, col, channel);
+          if (is_qk) w1.refill(a, a.k, row, tloc, from, col, kc + col);
+        }
+      }
+      if (slot < 0) continue;
+      const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+      float4 y0 = zero, y1 = zero;
+      if (live) {
+        y0 = w0.step(rows_at4_of<T, PARTS>(src, row, col));
+        if (is_qk) y1 = w1.step(rows_at4_of<T, PARTS>(a.k, row, col));
+        if (a.shift_state && a.taps > 1) {
+          w0.save(a, slot, channel);
+          if (is_qk) w1.save(a, slot, kc + col);
+        }
+      }
+      if (is_qk) {
+        const float rq = (1.0f / sqrtf(warp_sum(dot4(y0, y0)) + 1e-6f)) * (1.0f / sqrtf(static_cast<float>(a.dim)));
+        const float rk = 1.0f / sqrtf(warp_sum(dot4(y1, y1)) + 1e-6f);
+        y0 = scale4(y0, rq);
+        y1 = scale4(y1, rk);
+        const float kq = warp_sum(dot4(y0, y1));
+        const int64_t at = (row * a.kv_heads + unit) * a.dim_pad + c;
+        if (c < a.dim_pad) {
+          *reinterpret_cast<float4*>(a.q_out + at) = y0;
+          *reinterpret_cast<float4*>(a.k_out + at) = y1;
+        }
+        if (lane == 0) a.kq_out[row * a.kv_heads + unit] = kq;
+      } else if (live) {
+        *reinterpret_cast<float4*>(a.v_out + (row * a.heads + head) * a.vdim + vc) = y0;
+      }
+    }
+    return;
+  }
+  const int rest = unit - a.kv_heads - a.heads * vblocks;
+  for (int64_t row = row0; row < row1; ++row) {
+    if (rest == 0) {
+      for (int h = lane; h < a.heads; h += 32) a.beta_out[row * a.heads + h] = sigmoid_f(rows_at<T>(a.b, row, h));
+    } else {
+      const int cc = (rest - 1) * 128 + c;
+      if (cc < a.copy_cols) act_store4(static_cast<T*>(a.copy_out) + row * a.copy_ld + cc, rows_at4_of<T, PARTS>(a.copy, row, cc));
+    }
+  }
+}
+
 // The last taps - 1 inputs of every channel after a step of arbitrary portions: one thread per (sequence, channel).
 template <typename T>
 __global__ void __launch_bounds__(256) conv_state_kernel(const mdb_delta_prep_args a) {
@@ -183,44 +320,96 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const mdb_delta_prep_ar
   for (int j = 0; j < a.taps - 1; ++j) st[static_cast<int64_t>(j) * a.channels] = act_from_f<T>(keep[j]);
 }
 
-// g = exp(-exp(A_log) * softplus(x + dt_bias)), laid out [row][head][dim_pad] (padding channels: 1)
-__global__ void __launch_bounds__(256) channel_decay_kernel(const float* x, int64_t ldx,
-                                                            const float* a_log, const float* dt_bias,
-                                                            float* g, int64_t total, int heads, int dim, int dim_pad) {
+// One warp per (row, head).  g = exp(-exp(A_log) * softplus(x + dt_bias)), laid out [row][head][dim_pad] (padding
+// channels: 1), and, for the odd tokens of a portion, the cross products with the token before:
+// cross [row][head] = ((g k_prev) . k, (g k_prev) . q).  VEC: head rows of x start on 16-byte boundaries.
+template <bool VEC>
+__global__ void __launch_bounds__(128) channel_decay_kernel(const mdb_decay_args a) {
   pdl_launch_dependents();
   pdl_wait();
-  for (int64_t i = blockIdx.x * static_cast<int64_t>(256) + threadIdx.x; i < total; i += static_cast<int64_t>(gridDim.x) * 256) {
-    const int d = static_cast<int>(i % dim_pad);
-    const int64_t rh = i / dim_pad;
-    const int h = static_cast<int>(rh % heads);
-    float r = 1.f;
-    if (d < dim) r = expf(-expf(a_log[h]) * softplus_f(x[(rh / heads) * ldx + h * dim + d] + dt_bias[h * dim + d]));
-    g[i] = r;
+  const int lane = threadIdx.x & 31;
+  const int head = blockIdx.y * 4 + (threadIdx.x >> 5);
+  const int64_t row = blockIdx.x;
+  if (head >= a.heads) return;
+  const bool odd = ((static_cast<int>(row) - a.cu_q[a.row_seq[row]]) & 1) != 0;
+  const float* x = a.x + row * a.ldx + static_cast<int64_t>(head) * a.dim;
+  const float* bias = a.dt_bias + static_cast<int64_t>(head) * a.dim;
+  float* g = a.g + (row * a.heads + head) * a.dim_pad;
+  const int kvh = head / (a.heads / a.kv_heads);
+  const float* k = a.k + (row * a.kv_heads + kvh) * a.dim_pad;
+  const float* q = a.q + (row * a.kv_heads + kvh) * a.dim_pad;
+  const float* kp = k - static_cast<int64_t>(a.kv_heads) * a.dim_pad;      // read for odd tokens only
+  const float rate = -expf(a.a_log[head]);
+  float ck = 0.f, cq = 0.f;
+  for (int c = lane * 4; c < a.dim_pad; c += 128) {
+    float xv[4], bv[4], r[4];
+    if (VEC && c + 4 <= a.dim) {
+      const float4 x4 = *reinterpret_cast<const float4*>(x + c), b4 = *reinterpret_cast<const float4*>(bias + c);
+      xv[0] = x4.x; xv[1] = x4.y; xv[2] = x4.z; xv[3] = x4.w;
+      bv[0] = b4.x; bv[1] = b4.y; bv[2] = b4.z; bv[3] = b4.w;
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        xv[i] = c + i < a.dim ? x[c + i] : 0.f;
+        bv[i] = c + i < a.dim ? bias[c + i] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) r[i] = c + i < a.dim ? expf(rate * softplus_f(xv[i] + bv[i])) : 1.f;
+    *reinterpret_cast<float4*>(g + c) = make_float4(r[0], r[1], r[2], r[3]);
+    if (odd) {
+      const float4 k0 = *reinterpret_cast<const float4*>(kp + c), k1 = *reinterpret_cast<const float4*>(k + c);
+      const float4 q1 = *reinterpret_cast<const float4*>(q + c);
+      const float e0 = r[0] * k0.x, e1 = r[1] * k0.y, e2 = r[2] * k0.z, e3 = r[3] * k0.w;
+      ck += e0 * k1.x + e1 * k1.y + e2 * k1.z + e3 * k1.w;
+      cq += e0 * q1.x + e1 * q1.y + e2 * q1.z + e3 * q1.w;
+    }
+  }
+  if (odd) {
+    ck = warp_sum(ck);
+    cq = warp_sum(cq);
+    if (lane == 0) *reinterpret_cast<float2*>(a.cross + 2 * (row * a.heads + head)) = make_float2(ck, cq);
   }
 }
 
-// Before the mLSTM scan: q scaled, k, v as fp32 rows (key channels padded with zeros), and the two log gates.
-template <typename T>
-__global__ void __launch_bounds__(128) mlstm_prep_kernel(const mdb_mlstm_prep_args a) {
+// Before the mLSTM scan: q scaled, k, v as fp32 rows (key channels padded with zeros), and the two log gates.  Work
+// items of four channels; VEC: head rows of the projections start on 16-byte boundaries.
+template <typename T, bool VEC, bool PARTS>
+__global__ void __launch_bounds__(256) mlstm_prep_kernel(const mdb_mlstm_prep_args a) {
   pdl_launch_dependents();
   pdl_wait();
   const int64_t row = blockIdx.x;
   const int nq = a.heads * a.dim_pad, nv = a.heads * a.vdim;
+  const int iq = nq / 4, iv = (nv + 3) / 4;
   const float scale = 1.0f / sqrtf(static_cast<float>(a.dim));
-  for (int i = blockIdx.y * 128 + threadIdx.x; i < nq + nv + a.heads; i += gridDim.y * 128) {
-    if (i < nq) {
-      const int h = i / a.dim_pad, d = i % a.dim_pad;
-      float q = 0.f, k = 0.f;
-      if (d < a.dim) {
-        q = rows_at<T>(a.q, row, h * a.dim + d) * scale;
-        k = rows_at<T>(a.k, row, h * a.dim + d);
+  for (int i = blockIdx.y * 256 + threadIdx.x; i < iq + iv + a.heads; i += gridDim.y * 256) {
+    if (i < iq) {
+      const int h = i * 4 / a.dim_pad, d = i * 4 % a.dim_pad;
+      float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q;
+      if (VEC) {
+        if (d < a.dim) {
+          q = rows_at4_of<T, PARTS>(a.q, row, h * a.dim + d);
+          k = rows_at4_of<T, PARTS>(a.k, row, h * a.dim + d);
+        }
+      } else {
+        float* qe = &q.x;
+        float* ke = &k.x;
+        for (int e = 0; e < 4 && d + e < a.dim; ++e) {
+          qe[e] = rows_at<T>(a.q, row, h * a.dim + d + e);
+          ke[e] = rows_at<T>(a.k, row, h * a.dim + d + e);
+        }
       }
-      a.q_out[row * nq + i] = q;
-      a.k_out[row * nq + i] = k;
-    } else if (i < nq + nv) {
-      a.v_out[row * nv + (i - nq)] = rows_at<T>(a.v, row, i - nq);
+      *reinterpret_cast<float4*>(a.q_out + row * nq + i * 4) = make_float4(q.x * scale, q.y * scale, q.z * scale, q.w * scale);
+      *reinterpret_cast<float4*>(a.k_out + row * nq + i * 4) = k;
+    } else if (i < iq + iv) {
+      const int c = (i - iq) * 4;
+      if (VEC) {
+        *reinterpret_cast<float4*>(a.v_out + row * nv + c) = rows_at4_of<T, PARTS>(a.v, row, c);
+      } else {
+        for (int e = c; e < c + 4 && e < nv; ++e) a.v_out[row * nv + e] = rows_at<T>(a.v, row, e);
+      }
     } else {
-      const int h = i - nq - nv;
+      const int h = i - iq - iv;
       const float zi = rows_at<T>(a.i, row, h) + a.bias_i[h], zf = rows_at<T>(a.f, row, h) + a.bias_f[h];
       a.log_i[row * a.heads + h] = a.cap * tanhf(zi / a.cap);
       a.log_f[row * a.heads + h] = -softplus_f(-(a.cap * tanhf(zf / a.cap)));
@@ -233,26 +422,58 @@ __global__ void __launch_bounds__(128) mlstm_prep_kernel(const mdb_mlstm_prep_ar
 // ---------------------------------------------------------------------------
 enum { kScanDelta = MDB_SCAN_DELTA, kScanMlstm = MDB_SCAN_MLSTM };
 constexpr int kScanFusedThreads = 512, kScanFusedMaxDim = 256;
-constexpr int kScanBlockCols = 32;       // granularity of the copies of the mLSTM normaliser
+constexpr int kScanBlockCols = 32;       // columns of a CTA of the prompt form; granularity of the copies of the mLSTM maximum
+constexpr int kScanTokens = 16;          // tokens of a stage of the prompt form (even)
 
-// floats of one stage: k, q (and the decays) of tb tokens, their values for `cols` columns, two scalars per token
+// floats of one stage: k, q (and the decays) of tb tokens, their values for `cols` columns, four scalars per token
 __host__ __device__ constexpr int scan_stage_floats(int mode, int dp, int tb, int cols) {
   return tb * ((mode == kScanDelta ? 3 : 2) * dp + cols + 4);
 }
 
-// FUSED: every sequence brings one token and the CTA owns all columns of the head; the decay is computed from the raw
-// projection and the head's output is normalised, gated and stored as the next projection's input.
-template <typename T, int MODE, int NCH, int CPT, int TB, bool FUSED>
-__global__ void __launch_bounds__(FUSED ? kScanFusedThreads : 256) scan_kernel(const mdb_scan_args a, const int cols) {
-  constexpr int DP = NCH * 32;
+template <int NCH, int CPT>
+struct ScanState {
+  f32x2 v[CPT][NCH * 2];
+  // column col0 + i of a head's state (columns from `columns` on: zeros)
+  __device__ __forceinline__ void load(const float* state, int col0, int columns, int l8, bool fresh) {
+#pragma unroll
+    for (int i = 0; i < CPT; ++i)
+#pragma unroll
+      for (int c = 0; c < NCH; ++c) {
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (!fresh && col0 + i < columns)
+          x = *reinterpret_cast<const float4*>(state + static_cast<int64_t>(col0 + i) * (NCH * 32) + c * 32 + l8 * 4);
+        v[i][2 * c] = pack2(x.x, x.y);
+        v[i][2 * c + 1] = pack2(x.z, x.w);
+      }
+  }
+  __device__ __forceinline__ void store(float* state, int col0, int columns, int l8) const {
+#pragma unroll
+    for (int i = 0; i < CPT; ++i)
+      if (col0 + i < columns) {
+#pragma unroll
+        for (int c = 0; c < NCH; ++c) {
+          const float2 lo = unpack2(v[i][2 * c]), hi = unpack2(v[i][2 * c + 1]);
+          *reinterpret_cast<float4*>(state + static_cast<int64_t>(col0 + i) * (NCH * 32) + c * 32 + l8 * 4) =
+              make_float4(lo.x, lo.y, hi.x, hi.y);
+        }
+      }
+  }
+};
+
+// Prompt form: portions of any length, kScanBlockCols columns of one head per CTA, two tokens at a time.
+template <int MODE, int NCH, int CPT>
+__global__ void __launch_bounds__(kScanBlockCols / CPT * 8) scan_kernel(const mdb_scan_args a) {
+  constexpr int DP = NCH * 32, TB = kScanTokens, COLS = kScanBlockCols, THREADS = COLS / CPT * 8;
+  constexpr int VEC = MODE == kScanDelta ? 3 : 2;
+  constexpr int OFF_V = TB * VEC * DP, OFF_S = OFF_V + TB * COLS, STAGE = scan_stage_floats(MODE, DP, TB, COLS);
+  constexpr bool KEEP_K = NCH <= 8;      // the keys of a pair stay in registers between the two passes
   extern __shared__ __align__(16) float scan_smem[];
-  __shared__ float sh_gate[3 * TB];      // mLSTM: forget factor, input factor, exp(-m) per token of the block
-  __shared__ float red[32];
+  __shared__ float4 sh_gate[TB];         // mLSTM: forget factor, input factor, exp(-m) per token of the stage
   pdl_launch_dependents();
   pdl_wait();
   const int seq = blockIdx.z, head = blockIdx.y;
   const int l8 = threadIdx.x & 7, cg = threadIdx.x >> 3;
-  const int col0 = blockIdx.x * cols, mycol = col0 + cg * CPT;
+  const int col0 = blockIdx.x * COLS, mycol = col0 + cg * CPT;
   const int slot = a.state_slot[seq];
   if (slot < 0) return;
   if (slot >= a.num_slots) {
@@ -263,81 +484,64 @@ __global__ void __launch_bounds__(FUSED ? kScanFusedThreads : 256) scan_kernel(c
   if (t_end <= t_begin) return;
   const bool fresh = a.start[seq] == 0;
   const int kvh = head / (a.heads / a.kv_heads);
-  float* state = a.state + slot * a.state_slot_stride + static_cast<int64_t>(head) * a.vdim * DP;
-
-  f32x2 S[CPT][NCH * 2];
-#pragma unroll
-  for (int i = 0; i < CPT; ++i)
-#pragma unroll
-    for (int c = 0; c < NCH; ++c) {
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!fresh && mycol + i < a.vdim)
-        v = *reinterpret_cast<const float4*>(state + static_cast<int64_t>(mycol + i) * DP + c * 32 + l8 * 4);
-      S[i][2 * c] = pack2(v.x, v.y);
-      S[i][2 * c + 1] = pack2(v.z, v.w);
-    }
-  // mLSTM: the normaliser n and the running maximum m.  Each block of 32 columns keeps a copy of both, so that CTAs of
-  // one head never read what another writes.
-  f32x2 N[MODE == kScanMlstm ? NCH * 2 : 1];
+  const int columns = a.vdim + (MODE == kScanMlstm ? 1 : 0);
+  float* state = a.state + slot * a.state_slot_stride + static_cast<int64_t>(head) * columns * DP;
+  ScanState<NCH, CPT> S;
+  S.load(state, mycol, columns, l8, fresh);
+  // mLSTM: every block of 32 columns keeps a copy of the running maximum, so that no CTA reads what another writes
   float run_max = 0.f;
-  const int blocks = (a.vdim + kScanBlockCols - 1) / kScanBlockCols;
-  float* nstate = nullptr;
   float* mstate = nullptr;
   if (MODE == kScanMlstm) {
-    const int64_t hb = (static_cast<int64_t>(slot) * a.heads + head) * blocks;
-    nstate = a.nstate + hb * DP;
-    mstate = a.mstate + hb;
-    const int b0 = col0 / kScanBlockCols;
-#pragma unroll
-    for (int c = 0; c < NCH; ++c) {
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!fresh) v = *reinterpret_cast<const float4*>(nstate + static_cast<int64_t>(b0) * DP + c * 32 + l8 * 4);
-      N[2 * c] = pack2(v.x, v.y);
-      N[2 * c + 1] = pack2(v.z, v.w);
-    }
-    if (!fresh) run_max = mstate[b0];
+    mstate = a.mstate + (static_cast<int64_t>(slot) * a.heads + head) * ((columns + kScanBlockCols - 1) / kScanBlockCols) + blockIdx.x;
+    if (!fresh) run_max = *mstate;
   }
 
   const uint32_t smem0 = smem_u32(scan_smem);
-  const int stage_floats = scan_stage_floats(MODE, DP, TB, cols);
-  constexpr int kVec = MODE == kScanDelta ? 3 : 2;
-  const int off_v = TB * kVec * DP, off_s = off_v + TB * cols;
   auto stage = [&](int t0, int buf) {
     const int n = min(TB, t_end - t0);
-    const uint32_t base = smem0 + buf * stage_floats * 4;
-    for (int i = threadIdx.x; i < n * (DP / 4); i += blockDim.x) {
+    const uint32_t base = smem0 + buf * STAGE * 4;
+    float* st = scan_smem + buf * STAGE;
+    for (int i = threadIdx.x; i < n * (DP / 4); i += THREADS) {
       const int t = i / (DP / 4), c = i % (DP / 4);
       const int64_t krow = (static_cast<int64_t>(t0 + t) * a.kv_heads + kvh) * DP + c * 4;
       cp_async16(base + (t * DP + c * 4) * 4, a.k + krow);
       cp_async16(base + ((TB + t) * DP + c * 4) * 4, a.q + krow);
-      if (MODE == kScanDelta && !FUSED)
+      if (MODE == kScanDelta)
         cp_async16(base + ((2 * TB + t) * DP + c * 4) * 4, a.g + (static_cast<int64_t>(t0 + t) * a.heads + head) * DP + c * 4);
     }
-    if (MODE == kScanDelta && FUSED) {
-      for (int i = threadIdx.x; i < n * DP; i += blockDim.x) {
-        const int t = i / DP, d = i % DP;
-        float r = 1.f;
-        if (d < a.dim)
-          r = expf(-expf(a.a_log[head]) * softplus_f(rows_at<float>(a.raw_decay, t0 + t, head * a.dim + d) + a.dt_bias[head * a.dim + d]));
-        scan_smem[buf * stage_floats + (2 * TB + t) * DP + d] = r;
+    for (int i = threadIdx.x; i < n * COLS; i += THREADS) {
+      const int t = i / COLS, c = i % COLS;
+      if (col0 + c < a.vdim)
+        cp_async4(base + (OFF_V + t * COLS + c) * 4, a.v + (static_cast<int64_t>(t0 + t) * a.heads + head) * a.vdim + col0 + c);
+      else
+        st[OFF_V + t * COLS + c] = MODE == kScanMlstm && col0 + c == a.vdim ? 1.f : 0.f;
+    }
+    for (int i = threadIdx.x; i < n; i += THREADS) {
+      const int64_t th = static_cast<int64_t>(t0 + i) * a.heads + head;
+      const uint32_t dst = base + (OFF_S + 4 * i) * 4;
+      cp_async4(dst, a.s0 + th);
+      if (MODE == kScanDelta) {
+        cp_async4(dst + 4, a.s1 + static_cast<int64_t>(t0 + i) * a.kv_heads + kvh);
+        if (i & 1) {
+          cp_async4(dst + 8, a.cross + 2 * th);
+          cp_async4(dst + 12, a.cross + 2 * th + 1);
+        }
+      } else {
+        cp_async4(dst + 4, a.s1 + th);
       }
     }
-    for (int i = threadIdx.x; i < n * cols; i += blockDim.x) {
-      const int t = i / cols, c = i % cols;
-      if (col0 + c < a.vdim)
-        cp_async4(base + (off_v + t * cols + c) * 4, a.v + (static_cast<int64_t>(t0 + t) * a.heads + head) * a.vdim + col0 + c);
-      else
-        scan_smem[buf * stage_floats + off_v + t * cols + c] = 0.f;
-    }
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-      const int64_t t = t0 + i;
-      cp_async4(base + (off_s + 2 * i) * 4, a.s0 + t * a.heads + head);
-      cp_async4(base + (off_s + 2 * i + 1) * 4, MODE == kScanDelta ? a.s1 + t * a.kv_heads + kvh : a.s1 + t * a.heads + head);
+    if (n & 1) {
+      // the missing second token of the last pair changes nothing: no key, no query, no decay
+      for (int i = threadIdx.x; i < DP; i += THREADS) {
+        st[n * DP + i] = st[(TB + n) * DP + i] = 0.f;
+        if (MODE == kScanDelta) st[(2 * TB + n) * DP + i] = 1.f;
+      }
+      for (int i = threadIdx.x; i < COLS; i += THREADS) st[OFF_V + n * COLS + i] = 0.f;
+      if (threadIdx.x < 4) st[OFF_S + 4 * n + threadIdx.x] = 0.f;
     }
     cp_async_commit();
   };
 
-  float out[CPT];
   stage(t_begin, 0);
   int buf = 0;
   for (int t0 = t_begin; t0 < t_end; t0 += TB, buf ^= 1) {
@@ -349,13 +553,13 @@ __global__ void __launch_bounds__(FUSED ? kScanFusedThreads : 256) scan_kernel(c
       cp_async_wait<0>();
     }
     __syncthreads();
-    const float* st = scan_smem + buf * stage_floats;
-    const uint32_t st_addr = smem0 + buf * stage_floats * 4;
+    const float* st = scan_smem + buf * STAGE;
+    const uint32_t st_addr = smem0 + buf * STAGE * 4;
     if (MODE == kScanMlstm) {
-      // m_t = max(f_t + m_(t-1), i_t) over the block as a scan of the maps x -> max(x + F, I)
+      // m_t = max(f_t + m_(t-1), i_t) over the stage as a scan of the maps x -> max(x + F, I)
       if (threadIdx.x < 32) {
         const int l = threadIdx.x;
-        const float li = l < n ? st[off_s + 2 * l] : -INFINITY, lf = l < n ? st[off_s + 2 * l + 1] : 0.f;
+        const float li = l < n ? st[OFF_S + 4 * l] : -INFINITY, lf = l < n ? st[OFF_S + 4 * l + 1] : 0.f;
         float F = lf, I = li;
 #pragma unroll
         for (int o = 1; o < TB; o <<= 1) {
@@ -365,141 +569,294 @@ __global__ void __launch_bounds__(FUSED ? kScanFusedThreads : 256) scan_kernel(c
         const float m = fmaxf(F + run_max, I);
         float mp = __shfl_up_sync(0xffffffffu, m, 1);
         if (l == 0) mp = run_max;
-        if (l < n) {
-          sh_gate[l] = expf(lf + mp - m);
-          sh_gate[TB + l] = expf(li - m);
-          sh_gate[2 * TB + l] = expf(-m);
-        }
+        if (l < n) sh_gate[l] = make_float4(expf(lf + mp - m), expf(li - m), expf(-m), 0.f);
+        else if (l < TB) sh_gate[l] = make_float4(1.f, 0.f, 0.f, 0.f);
         run_max = __shfl_sync(0xffffffffu, m, n - 1);
       }
       __syncthreads();
     }
-    for (int t = 0; t < n; ++t) {
+    for (int t = 0; t < n; t += 2) {
       const uint32_t ka = st_addr + (t * DP + l8 * 4) * 4, qa = ka + TB * DP * 4;
+      float o1[CPT], o2[CPT];
       if (MODE == kScanDelta) {
         const uint32_t ga = ka + 2 * TB * DP * 4;
-        f32x2 K[NCH * 2], A[CPT], B[CPT];
+        f32x2 K1[KEEP_K ? NCH * 2 : 1], K2[KEEP_K ? NCH * 2 : 1];
+        f32x2 A1[CPT], B1[CPT], A2[CPT], B2[CPT];
 #pragma unroll
-        for (int i = 0; i < CPT; ++i) A[i] = B[i] = 0ull;
+        for (int i = 0; i < CPT; ++i) A1[i] = B1[i] = A2[i] = B2[i] = 0ull;
 #pragma unroll
         for (int c = 0; c < NCH; ++c) {
-          f32x2 q0, q1, g0, g1;
-          lds2(ka + c * 128, K[2 * c], K[2 * c + 1]);
-          lds2(qa + c * 128, q0, q1);
-          lds2(ga + c * 128, g0, g1);
+          f32x2 k1[2], q1[2], g1[2], k2[2], q2[2], g2[2];
+          lds2(ka + c * 128, k1[0], k1[1]);
+          lds2(qa + c * 128, q1[0], q1[1]);
+          lds2(ga + c * 128, g1[0], g1[1]);
+          lds2(ka + DP * 4 + c * 128, k2[0], k2[1]);
+          lds2(qa + DP * 4 + c * 128, q2[0], q2[1]);
+          lds2(ga + DP * 4 + c * 128, g2[0], g2[1]);
 #pragma unroll
-          for (int i = 0; i < CPT; ++i) {
-            S[i][2 * c] = mul2(S[i][2 * c], g0);
-            S[i][2 * c + 1] = mul2(S[i][2 * c + 1], g1);
-            A[i] = fma2(S[i][2 * c], K[2 * c], A[i]);
-            B[i] = fma2(S[i][2 * c], q0, B[i]);
-            A[i] = fma2(S[i][2 * c + 1], K[2 * c + 1], A[i]);
-            B[i] = fma2(S[i][2 * c + 1], q1, B[i]);
+          for (int e = 0; e < 2; ++e) {
+            if (KEEP_K) {
+              K1[KEEP_K ? 2 * c + e : 0] = mul2(g2[e], k1[e]);
+              K2[KEEP_K ? 2 * c + e : 0] = k2[e];
+            }
+#pragma unroll
+            for (int i = 0; i < CPT; ++i) {
+              f32x2 s = mul2(S.v[i][2 * c + e], g1[e]);
+              A1[i] = fma2(s, k1[e], A1[i]);
+              B1[i] = fma2(s, q1[e], B1[i]);
+              s = mul2(s, g2[e]);
+              A2[i] = fma2(s, k2[e], A2[i]);
+              B2[i] = fma2(s, q2[e], B2[i]);
+              S.v[i][2 * c + e] = s;
+            }
           }
         }
-        const float beta = st[off_s + 2 * t], kq = st[off_s + 2 * t + 1];
-        float ra[CPT], rb[CPT];
+        float r[4 * CPT];
 #pragma unroll
         for (int i = 0; i < CPT; ++i) {
-          const float2 x = unpack2(A[i]), y = unpack2(B[i]);
-          ra[i] = x.x + x.y;
-          rb[i] = y.x + y.y;
+          const float2 w = unpack2(A1[i]), x = unpack2(B1[i]), y = unpack2(A2[i]), z = unpack2(B2[i]);
+          r[4 * i] = w.x + w.y; r[4 * i + 1] = x.x + x.y; r[4 * i + 2] = y.x + y.y; r[4 * i + 3] = z.x + z.y;
         }
 #pragma unroll
         for (int o = 4; o > 0; o >>= 1)
 #pragma unroll
-          for (int i = 0; i < CPT; ++i) {
-            ra[i] += __shfl_xor_sync(0xffffffffu, ra[i], o);
-            rb[i] += __shfl_xor_sync(0xffffffffu, rb[i], o);
-          }
+          for (int i = 0; i < 4 * CPT; ++i) r[i] += __shfl_xor_sync(0xffffffffu, r[i], o);
+        const float4 s1 = *reinterpret_cast<const float4*>(st + OFF_S + 4 * t), s2 = *reinterpret_cast<const float4*>(st + OFF_S + 4 * t + 4);
 #pragma unroll
         for (int i = 0; i < CPT; ++i) {
-          const float u = beta * (st[off_v + t * cols + cg * CPT + i] - ra[i]);
-          out[i] = fmaf(kq, u, rb[i]);
-          const f32x2 u2 = pack2(u, u);
+          const float v1 = st[OFF_V + t * COLS + cg * CPT + i], v2 = st[OFF_V + (t + 1) * COLS + cg * CPT + i];
+          const float u1 = s1.x * (v1 - r[4 * i]);
+          const float u2 = s2.x * (v2 - fmaf(s2.z, u1, r[4 * i + 2]));
+          o1[i] = fmaf(s1.y, u1, r[4 * i + 1]);
+          o2[i] = fmaf(s2.y, u2, fmaf(s2.w, u1, r[4 * i + 3]));
+          const f32x2 p1 = pack2(u1, u1), p2 = pack2(u2, u2);
+          if (KEEP_K) {
 #pragma unroll
-          for (int c = 0; c < NCH * 2; ++c) S[i][c] = fma2(K[c], u2, S[i][c]);
+            for (int c = 0; c < NCH * 2; ++c) S.v[i][c] = fma2(K2[KEEP_K ? c : 0], p2, fma2(K1[KEEP_K ? c : 0], p1, S.v[i][c]));
+          } else {
+#pragma unroll
+            for (int c = 0; c < NCH; ++c) {
+              f32x2 k1[2], k2[2], g2[2];
+              lds2(ka + c * 128, k1[0], k1[1]);
+              lds2(ka + DP * 4 + c * 128, k2[0], k2[1]);
+              lds2(ga + DP * 4 + c * 128, g2[0], g2[1]);
+#pragma unroll
+              for (int e = 0; e < 2; ++e)
+                S.v[i][2 * c + e] = fma2(k2[e], p2, fma2(mul2(g2[e], k1[e]), p1, S.v[i][2 * c + e]));
+            }
+          }
         }
       } else {
-        const float fa = sh_gate[t], ib = sh_gate[TB + t], em = sh_gate[2 * TB + t];
-        const f32x2 f2 = pack2(fa, fa), i2 = pack2(ib, ib);
-        f32x2 B[CPT], vb[CPT], D = 0ull;
+        const float4 ga = sh_gate[t], gb = sh_gate[t + 1 < TB ? t + 1 : t];
+        const f32x2 f1 = pack2(ga.x, ga.x), f2 = pack2(gb.x, gb.x);
+        f32x2 v1[CPT], v2[CPT], B1[CPT], B2[CPT];
 #pragma unroll
         for (int i = 0; i < CPT; ++i) {
-          const float v = st[off_v + t * cols + cg * CPT + i] * ib;
-          vb[i] = pack2(v, v);
-          B[i] = 0ull;
+          const float x = st[OFF_V + t * COLS + cg * CPT + i] * ga.y, y = st[OFF_V + (t + 1) * COLS + cg * CPT + i] * gb.y;
+          v1[i] = pack2(x, x);
+          v2[i] = pack2(y, y);
+          B1[i] = B2[i] = 0ull;
         }
 #pragma unroll
         for (int c = 0; c < NCH; ++c) {
-          f32x2 k0, k1, q0, q1;
-          lds2(ka + c * 128, k0, k1);
-          lds2(qa + c * 128, q0, q1);
+          f32x2 k1[2], q1[2], k2[2], q2[2];
+          lds2(ka + c * 128, k1[0], k1[1]);
+          lds2(qa + c * 128, q1[0], q1[1]);
+          lds2(ka + DP * 4 + c * 128, k2[0], k2[1]);
+          lds2(qa + DP * 4 + c * 128, q2[0], q2[1]);
 #pragma unroll
-          for (int i = 0; i < CPT; ++i) {
-            S[i][2 * c] = fma2(k0, vb[i], mul2(S[i][2 * c], f2));
-            S[i][2 * c + 1] = fma2(k1, vb[i], mul2(S[i][2 * c + 1], f2));
-            B[i] = fma2(S[i][2 * c], q0, B[i]);
-            B[i] = fma2(S[i][2 * c + 1], q1, B[i]);
-          }
-          N[2 * c] = fma2(k0, i2, mul2(N[2 * c], f2));
-          N[2 * c + 1] = fma2(k1, i2, mul2(N[2 * c + 1], f2));
-          D = fma2(N[2 * c], q0, D);
-          D = fma2(N[2 * c + 1], q1, D);
+          for (int e = 0; e < 2; ++e)
+#pragma unroll
+            for (int i = 0; i < CPT; ++i) {
+              f32x2 s = fma2(k1[e], v1[i], mul2(S.v[i][2 * c + e], f1));
+              B1[i] = fma2(s, q1[e], B1[i]);
+              s = fma2(k2[e], v2[i], mul2(s, f2));
+              B2[i] = fma2(s, q2[e], B2[i]);
+              S.v[i][2 * c + e] = s;
+            }
         }
-        const float2 dd = unpack2(D);
-        const float den = fmaxf(fabsf(sum8(dd.x + dd.y)), em) + 1e-6f;
-        const float inv = 1.0f / den;
+        float r[2 * CPT];
 #pragma unroll
         for (int i = 0; i < CPT; ++i) {
-          const float2 y = unpack2(B[i]);
-          out[i] = sum8(y.x + y.y) * inv;
+          const float2 x = unpack2(B1[i]), y = unpack2(B2[i]);
+          r[2 * i] = x.x + x.y; r[2 * i + 1] = y.x + y.y;
+        }
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1)
+#pragma unroll
+          for (int i = 0; i < 2 * CPT; ++i) r[i] += __shfl_xor_sync(0xffffffffu, r[i], o);
+#pragma unroll
+        for (int i = 0; i < CPT; ++i) {
+          o1[i] = r[2 * i];
+          o2[i] = r[2 * i + 1];
+          if (mycol + i == a.vdim) {         // the normaliser's column
+            const int64_t th = static_cast<int64_t>(t0 + t) * a.heads + head;
+            if (l8 == 0) {
+              a.den[th] = fmaxf(fabsf(o1[i]), ga.z) + 1e-6f;
+              if (t + 1 < n) a.den[th + a.heads] = fmaxf(fabsf(o2[i]), gb.z) + 1e-6f;
+            }
+          }
         }
       }
-      if (!FUSED) {
-        float* orow = a.out + (static_cast<int64_t>(t0 + t) * a.heads + head) * a.vdim + mycol;
+      float* orow = a.out + (static_cast<int64_t>(t0 + t) * a.heads + head) * a.vdim + mycol;
 #pragma unroll
-        for (int i = 0; i < CPT; ++i)
-          if (l8 == i && mycol + i < a.vdim) orow[i] = out[i];
-      }
+      for (int i = 0; i < CPT; ++i)
+        if (mycol + i < a.vdim) {
+          if (l8 == i) orow[i] = o1[i];
+          if (l8 == CPT + i && t + 1 < n) orow[static_cast<int64_t>(a.heads) * a.vdim + i] = o2[i];
+        }
     }
     __syncthreads();       // the stage may be refilled
   }
+  S.store(state, mycol, columns, l8);
+  if (MODE == kScanMlstm && threadIdx.x == 0) *mstate = run_max;
+}
 
+// One-token form: every sequence brings one token and a CTA owns all columns of a head.  The decay is computed from the
+// raw projection, and the head's output is normalised, gated and stored as the next projection's input.  The state is
+// fetched into L2 before the wait for the preceding kernel (a prefetch reads nothing that could be stale).
+template <typename T, int MODE, int NCH, int CPT>
+__global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb_scan_args a) {
+  constexpr int DP = NCH * 32;
+  __shared__ __align__(16) float sh[3 * DP];       // k, q, decay
+  __shared__ float red[kScanFusedThreads / 32];
+  pdl_launch_dependents();
+  const int seq = blockIdx.y, head = blockIdx.x;
+  const int l8 = threadIdx.x & 7, cg = threadIdx.x >> 3, mycol = cg * CPT;
+  const int columns = a.vdim + (MODE == kScanMlstm ? 1 : 0);
+  const int slot = a.state_slot[seq];               // a step input, written by no kernel
+  const bool ok = slot >= 0 && slot < a.num_slots;
+  float* state = a.state + (ok ? slot : 0) * a.state_slot_stride + static_cast<int64_t>(head) * columns * DP;
+  if (ok)
+    for (int i = threadIdx.x; i < columns * DP / 32; i += blockDim.x)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(state + i * 32));
+  pdl_wait();
+  if (!ok) {
+    if (slot >= a.num_slots && threadIdx.x == 0) report_status(MDB_STATUS_BAD_SLOT);
+    return;
+  }
+  const int64_t t = a.cu_q[seq];
+  const bool fresh = a.start[seq] == 0;
+  const int kvh = head / (a.heads / a.kv_heads);
+  ScanState<NCH, CPT> S;
+  S.load(state, mycol, a.vdim, l8, fresh);
+  ScanState<MODE == kScanMlstm ? NCH : 1, 1> N;      // the normaliser, in every column group
+  float m_old = 0.f;
+  const int blocks = (columns + kScanBlockCols - 1) / kScanBlockCols;
+  float* mstate = nullptr;
+  if constexpr (MODE == kScanMlstm) {
+    N.load(state, a.vdim, columns, l8, fresh);
+    mstate = a.mstate + (static_cast<int64_t>(slot) * a.heads + head) * blocks;
+    if (!fresh) m_old = mstate[0];
+  }
+  const float s0 = a.s0[t * a.heads + head];
+  const float s1 = MODE == kScanDelta ? a.s1[t * a.kv_heads + kvh] : a.s1[t * a.heads + head];
+  float v[CPT];
+#pragma unroll
+  for (int i = 0; i < CPT; ++i) v[i] = mycol + i < a.vdim ? a.v[(t * a.heads + head) * a.vdim + mycol + i] : 0.f;
+  for (int d = threadIdx.x; d < DP; d += blockDim.x) {
+    sh[d] = a.k[(t * a.kv_heads + kvh) * DP + d];
+    sh[DP + d] = a.q[(t * a.kv_heads + kvh) * DP + d];
+    if (MODE == kScanDelta) {
+      float r = 1.f;
+      if (d < a.dim)
+        r = expf(-expf(a.a_log[head]) * softplus_f(rows_at<float>(a.raw_decay, t, head * a.dim + d) + a.dt_bias[head * a.dim + d]));
+      sh[2 * DP + d] = r;
+    }
+  }
+  __syncthreads();
+  const uint32_t ka = smem_u32(sh) + l8 * 16;
+  float out[CPT];
+  if (MODE == kScanDelta) {
+    f32x2 A[CPT], B[CPT];
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) A[i] = B[i] = 0ull;
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+      f32x2 k[2], q[2], g[2];
+      lds2(ka + c * 128, k[0], k[1]);
+      lds2(ka + DP * 4 + c * 128, q[0], q[1]);
+      lds2(ka + DP * 8 + c * 128, g[0], g[1]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+#pragma unroll
+        for (int i = 0; i < CPT; ++i) {
+          const f32x2 s = mul2(S.v[i][2 * c + e], g[e]);
+          A[i] = fma2(s, k[e], A[i]);
+          B[i] = fma2(s, q[e], B[i]);
+          S.v[i][2 * c + e] = s;
+        }
+    }
+    f32x2 u2[CPT];
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) {
+      const float2 x = unpack2(A[i]), y = unpack2(B[i]);
+      const float u = s0 * (v[i] - sum8(x.x + x.y));
+      out[i] = fmaf(s1, u, sum8(y.x + y.y));
+      u2[i] = pack2(u, u);
+    }
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+      f32x2 k[2];
+      lds2(ka + c * 128, k[0], k[1]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+#pragma unroll
+        for (int i = 0; i < CPT; ++i) S.v[i][2 * c + e] = fma2(k[e], u2[i], S.v[i][2 * c + e]);
+    }
+  } else {
+    const float m_new = fmaxf(s1 + m_old, s0);
+    const float fa = expf(s1 + m_old - m_new), ib = expf(s0 - m_new), em = expf(-m_new);
+    const f32x2 f2 = pack2(fa, fa), i2 = pack2(ib, ib);
+    f32x2 B[CPT], vb[CPT], D = 0ull;
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) {
+      vb[i] = pack2(v[i] * ib, v[i] * ib);
+      B[i] = 0ull;
+    }
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+      f32x2 k[2], q[2];
+      lds2(ka + c * 128, k[0], k[1]);
+      lds2(ka + DP * 4 + c * 128, q[0], q[1]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+#pragma unroll
+        for (int i = 0; i < CPT; ++i) {
+          S.v[i][2 * c + e] = fma2(k[e], vb[i], mul2(S.v[i][2 * c + e], f2));
+          B[i] = fma2(S.v[i][2 * c + e], q[e], B[i]);
+        }
+        if constexpr (MODE == kScanMlstm) {
+          N.v[0][2 * c + e] = fma2(k[e], i2, mul2(N.v[0][2 * c + e], f2));
+          D = fma2(N.v[0][2 * c + e], q[e], D);
+        }
+      }
+    }
+    const float2 dd = unpack2(D);
+    const float inv = 1.0f / (fmaxf(fabsf(sum8(dd.x + dd.y)), em) + 1e-6f);
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) {
+      const float2 y = unpack2(B[i]);
+      out[i] = sum8(y.x + y.y) * inv;
+    }
+    if constexpr (MODE == kScanMlstm) {
+      __syncthreads();             // every column group has read the normaliser and the maximum
+      if (cg == 0) N.store(state, a.vdim, columns, l8);
+      for (int b = threadIdx.x; b < blocks; b += blockDim.x) mstate[b] = m_new;
+    }
+  }
+  S.store(state, mycol, a.vdim, l8);
+  float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < CPT; ++i)
-    if (mycol + i < a.vdim) {
+    if (l8 == i && mycol + i < a.vdim) ss = out[i] * out[i];
+  const float rstd = 1.0f / sqrtf(cta_sum(ss, red) / static_cast<float>(a.vdim) + a.eps);
+  T* y = static_cast<T*>(a.y) + t * a.ldy + static_cast<int64_t>(head) * a.vdim;
+  const float* w = a.norm + static_cast<int64_t>(head) * a.norm_head_stride;
 #pragma unroll
-      for (int c = 0; c < NCH; ++c) {
-        const float2 lo = unpack2(S[i][2 * c]), hi = unpack2(S[i][2 * c + 1]);
-        *reinterpret_cast<float4*>(state + static_cast<int64_t>(mycol + i) * DP + c * 32 + l8 * 4) = make_float4(lo.x, lo.y, hi.x, hi.y);
-      }
-    }
-  if (MODE == kScanMlstm) {
-    // refresh the copies of the column blocks this CTA covers (the first column group of each)
-    for (int b = col0 / kScanBlockCols; b < blocks && b * kScanBlockCols < col0 + cols; ++b) {
-      if (cg != 0) break;
-#pragma unroll
-      for (int c = 0; c < NCH; ++c) {
-        const float2 lo = unpack2(N[2 * c]), hi = unpack2(N[2 * c + 1]);
-        *reinterpret_cast<float4*>(nstate + static_cast<int64_t>(b) * DP + c * 32 + l8 * 4) = make_float4(lo.x, lo.y, hi.x, hi.y);
-      }
-      if (threadIdx.x == 0) mstate[b] = run_max;
-    }
-  }
-  if (FUSED) {
-    float ss = 0.f;
-#pragma unroll
-    for (int i = 0; i < CPT; ++i)
-      if (l8 == i && mycol + i < a.vdim) ss = out[i] * out[i];
-    const float rstd = 1.0f / sqrtf(cta_sum(ss, red) / static_cast<float>(a.vdim) + a.eps);
-    T* y = static_cast<T*>(a.y) + static_cast<int64_t>(t_begin) * a.ldy + static_cast<int64_t>(head) * a.vdim;
-    const float* w = a.norm + static_cast<int64_t>(head) * a.norm_head_stride;
-#pragma unroll
-    for (int i = 0; i < CPT; ++i)
-      if (l8 == i && mycol + i < a.vdim)
-        y[mycol + i] = act_from_f<T>(out[i] * rstd * w[mycol + i] * sigmoid_f(rows_at<T>(a.gate, t_begin, head * a.vdim + mycol + i)));
-  }
+  for (int i = 0; i < CPT; ++i)
+    if (l8 == i && mycol + i < a.vdim)
+      y[mycol + i] = act_from_f<T>(out[i] * rstd * w[mycol + i] * sigmoid_f(rows_at<T>(a.gate, t, head * a.vdim + mycol + i)));
 }
 
 }  // namespace mdb
@@ -508,55 +865,56 @@ using namespace mdb;
 
 namespace {
 
-// at most 64 state registers per thread whatever the key size
-constexpr int scan_cols_per_thread(int dim_pad) { return dim_pad <= 128 ? 4 : (dim_pad <= 256 ? 2 : 1); }
-// column groups (of eight lanes) of a CTA that owns a whole head
-constexpr int scan_fused_groups(int vdim, int cpt) { return ((vdim + cpt - 1) / cpt + 3) / 4 * 4; }
+// One-token form: at most 64 state registers per thread whatever the key size.
+constexpr int scan_token_cols(int dim_pad) { return dim_pad <= 128 ? 4 : 2; }
+constexpr int scan_token_groups(int vdim, int cpt) { return ((vdim + cpt - 1) / cpt + 3) / 4 * 4; }
 
-template <typename T, int MODE, int NCH, int CPT, int TB, bool FUSED>
-int launch_scan_form(const mdb_scan_args& a, cudaStream_t st) {
-  constexpr int DP = NCH * 32;
-  int groups;                                     // column groups (of eight lanes) per CTA
-  if (FUSED) groups = scan_fused_groups(a.vdim, CPT);
-  else groups = kScanBlockCols / CPT;
-  const int threads = groups * 8, cols = groups * CPT;
-  if (FUSED && threads > kScanFusedThreads) return MDB_ERR_UNSUPPORTED;
-  const int smem = 2 * scan_stage_floats(MODE, DP, TB, cols) * 4;
-  if (smem > 200 * 1024) return MDB_ERR_UNSUPPORTED;
+template <typename T, int MODE, int NCH>
+int launch_scan_token(const mdb_scan_args& a, cudaStream_t st) {
+  if constexpr (NCH * 32 > kScanFusedMaxDim) {
+    return MDB_ERR_UNSUPPORTED;
+  } else {
+    constexpr int CPT = scan_token_cols(NCH * 32);
+    const int threads = scan_token_groups(a.vdim, CPT) * 8;
+    if (threads > kScanFusedThreads) return MDB_ERR_UNSUPPORTED;
+    return mdb_launch(scan_token_kernel<T, MODE, NCH, CPT>, dim3(a.heads, a.bs), dim3(threads), 0, st, a);
+  }
+}
+
+template <int MODE, int NCH>
+int launch_scan_prompt(const mdb_scan_args& a, cudaStream_t st) {
+  constexpr int CPT = NCH > 8 ? 1 : (MODE == kScanMlstm ? (NCH <= 4 ? 4 : 2) : (NCH <= 4 ? 2 : 1));
+  constexpr int smem = 2 * scan_stage_floats(MODE, NCH * 32, kScanTokens, kScanBlockCols) * 4;
+  static_assert(smem <= 227 * 1024, "shared memory of the scan");
   static PerDeviceOnce attr_once;
   const int dev = attr_once.slot();
   if (dev < 0) return MDB_ERR_CUDA;
   if (!attr_once.done[dev]) {
-    if (cudaFuncSetAttribute(scan_kernel<T, MODE, NCH, CPT, TB, FUSED>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) !=
-        cudaSuccess)
+    if (cudaFuncSetAttribute(scan_kernel<MODE, NCH, CPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
       return MDB_ERR_CUDA;
     attr_once.done[dev] = true;
   }
-  const dim3 grid(FUSED ? 1 : (a.vdim + cols - 1) / cols, a.heads, a.bs);
-  return mdb_launch(scan_kernel<T, MODE, NCH, CPT, TB, FUSED>, grid, dim3(threads), smem, st, a, cols);
+  const int columns = a.vdim + (MODE == kScanMlstm ? 1 : 0);
+  const dim3 grid((columns + kScanBlockCols - 1) / kScanBlockCols, a.heads, a.bs);
+  return mdb_launch(scan_kernel<MODE, NCH, CPT>, grid, dim3(kScanBlockCols / CPT * 8), smem, st, a);
 }
 
-template <typename T, int MODE, int NCH>
+template <int MODE, int NCH>
 int launch_scan_dim(const mdb_scan_args& a, cudaStream_t st) {
-  constexpr int CPT = scan_cols_per_thread(NCH * 32);
-  constexpr int TB = NCH <= 4 ? 16 : 8;
-  if (a.fused) {
-    if constexpr (NCH * 32 <= kScanFusedMaxDim) return launch_scan_form<T, MODE, NCH, CPT, 1, true>(a, st);
-    else return MDB_ERR_UNSUPPORTED;
-  }
-  return launch_scan_form<float, MODE, NCH, CPT, TB, false>(a, st);     // the activation type plays no part here
+  if (!a.fused) return launch_scan_prompt<MODE, NCH>(a, st);
+  return a.dtype == MDB_F32 ? launch_scan_token<float, MODE, NCH>(a, st) : launch_scan_token<bf16, MODE, NCH>(a, st);
 }
 
-template <typename T, int MODE>
+template <int MODE>
 int launch_scan(const mdb_scan_args& a, cudaStream_t st) {
   switch (a.dim_pad) {
-    case 32: return launch_scan_dim<T, MODE, 1>(a, st);
-    case 64: return launch_scan_dim<T, MODE, 2>(a, st);
-    case 96: return launch_scan_dim<T, MODE, 3>(a, st);
-    case 128: return launch_scan_dim<T, MODE, 4>(a, st);
-    case 192: return launch_scan_dim<T, MODE, 6>(a, st);
-    case 256: return launch_scan_dim<T, MODE, 8>(a, st);
-    case 512: return launch_scan_dim<T, MODE, 16>(a, st);
+    case 32: return launch_scan_dim<MODE, 1>(a, st);
+    case 64: return launch_scan_dim<MODE, 2>(a, st);
+    case 96: return launch_scan_dim<MODE, 3>(a, st);
+    case 128: return launch_scan_dim<MODE, 4>(a, st);
+    case 192: return launch_scan_dim<MODE, 6>(a, st);
+    case 256: return launch_scan_dim<MODE, 8>(a, st);
+    case 512: return launch_scan_dim<MODE, 16>(a, st);
     default: return MDB_ERR_UNSUPPORTED;
   }
 }
@@ -574,10 +932,10 @@ int mdb_scan_dim_pad(int dim) {
   return 0;
 }
 
-int mdb_scan_blocks(int vdim) { return (vdim + kScanBlockCols - 1) / kScanBlockCols; }
+int mdb_scan_blocks(int vdim) { return (vdim + 1 + kScanBlockCols - 1) / kScanBlockCols; }
 
 int mdb_scan_fusable(int dim_pad, int vdim) {
-  return dim_pad <= kScanFusedMaxDim && scan_fused_groups(vdim, scan_cols_per_thread(dim_pad)) * 8 <= kScanFusedThreads ? 1 : 0;
+  return dim_pad <= kScanFusedMaxDim && scan_token_groups(vdim, scan_token_cols(dim_pad)) * 8 <= kScanFusedThreads ? 1 : 0;
 }
 
 int mdb_delta_prep(const mdb_delta_prep_args* args, mdb_stream_t stream) {
@@ -595,25 +953,45 @@ int mdb_delta_prep(const mdb_delta_prep_args* args, mdb_stream_t stream) {
               MDB_ERR_ARG);
   MDB_REQUIRE(a.taps <= kMaxTaps, MDB_ERR_UNSUPPORTED);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const int units = a.kv_heads + a.heads + 1 + (a.copy_cols + 127) / 128;
-  const dim3 grid(a.m, (units + kPrepWarps - 1) / kPrepWarps);
-  int rc = a.dtype == MDB_F32 ? mdb_launch(delta_prep_kernel<float>, grid, dim3(kPrepWarps * 32), 0, st, a)
-                              : mdb_launch(delta_prep_kernel<bf16>, grid, dim3(kPrepWarps * 32), 0, st, a);
+  int rc;
+  if (a.dim % 4 == 0 && a.vdim % 4 == 0 && a.dim <= 128 && a.dim_pad <= 128 && a.taps <= 4 && rows_ok(a.q) && rows_ok(a.k) && rows_ok(a.v) &&
+      a.conv_slot_stride % 4 == 0 && mdb_aligned16(a.v_out) && (a.q.parts != nullptr) == (a.k.parts != nullptr) &&
+      (a.q.parts != nullptr) == (a.v.parts != nullptr) && (a.copy_cols == 0 || (a.q.parts != nullptr) == (a.copy.parts != nullptr)) &&
+      (a.dtype == MDB_BF16 || a.q.parts == nullptr)) {
+    const int run = a.m >= 1024 ? 8 : 1;
+    const int units = a.kv_heads + a.heads * ((a.vdim + 127) / 128) + 1 + (a.copy_cols + 127) / 128;
+    const dim3 grid((a.m + run - 1) / run, (units + kPrepWarps - 1) / kPrepWarps);
+    const bool parts = a.q.parts != nullptr;
+    const dim3 block(kPrepWarps * 32);
+    if (a.dtype == MDB_F32) rc = mdb_launch(delta_prep_rows_kernel<float, false>, grid, block, 0, st, a, run);
+    else if (parts) rc = mdb_launch(delta_prep_rows_kernel<bf16, true>, grid, block, 0, st, a, run);
+    else rc = mdb_launch(delta_prep_rows_kernel<bf16, false>, grid, block, 0, st, a, run);
+  } else {
+    const int units = a.kv_heads + a.heads + 1 + (a.copy_cols + 127) / 128;
+    const dim3 grid(a.m, (units + kPrepWarps - 1) / kPrepWarps);
+    rc = a.dtype == MDB_F32 ? mdb_launch(delta_prep_kernel<float>, grid, dim3(kPrepWarps * 32), 0, st, a)
+                            : mdb_launch(delta_prep_kernel<bf16>, grid, dim3(kPrepWarps * 32), 0, st, a);
+  }
   if (rc != MDB_OK || a.shift_state || a.taps < 2) return rc;
   const dim3 cgrid((a.channels + 255) / 256, a.bs);
   return a.dtype == MDB_F32 ? mdb_launch(conv_state_kernel<float>, cgrid, dim3(256), 0, st, a)
                             : mdb_launch(conv_state_kernel<bf16>, cgrid, dim3(256), 0, st, a);
 }
 
-int mdb_channel_decay(const float* x, int64_t ldx, const float* a_log, const float* dt_bias, float* g, int m, int heads,
-                      int dim, int dim_pad, mdb_stream_t stream) {
-  MDB_REQUIRE(m >= 0 && heads > 0 && dim > 0 && dim_pad >= dim, MDB_ERR_ARG);
-  if (m == 0) return MDB_OK;
-  MDB_REQUIRE(x && a_log && dt_bias && g && ldx >= static_cast<int64_t>(heads) * dim, MDB_ERR_ARG);
-  const int64_t total = static_cast<int64_t>(m) * heads * dim_pad;
-  const int64_t blocks = (total + 255) / 256;
-  return mdb_launch(channel_decay_kernel, dim3(static_cast<int>(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0,
-                    static_cast<cudaStream_t>(stream), x, ldx, a_log, dt_bias, g, total, heads, dim, dim_pad);
+int mdb_channel_decay(const mdb_decay_args* args, mdb_stream_t stream) {
+  MDB_REQUIRE(args != nullptr, MDB_ERR_ARG);
+  const mdb_decay_args a = *args;
+  MDB_REQUIRE(a.m >= 0 && a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.dim_pad >= a.dim, MDB_ERR_ARG);
+  if (a.m == 0) return MDB_OK;
+  MDB_REQUIRE(a.x && a.a_log && a.dt_bias && a.q && a.k && a.g && a.cross && a.row_seq && a.cu_q &&
+                  a.ldx >= static_cast<int64_t>(a.heads) * a.dim,
+              MDB_ERR_ARG);
+  MDB_REQUIRE(a.dim_pad % 4 == 0 && mdb_aligned16(a.g) && mdb_aligned16(a.q) && mdb_aligned16(a.k), MDB_ERR_ALIGN);
+  const dim3 grid(a.m, (a.heads + 3) / 4);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (a.dim % 4 == 0 && a.ldx % 4 == 0 && mdb_aligned16(a.x) && mdb_aligned16(a.dt_bias))
+    return mdb_launch(channel_decay_kernel<true>, grid, dim3(128), 0, st, a);
+  return mdb_launch(channel_decay_kernel<false>, grid, dim3(128), 0, st, a);
 }
 
 int mdb_mlstm_prep(const mdb_mlstm_prep_args* args, mdb_stream_t stream) {
@@ -624,11 +1002,18 @@ int mdb_mlstm_prep(const mdb_mlstm_prep_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(rows_present(a.q) && rows_present(a.k) && rows_present(a.v) && rows_present(a.i) && rows_present(a.f) &&
                   a.bias_i && a.bias_f && a.q_out && a.k_out && a.v_out && a.log_i && a.log_f,
               MDB_ERR_ARG);
-  const int items = a.heads * (a.dim_pad + a.vdim + 1);
-  const dim3 grid(a.m, (items + 511) / 512);
+  const int items = a.heads * a.dim_pad / 4 + (a.heads * a.vdim + 3) / 4 + a.heads;
+  const dim3 grid(a.m, a.m >= 1024 ? 1 : (items + 255) / 256);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return a.dtype == MDB_F32 ? mdb_launch(mlstm_prep_kernel<float>, grid, dim3(128), 0, st, a)
-                            : mdb_launch(mlstm_prep_kernel<bf16>, grid, dim3(128), 0, st, a);
+  const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && rows_ok(a.q) && rows_ok(a.k) && rows_ok(a.v) && mdb_aligned16(a.v_out);
+  const bool parts = a.q.parts != nullptr;
+  if ((a.k.parts != nullptr) != parts || (a.v.parts != nullptr) != parts || (parts && a.dtype == MDB_F32)) return MDB_ERR_UNSUPPORTED;
+  if (a.dtype == MDB_F32)
+    return vec ? mdb_launch(mlstm_prep_kernel<float, true, false>, grid, dim3(256), 0, st, a)
+               : mdb_launch(mlstm_prep_kernel<float, false, false>, grid, dim3(256), 0, st, a);
+  if (!vec) return mdb_launch(mlstm_prep_kernel<bf16, false, false>, grid, dim3(256), 0, st, a);
+  return parts ? mdb_launch(mlstm_prep_kernel<bf16, true, true>, grid, dim3(256), 0, st, a)
+               : mdb_launch(mlstm_prep_kernel<bf16, true, false>, grid, dim3(256), 0, st, a);
 }
 
 int mdb_scan(const mdb_scan_args* args, mdb_stream_t stream) {
@@ -638,21 +1023,19 @@ int mdb_scan(const mdb_scan_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(a.bs >= 0 && a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.vdim > 0, MDB_ERR_ARG);
   if (a.bs == 0) return MDB_OK;
   MDB_REQUIRE(a.q && a.k && a.v && a.s0 && a.s1 && a.state && seqs_ok(a.cu_q, a.start, a.state_slot), MDB_ERR_ARG);
-  MDB_REQUIRE(a.mode != MDB_SCAN_MLSTM || (a.nstate && a.mstate && a.kv_heads == a.heads), MDB_ERR_ARG);
+  MDB_REQUIRE(a.mode != MDB_SCAN_MLSTM || (a.mstate && a.kv_heads == a.heads), MDB_ERR_ARG);
   if (a.fused) {
     MDB_REQUIRE(rows_present(a.gate) && a.norm && a.y, MDB_ERR_ARG);
     MDB_REQUIRE(a.mode != MDB_SCAN_DELTA || (rows_present(a.raw_decay) && a.a_log && a.dt_bias), MDB_ERR_ARG);
   } else {
-    MDB_REQUIRE(a.out != nullptr && (a.mode != MDB_SCAN_DELTA || a.g != nullptr), MDB_ERR_ARG);
+    MDB_REQUIRE(a.out != nullptr && (a.mode == MDB_SCAN_DELTA ? a.g && a.cross : a.den != nullptr), MDB_ERR_ARG);
   }
-  MDB_REQUIRE(mdb_aligned16(a.q) && mdb_aligned16(a.k) && mdb_aligned16(a.g) && mdb_aligned16(a.state) && mdb_aligned16(a.nstate) &&
+  MDB_REQUIRE(mdb_aligned16(a.q) && mdb_aligned16(a.k) && mdb_aligned16(a.g) && mdb_aligned16(a.state) &&
                   a.state_slot_stride % 4 == 0,
               MDB_ERR_ALIGN);
   MDB_REQUIRE(a.heads <= 65535 && a.bs <= 65535, MDB_ERR_UNSUPPORTED);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (a.dtype == MDB_F32)
-    return a.mode == MDB_SCAN_DELTA ? launch_scan<float, kScanDelta>(a, st) : launch_scan<float, kScanMlstm>(a, st);
-  return a.mode == MDB_SCAN_DELTA ? launch_scan<bf16, kScanDelta>(a, st) : launch_scan<bf16, kScanMlstm>(a, st);
+  return a.mode == MDB_SCAN_DELTA ? launch_scan<kScanDelta>(a, st) : launch_scan<kScanMlstm>(a, st);
 }
 
 }  // extern "C"

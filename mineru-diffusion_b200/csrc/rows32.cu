@@ -59,6 +59,19 @@ __device__ __forceinline__ float4 rows_at4(const mdb_rows& s, int64_t row, int c
   }
   return act_load4(static_cast<const T*>(s.x) + off);
 }
+// The form known at compile time: kernels that read many places keep the slice loop out of their row form.
+template <typename T, bool PARTS>
+__device__ __forceinline__ float4 rows_at4_of(const mdb_rows& s, int64_t row, int col) {
+  const int64_t off = row * s.ld + s.col + col;
+  if (!PARTS) return act_load4(static_cast<const T*>(s.x) + off);
+  float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+  for (int p = 0; p < s.nparts; ++p) {
+    const float4 v = *reinterpret_cast<const float4*>(s.parts + p * s.part_stride + off);
+    a.x += v.x; a.y += v.y; a.z += v.z; a.w += v.w;
+  }
+  return make_float4(act_to_f(act_from_f<T>(a.x)), act_to_f(act_from_f<T>(a.y)), act_to_f(act_from_f<T>(a.z)), act_to_f(act_from_f<T>(a.w)));
+}
 __host__ __device__ __forceinline__ bool rows_present(const mdb_rows& s) { return s.x != nullptr || s.parts != nullptr; }
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
@@ -179,23 +192,40 @@ __global__ void __launch_bounds__(kRmsRowsThreads) rms_rows_kernel(const RmsSegm
   }
 }
 
-// Behind a recurrence: one warp per (row, head).  y = o / rms(o) * weight * sigmoid(gate).
-template <typename T>
+// Behind a recurrence: one warp per (row, head).  y = o' / rms(o') * weight * sigmoid(gate), o' = o / den where there is
+// a den.  VEC: heads in multiples of four, everything 16-byte aligned.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(128) gated_norm_kernel(const mdb_gated_norm_args a) {
   pdl_launch_dependents();
   pdl_wait();
-  const int64_t item = static_cast<int64_t>(blockIdx.x) * 4 + (threadIdx.x >> 5);
-  if (item >= static_cast<int64_t>(a.m) * a.heads) return;
-  const int64_t row = item / a.heads;
-  const int head = static_cast<int>(item % a.heads), lane = threadIdx.x & 31;
+  const int64_t row = blockIdx.x;
+  const int head = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (head >= a.heads) return;
   const float* o = a.o + (row * a.heads + head) * a.vdim;
-  float ss = 0.f;
-  for (int c = lane; c < a.vdim; c += 32) ss += o[c] * o[c];
-  const float rstd = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(a.vdim) + a.eps);
+  const float inv = a.den != nullptr ? 1.0f / a.den[row * a.heads + head] : 1.0f;
   const float* w = a.weight + static_cast<int64_t>(head) * a.weight_head_stride;
   T* y = static_cast<T*>(a.y) + row * a.ldy + static_cast<int64_t>(head) * a.vdim;
-  for (int c = lane; c < a.vdim; c += 32)
-    y[c] = act_from_f<T>(o[c] * rstd * w[c] * sigmoid_f(rows_at<T>(a.gate, row, head * a.vdim + c)));
+  float ss = 0.f;
+  if (VEC) {
+    for (int c = lane * 4; c < a.vdim; c += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(o + c);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int c = lane; c < a.vdim; c += 32) ss += o[c] * o[c];
+  }
+  const float rstd = inv / sqrtf(warp_sum(ss) * inv * inv / static_cast<float>(a.vdim) + a.eps);
+  if (VEC) {
+    for (int c = lane * 4; c < a.vdim; c += 128) {
+      const float4 v = *reinterpret_cast<const float4*>(o + c), wv = *reinterpret_cast<const float4*>(w + c);
+      const float4 g = rows_at4<T>(a.gate, row, head * a.vdim + c);
+      act_store4(y + c, make_float4(v.x * rstd * wv.x * sigmoid_f(g.x), v.y * rstd * wv.y * sigmoid_f(g.y),
+                                    v.z * rstd * wv.z * sigmoid_f(g.z), v.w * rstd * wv.w * sigmoid_f(g.w)));
+    }
+  } else {
+    for (int c = lane; c < a.vdim; c += 32)
+      y[c] = act_from_f<T>(o[c] * rstd * w[c] * sigmoid_f(rows_at<T>(a.gate, row, head * a.vdim + c)));
+  }
 }
 
 // Row r of the output = the latent of token r - cu[seq] of its sequence, read through the page table.
@@ -322,11 +352,15 @@ int mdb_gated_norm(const mdb_gated_norm_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(a.m >= 0 && a.heads > 0 && a.vdim > 0, MDB_ERR_ARG);
   if (a.m == 0) return MDB_OK;
   MDB_REQUIRE(a.o && a.weight && a.y && rows_present(a.gate) && a.ldy >= static_cast<int64_t>(a.heads) * a.vdim, MDB_ERR_ARG);
-  const int64_t items = static_cast<int64_t>(a.m) * a.heads;
-  const int grid = static_cast<int>((items + 3) / 4);
+  const dim3 grid(a.m, (a.heads + 3) / 4);
+  const bool vec = a.vdim % 4 == 0 && rows_ok(a.gate) && a.ldy % 4 == 0 && mdb_aligned16(a.o) && mdb_aligned16(a.y) &&
+                   mdb_aligned16(a.weight) && a.weight_head_stride % 4 == 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (a.dtype == MDB_F32) return mdb_launch(gated_norm_kernel<float>, dim3(grid), dim3(128), 0, st, a);
-  return mdb_launch(gated_norm_kernel<bf16>, dim3(grid), dim3(128), 0, st, a);
+  if (a.dtype == MDB_F32)
+    return vec ? mdb_launch(gated_norm_kernel<float, true>, grid, dim3(128), 0, st, a)
+               : mdb_launch(gated_norm_kernel<float, false>, grid, dim3(128), 0, st, a);
+  return vec ? mdb_launch(gated_norm_kernel<bf16, true>, grid, dim3(128), 0, st, a)
+             : mdb_launch(gated_norm_kernel<bf16, false>, grid, dim3(128), 0, st, a);
 }
 
 int mdb_gather_latents(int dtype, const void* cache, const int32_t* block_table, int table_stride, int num_pages,

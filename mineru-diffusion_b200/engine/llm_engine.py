@@ -29,6 +29,10 @@ class LLMEngine:
         """Engine with the runner of the configuration's design."""
         return cls(config, registry.of_config(config.decoder_config).load("runner")(config, **runner_args))
 
+    def new_request(self, token_ids: list[int], params) -> Sequence:
+        """A request of the kind the configuration's design decodes."""
+        return registry.of_config(self.config.decoder_config).load("request")(token_ids, params, self.config)
+
     def add_sequence(self, seq: Sequence):
         self.scheduler.add(seq)
 

@@ -19,6 +19,7 @@ class Architecture:
     read_config: Callable[[dict], object]     # parsed config.json -> config_type
     runner: str                               # "module:class", imported on first use
     scheduler: str
+    request: str                              # makes a request from (token ids, SamplingParams, Config)
 
     def load(self, which: str):
         module, name = getattr(self, which).split(":")
@@ -56,6 +57,17 @@ def read_config(raw: dict):
     return by_name(name).read_config(raw) if name is not None else _read_sdar(raw)
 
 
-register(Architecture("sdar", object, _read_sdar, ".model_runner:ModelRunner", ".scheduler:Scheduler"))
+def sdar_request(token_ids, params, config):
+    from .sequence import Sequence
+    return Sequence(token_ids, params, denoising_block_size=config.block_size, mask_token_id=config.mask_token_id)
+
+
+def causal_request(token_ids, params, config):
+    from .causal_scheduler import CausalSequence
+    return CausalSequence(token_ids, params)
+
+
+register(Architecture("sdar", object, _read_sdar, ".model_runner:ModelRunner", ".scheduler:Scheduler",
+                      ".registry:sdar_request"))
 register(Architecture("Zikunex", HybridConfig, HybridConfig.from_json, ".causal_runner:CausalModelRunner",
-                      ".causal_scheduler:CausalScheduler"))
+                      ".causal_scheduler:CausalScheduler", ".registry:causal_request"))

@@ -395,9 +395,10 @@ class HybridEngine:
                      norm=lw["norm"], y=y)
         else:
             g = self.buf("scan_g", m, heads, dp, dtype=f32)
-            ops.channel_decay(raw, lw["a_log"], lw["dt_bias"], g, dim)
+            cross = self.buf("scan_cross", m, heads, 2, dtype=f32)
+            ops.channel_decay(raw, lw["a_log"], lw["dt_bias"], q, k, self._portions(b), g, cross, dim)
             o = self.buf("scan_o", m, heads, vdim, dtype=f32)
-            ops.scan(*common, g=g, out=o)
+            ops.scan(*common, g=g, cross=cross, out=o)
             ops.gated_norm(o, gate, lw["norm"], False, eps, y)
         return self._linear("mix_out", y, lw["o"])
 
@@ -414,14 +415,14 @@ class HybridEngine:
         ops.mlstm_prep(self.dtype, m, heads, dim, vdim, x.cols(q0), x.cols(k0), x.cols(v0), x.cols(i0), x.cols(f0),
                        lw["bias_i"], lw["bias_f"], mx.gate_cap, outs)
         y = self.buf(f"mix_o_{heads * vdim}", m, lw["o"].shape[1])
-        common = dict(nstate=st["n"], mstate=st["m"])
         args = (ops.SCAN_MLSTM, self.dtype, b.bs, heads, heads, dim, vdim, *outs, st["s"], self._portions(b))
         if fused:
-            ops.scan(*args, eps=eps, gate=x.cols(g0), norm=lw["norm"], per_head_norm=True, y=y, **common)
+            ops.scan(*args, eps=eps, gate=x.cols(g0), norm=lw["norm"], per_head_norm=True, y=y, mstate=st["m"])
         else:
             o = self.buf("scan_o", m, heads, vdim, dtype=f32)
-            ops.scan(*args, out=o, **common)
-            ops.gated_norm(o, x.cols(g0), lw["norm"], True, eps, y)
+            den = self.buf("scan_den", m, heads, dtype=f32)
+            ops.scan(*args, out=o, den=den, mstate=st["m"])
+            ops.gated_norm(o, x.cols(g0), lw["norm"], True, eps, y, den=den)
         return self._linear("mix_out", y, lw["o"])
 
     def _latent_attention(self, li: int, mx: LatentAttentionSpec, lw: dict, h: torch.Tensor, b: StepBatch) -> ops.Rows:
@@ -491,8 +492,7 @@ def state_shapes(mx, dtype: torch.dtype) -> dict[str, tuple]:
         channels = 2 * mx.kv_heads * mx.dim + mx.heads * mx.vdim
         return {"s": ((mx.heads, mx.vdim, dp), torch.float32), "conv": ((mx.conv - 1, channels), dtype)}
     blocks = ops.scan_blocks(mx.vdim)
-    return {"s": ((mx.heads, mx.vdim, dp), torch.float32), "n": ((mx.heads, blocks, dp), torch.float32),
-            "m": ((mx.heads, blocks), torch.float32)}
+    return {"s": ((mx.heads, mx.vdim + 1, dp), torch.float32), "m": ((mx.heads, blocks), torch.float32)}
 
 
 def bytes_per_page(cfg: HybridConfig, dtype: torch.dtype) -> int:

@@ -640,11 +640,13 @@ def rms_rows(segments: list, m: int, dtype: torch.dtype) -> None:
     _lib.check(_lib.lib().mdb_rms_rows(_DTYPES[dtype], arr, len(segments), m, _stream()), "mdb_rms_rows")
 
 
-def gated_norm(o: torch.Tensor, gate: Rows, weight: torch.Tensor, per_head_weight: bool, eps: float, out: torch.Tensor) -> None:
-    """o [m, heads, vdim] fp32, normalised per head, times weight, times sigmoid(gate), into out [m, heads * vdim]."""
+def gated_norm(o: torch.Tensor, gate: Rows, weight: torch.Tensor, per_head_weight: bool, eps: float, out: torch.Tensor,
+               den: torch.Tensor | None = None) -> None:
+    """o [m, heads, vdim] fp32, divided by den [m, heads] if given, normalised per head, times weight, times sigmoid(gate),
+    into out [m, heads * vdim]."""
     m, heads, vdim = o.shape
-    a = _lib.GatedNormArgs(_act_dtype(out, "out"), m, heads, vdim, o.data_ptr(), gate.c(), weight.data_ptr(), out.data_ptr(),
-                           _rows(out, "out"), vdim if per_head_weight else 0, eps)
+    a = _lib.GatedNormArgs(_act_dtype(out, "out"), m, heads, vdim, o.data_ptr(), _ptr(den), gate.c(), weight.data_ptr(),
+                           out.data_ptr(), _rows(out, "out"), vdim if per_head_weight else 0, eps)
     _lib.check(_lib.lib().mdb_gated_norm(a, _stream()), "mdb_gated_norm")
 
 
@@ -683,11 +685,15 @@ def delta_prep(dtype: torch.dtype, m: int, bs: int, heads: int, kv_heads: int, d
     _lib.check(_lib.lib().mdb_delta_prep(a, _stream()), "mdb_delta_prep")
 
 
-def channel_decay(x: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, out: torch.Tensor, dim: int) -> None:
-    """out [m, heads, dim_pad] = exp(-exp(a_log) softplus(x + dt_bias)); x fp32 [m, >= heads * dim]."""
+def channel_decay(x: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, q: torch.Tensor, k: torch.Tensor,
+                  portions: tuple, out: torch.Tensor, cross: torch.Tensor, dim: int) -> None:
+    """out [m, heads, dim_pad] = exp(-exp(a_log) softplus(x + dt_bias)); x fp32 [m, >= heads * dim]; cross [m, heads, 2]: the
+    products of a portion's odd tokens with the token before (q, k of ``delta_prep``)."""
     m, heads, dp = out.shape
-    _lib.check(_lib.lib().mdb_channel_decay(x.data_ptr(), _rows(x, "x"), a_log.data_ptr(), dt_bias.data_ptr(),
-                                            out.data_ptr(), m, heads, dim, dp, _stream()), "mdb_channel_decay")
+    row_seq, cu_q, _, _ = portions
+    a = _lib.DecayArgs(m, heads, q.shape[1], dim, dp, x.data_ptr(), _rows(x, "x"), a_log.data_ptr(), dt_bias.data_ptr(),
+                       q.data_ptr(), k.data_ptr(), out.data_ptr(), cross.data_ptr(), row_seq.data_ptr(), cu_q.data_ptr())
+    _lib.check(_lib.lib().mdb_channel_decay(a, _stream()), "mdb_channel_decay")
 
 
 def mlstm_prep(dtype: torch.dtype, m: int, heads: int, dim: int, vdim: int, q: Rows, k: Rows, v: Rows, i: Rows, f: Rows,
@@ -703,16 +709,17 @@ SCAN_DELTA, SCAN_MLSTM = 0, 1
 
 
 def scan(mode: int, dtype: torch.dtype, bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q, k, v, s0, s1, state,
-         portions: tuple, eps: float = 0.0, g=None, nstate=None, mstate=None, out=None, raw_decay: Rows | None = None,
+         portions: tuple, eps: float = 0.0, g=None, cross=None, mstate=None, den=None, out=None, raw_decay: Rows | None = None,
          a_log=None, dt_bias=None, gate: Rows | None = None, norm=None, per_head_norm: bool = False, y=None) -> None:
-    """The recurrence over every sequence's portion; ``state`` [slots, heads, vdim, dim_pad] fp32.  With ``y`` the fused
-    one-token form runs (decay from ``raw_decay``, gated norm into ``y``), else ``out`` [m, heads, vdim] fp32 is written."""
+    """The recurrence over every sequence's portion; ``state`` [slots, heads, vdim (mLSTM: + 1), dim_pad] fp32.  With ``y``
+    the fused one-token form runs (decay from ``raw_decay``, gated norm into ``y``), else ``out`` [m, heads, vdim] fp32
+    (mLSTM: and ``den`` [m, heads]) is written."""
     _, cu_q, start, slot = portions
     a = _lib.ScanArgs(
         mode=mode, dtype=_DTYPES[dtype], fused=int(y is not None), bs=bs, heads=heads, kv_heads=kv_heads, dim=dim,
         dim_pad=q.shape[-1], vdim=vdim, eps=eps, q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), g=_ptr(g), s0=s0.data_ptr(),
         s1=s1.data_ptr(), state=state.data_ptr(), state_slot_stride=state.stride(0), num_slots=state.shape[0],
-        nstate=_ptr(nstate), mstate=_ptr(mstate), cu_q=cu_q.data_ptr(), start=start.data_ptr(), state_slot=slot.data_ptr(),
+        mstate=_ptr(mstate), cross=_ptr(cross), den=_ptr(den), cu_q=cu_q.data_ptr(), start=start.data_ptr(), state_slot=slot.data_ptr(),
         out=_ptr(out), raw_decay=_rows_c(raw_decay), a_log=_ptr(a_log), dt_bias=_ptr(dt_bias), gate=_rows_c(gate),
         norm=_ptr(norm), norm_head_stride=vdim if per_head_norm else 0, y=_ptr(y), ldy=0 if y is None else _rows(y, "y"))
     _lib.check(_lib.lib().mdb_scan(a, _stream()), "mdb_scan")

@@ -149,9 +149,9 @@ def _delta_run(case, H, KH, D, DV, counts, dtype, fused=False):
                      norm=torch.ones(DV, device=DEV), y=y)
             outs.append(y.float().view(1, H, DV))
         else:
-            g, o = torch.zeros(n, H, dp, device=DEV), torch.zeros(n, H, DV, device=DEV)
-            ops.channel_decay(r, a_log.to(DEV), dt.to(DEV), g, D)
-            ops.scan(*common, g=g, out=o)
+            g, o, cross = torch.zeros(n, H, dp, device=DEV), torch.zeros(n, H, DV, device=DEV), torch.full((n, H, 2), 9.0, device=DEV)
+            ops.channel_decay(r, a_log.to(DEV), dt.to(DEV), q, k, p, g, cross, D)
+            ops.scan(*common, g=g, cross=cross, out=o)
             outs.append(orc.rms(o, 1e-5) if fused else o)
         at += n
     torch.cuda.synchronize()
@@ -187,8 +187,10 @@ def test_delta_remembers_a_far_key():
     v = torch.randn(T, 1, DV, generator=gen(1))
     one, z = torch.ones(T, 1), (k * q).sum(-1)
     state, o = torch.zeros(1, 1, DV, D, device=DEV), torch.zeros(T, 1, DV, device=DEV)
+    cross = torch.zeros(T, 1, 2)
+    cross[1:, :, 0], cross[1:, :, 1] = (k[:-1] * k[1:]).sum(-1), (k[:-1] * q[1:]).sum(-1)
     ops.scan(ops.SCAN_DELTA, F32, 1, 1, 1, D, DV, q.to(DEV), k.to(DEV), v.to(DEV), one.to(DEV), z.to(DEV), state,
-             portions_of([T], slots=[0]), g=torch.ones(T, 1, D, device=DEV), out=o)
+             portions_of([T], slots=[0]), g=torch.ones(T, 1, D, device=DEV), cross=cross.to(DEV), out=o)
     o = o.cpu()
     assert float(o[:3].abs().max()) == 0 and float((o[3:, 0] - v[3, 0]).abs().max()) < 1e-5
 
@@ -206,7 +208,7 @@ def test_mlstm_scan_in_portions(dtype, H, D, DV, cap):
     dp, nb = ops.scan_dim_pad(D), ops.scan_blocks(DV)
     w = 0.5 + torch.rand(H * DV, generator=gen(4))
     for counts in ([T], [2, 33, 1, 1, 2, 31], [1] * 12 + [58]):
-        st = (torch.full((2, H, DV, dp), 3.0, device=DEV), torch.full((2, H, nb, dp), 3.0, device=DEV), torch.full((2, H, nb), 3.0, device=DEV))
+        state, mst = torch.full((2, H, DV + 1, dp), 3.0, device=DEV), torch.full((2, H, nb), 3.0, device=DEV)
         outs, normed, at = [], [], 0
         for n in counts:
             p = portions_of([n], [at], [1])
@@ -214,17 +216,17 @@ def test_mlstm_scan_in_portions(dtype, H, D, DV, cap):
             q, k, v = (torch.full((n, H, dp), 9.0, device=DEV), torch.full((n, H, dp), 9.0, device=DEV), torch.zeros(n, H, DV, device=DEV))
             gi, gf = torch.zeros(n, H, device=DEV), torch.zeros(n, H, device=DEV)
             ops.mlstm_prep(dtype, n, H, D, DV, r["q"], r["k"], r["v"], r["i"], r["f"], bi.to(DEV), bf.to(DEV), cap, (q, k, v, gi, gf))
-            args = (ops.SCAN_MLSTM, dtype, 1, H, H, D, DV, q, k, v, gi, gf, st[0], p)
+            args = (ops.SCAN_MLSTM, dtype, 1, H, H, D, DV, q, k, v, gi, gf, state, p)
             if n == 1 and ops.scan_fusable(dp, DV):
                 y = torch.zeros(1, H * DV, dtype=dtype, device=DEV)
                 gate = torch.full((1, (H * DV + 3) // 4 * 4), 100.0, dtype=dtype, device=DEV)
-                ops.scan(*args, nstate=st[1], mstate=st[2], eps=1e-5, gate=ops.Rows(gate), norm=w.to(DEV), per_head_norm=True, y=y)
+                ops.scan(*args, mstate=mst, eps=1e-5, gate=ops.Rows(gate), norm=w.to(DEV), per_head_norm=True, y=y)
                 normed.append((at, y.float().view(H, DV)))
                 outs.append(torch.zeros(1, H, DV, device=DEV))
             else:
-                o = torch.zeros(n, H, DV, device=DEV)
-                ops.scan(*args, nstate=st[1], mstate=st[2], out=o)
-                outs.append(o)
+                o, den = torch.zeros(n, H, DV, device=DEV), torch.zeros(n, H, device=DEV)
+                ops.scan(*args, mstate=mst, out=o, den=den)
+                outs.append(o / den[..., None])
             at += n
         got = torch.cat(outs)
         keep = [t for t in range(T) if t not in {a for a, _ in normed}]
@@ -242,8 +244,10 @@ def test_scans_of_unequal_portions_in_one_batch():
     g, k = torch.sigmoid(g + 2), torch.nn.functional.normalize(k, dim=-1)
     v, beta, kq = torch.randn(T, H, DV, generator=gen(4)), torch.rand(T, H, generator=gen(5)), (q * k).sum(-1)
     state, o = torch.zeros(3, H, DV, D, device=DEV), torch.full((T, H, DV), 4.0, device=DEV)
+    cross = torch.zeros(T, H, 2)
+    cross[1:, :, 0], cross[1:, :, 1] = (g[1:] * k[:-1] * k[1:]).sum(-1), (g[1:] * k[:-1] * q[1:]).sum(-1)
     ops.scan(ops.SCAN_DELTA, F32, 4, H, H, D, DV, *(t.to(DEV) for t in (q, k, v, beta, kq)), state, portions_of(counts, slots=slots),
-             g=g.to(DEV), out=o)
+             g=g.to(DEV), cross=cross.to(DEV), out=o)
     at = 0
     for n, s in zip(counts, slots):
         r = slice(at, at + n)
