@@ -174,6 +174,13 @@ struct ConvWindow {
   float4 x[3];         // inputs 3, 2 and 1 tokens ago
   float4 w[4];         // taps of the four channels: w[j] belongs to the input 3 - j tokens ago
   __device__ __forceinline__ void load_taps(const float* weights, int col, int taps) {
+    if (taps == 4) {
+      const float4* p = reinterpret_cast<const float4*>(weights + static_cast<int64_t>(col) * 4);
+      const float4 a = p[0], b = p[1], c = p[2], d = p[3];
+      w[0] = make_float4(a.x, b.x, c.x, d.x); w[1] = make_float4(a.y, b.y, c.y, d.y);
+      w[2] = make_float4(a.z, b.z, c.z, d.z); w[3] = make_float4(a.w, b.w, c.w, d.w);
+      return;
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int t = j - (4 - taps);
@@ -204,8 +211,9 @@ struct ConvWindow {
     y.z = fmaf(w[3].z, now.z, fmaf(w[2].z, x[2].z, fmaf(w[1].z, x[1].z, w[0].z * x[0].z)));
     y.w = fmaf(w[3].w, now.w, fmaf(w[2].w, x[2].w, fmaf(w[1].w, x[1].w, w[0].w * x[0].w)));
     x[0] = x[1]; x[1] = x[2]; x[2] = now;
-    y.x = y.x / (1.0f + expf(-y.x)); y.y = y.y / (1.0f + expf(-y.y));
-    y.z = y.z / (1.0f + expf(-y.z)); y.w = y.w / (1.0f + expf(-y.w));
+    // silu; the approximate division and exponential are good to a few units in the last place of fp32
+    y.x = __fdividef(y.x, 1.0f + __expf(-y.x)); y.y = __fdividef(y.y, 1.0f + __expf(-y.y));
+    y.z = __fdividef(y.z, 1.0f + __expf(-y.z)); y.w = __fdividef(y.w, 1.0f + __expf(-y.w));
     return y;
   }
   // one-token portions: the last taps - 1 inputs back into the slot
@@ -221,7 +229,7 @@ __device__ __forceinline__ float dot4(float4 a, float4 b) { return a.x * b.x + a
 __device__ __forceinline__ float4 scale4(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
 
 template <typename T, bool PARTS>
-__global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_rows_kernel(const mdb_delta_prep_args a, const int run) {
+__global__ void __launch_bounds__(kPrepWarps * 32, 4) delta_prep_rows_kernel(const mdb_delta_prep_args a, const int run) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31, c = lane * 4;
@@ -241,9 +249,26 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_rows_kernel(const 
       w0.load_taps(is_qk ? a.conv_q : a.conv_v, col, a.taps);
       if (is_qk) w1.load_taps(a.conv_k, col, a.taps);
     }
+    const float q_scale = 1.0f / sqrtf(static_cast<float>(a.dim));
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     int seq = -1, slot = -1;
+    // the next row's inputs are requested before this row's are used
+    float4 next0 = zero, next1 = zero;
+    int next_seq = a.row_seq[row0];
+    if (live) {
+      next0 = rows_at4_of<T, PARTS>(src, row0, col);
+      if (is_qk) next1 = rows_at4_of<T, PARTS>(a.k, row0, col);
+    }
     for (int64_t row = row0; row < row1; ++row) {
-      const int s = a.row_seq[row];
+      const int s = next_seq;
+      const float4 in0 = next0, in1 = next1;
+      if (row + 1 < row1) {
+        next_seq = a.row_seq[row + 1];
+        if (live) {
+          next0 = rows_at4_of<T, PARTS>(src, row + 1, col);
+          if (is_qk) next1 = rows_at4_of<T, PARTS>(a.k, row + 1, col);
+        }
+      }
       if (s != seq) {
         seq = s;
         slot = a.state_slot[s];
@@ -258,22 +283,27 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_rows_kernel(const 
         }
       }
       if (slot < 0) continue;
-      const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
       float4 y0 = zero, y1 = zero;
       if (live) {
-        y0 = w0.step(rows_at4_of<T, PARTS>(src, row, col));
-        if (is_qk) y1 = w1.step(rows_at4_of<T, PARTS>(a.k, row, col));
+        y0 = w0.step(in0);
+        if (is_qk) y1 = w1.step(in1);
         if (a.shift_state && a.taps > 1) {
           w0.save(a, slot, channel);
           if (is_qk) w1.save(a, slot, kc + col);
         }
       }
       if (is_qk) {
-        const float rq = (1.0f / sqrtf(warp_sum(dot4(y0, y0)) + 1e-6f)) * (1.0f / sqrtf(static_cast<float>(a.dim)));
-        const float rk = 1.0f / sqrtf(warp_sum(dot4(y1, y1)) + 1e-6f);
+        float qq = dot4(y0, y0), kk = dot4(y1, y1), qk = dot4(y0, y1);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+          qq += __shfl_xor_sync(0xffffffffu, qq, o);
+          kk += __shfl_xor_sync(0xffffffffu, kk, o);
+          qk += __shfl_xor_sync(0xffffffffu, qk, o);
+        }
+        const float rq = (1.0f / sqrtf(qq + 1e-6f)) * q_scale, rk = 1.0f / sqrtf(kk + 1e-6f);
         y0 = scale4(y0, rq);
         y1 = scale4(y1, rk);
-        const float kq = warp_sum(dot4(y0, y1));
+        const float kq = qk * rq * rk;
         const int64_t at = (row * a.kv_heads + unit) * a.dim_pad + c;
         if (c < a.dim_pad) {
           *reinterpret_cast<float4*>(a.q_out + at) = y0;
@@ -320,7 +350,7 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const mdb_delta_prep_ar
   for (int j = 0; j < a.taps - 1; ++j) st[static_cast<int64_t>(j) * a.channels] = act_from_f<T>(keep[j]);
 }
 
-// One warp per (row, head).  g = exp(-exp(A_log) * softplus(x + dt_bias)), laid out [row][head][dim_pad] (padding
+// A warp per (row, head).  g = exp(-exp(A_log) * softplus(x + dt_bias)), laid out [row][head][dim_pad] (padding
 // channels: 1), and, for the odd tokens of a portion, the cross products with the token before:
 // cross [row][head] = ((g k_prev) . k, (g k_prev) . q).  VEC: head rows of x start on 16-byte boundaries.
 template <bool VEC>
@@ -328,47 +358,48 @@ __global__ void __launch_bounds__(128) channel_decay_kernel(const mdb_decay_args
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
-  const int head = blockIdx.y * 4 + (threadIdx.x >> 5);
   const int64_t row = blockIdx.x;
-  if (head >= a.heads) return;
   const bool odd = ((static_cast<int>(row) - a.cu_q[a.row_seq[row]]) & 1) != 0;
-  const float* x = a.x + row * a.ldx + static_cast<int64_t>(head) * a.dim;
-  const float* bias = a.dt_bias + static_cast<int64_t>(head) * a.dim;
-  float* g = a.g + (row * a.heads + head) * a.dim_pad;
-  const int kvh = head / (a.heads / a.kv_heads);
-  const float* k = a.k + (row * a.kv_heads + kvh) * a.dim_pad;
-  const float* q = a.q + (row * a.kv_heads + kvh) * a.dim_pad;
-  const float* kp = k - static_cast<int64_t>(a.kv_heads) * a.dim_pad;      // read for odd tokens only
-  const float rate = -expf(a.a_log[head]);
-  float ck = 0.f, cq = 0.f;
-  for (int c = lane * 4; c < a.dim_pad; c += 128) {
-    float xv[4], bv[4], r[4];
-    if (VEC && c + 4 <= a.dim) {
-      const float4 x4 = *reinterpret_cast<const float4*>(x + c), b4 = *reinterpret_cast<const float4*>(bias + c);
-      xv[0] = x4.x; xv[1] = x4.y; xv[2] = x4.z; xv[3] = x4.w;
-      bv[0] = b4.x; bv[1] = b4.y; bv[2] = b4.z; bv[3] = b4.w;
-    } else {
+#pragma unroll 2
+  for (int head = blockIdx.y * 4 + (threadIdx.x >> 5); head < a.heads; head += gridDim.y * 4) {
+    const float* x = a.x + row * a.ldx + static_cast<int64_t>(head) * a.dim;
+    const float* bias = a.dt_bias + static_cast<int64_t>(head) * a.dim;
+    float* g = a.g + (row * a.heads + head) * a.dim_pad;
+    const int kvh = head / (a.heads / a.kv_heads);
+    const float* k = a.k + (row * a.kv_heads + kvh) * a.dim_pad;
+    const float* q = a.q + (row * a.kv_heads + kvh) * a.dim_pad;
+    const float* kp = k - static_cast<int64_t>(a.kv_heads) * a.dim_pad;      // read for odd tokens only
+    const float rate = -expf(a.a_log[head]);
+    float ck = 0.f, cq = 0.f;
+    for (int c = lane * 4; c < a.dim_pad; c += 128) {
+      float xv[4], bv[4], r[4];
+      if (VEC && c + 4 <= a.dim) {
+        const float4 x4 = *reinterpret_cast<const float4*>(x + c), b4 = *reinterpret_cast<const float4*>(bias + c);
+        xv[0] = x4.x; xv[1] = x4.y; xv[2] = x4.z; xv[3] = x4.w;
+        bv[0] = b4.x; bv[1] = b4.y; bv[2] = b4.z; bv[3] = b4.w;
+      } else {
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        xv[i] = c + i < a.dim ? x[c + i] : 0.f;
-        bv[i] = c + i < a.dim ? bias[c + i] : 0.f;
+        for (int i = 0; i < 4; ++i) {
+          xv[i] = c + i < a.dim ? x[c + i] : 0.f;
+          bv[i] = c + i < a.dim ? bias[c + i] : 0.f;
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) r[i] = c + i < a.dim ? expf(rate * softplus_f(xv[i] + bv[i])) : 1.f;
+      *reinterpret_cast<float4*>(g + c) = make_float4(r[0], r[1], r[2], r[3]);
+      if (odd) {
+        const float4 k0 = *reinterpret_cast<const float4*>(kp + c), k1 = *reinterpret_cast<const float4*>(k + c);
+        const float4 q1 = *reinterpret_cast<const float4*>(q + c);
+        const float e0 = r[0] * k0.x, e1 = r[1] * k0.y, e2 = r[2] * k0.z, e3 = r[3] * k0.w;
+        ck += e0 * k1.x + e1 * k1.y + e2 * k1.z + e3 * k1.w;
+        cq += e0 * q1.x + e1 * q1.y + e2 * q1.z + e3 * q1.w;
       }
     }
-#pragma unroll
-    for (int i = 0; i < 4; ++i) r[i] = c + i < a.dim ? expf(rate * softplus_f(xv[i] + bv[i])) : 1.f;
-    *reinterpret_cast<float4*>(g + c) = make_float4(r[0], r[1], r[2], r[3]);
     if (odd) {
-      const float4 k0 = *reinterpret_cast<const float4*>(kp + c), k1 = *reinterpret_cast<const float4*>(k + c);
-      const float4 q1 = *reinterpret_cast<const float4*>(q + c);
-      const float e0 = r[0] * k0.x, e1 = r[1] * k0.y, e2 = r[2] * k0.z, e3 = r[3] * k0.w;
-      ck += e0 * k1.x + e1 * k1.y + e2 * k1.z + e3 * k1.w;
-      cq += e0 * q1.x + e1 * q1.y + e2 * q1.z + e3 * q1.w;
+      ck = warp_sum(ck);
+      cq = warp_sum(cq);
+      if (lane == 0) *reinterpret_cast<float2*>(a.cross + 2 * (row * a.heads + head)) = make_float2(ck, cq);
     }
-  }
-  if (odd) {
-    ck = warp_sum(ck);
-    cq = warp_sum(cq);
-    if (lane == 0) *reinterpret_cast<float2*>(a.cross + 2 * (row * a.heads + head)) = make_float2(ck, cq);
   }
 }
 
@@ -955,10 +986,11 @@ int mdb_delta_prep(const mdb_delta_prep_args* args, mdb_stream_t stream) {
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   int rc;
   if (a.dim % 4 == 0 && a.vdim % 4 == 0 && a.dim <= 128 && a.dim_pad <= 128 && a.taps <= 4 && rows_ok(a.q) && rows_ok(a.k) && rows_ok(a.v) &&
-      a.conv_slot_stride % 4 == 0 && mdb_aligned16(a.v_out) && (a.q.parts != nullptr) == (a.k.parts != nullptr) &&
+      a.conv_slot_stride % 4 == 0 && mdb_aligned16(a.v_out) && mdb_aligned16(a.conv_q) && mdb_aligned16(a.conv_k) &&
+      mdb_aligned16(a.conv_v) && (a.q.parts != nullptr) == (a.k.parts != nullptr) &&
       (a.q.parts != nullptr) == (a.v.parts != nullptr) && (a.copy_cols == 0 || (a.q.parts != nullptr) == (a.copy.parts != nullptr)) &&
       (a.dtype == MDB_BF16 || a.q.parts == nullptr)) {
-    const int run = a.m >= 1024 ? 8 : 1;
+    const int run = a.m >= 4096 ? 32 : (a.m >= 1024 ? 8 : 1);      // rows a warp walks
     const int units = a.kv_heads + a.heads * ((a.vdim + 127) / 128) + 1 + (a.copy_cols + 127) / 128;
     const dim3 grid((a.m + run - 1) / run, (units + kPrepWarps - 1) / kPrepWarps);
     const bool parts = a.q.parts != nullptr;
@@ -987,7 +1019,7 @@ int mdb_channel_decay(const mdb_decay_args* args, mdb_stream_t stream) {
                   a.ldx >= static_cast<int64_t>(a.heads) * a.dim,
               MDB_ERR_ARG);
   MDB_REQUIRE(a.dim_pad % 4 == 0 && mdb_aligned16(a.g) && mdb_aligned16(a.q) && mdb_aligned16(a.k), MDB_ERR_ALIGN);
-  const dim3 grid(a.m, (a.heads + 3) / 4);
+  const dim3 grid(a.m, a.m >= 1024 ? 1 : (a.heads + 3) / 4);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (a.dim % 4 == 0 && a.ldx % 4 == 0 && mdb_aligned16(a.x) && mdb_aligned16(a.dt_bias))
     return mdb_launch(channel_decay_kernel<true>, grid, dim3(128), 0, st, a);

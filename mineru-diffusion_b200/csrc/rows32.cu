@@ -161,7 +161,7 @@ struct RmsSegments {
   mdb_rms_segment s[MDB_MAX_RMS_SEGMENTS];
 };
 constexpr int kRmsRowsThreads = 128;
-template <typename T>
+template <typename T, bool PARTS>
 __global__ void __launch_bounds__(kRmsRowsThreads) rms_rows_kernel(const RmsSegments segs) {
   pdl_launch_dependents();
   pdl_wait();
@@ -178,53 +178,86 @@ __global__ void __launch_bounds__(kRmsRowsThreads) rms_rows_kernel(const RmsSegm
     }
     out_row = slot;
   }
+  T* out = static_cast<T*>(s.out) + out_row * s.ld_out;
+  // columns n .. n_pad of the projection are zeros; the first kKeep pieces of the row stay in registers
+  constexpr int kKeep = 4;
+  float4 v[kKeep];
   float ss = 0.f;
-  for (int c = threadIdx.x * 4; c < s.n_pad; c += kRmsRowsThreads * 4) {
-    const float4 x = rows_at4<T>(s.src, row, c);        // columns n .. n_pad of the projection are zeros
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int c = (threadIdx.x + i * kRmsRowsThreads) * 4;
+    v[i] = c < s.n_pad ? rows_at4_of<T, PARTS>(s.src, row, c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+  for (int c = (threadIdx.x + kKeep * kRmsRowsThreads) * 4; c < s.n_pad; c += kRmsRowsThreads * 4) {
+    const float4 x = rows_at4_of<T, PARTS>(s.src, row, c);
     ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
   }
   const float rstd = 1.0f / sqrtf(cta_sum(ss, red) / static_cast<float>(s.n) + s.eps);
-  T* out = static_cast<T*>(s.out) + out_row * s.ld_out;
-  for (int c = threadIdx.x * 4; c < s.n_pad; c += kRmsRowsThreads * 4) {
-    const float4 x = rows_at4<T>(s.src, row, c);
+  auto put = [&](int c, float4 x) {
     const float4 w = *reinterpret_cast<const float4*>(s.weight + c);
     act_store4(out + c, make_float4(x.x * rstd * w.x, x.y * rstd * w.y, x.z * rstd * w.z, x.w * rstd * w.w));
+  };
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int c = (threadIdx.x + i * kRmsRowsThreads) * 4;
+    if (c < s.n_pad) put(c, v[i]);
   }
+  for (int c = (threadIdx.x + kKeep * kRmsRowsThreads) * 4; c < s.n_pad; c += kRmsRowsThreads * 4)
+    put(c, rows_at4_of<T, PARTS>(s.src, row, c));
 }
 
-// Behind a recurrence: one warp per (row, head).  y = o' / rms(o') * weight * sigmoid(gate), o' = o / den where there is
-// a den.  VEC: heads in multiples of four, everything 16-byte aligned.
-template <typename T, bool VEC>
+// Behind a recurrence: a warp per (row, head).  y = o' / rms(o') * weight * sigmoid(gate), o' = o / den where there is
+// a den.  VEC: heads in multiples of four, everything 16-byte aligned; up to 256 values stay in registers between the
+// two passes, and the gate is requested with them.
+template <typename T, bool VEC, bool PARTS>
 __global__ void __launch_bounds__(128) gated_norm_kernel(const mdb_gated_norm_args a) {
   pdl_launch_dependents();
   pdl_wait();
   const int64_t row = blockIdx.x;
-  const int head = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (head >= a.heads) return;
-  const float* o = a.o + (row * a.heads + head) * a.vdim;
-  const float inv = a.den != nullptr ? 1.0f / a.den[row * a.heads + head] : 1.0f;
-  const float* w = a.weight + static_cast<int64_t>(head) * a.weight_head_stride;
-  T* y = static_cast<T*>(a.y) + row * a.ldy + static_cast<int64_t>(head) * a.vdim;
-  float ss = 0.f;
-  if (VEC) {
-    for (int c = lane * 4; c < a.vdim; c += 128) {
-      const float4 v = *reinterpret_cast<const float4*>(o + c);
-      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  const int lane = threadIdx.x & 31;
+  constexpr int kKeep = 2;
+#pragma unroll 2
+  for (int head = blockIdx.y * 4 + (threadIdx.x >> 5); head < a.heads; head += gridDim.y * 4) {
+    const float* o = a.o + (row * a.heads + head) * a.vdim;
+    const float den = a.den != nullptr ? a.den[row * a.heads + head] : 1.0f;
+    const float* w = a.weight + static_cast<int64_t>(head) * a.weight_head_stride;
+    T* y = static_cast<T*>(a.y) + row * a.ldy + static_cast<int64_t>(head) * a.vdim;
+    float ss = 0.f;
+    if (VEC) {
+      float4 v[kKeep], g[kKeep];
+#pragma unroll
+      for (int i = 0; i < kKeep; ++i) {
+        const int c = lane * 4 + 128 * i;
+        v[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < a.vdim) {
+          v[i] = *reinterpret_cast<const float4*>(o + c);
+          g[i] = rows_at4_of<T, PARTS>(a.gate, row, head * a.vdim + c);
+        }
+        ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+      }
+      for (int c = lane * 4 + 128 * kKeep; c < a.vdim; c += 128) {
+        const float4 x = *reinterpret_cast<const float4*>(o + c);
+        ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+      }
+      const float inv = 1.0f / den, rstd = inv / sqrtf(warp_sum(ss) * inv * inv / static_cast<float>(a.vdim) + a.eps);
+      auto put = [&](int c, float4 x, float4 gv) {
+        const float4 wv = *reinterpret_cast<const float4*>(w + c);
+        act_store4(y + c, make_float4(x.x * rstd * wv.x * sigmoid_f(gv.x), x.y * rstd * wv.y * sigmoid_f(gv.y),
+                                      x.z * rstd * wv.z * sigmoid_f(gv.z), x.w * rstd * wv.w * sigmoid_f(gv.w)));
+      };
+#pragma unroll
+      for (int i = 0; i < kKeep; ++i)
+        if (lane * 4 + 128 * i < a.vdim) put(lane * 4 + 128 * i, v[i], g[i]);
+      for (int c = lane * 4 + 128 * kKeep; c < a.vdim; c += 128)
+        put(c, *reinterpret_cast<const float4*>(o + c), rows_at4_of<T, PARTS>(a.gate, row, head * a.vdim + c));
+    } else {
+      for (int c = lane; c < a.vdim; c += 32) ss += o[c] * o[c];
+      const float inv = 1.0f / den, rstd = inv / sqrtf(warp_sum(ss) * inv * inv / static_cast<float>(a.vdim) + a.eps);
+      for (int c = lane; c < a.vdim; c += 32)
+        y[c] = act_from_f<T>(o[c] * rstd * w[c] * sigmoid_f(rows_at<T>(a.gate, row, head * a.vdim + c)));
     }
-  } else {
-    for (int c = lane; c < a.vdim; c += 32) ss += o[c] * o[c];
-  }
-  const float rstd = inv / sqrtf(warp_sum(ss) * inv * inv / static_cast<float>(a.vdim) + a.eps);
-  if (VEC) {
-    for (int c = lane * 4; c < a.vdim; c += 128) {
-      const float4 v = *reinterpret_cast<const float4*>(o + c), wv = *reinterpret_cast<const float4*>(w + c);
-      const float4 g = rows_at4<T>(a.gate, row, head * a.vdim + c);
-      act_store4(y + c, make_float4(v.x * rstd * wv.x * sigmoid_f(g.x), v.y * rstd * wv.y * sigmoid_f(g.y),
-                                    v.z * rstd * wv.z * sigmoid_f(g.z), v.w * rstd * wv.w * sigmoid_f(g.w)));
-    }
-  } else {
-    for (int c = lane; c < a.vdim; c += 32)
-      y[c] = act_from_f<T>(o[c] * rstd * w[c] * sigmoid_f(rows_at<T>(a.gate, row, head * a.vdim + c)));
   }
 }
 
@@ -342,8 +375,12 @@ int mdb_rms_rows(int dtype, const mdb_rms_segment* segments, int nseg, int m, md
     segs.s[i] = s;
   }
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (dtype == MDB_F32) return mdb_launch(rms_rows_kernel<float>, dim3(m, nseg), dim3(kRmsRowsThreads), 0, st, segs);
-  return mdb_launch(rms_rows_kernel<bf16>, dim3(m, nseg), dim3(kRmsRowsThreads), 0, st, segs);
+  const bool parts = segs.s[0].src.parts != nullptr;
+  for (int i = 1; i < nseg; ++i) MDB_REQUIRE((segs.s[i].src.parts != nullptr) == parts, MDB_ERR_UNSUPPORTED);
+  const dim3 grid(m, nseg), block(kRmsRowsThreads);
+  if (dtype == MDB_F32)
+    return parts ? mdb_launch(rms_rows_kernel<float, true>, grid, block, 0, st, segs) : mdb_launch(rms_rows_kernel<float, false>, grid, block, 0, st, segs);
+  return parts ? mdb_launch(rms_rows_kernel<bf16, true>, grid, block, 0, st, segs) : mdb_launch(rms_rows_kernel<bf16, false>, grid, block, 0, st, segs);
 }
 
 int mdb_gated_norm(const mdb_gated_norm_args* args, mdb_stream_t stream) {
@@ -352,15 +389,18 @@ int mdb_gated_norm(const mdb_gated_norm_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(a.m >= 0 && a.heads > 0 && a.vdim > 0, MDB_ERR_ARG);
   if (a.m == 0) return MDB_OK;
   MDB_REQUIRE(a.o && a.weight && a.y && rows_present(a.gate) && a.ldy >= static_cast<int64_t>(a.heads) * a.vdim, MDB_ERR_ARG);
-  const dim3 grid(a.m, (a.heads + 3) / 4);
+  // many rows: a CTA takes all heads of its row
+  const dim3 grid(a.m, a.m >= 1024 ? 1 : (a.heads + 3) / 4);
   const bool vec = a.vdim % 4 == 0 && rows_ok(a.gate) && a.ldy % 4 == 0 && mdb_aligned16(a.o) && mdb_aligned16(a.y) &&
                    mdb_aligned16(a.weight) && a.weight_head_stride % 4 == 0;
+  const bool parts = a.gate.parts != nullptr;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (a.dtype == MDB_F32)
-    return vec ? mdb_launch(gated_norm_kernel<float, true>, grid, dim3(128), 0, st, a)
-               : mdb_launch(gated_norm_kernel<float, false>, grid, dim3(128), 0, st, a);
-  return vec ? mdb_launch(gated_norm_kernel<bf16, true>, grid, dim3(128), 0, st, a)
-             : mdb_launch(gated_norm_kernel<bf16, false>, grid, dim3(128), 0, st, a);
+    return vec && !parts ? mdb_launch(gated_norm_kernel<float, true, false>, grid, dim3(128), 0, st, a)
+                         : mdb_launch(gated_norm_kernel<float, false, true>, grid, dim3(128), 0, st, a);
+  if (!vec) return mdb_launch(gated_norm_kernel<bf16, false, true>, grid, dim3(128), 0, st, a);
+  return parts ? mdb_launch(gated_norm_kernel<bf16, true, true>, grid, dim3(128), 0, st, a)
+               : mdb_launch(gated_norm_kernel<bf16, true, false>, grid, dim3(128), 0, st, a);
 }
 
 int mdb_gather_latents(int dtype, const void* cache, const int32_t* block_table, int table_stride, int num_pages,
