@@ -422,7 +422,7 @@ typedef struct {
 } mdb_gated_norm_args;
 int mdb_gated_norm(const mdb_gated_norm_args* args, mdb_stream_t stream);
 
-/* Key channels of a recurrent head as the state stores them (a multiple of 32; 0: not supported), and the number of
+/* Key channels of a recurrent head as the state stores them (a multiple of 64; 0: not supported), and the number of
  * copies of the mLSTM maximum a head keeps. */
 int mdb_scan_dim_pad(int dim);
 int mdb_scan_blocks(int vdim);

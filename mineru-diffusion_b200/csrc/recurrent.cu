@@ -1,12 +1,12 @@
 // Recurrent mixers with a matrix state per head: the gated delta rule with one decay per key channel, and the mLSTM
-// matrix memory.  One scan kernel serves prompts, portions of prompts and decoding; the state lives in fp32 in a slot
+// matrix memory.  A scan kernel each for prompts and their portions, one for single tokens; the state lives in fp32 in a slot
 // per sequence and every product of the recurrence is an fp32 FMA (packed two at a time, fma.rn.f32x2).
 //
-// State layout: [slot][head][value column][key channel padded to a multiple of 32], so a value column is contiguous.
+// State layout: [slot][head][value column][key channel padded to a multiple of 64], so a value column is contiguous.
 // The columns of a head are independent of one another (the delta rule's correction of a column only needs that
-// column), so a CTA owns a block of columns: eight lanes share a column, each holding every eighth float4 of it in
-// registers, CPT columns per thread.  k, q and the decays of a block of tokens come through a double-buffered
-// shared-memory stage (cp.async).
+// column), so a CTA owns a block of columns: eight lanes (mLSTM prompts: sixteen) share a column, each holding every
+// eighth (sixteenth) float4 of it in registers, CPT columns per thread.  k, q and the decays of a block of tokens come
+// through a double-buffered shared-memory stage (cp.async).
 //
 // The read-out of the delta rule is rewritten so that both products with the old state share one reduction,
 //   a = (g S)^T k,  b = (g S)^T q,  u = beta (v - a),  o = b + (k . q) u,  S <- g S + k u^T,
@@ -42,8 +42,10 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
   return r;
 }
-__device__ __forceinline__ void lds2(uint32_t addr, f32x2& a, f32x2& b) {
-  asm volatile("ld.shared.v2.u64 {%0, %1}, [%2];" : "=l"(a), "=l"(b) : "r"(addr));
+__device__ __forceinline__ void lds2(const float* p, f32x2& a, f32x2& b) {      // four floats of shared memory
+  const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(p);
+  a = v.x;
+  b = v.y;
 }
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
@@ -453,7 +455,7 @@ __global__ void __launch_bounds__(256) mlstm_prep_kernel(const mdb_mlstm_prep_ar
 // ---------------------------------------------------------------------------
 enum { kScanDelta = MDB_SCAN_DELTA, kScanMlstm = MDB_SCAN_MLSTM };
 constexpr int kScanFusedThreads = 512, kScanFusedMaxDim = 256;
-constexpr int kScanBlockCols = 32;       // columns of a CTA of the prompt form; granularity of the copies of the mLSTM maximum
+constexpr int kScanBlockCols = 16;       // granularity of the copies of the mLSTM maximum; narrowest block of a prompt CTA
 constexpr int kScanTokens = 16;          // tokens of a stage of the prompt form (even)
 
 // floats of one stage: k, q (and the decays) of tb tokens, their values for `cols` columns, four scalars per token
@@ -491,68 +493,63 @@ struct ScanState {
   }
 };
 
-// Prompt form: portions of any length, kScanBlockCols columns of one head per CTA, two tokens at a time.
-template <int MODE, int NCH, int CPT>
-__global__ void __launch_bounds__(kScanBlockCols / CPT * 8) scan_kernel(const mdb_scan_args a) {
-  constexpr int DP = NCH * 32, TB = kScanTokens, COLS = kScanBlockCols, THREADS = COLS / CPT * 8;
-  constexpr int VEC = MODE == kScanDelta ? 3 : 2;
-  constexpr int OFF_V = TB * VEC * DP, OFF_S = OFF_V + TB * COLS, STAGE = scan_stage_floats(MODE, DP, TB, COLS);
-  constexpr bool KEEP_K = NCH <= 8;      // the keys of a pair stay in registers between the two passes
-  extern __shared__ __align__(16) float scan_smem[];
-  __shared__ float4 sh_gate[TB];         // mLSTM: forget factor, input factor, exp(-m) per token of the stage
-  pdl_launch_dependents();
-  pdl_wait();
-  const int seq = blockIdx.z, head = blockIdx.y;
-  const int l8 = threadIdx.x & 7, cg = threadIdx.x >> 3;
-  const int col0 = blockIdx.x * COLS, mycol = col0 + cg * CPT;
-  const int slot = a.state_slot[seq];
-  if (slot < 0) return;
-  if (slot >= a.num_slots) {
+// What a CTA of the prompt form works on: COLS columns of one head of one sequence.
+struct ScanJob {
+  bool live, fresh;
+  int head, kvh, slot, t_begin, t_end, col0, columns;
+  float* state;       // the head's columns
+};
+template <int MODE, int DP, int COLS>
+__device__ __forceinline__ ScanJob scan_job(const mdb_scan_args& a) {
+  ScanJob w = {};
+  const int seq = blockIdx.z;
+  w.head = blockIdx.y;
+  w.col0 = blockIdx.x * COLS;
+  w.slot = a.state_slot[seq];
+  if (w.slot < 0) return w;
+  if (w.slot >= a.num_slots) {
     if (threadIdx.x == 0) report_status(MDB_STATUS_BAD_SLOT);
-    return;
+    return w;
   }
-  const int t_begin = a.cu_q[seq], t_end = a.cu_q[seq + 1];
-  if (t_end <= t_begin) return;
-  const bool fresh = a.start[seq] == 0;
-  const int kvh = head / (a.heads / a.kv_heads);
-  const int columns = a.vdim + (MODE == kScanMlstm ? 1 : 0);
-  float* state = a.state + slot * a.state_slot_stride + static_cast<int64_t>(head) * columns * DP;
-  ScanState<NCH, CPT> S;
-  S.load(state, mycol, columns, l8, fresh);
-  // mLSTM: every block of 32 columns keeps a copy of the running maximum, so that no CTA reads what another writes
-  float run_max = 0.f;
-  float* mstate = nullptr;
-  if (MODE == kScanMlstm) {
-    mstate = a.mstate + (static_cast<int64_t>(slot) * a.heads + head) * ((columns + kScanBlockCols - 1) / kScanBlockCols) + blockIdx.x;
-    if (!fresh) run_max = *mstate;
-  }
+  w.t_begin = a.cu_q[seq];
+  w.t_end = a.cu_q[seq + 1];
+  w.live = w.t_end > w.t_begin;
+  w.fresh = a.start[seq] == 0;
+  w.kvh = w.head / (a.heads / a.kv_heads);
+  w.columns = a.vdim + (MODE == kScanMlstm ? 1 : 0);
+  w.state = a.state + w.slot * a.state_slot_stride + static_cast<int64_t>(w.head) * w.columns * DP;
+  return w;
+}
 
-  const uint32_t smem0 = smem_u32(scan_smem);
-  auto stage = [&](int t0, int buf) {
-    const int n = min(TB, t_end - t0);
-    const uint32_t base = smem0 + buf * STAGE * 4;
-    float* st = scan_smem + buf * STAGE;
-    for (int i = threadIdx.x; i < n * (DP / 4); i += THREADS) {
+template <int MODE, int DP, int COLS>
+struct ScanStage {
+  static constexpr int TB = kScanTokens, VEC = MODE == kScanDelta ? 3 : 2;
+  static constexpr int OFF_V = TB * VEC * DP, OFF_S = OFF_V + TB * COLS, FLOATS = scan_stage_floats(MODE, DP, TB, COLS);
+  // requests the operands of tokens [t0, t0 + TB) into the buffer at st
+  static __device__ __forceinline__ void fill(const mdb_scan_args& a, const ScanJob& w, int t0, float* st) {
+    const int n = min(TB, w.t_end - t0), step = blockDim.x;
+    const uint32_t base = smem_u32(st);
+    for (int i = threadIdx.x; i < n * (DP / 4); i += step) {
       const int t = i / (DP / 4), c = i % (DP / 4);
-      const int64_t krow = (static_cast<int64_t>(t0 + t) * a.kv_heads + kvh) * DP + c * 4;
+      const int64_t krow = (static_cast<int64_t>(t0 + t) * a.kv_heads + w.kvh) * DP + c * 4;
       cp_async16(base + (t * DP + c * 4) * 4, a.k + krow);
       cp_async16(base + ((TB + t) * DP + c * 4) * 4, a.q + krow);
       if (MODE == kScanDelta)
-        cp_async16(base + ((2 * TB + t) * DP + c * 4) * 4, a.g + (static_cast<int64_t>(t0 + t) * a.heads + head) * DP + c * 4);
+        cp_async16(base + ((2 * TB + t) * DP + c * 4) * 4, a.g + (static_cast<int64_t>(t0 + t) * a.heads + w.head) * DP + c * 4);
     }
-    for (int i = threadIdx.x; i < n * COLS; i += THREADS) {
+    for (int i = threadIdx.x; i < n * COLS; i += step) {
       const int t = i / COLS, c = i % COLS;
-      if (col0 + c < a.vdim)
-        cp_async4(base + (OFF_V + t * COLS + c) * 4, a.v + (static_cast<int64_t>(t0 + t) * a.heads + head) * a.vdim + col0 + c);
+      if (w.col0 + c < a.vdim)
+        cp_async4(base + (OFF_V + t * COLS + c) * 4, a.v + (static_cast<int64_t>(t0 + t) * a.heads + w.head) * a.vdim + w.col0 + c);
       else
-        st[OFF_V + t * COLS + c] = MODE == kScanMlstm && col0 + c == a.vdim ? 1.f : 0.f;
+        st[OFF_V + t * COLS + c] = MODE == kScanMlstm && w.col0 + c == a.vdim ? 1.f : 0.f;
     }
-    for (int i = threadIdx.x; i < n; i += THREADS) {
-      const int64_t th = static_cast<int64_t>(t0 + i) * a.heads + head;
+    for (int i = threadIdx.x; i < n; i += step) {
+      const int64_t th = static_cast<int64_t>(t0 + i) * a.heads + w.head;
       const uint32_t dst = base + (OFF_S + 4 * i) * 4;
       cp_async4(dst, a.s0 + th);
       if (MODE == kScanDelta) {
-        cp_async4(dst + 4, a.s1 + static_cast<int64_t>(t0 + i) * a.kv_heads + kvh);
+        cp_async4(dst + 4, a.s1 + static_cast<int64_t>(t0 + i) * a.kv_heads + w.kvh);
         if (i & 1) {
           cp_async4(dst + 8, a.cross + 2 * th);
           cp_async4(dst + 12, a.cross + 2 * th + 1);
@@ -563,184 +560,260 @@ __global__ void __launch_bounds__(kScanBlockCols / CPT * 8) scan_kernel(const md
     }
     if (n & 1) {
       // the missing second token of the last pair changes nothing: no key, no query, no decay
-      for (int i = threadIdx.x; i < DP; i += THREADS) {
+      for (int i = threadIdx.x; i < DP; i += step) {
         st[n * DP + i] = st[(TB + n) * DP + i] = 0.f;
         if (MODE == kScanDelta) st[(2 * TB + n) * DP + i] = 1.f;
       }
-      for (int i = threadIdx.x; i < COLS; i += THREADS) st[OFF_V + n * COLS + i] = 0.f;
+      for (int i = threadIdx.x; i < COLS; i += step) st[OFF_V + n * COLS + i] = 0.f;
       if (threadIdx.x < 4) st[OFF_S + 4 * n + threadIdx.x] = 0.f;
     }
     cp_async_commit();
-  };
-
-  stage(t_begin, 0);
-  int buf = 0;
-  for (int t0 = t_begin; t0 < t_end; t0 += TB, buf ^= 1) {
-    const int n = min(TB, t_end - t0);
-    if (t0 + TB < t_end) {
-      stage(t0 + TB, buf ^ 1);
+  }
+  // on return the tokens from t0 on are in buffer buf for the whole CTA, and the next ones have been requested
+  static __device__ __forceinline__ void turn(const mdb_scan_args& a, const ScanJob& w, int t0, float* smem, int buf) {
+    if (t0 + TB < w.t_end) {
+      fill(a, w, t0 + TB, smem + (buf ^ 1) * FLOATS);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
     }
     __syncthreads();
-    const float* st = scan_smem + buf * STAGE;
-    const uint32_t st_addr = smem0 + buf * STAGE * 4;
-    if (MODE == kScanMlstm) {
-      // m_t = max(f_t + m_(t-1), i_t) over the stage as a scan of the maps x -> max(x + F, I)
-      if (threadIdx.x < 32) {
-        const int l = threadIdx.x;
-        const float li = l < n ? st[OFF_S + 4 * l] : -INFINITY, lf = l < n ? st[OFF_S + 4 * l + 1] : 0.f;
-        float F = lf, I = li;
-#pragma unroll
-        for (int o = 1; o < TB; o <<= 1) {
-          const float Fp = __shfl_up_sync(0xffffffffu, F, o), Ip = __shfl_up_sync(0xffffffffu, I, o);
-          if (l >= o) { I = fmaxf(Ip + F, I); F += Fp; }
-        }
-        const float m = fmaxf(F + run_max, I);
-        float mp = __shfl_up_sync(0xffffffffu, m, 1);
-        if (l == 0) mp = run_max;
-        if (l < n) sh_gate[l] = make_float4(expf(lf + mp - m), expf(li - m), expf(-m), 0.f);
-        else if (l < TB) sh_gate[l] = make_float4(1.f, 0.f, 0.f, 0.f);
-        run_max = __shfl_sync(0xffffffffu, m, n - 1);
-      }
-      __syncthreads();
-    }
+  }
+};
+
+// Delta rule, prompt form: portions of any length, two tokens at a time, eight lanes per column.
+template <int NCH, int CPT, int COLS>
+__global__ void __launch_bounds__(COLS / CPT * 8) delta_scan_kernel(const mdb_scan_args a) {
+  constexpr int DP = NCH * 32;
+  using Stage = ScanStage<kScanDelta, DP, COLS>;
+  constexpr int TB = Stage::TB;
+  constexpr bool KEEP_K = NCH <= 8;      // the keys of a pair stay in registers between the two passes
+  extern __shared__ __align__(16) float scan_smem[];
+  pdl_launch_dependents();
+  pdl_wait();
+  const ScanJob w = scan_job<kScanDelta, DP, COLS>(a);
+  if (!w.live) return;
+  const int l8 = threadIdx.x & 7, cg = threadIdx.x >> 3, mycol = w.col0 + cg * CPT;
+  ScanState<NCH, CPT> S;
+  S.load(w.state, mycol, w.columns, l8, w.fresh);
+  Stage::fill(a, w, w.t_begin, scan_smem);
+  int buf = 0;
+  for (int t0 = w.t_begin; t0 < w.t_end; t0 += TB, buf ^= 1) {
+    const int n = min(TB, w.t_end - t0);
+    Stage::turn(a, w, t0, scan_smem, buf);
+    const float* st = scan_smem + buf * Stage::FLOATS;
     for (int t = 0; t < n; t += 2) {
-      const uint32_t ka = st_addr + (t * DP + l8 * 4) * 4, qa = ka + TB * DP * 4;
-      float o1[CPT], o2[CPT];
-      if (MODE == kScanDelta) {
-        const uint32_t ga = ka + 2 * TB * DP * 4;
-        f32x2 K1[KEEP_K ? NCH * 2 : 1], K2[KEEP_K ? NCH * 2 : 1];
-        f32x2 A1[CPT], B1[CPT], A2[CPT], B2[CPT];
+      const float* ka = st + t * DP + l8 * 4;
+      const float* qa = ka + TB * DP;
+      const float* ga = ka + 2 * TB * DP;
+      f32x2 K1[KEEP_K ? NCH * 2 : 1], K2[KEEP_K ? NCH * 2 : 1];
+      f32x2 A1[CPT], B1[CPT], A2[CPT], B2[CPT];
 #pragma unroll
-        for (int i = 0; i < CPT; ++i) A1[i] = B1[i] = A2[i] = B2[i] = 0ull;
+      for (int i = 0; i < CPT; ++i) A1[i] = B1[i] = A2[i] = B2[i] = 0ull;
 #pragma unroll
-        for (int c = 0; c < NCH; ++c) {
-          f32x2 k1[2], q1[2], g1[2], k2[2], q2[2], g2[2];
-          lds2(ka + c * 128, k1[0], k1[1]);
-          lds2(qa + c * 128, q1[0], q1[1]);
-          lds2(ga + c * 128, g1[0], g1[1]);
-          lds2(ka + DP * 4 + c * 128, k2[0], k2[1]);
-          lds2(qa + DP * 4 + c * 128, q2[0], q2[1]);
-          lds2(ga + DP * 4 + c * 128, g2[0], g2[1]);
+      for (int c = 0; c < NCH; ++c) {
+        f32x2 k1[2], q1[2], g1[2], k2[2], q2[2], g2[2];
+        lds2(ka + c * 32, k1[0], k1[1]);
+        lds2(qa + c * 32, q1[0], q1[1]);
+        lds2(ga + c * 32, g1[0], g1[1]);
+        lds2(ka + DP + c * 32, k2[0], k2[1]);
+        lds2(qa + DP + c * 32, q2[0], q2[1]);
+        lds2(ga + DP + c * 32, g2[0], g2[1]);
 #pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            if (KEEP_K) {
-              K1[KEEP_K ? 2 * c + e : 0] = mul2(g2[e], k1[e]);
-              K2[KEEP_K ? 2 * c + e : 0] = k2[e];
-            }
-#pragma unroll
-            for (int i = 0; i < CPT; ++i) {
-              f32x2 s = mul2(S.v[i][2 * c + e], g1[e]);
-              A1[i] = fma2(s, k1[e], A1[i]);
-              B1[i] = fma2(s, q1[e], B1[i]);
-              s = mul2(s, g2[e]);
-              A2[i] = fma2(s, k2[e], A2[i]);
-              B2[i] = fma2(s, q2[e], B2[i]);
-              S.v[i][2 * c + e] = s;
-            }
-          }
-        }
-        float r[4 * CPT];
-#pragma unroll
-        for (int i = 0; i < CPT; ++i) {
-          const float2 w = unpack2(A1[i]), x = unpack2(B1[i]), y = unpack2(A2[i]), z = unpack2(B2[i]);
-          r[4 * i] = w.x + w.y; r[4 * i + 1] = x.x + x.y; r[4 * i + 2] = y.x + y.y; r[4 * i + 3] = z.x + z.y;
-        }
-#pragma unroll
-        for (int o = 4; o > 0; o >>= 1)
-#pragma unroll
-          for (int i = 0; i < 4 * CPT; ++i) r[i] += __shfl_xor_sync(0xffffffffu, r[i], o);
-        const float4 s1 = *reinterpret_cast<const float4*>(st + OFF_S + 4 * t), s2 = *reinterpret_cast<const float4*>(st + OFF_S + 4 * t + 4);
-#pragma unroll
-        for (int i = 0; i < CPT; ++i) {
-          const float v1 = st[OFF_V + t * COLS + cg * CPT + i], v2 = st[OFF_V + (t + 1) * COLS + cg * CPT + i];
-          const float u1 = s1.x * (v1 - r[4 * i]);
-          const float u2 = s2.x * (v2 - fmaf(s2.z, u1, r[4 * i + 2]));
-          o1[i] = fmaf(s1.y, u1, r[4 * i + 1]);
-          o2[i] = fmaf(s2.y, u2, fmaf(s2.w, u1, r[4 * i + 3]));
-          const f32x2 p1 = pack2(u1, u1), p2 = pack2(u2, u2);
+        for (int e = 0; e < 2; ++e) {
           if (KEEP_K) {
-#pragma unroll
-            for (int c = 0; c < NCH * 2; ++c) S.v[i][c] = fma2(K2[KEEP_K ? c : 0], p2, fma2(K1[KEEP_K ? c : 0], p1, S.v[i][c]));
-          } else {
-#pragma unroll
-            for (int c = 0; c < NCH; ++c) {
-              f32x2 k1[2], k2[2], g2[2];
-              lds2(ka + c * 128, k1[0], k1[1]);
-              lds2(ka + DP * 4 + c * 128, k2[0], k2[1]);
-              lds2(ga + DP * 4 + c * 128, g2[0], g2[1]);
-#pragma unroll
-              for (int e = 0; e < 2; ++e)
-                S.v[i][2 * c + e] = fma2(k2[e], p2, fma2(mul2(g2[e], k1[e]), p1, S.v[i][2 * c + e]));
-            }
+            K1[KEEP_K ? 2 * c + e : 0] = mul2(g2[e], k1[e]);
+            K2[KEEP_K ? 2 * c + e : 0] = k2[e];
           }
-        }
-      } else {
-        const float4 ga = sh_gate[t], gb = sh_gate[t + 1 < TB ? t + 1 : t];
-        const f32x2 f1 = pack2(ga.x, ga.x), f2 = pack2(gb.x, gb.x);
-        f32x2 v1[CPT], v2[CPT], B1[CPT], B2[CPT];
 #pragma unroll
-        for (int i = 0; i < CPT; ++i) {
-          const float x = st[OFF_V + t * COLS + cg * CPT + i] * ga.y, y = st[OFF_V + (t + 1) * COLS + cg * CPT + i] * gb.y;
-          v1[i] = pack2(x, x);
-          v2[i] = pack2(y, y);
-          B1[i] = B2[i] = 0ull;
-        }
-#pragma unroll
-        for (int c = 0; c < NCH; ++c) {
-          f32x2 k1[2], q1[2], k2[2], q2[2];
-          lds2(ka + c * 128, k1[0], k1[1]);
-          lds2(qa + c * 128, q1[0], q1[1]);
-          lds2(ka + DP * 4 + c * 128, k2[0], k2[1]);
-          lds2(qa + DP * 4 + c * 128, q2[0], q2[1]);
-#pragma unroll
-          for (int e = 0; e < 2; ++e)
-#pragma unroll
-            for (int i = 0; i < CPT; ++i) {
-              f32x2 s = fma2(k1[e], v1[i], mul2(S.v[i][2 * c + e], f1));
-              B1[i] = fma2(s, q1[e], B1[i]);
-              s = fma2(k2[e], v2[i], mul2(s, f2));
-              B2[i] = fma2(s, q2[e], B2[i]);
-              S.v[i][2 * c + e] = s;
-            }
-        }
-        float r[2 * CPT];
-#pragma unroll
-        for (int i = 0; i < CPT; ++i) {
-          const float2 x = unpack2(B1[i]), y = unpack2(B2[i]);
-          r[2 * i] = x.x + x.y; r[2 * i + 1] = y.x + y.y;
-        }
-#pragma unroll
-        for (int o = 4; o > 0; o >>= 1)
-#pragma unroll
-          for (int i = 0; i < 2 * CPT; ++i) r[i] += __shfl_xor_sync(0xffffffffu, r[i], o);
-#pragma unroll
-        for (int i = 0; i < CPT; ++i) {
-          o1[i] = r[2 * i];
-          o2[i] = r[2 * i + 1];
-          if (mycol + i == a.vdim) {         // the normaliser's column
-            const int64_t th = static_cast<int64_t>(t0 + t) * a.heads + head;
-            if (l8 == 0) {
-              a.den[th] = fmaxf(fabsf(o1[i]), ga.z) + 1e-6f;
-              if (t + 1 < n) a.den[th + a.heads] = fmaxf(fabsf(o2[i]), gb.z) + 1e-6f;
-            }
+          for (int i = 0; i < CPT; ++i) {
+            f32x2 s = mul2(S.v[i][2 * c + e], g1[e]);
+            A1[i] = fma2(s, k1[e], A1[i]);
+            B1[i] = fma2(s, q1[e], B1[i]);
+            s = mul2(s, g2[e]);
+            A2[i] = fma2(s, k2[e], A2[i]);
+            B2[i] = fma2(s, q2[e], B2[i]);
+            S.v[i][2 * c + e] = s;
           }
         }
       }
-      float* orow = a.out + (static_cast<int64_t>(t0 + t) * a.heads + head) * a.vdim + mycol;
+      float r[4 * CPT];
 #pragma unroll
-      for (int i = 0; i < CPT; ++i)
-        if (mycol + i < a.vdim) {
-          if (l8 == i) orow[i] = o1[i];
-          if (l8 == CPT + i && t + 1 < n) orow[static_cast<int64_t>(a.heads) * a.vdim + i] = o2[i];
+      for (int i = 0; i < CPT; ++i) {
+        const float2 x0 = unpack2(A1[i]), x1 = unpack2(B1[i]), x2 = unpack2(A2[i]), x3 = unpack2(B2[i]);
+        r[4 * i] = x0.x + x0.y; r[4 * i + 1] = x1.x + x1.y; r[4 * i + 2] = x2.x + x2.y; r[4 * i + 3] = x3.x + x3.y;
+      }
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1)
+#pragma unroll
+        for (int i = 0; i < 4 * CPT; ++i) r[i] += __shfl_xor_sync(0xffffffffu, r[i], o);
+      const float4 s1 = *reinterpret_cast<const float4*>(st + Stage::OFF_S + 4 * t);
+      const float4 s2 = *reinterpret_cast<const float4*>(st + Stage::OFF_S + 4 * t + 4);
+      float* orow = a.out + (static_cast<int64_t>(t0 + t) * a.heads + w.head) * a.vdim + mycol;
+#pragma unroll
+      for (int i = 0; i < CPT; ++i) {
+        const float v1 = st[Stage::OFF_V + t * COLS + cg * CPT + i], v2 = st[Stage::OFF_V + (t + 1) * COLS + cg * CPT + i];
+        const float u1 = s1.x * (v1 - r[4 * i]);
+        const float u2 = s2.x * (v2 - fmaf(s2.z, u1, r[4 * i + 2]));
+        const f32x2 p1 = pack2(u1, u1), p2 = pack2(u2, u2);
+        if (KEEP_K) {
+#pragma unroll
+          for (int c = 0; c < NCH * 2; ++c) S.v[i][c] = fma2(K2[KEEP_K ? c : 0], p2, fma2(K1[KEEP_K ? c : 0], p1, S.v[i][c]));
+        } else {
+#pragma unroll
+          for (int c = 0; c < NCH; ++c) {
+            f32x2 k1[2], k2[2], g2[2];
+            lds2(ka + c * 32, k1[0], k1[1]);
+            lds2(ka + DP + c * 32, k2[0], k2[1]);
+            lds2(ga + DP + c * 32, g2[0], g2[1]);
+#pragma unroll
+            for (int e = 0; e < 2; ++e) S.v[i][2 * c + e] = fma2(k2[e], p2, fma2(mul2(g2[e], k1[e]), p1, S.v[i][2 * c + e]));
+          }
         }
+        if (mycol + i < a.vdim) {
+          if (l8 == i) orow[i] = fmaf(s1.y, u1, r[4 * i + 1]);
+          if (l8 == CPT + i && t + 1 < n) orow[static_cast<int64_t>(a.heads) * a.vdim + i] = fmaf(s2.y, u2, fmaf(s2.w, u1, r[4 * i + 3]));
+        }
+      }
     }
     __syncthreads();       // the stage may be refilled
   }
-  S.store(state, mycol, columns, l8);
-  if (MODE == kScanMlstm && threadIdx.x == 0) *mstate = run_max;
+  S.store(w.state, mycol, w.columns, l8);
+}
+
+// Sums V values per lane over the 16 lanes of a column group, halving the values a lane carries at every exchange:
+// lane l of the group returns the total of value l * V / 16.
+template <int V>
+__device__ __forceinline__ float reduce_scatter16(float (&r)[V], int l16) {
+#pragma unroll
+  for (int o = 8, cur = V; o > 0; o >>= 1) {
+    if (cur > 1) {
+      cur >>= 1;
+      const bool upper = (l16 & o) != 0;
+#pragma unroll
+      for (int j = 0; j < cur; ++j) {
+        const float send = upper ? r[j] : r[j + cur], keep = upper ? r[j + cur] : r[j];
+        r[j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+      }
+    } else {
+      r[0] += __shfl_xor_sync(0xffffffffu, r[0], o);
+    }
+  }
+  return r[0];
+}
+
+// mLSTM, prompt form: sixteen lanes per CPT columns (a shared-memory read costs the same whatever the lanes do with it, so
+// a lane's channels serve four columns), sums handed out one per lane.
+template <int DP, int CPT, int COLS>
+__global__ void __launch_bounds__(COLS / CPT * 16) mlstm_scan_kernel(const mdb_scan_args a) {
+  constexpr int NR = DP / 64;            // float4 per lane and column
+  using Stage = ScanStage<kScanMlstm, DP, COLS>;
+  constexpr int TB = Stage::TB, OFF_V = Stage::OFF_V, OFF_S = Stage::OFF_S;
+  constexpr int VALS = 2 * CPT, PER = 16 / VALS;      // sums of a pair of tokens; lanes per sum
+  extern __shared__ __align__(16) float scan_smem[];
+  __shared__ float4 sh_gate[TB];         // forget factor, input factor, exp(-m) per token of the stage
+  pdl_launch_dependents();
+  pdl_wait();
+  const ScanJob w = scan_job<kScanMlstm, DP, COLS>(a);
+  if (!w.live) return;
+  const int l16 = threadIdx.x & 15, cg = threadIdx.x >> 4, mycol = w.col0 + cg * CPT;
+  f32x2 S[CPT][2 * NR];
+#pragma unroll
+  for (int i = 0; i < CPT; ++i)
+#pragma unroll
+    for (int c = 0; c < NR; ++c) {
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!w.fresh && mycol + i < w.columns)
+        x = *reinterpret_cast<const float4*>(w.state + static_cast<int64_t>(mycol + i) * DP + c * 64 + l16 * 4);
+      S[i][2 * c] = pack2(x.x, x.y);
+      S[i][2 * c + 1] = pack2(x.z, x.w);
+    }
+  // every block of columns keeps a copy of the running maximum, so that no CTA reads what another writes
+  const int blocks = (w.columns + kScanBlockCols - 1) / kScanBlockCols, block0 = w.col0 / kScanBlockCols;
+  float* mstate = a.mstate + (static_cast<int64_t>(w.slot) * a.heads + w.head) * blocks;
+  float run_max = w.fresh ? 0.f : mstate[block0];
+  Stage::fill(a, w, w.t_begin, scan_smem);
+  int buf = 0;
+  for (int t0 = w.t_begin; t0 < w.t_end; t0 += TB, buf ^= 1) {
+    const int n = min(TB, w.t_end - t0);
+    Stage::turn(a, w, t0, scan_smem, buf);
+    const float* st = scan_smem + buf * Stage::FLOATS;
+    // m_t = max(f_t + m_(t-1), i_t) over the stage as a scan of the maps x -> max(x + F, I)
+    if (threadIdx.x < 32) {
+      const int l = threadIdx.x;
+      const float li = l < n ? st[OFF_S + 4 * l] : -INFINITY, lf = l < n ? st[OFF_S + 4 * l + 1] : 0.f;
+      float F = lf, I = li;
+#pragma unroll
+      for (int o = 1; o < TB; o <<= 1) {
+        const float Fp = __shfl_up_sync(0xffffffffu, F, o), Ip = __shfl_up_sync(0xffffffffu, I, o);
+        if (l >= o) { I = fmaxf(Ip + F, I); F += Fp; }
+      }
+      const float m = fmaxf(F + run_max, I);
+      float mp = __shfl_up_sync(0xffffffffu, m, 1);
+      if (l == 0) mp = run_max;
+      if (l < n) sh_gate[l] = make_float4(expf(lf + mp - m), expf(li - m), expf(-m), 0.f);
+      else if (l < TB) sh_gate[l] = make_float4(1.f, 0.f, 0.f, 0.f);
+      run_max = __shfl_sync(0xffffffffu, m, n - 1);
+    }
+    __syncthreads();
+    for (int t = 0; t < n; t += 2) {
+      const float* k1p = st + t * DP + l16 * 4;
+      const float* k2p = k1p + DP;
+      const float4 ga = sh_gate[t], gb = sh_gate[t + 1];
+      const f32x2 f1 = pack2(ga.x, ga.x), f2 = pack2(gb.x, gb.x);
+      f32x2 v1[CPT], v2[CPT], acc[CPT][2];
+#pragma unroll
+      for (int i = 0; i < CPT; ++i) {
+        const float y1 = st[OFF_V + t * COLS + cg * CPT + i] * ga.y, y2 = st[OFF_V + (t + 1) * COLS + cg * CPT + i] * gb.y;
+        v1[i] = pack2(y1, y1);
+        v2[i] = pack2(y2, y2);
+        acc[i][0] = acc[i][1] = 0ull;
+      }
+#pragma unroll
+      for (int c = 0; c < NR; ++c) {
+        f32x2 k1[2], q1[2], k2[2], q2[2];
+        lds2(k1p + c * 64, k1[0], k1[1]);
+        lds2(k1p + TB * DP + c * 64, q1[0], q1[1]);
+        lds2(k2p + c * 64, k2[0], k2[1]);
+        lds2(k2p + TB * DP + c * 64, q2[0], q2[1]);
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+#pragma unroll
+          for (int i = 0; i < CPT; ++i) {
+            f32x2 s = fma2(k1[e], v1[i], mul2(S[i][2 * c + e], f1));
+            acc[i][0] = fma2(s, q1[e], acc[i][0]);
+            s = fma2(k2[e], v2[i], mul2(s, f2));
+            acc[i][1] = fma2(s, q2[e], acc[i][1]);
+            S[i][2 * c + e] = s;
+          }
+      }
+      float r[VALS];
+#pragma unroll
+      for (int i = 0; i < VALS; ++i) {
+        const float2 x = unpack2(acc[i / 2][i % 2]);
+        r[i] = x.x + x.y;
+      }
+      const float sum = reduce_scatter16<VALS>(r, l16);
+      const int mine = l16 / PER, col = mine >> 1, kind = mine & 1;      // kind: first or second token of the pair
+      if (l16 % PER == 0 && t + kind < n) {
+        const int64_t th = static_cast<int64_t>(t0 + t + kind) * a.heads + w.head;
+        if (mycol + col < a.vdim) a.out[th * a.vdim + mycol + col] = sum;
+        else if (mycol + col == a.vdim) a.den[th] = fmaxf(fabsf(sum), kind ? gb.z : ga.z) + 1e-6f;      // the normaliser's column
+      }
+    }
+    __syncthreads();       // the stage may be refilled
+  }
+#pragma unroll
+  for (int i = 0; i < CPT; ++i)
+    if (mycol + i < w.columns) {
+#pragma unroll
+      for (int c = 0; c < NR; ++c) {
+        const float2 lo = unpack2(S[i][2 * c]), hi = unpack2(S[i][2 * c + 1]);
+        *reinterpret_cast<float4*>(w.state + static_cast<int64_t>(mycol + i) * DP + c * 64 + l16 * 4) = make_float4(lo.x, lo.y, hi.x, hi.y);
+      }
+    }
+  if (threadIdx.x == 0)
+    for (int b = block0; b < blocks && b * kScanBlockCols < w.col0 + COLS; ++b) mstate[b] = run_max;
 }
 
 // One-token form: every sequence brings one token and a CTA owns all columns of a head.  The decay is computed from the
@@ -796,7 +869,7 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
     }
   }
   __syncthreads();
-  const uint32_t ka = smem_u32(sh) + l8 * 16;
+  const float* ka = sh + l8 * 4;
   float out[CPT];
   if (MODE == kScanDelta) {
     f32x2 A[CPT], B[CPT];
@@ -805,9 +878,9 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
 #pragma unroll
     for (int c = 0; c < NCH; ++c) {
       f32x2 k[2], q[2], g[2];
-      lds2(ka + c * 128, k[0], k[1]);
-      lds2(ka + DP * 4 + c * 128, q[0], q[1]);
-      lds2(ka + DP * 8 + c * 128, g[0], g[1]);
+      lds2(ka + c * 32, k[0], k[1]);
+      lds2(ka + DP + c * 32, q[0], q[1]);
+      lds2(ka + 2 * DP + c * 32, g[0], g[1]);
 #pragma unroll
       for (int e = 0; e < 2; ++e)
 #pragma unroll
@@ -829,7 +902,7 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
 #pragma unroll
     for (int c = 0; c < NCH; ++c) {
       f32x2 k[2];
-      lds2(ka + c * 128, k[0], k[1]);
+      lds2(ka + c * 32, k[0], k[1]);
 #pragma unroll
       for (int e = 0; e < 2; ++e)
 #pragma unroll
@@ -848,8 +921,8 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
 #pragma unroll
     for (int c = 0; c < NCH; ++c) {
       f32x2 k[2], q[2];
-      lds2(ka + c * 128, k[0], k[1]);
-      lds2(ka + DP * 4 + c * 128, q[0], q[1]);
+      lds2(ka + c * 32, k[0], k[1]);
+      lds2(ka + DP + c * 32, q[0], q[1]);
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
 #pragma unroll
@@ -912,40 +985,42 @@ int launch_scan_token(const mdb_scan_args& a, cudaStream_t st) {
   }
 }
 
-template <int MODE, int NCH>
+template <int MODE, int DP, int COLS>
 int launch_scan_prompt(const mdb_scan_args& a, cudaStream_t st) {
-  constexpr int CPT = NCH > 8 ? 1 : (MODE == kScanMlstm ? (NCH <= 4 ? 4 : 2) : (NCH <= 4 ? 2 : 1));
-  constexpr int smem = 2 * scan_stage_floats(MODE, NCH * 32, kScanTokens, kScanBlockCols) * 4;
+  constexpr int smem = 2 * ScanStage<MODE, DP, COLS>::FLOATS * 4;
   static_assert(smem <= 227 * 1024, "shared memory of the scan");
+  constexpr int DELTA_CPT = DP <= 128 ? 2 : 1, MLSTM_CPT = DP <= 256 ? 4 : 2;
+  constexpr int threads = MODE == kScanDelta ? COLS / DELTA_CPT * 8 : COLS / MLSTM_CPT * 16;
+  void (*kernel)(mdb_scan_args);
+  if constexpr (MODE == kScanDelta) kernel = delta_scan_kernel<DP / 32, DELTA_CPT, COLS>;
+  else kernel = mlstm_scan_kernel<DP, MLSTM_CPT, COLS>;
   static PerDeviceOnce attr_once;
   const int dev = attr_once.slot();
   if (dev < 0) return MDB_ERR_CUDA;
   if (!attr_once.done[dev]) {
-    if (cudaFuncSetAttribute(scan_kernel<MODE, NCH, CPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
-      return MDB_ERR_CUDA;
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return MDB_ERR_CUDA;
     attr_once.done[dev] = true;
   }
   const int columns = a.vdim + (MODE == kScanMlstm ? 1 : 0);
-  const dim3 grid((columns + kScanBlockCols - 1) / kScanBlockCols, a.heads, a.bs);
-  return mdb_launch(scan_kernel<MODE, NCH, CPT>, grid, dim3(kScanBlockCols / CPT * 8), smem, st, a);
+  return mdb_launch(kernel, dim3((columns + COLS - 1) / COLS, a.heads, a.bs), dim3(threads), smem, st, a);
 }
 
-template <int MODE, int NCH>
+template <int MODE, int DP>
 int launch_scan_dim(const mdb_scan_args& a, cudaStream_t st) {
-  if (!a.fused) return launch_scan_prompt<MODE, NCH>(a, st);
-  return a.dtype == MDB_F32 ? launch_scan_token<float, MODE, NCH>(a, st) : launch_scan_token<bf16, MODE, NCH>(a, st);
+  if (a.fused) return a.dtype == MDB_F32 ? launch_scan_token<float, MODE, DP / 32>(a, st) : launch_scan_token<bf16, MODE, DP / 32>(a, st);
+  // blocks of 32 columns while they fill the SMs, narrower ones (more re-reads of k, q and g) below that
+  const int64_t wide = static_cast<int64_t>((a.vdim + 31) / 32) * a.heads * a.bs;
+  return wide >= 148 ? launch_scan_prompt<MODE, DP, 32>(a, st) : launch_scan_prompt<MODE, DP, 16>(a, st);
 }
 
 template <int MODE>
 int launch_scan(const mdb_scan_args& a, cudaStream_t st) {
   switch (a.dim_pad) {
-    case 32: return launch_scan_dim<MODE, 1>(a, st);
-    case 64: return launch_scan_dim<MODE, 2>(a, st);
-    case 96: return launch_scan_dim<MODE, 3>(a, st);
-    case 128: return launch_scan_dim<MODE, 4>(a, st);
-    case 192: return launch_scan_dim<MODE, 6>(a, st);
-    case 256: return launch_scan_dim<MODE, 8>(a, st);
-    case 512: return launch_scan_dim<MODE, 16>(a, st);
+    case 64: return launch_scan_dim<MODE, 64>(a, st);
+    case 128: return launch_scan_dim<MODE, 128>(a, st);
+    case 192: return launch_scan_dim<MODE, 192>(a, st);
+    case 256: return launch_scan_dim<MODE, 256>(a, st);
+    case 512: return launch_scan_dim<MODE, 512>(a, st);
     default: return MDB_ERR_UNSUPPORTED;
   }
 }
@@ -957,7 +1032,7 @@ bool seqs_ok(const int32_t* cu_q, const int32_t* start, const int32_t* slot) { r
 extern "C" {
 
 int mdb_scan_dim_pad(int dim) {
-  static const int sizes[] = {32, 64, 96, 128, 192, 256, 512};
+  static const int sizes[] = {64, 128, 192, 256, 512};
   for (int s : sizes)
     if (dim <= s) return s;
   return 0;

@@ -178,7 +178,7 @@ def test_delta_scan_fused_token(H, KH, D, DV, taps):
 
 def test_delta_remembers_a_far_key():
     """A value written under one key long ago, no decay and orthogonal writes since, comes back whole."""
-    ops, T, D, DV = pkg.ops, 400, 32, 16
+    ops, T, D, DV = pkg.ops, 400, 64, 16
     k = torch.zeros(T, 1, D)
     k[:, 0, 1:] = torch.nn.functional.normalize(torch.randn(T, D - 1, generator=gen(0)), dim=-1)
     k[3, 0], k[3, 0, 0] = 0.0, 1.0
