@@ -142,8 +142,8 @@ def work_of(name: str, a: tuple, k: dict, ctx: dict):
         m, heads, dim, vdim = a[1:5]
         return "mlstm inputs", m * heads * (2 * dim + vdim) * (e + 4), 0, 0
     if name == "channel_decay":
-        m, heads, dp = a[6].shape          # projection in, decay out, and for every second token its key, query and the key before
-        return "decay", m * heads * dp * 8 + m * a[3].shape[1] * dp * 6, 0, 0
+        m, heads, dp = a[7].shape          # projection in, decay out, key and query, for every second token the key before
+        return "decay", m * heads * dp * 8 + m * a[3].shape[1] * dp * 10, 0, 0
     if name == "gated_norm":
         m, h, v = a[0].shape
         return "gated norm", m * h * v * (4 + 2 * e), 0, 0

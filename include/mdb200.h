@@ -430,9 +430,9 @@ int mdb_scan_blocks(int vdim);
 int mdb_scan_fusable(int dim_pad, int vdim);
 
 /* Inputs of the delta scan: causal short convolution over time per channel (weights fp32 [channels][taps], the last
- * tap is the current token's) and silu of q, k, v; q and k as unit vectors (q times dim^-1/2), k . q, beta =
- * sigmoid(b).  conv_state [slot][taps - 1][channels] of the activation type, channels ordered q | k | v, holds the
- * last inputs and is moved on: in the same kernel when shift_state is set (every portion is one token), else by a
+ * tap is the current token's) and silu of q, k, v; q and k as unit vectors (q times dim^-1/2), beta = sigmoid(b).
+ * conv_state [slot][taps - 1][channels] of the activation type, channels ordered q | k | v, holds the last inputs and is
+ * moved on: in the same kernel when shift_state is set (every portion is one token), else by a
  * second one.  copy_cols columns of `copy` are written to copy_out (materialises split-k slices). */
 typedef struct {
   int32_t dtype, m, bs, heads, kv_heads, dim, dim_pad, vdim, taps, channels, shift_state, copy_cols;
@@ -452,13 +452,12 @@ typedef struct {
   float* k_out;
   float* v_out;    /* [m][heads][vdim] */
   float* beta_out; /* [m][heads] */
-  float* kq_out;   /* [m][kv_heads] */
 } mdb_delta_prep_args;
 int mdb_delta_prep(const mdb_delta_prep_args* args, mdb_stream_t stream);
 
-/* g [m][heads][dim_pad] = exp(-exp(a_log[h]) * softplus(x + dt_bias)), x [m] rows of heads * dim columns; cross
- * [m][heads][2], written for the odd tokens of every portion: ((g k_prev) . k, (g k_prev) . q) with the outputs of
- * mdb_delta_prep. */
+/* g [m][heads][dim_pad] = exp(-exp(a_log[h]) * softplus(x + dt_bias)), x [m] rows of heads * dim columns; scalars
+ * [m][heads][4] = (k . q, (g k_prev) . k, (g k_prev) . q, beta) with the outputs of mdb_delta_prep; the products with the
+ * token before are written for the odd tokens of every portion. */
 typedef struct {
   int32_t m, heads, kv_heads, dim, dim_pad;
   const float* x;
@@ -467,8 +466,9 @@ typedef struct {
   const float* dt_bias;
   const float* q;
   const float* k;
+  const float* beta;
   float* g;
-  float* cross;
+  float* scalars;
   const int32_t* row_seq;
   const int32_t* cu_q;
 } mdb_decay_args;
@@ -491,7 +491,8 @@ typedef struct {
 int mdb_mlstm_prep(const mdb_mlstm_prep_args* args, mdb_stream_t stream);
 
 /* The recurrences over every sequence's portion; state [slot][heads][vdim][dim_pad] fp32 is read and written.
- * DELTA: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; s0 = beta, s1 = k . q.  MLSTM: m' = max(f + m, i);
+ * DELTA: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; beta comes
+ * with the scalars of mdb_channel_decay, in the fused form as s0.  MLSTM: m' = max(f + m, i);
  * S, n <- exp(f + m - m') (.) + exp(i - m') k (v^T, 1); o = S^T q, den [m][heads] = max(|n . q|, exp(-m')) + 1e-6;
  * s0 = i, s1 = f; its state has one more column per head (vdim + 1), which is n; mstate [slot][heads][mdb_scan_blocks].
  * out [m][heads][vdim] fp32; with `fused` (every portion is one token) the decay comes from raw_decay + dt_bias and
@@ -509,7 +510,7 @@ typedef struct {
   float* state;
   int64_t state_slot_stride, num_slots;
   float* mstate;
-  const float* cross; /* DELTA: of mdb_channel_decay */
+  const float* scalars; /* DELTA: of mdb_channel_decay */
   float* den;         /* MLSTM */
   const int32_t* cu_q;
   const int32_t* start;

@@ -41,10 +41,10 @@ DeltaPrepArgs = _struct("DeltaPrepArgs", [(n, _i) for n in (
     "dtype", "m", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim", "taps", "channels", "shift_state", "copy_cols")] + [
     ("q", Rows), ("k", Rows), ("v", Rows), ("b", Rows), ("copy", Rows), ("copy_out", _p), ("copy_ld", _i64), ("conv_q", _p),
     ("conv_k", _p), ("conv_v", _p), ("conv_state", _p), ("conv_slot_stride", _i64), ("num_slots", _i64), ("row_seq", _p),
-    ("cu_q", _p), ("start", _p), ("state_slot", _p), ("q_out", _p), ("k_out", _p), ("v_out", _p), ("beta_out", _p),
-    ("kq_out", _p)])
+    ("cu_q", _p), ("start", _p), ("state_slot", _p), ("q_out", _p), ("k_out", _p), ("v_out", _p), ("beta_out", _p)])
 DecayArgs = _struct("DecayArgs", [(n, _i) for n in ("m", "heads", "kv_heads", "dim", "dim_pad")] + [
-    ("x", _p), ("ldx", _i64), ("a_log", _p), ("dt_bias", _p), ("q", _p), ("k", _p), ("g", _p), ("cross", _p), ("row_seq", _p),
+    ("x", _p), ("ldx", _i64), ("a_log", _p), ("dt_bias", _p), ("q", _p), ("k", _p), ("beta", _p), ("g", _p), ("scalars", _p),
+    ("row_seq", _p),
     ("cu_q", _p)])
 MlstmPrepArgs = _struct("MlstmPrepArgs", [(n, _i) for n in ("dtype", "m", "heads", "dim", "dim_pad", "vdim")] + [
     ("q", Rows), ("k", Rows), ("v", Rows), ("i", Rows), ("f", Rows), ("bias_i", _p), ("bias_f", _p), ("q_out", _p),
@@ -52,7 +52,7 @@ MlstmPrepArgs = _struct("MlstmPrepArgs", [(n, _i) for n in ("dtype", "m", "heads
 ScanArgs = _struct("ScanArgs", [(n, _i) for n in (
     "mode", "dtype", "fused", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim")] + [
     ("eps", _f), ("q", _p), ("k", _p), ("v", _p), ("g", _p), ("s0", _p), ("s1", _p), ("state", _p),
-    ("state_slot_stride", _i64), ("num_slots", _i64), ("mstate", _p), ("cross", _p),
+    ("state_slot_stride", _i64), ("num_slots", _i64), ("mstate", _p), ("scalars", _p),
     ("den", _p), ("cu_q", _p), ("start", _p),
     ("state_slot", _p), ("out", _p), ("raw_decay", Rows), ("a_log", _p), ("dt_bias", _p), ("gate", Rows), ("norm", _p),
     ("norm_head_stride", _i64), ("y", _p), ("ldy", _i64)])

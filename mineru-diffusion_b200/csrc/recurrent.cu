@@ -12,7 +12,7 @@
 //   a = (g S)^T k,  b = (g S)^T q,  u = beta (v - a),  o = b + (k . q) u,  S <- g S + k u^T,
 // and prompts take two tokens per reduction: with S' = g2 g1 S the second token's products are
 //   a2 = S'^T k2 + ((g2 k1) . k2) u1,  b2 = S'^T q2 + ((g2 k1) . q2) u1,  S <- S' + (g2 k1) u1^T + k2 u2^T,
-// the same number of FMAs per token with half the dependent shuffle reductions; the two cross products per token are
+// the same number of FMAs per token with half the dependent shuffle reductions; these products of keys and queries are
 // computed beforehand, with the decays.
 //
 // mLSTM: the normaliser n is one more column of the state (its value is 1 for every token); the division by
@@ -65,8 +65,8 @@ __device__ __forceinline__ float sum8(float v) {
 }
 
 // ---------------------------------------------------------------------------
-// Before the delta scan: short convolution + silu of q, k and v, unit norm of q and k, k . q, sigmoid of beta.
-// Units of a row, one warp each: kv_heads (q and k of one head), heads (v of one head), one for beta, and, where the
+// Before the delta scan: short convolution + silu of q, k and v, unit norm of q and k, sigmoid of beta.
+// Units of a row, one warp each: q and k of a head (together or apart), v of a head, one for beta, and, where the
 // projection came as split-k slices, the copy of its low-rank columns for the GEMM that follows.
 // ---------------------------------------------------------------------------
 constexpr int kPrepWarps = 4;
@@ -120,7 +120,7 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const mdb_d
     float* qo = a.q_out + (row * a.kv_heads + unit) * a.dim_pad;
     float* ko = a.k_out + (row * a.kv_heads + unit) * a.dim_pad;
     const int kq_channels = a.kv_heads * a.dim;
-    float sq = 0.f, sk = 0.f, dot = 0.f;
+    float sq = 0.f, sk = 0.f;
     for (int d = lane; d < a.dim_pad; d += 32) {
       float q = 0.f, k = 0.f;
       if (d < a.dim) {
@@ -138,13 +138,9 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const mdb_d
     const float rq = (1.0f / sqrtf(warp_sum(sq) + 1e-6f)) * (1.0f / sqrtf(static_cast<float>(a.dim)));
     const float rk = 1.0f / sqrtf(warp_sum(sk) + 1e-6f);
     for (int d = lane; d < a.dim_pad; d += 32) {       // a lane re-reads what it wrote itself
-      const float q = qo[d] * rq, k = ko[d] * rk;
-      qo[d] = q;
-      ko[d] = k;
-      dot += q * k;
+      qo[d] *= rq;
+      ko[d] *= rk;
     }
-    dot = warp_sum(dot);
-    if (lane == 0) a.kq_out[row * a.kv_heads + unit] = dot;
     return;
   }
   const int vu = unit - a.kv_heads;
@@ -231,46 +227,36 @@ __device__ __forceinline__ float dot4(float4 a, float4 b) { return a.x * b.x + a
 __device__ __forceinline__ float4 scale4(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
 
 template <typename T, bool PARTS>
-__global__ void __launch_bounds__(kPrepWarps * 32, 4) delta_prep_rows_kernel(const mdb_delta_prep_args a, const int run) {
+__global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_rows_kernel(const mdb_delta_prep_args a, const int run) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31, c = lane * 4;
-  const int unit = blockIdx.y * kPrepWarps + (threadIdx.x >> 5);
-  const int64_t row0 = static_cast<int64_t>(blockIdx.x) * run, row1 = min(row0 + run, static_cast<int64_t>(a.m));
+  const int unit = blockIdx.x * kPrepWarps + (threadIdx.x >> 5);
+  const int64_t row0 = static_cast<int64_t>(blockIdx.y) * run, row1 = min(row0 + run, static_cast<int64_t>(a.m));
   const int vblocks = (a.vdim + 127) / 128;        // a head's values in blocks of 128
-  const bool is_qk = unit < a.kv_heads, is_v = !is_qk && unit < a.kv_heads + a.heads * vblocks;
-  const int kc = a.kv_heads * a.dim;
-  if (is_qk || is_v) {
-    const int vu = unit - a.kv_heads, head = vu / vblocks, vc = (vu % vblocks) * 128 + c;
-    const bool live = is_qk ? c < a.dim : vc < a.vdim;
-    const int col = is_qk ? unit * a.dim + c : head * a.vdim + vc;
-    const mdb_rows& src = is_qk ? a.q : a.v;
-    const int channel = is_qk ? col : 2 * kc + col;
-    ConvWindow<T, PARTS> w0, w1;
-    if (live) {
-      w0.load_taps(is_qk ? a.conv_q : a.conv_v, col, a.taps);
-      if (is_qk) w1.load_taps(a.conv_k, col, a.taps);
-    }
-    const float q_scale = 1.0f / sqrtf(static_cast<float>(a.dim));
+  const int qk_units = 2 * a.kv_heads, kc = a.kv_heads * a.dim;
+  if (unit < qk_units + a.heads * vblocks) {
+    const int stream = unit < a.kv_heads ? 0 : (unit < qk_units ? 1 : 2);      // q, k or v
+    const int vu = unit - qk_units, head = stream == 2 ? vu / vblocks : unit - stream * a.kv_heads;
+    const int hc = stream == 2 ? (vu % vblocks) * 128 + c : c;       // first of the lane's channels in its head
+    const int dim = stream == 2 ? a.vdim : a.dim;
+    const bool live = hc < dim;
+    const int col = head * dim + hc, channel = stream * kc + col;
+    // by value: a reference picked at run time would be read through memory at every use
+    mdb_rows src = a.q;
+    if (stream == 1) src = a.k;
+    if (stream == 2) src = a.v;
+    ConvWindow<T, PARTS> win;
+    if (live) win.load_taps(stream == 0 ? a.conv_q : (stream == 1 ? a.conv_k : a.conv_v), col, a.taps);
+    const float unit_scale = stream == 0 ? 1.0f / sqrtf(static_cast<float>(a.dim)) : 1.0f;
+    const int out_dim = stream == 2 ? a.vdim : a.dim_pad, out_heads = stream == 2 ? a.heads : a.kv_heads;
+    float* out = (stream == 0 ? a.q_out : (stream == 1 ? a.k_out : a.v_out)) + static_cast<int64_t>(head) * out_dim + hc;
+    const int64_t out_ld = static_cast<int64_t>(out_heads) * out_dim;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     int seq = -1, slot = -1;
-    // the next row's inputs are requested before this row's are used
-    float4 next0 = zero, next1 = zero;
-    int next_seq = a.row_seq[row0];
-    if (live) {
-      next0 = rows_at4_of<T, PARTS>(src, row0, col);
-      if (is_qk) next1 = rows_at4_of<T, PARTS>(a.k, row0, col);
-    }
     for (int64_t row = row0; row < row1; ++row) {
-      const int s = next_seq;
-      const float4 in0 = next0, in1 = next1;
-      if (row + 1 < row1) {
-        next_seq = a.row_seq[row + 1];
-        if (live) {
-          next0 = rows_at4_of<T, PARTS>(src, row + 1, col);
-          if (is_qk) next1 = rows_at4_of<T, PARTS>(a.k, row + 1, col);
-        }
-      }
+      const int s = a.row_seq[row];
+      const float4 in = live ? rows_at4_of<T, PARTS>(src, row, col) : zero;
       if (s != seq) {
         seq = s;
         slot = a.state_slot[s];
@@ -278,55 +264,34 @@ __global__ void __launch_bounds__(kPrepWarps * 32, 4) delta_prep_rows_kernel(con
           if (lane == 0) report_status(MDB_STATUS_BAD_SLOT);
           slot = -1;
         }
-        if (slot >= 0 && live) {
-          const int from = a.start[s] == 0 ? -1 : slot, tloc = static_cast<int>(row) - a.cu_q[s];
-          w0.refill(a, src, row, tloc, from, col, channel);
-          if (is_qk) w1.refill(a, a.k, row, tloc, from, col, kc + col);
-        }
+        if (slot >= 0 && live)
+          win.refill(a, src, row, static_cast<int>(row) - a.cu_q[s], a.start[s] == 0 ? -1 : slot, col, channel);
       }
       if (slot < 0) continue;
-      float4 y0 = zero, y1 = zero;
+      float4 y = zero;
       if (live) {
-        y0 = w0.step(in0);
-        if (is_qk) y1 = w1.step(in1);
-        if (a.shift_state && a.taps > 1) {
-          w0.save(a, slot, channel);
-          if (is_qk) w1.save(a, slot, kc + col);
-        }
+        y = win.step(in);
+        if (a.shift_state && a.taps > 1) win.save(a, slot, channel);
       }
-      if (is_qk) {
-        float qq = dot4(y0, y0), kk = dot4(y1, y1), qk = dot4(y0, y1);
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          qq += __shfl_xor_sync(0xffffffffu, qq, o);
-          kk += __shfl_xor_sync(0xffffffffu, kk, o);
-          qk += __shfl_xor_sync(0xffffffffu, qk, o);
-        }
-        const float rq = (1.0f / sqrtf(qq + 1e-6f)) * q_scale, rk = 1.0f / sqrtf(kk + 1e-6f);
-        y0 = scale4(y0, rq);
-        y1 = scale4(y1, rk);
-        const float kq = qk * rq * rk;
-        const int64_t at = (row * a.kv_heads + unit) * a.dim_pad + c;
-        if (c < a.dim_pad) {
-          *reinterpret_cast<float4*>(a.q_out + at) = y0;
-          *reinterpret_cast<float4*>(a.k_out + at) = y1;
-        }
-        if (lane == 0) a.kq_out[row * a.kv_heads + unit] = kq;
-      } else if (live) {
-        *reinterpret_cast<float4*>(a.v_out + (row * a.heads + head) * a.vdim + vc) = y0;
-      }
+      if (stream < 2) y = scale4(y, (1.0f / sqrtf(warp_sum(dot4(y, y)) + 1e-6f)) * unit_scale);
+      if (hc < out_dim) *reinterpret_cast<float4*>(out + row * out_ld) = y;
     }
     return;
   }
-  const int rest = unit - a.kv_heads - a.heads * vblocks;
-  for (int64_t row = row0; row < row1; ++row) {
-    if (rest == 0) {
-      for (int h = lane; h < a.heads; h += 32) a.beta_out[row * a.heads + h] = sigmoid_f(rows_at<T>(a.b, row, h));
-    } else {
-      const int cc = (rest - 1) * 128 + c;
-      if (cc < a.copy_cols) act_store4(static_cast<T*>(a.copy_out) + row * a.copy_ld + cc, rows_at4_of<T, PARTS>(a.copy, row, cc));
+  const int rest = unit - qk_units - a.heads * vblocks;
+  if (rest == 0) {
+    const int n = static_cast<int>(row1 - row0) * a.heads;
+#pragma unroll 4
+    for (int i = lane; i < n; i += 32) {
+      const int64_t row = row0 + i / a.heads;
+      a.beta_out[row * a.heads + i % a.heads] = sigmoid_f(rows_at<T>(a.b, row, i % a.heads));
     }
+    return;
   }
+  const int cc = (rest - 1) * 128 + c;
+  if (cc < a.copy_cols)
+    for (int64_t row = row0; row < row1; ++row)
+      act_store4(static_cast<T*>(a.copy_out) + row * a.copy_ld + cc, rows_at4_of<T, PARTS>(a.copy, row, cc));
 }
 
 // The last taps - 1 inputs of every channel after a step of arbitrary portions: one thread per (sequence, channel).
@@ -353,8 +318,8 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const mdb_delta_prep_ar
 }
 
 // A warp per (row, head).  g = exp(-exp(A_log) * softplus(x + dt_bias)), laid out [row][head][dim_pad] (padding
-// channels: 1), and, for the odd tokens of a portion, the cross products with the token before:
-// cross [row][head] = ((g k_prev) . k, (g k_prev) . q).  VEC: head rows of x start on 16-byte boundaries.
+// channels: 1), and the scalars of the scan, [row][head][4] = (k . q, (g k_prev) . k, (g k_prev) . q, beta): the middle two
+// are the products with the token before and exist for the odd tokens of a portion.  VEC: head rows of x start on 16-byte boundaries.
 template <bool VEC>
 __global__ void __launch_bounds__(128) channel_decay_kernel(const mdb_decay_args a) {
   pdl_launch_dependents();
@@ -372,7 +337,7 @@ __global__ void __launch_bounds__(128) channel_decay_kernel(const mdb_decay_args
     const float* q = a.q + (row * a.kv_heads + kvh) * a.dim_pad;
     const float* kp = k - static_cast<int64_t>(a.kv_heads) * a.dim_pad;      // read for odd tokens only
     const float rate = -expf(a.a_log[head]);
-    float ck = 0.f, cq = 0.f;
+    float kq = 0.f, ck = 0.f, cq = 0.f;
     for (int c = lane * 4; c < a.dim_pad; c += 128) {
       float xv[4], bv[4], r[4];
       if (VEC && c + 4 <= a.dim) {
@@ -389,19 +354,22 @@ __global__ void __launch_bounds__(128) channel_decay_kernel(const mdb_decay_args
 #pragma unroll
       for (int i = 0; i < 4; ++i) r[i] = c + i < a.dim ? expf(rate * softplus_f(xv[i] + bv[i])) : 1.f;
       *reinterpret_cast<float4*>(g + c) = make_float4(r[0], r[1], r[2], r[3]);
+      const float4 k1 = *reinterpret_cast<const float4*>(k + c), q1 = *reinterpret_cast<const float4*>(q + c);
+      kq += dot4(k1, q1);
       if (odd) {
-        const float4 k0 = *reinterpret_cast<const float4*>(kp + c), k1 = *reinterpret_cast<const float4*>(k + c);
-        const float4 q1 = *reinterpret_cast<const float4*>(q + c);
-        const float e0 = r[0] * k0.x, e1 = r[1] * k0.y, e2 = r[2] * k0.z, e3 = r[3] * k0.w;
-        ck += e0 * k1.x + e1 * k1.y + e2 * k1.z + e3 * k1.w;
-        cq += e0 * q1.x + e1 * q1.y + e2 * q1.z + e3 * q1.w;
+        const float4 k0 = *reinterpret_cast<const float4*>(kp + c);
+        const float4 e = make_float4(r[0] * k0.x, r[1] * k0.y, r[2] * k0.z, r[3] * k0.w);
+        ck += dot4(e, k1);
+        cq += dot4(e, q1);
       }
     }
+    kq = warp_sum(kq);
     if (odd) {
       ck = warp_sum(ck);
       cq = warp_sum(cq);
-      if (lane == 0) *reinterpret_cast<float2*>(a.cross + 2 * (row * a.heads + head)) = make_float2(ck, cq);
     }
+    if (lane == 0)
+      *reinterpret_cast<float4*>(a.scalars + 4 * (row * a.heads + head)) = make_float4(kq, ck, cq, a.beta[row * a.heads + head]);
   }
 }
 
@@ -547,14 +515,10 @@ struct ScanStage {
     for (int i = threadIdx.x; i < n; i += step) {
       const int64_t th = static_cast<int64_t>(t0 + i) * a.heads + w.head;
       const uint32_t dst = base + (OFF_S + 4 * i) * 4;
-      cp_async4(dst, a.s0 + th);
       if (MODE == kScanDelta) {
-        cp_async4(dst + 4, a.s1 + static_cast<int64_t>(t0 + i) * a.kv_heads + w.kvh);
-        if (i & 1) {
-          cp_async4(dst + 8, a.cross + 2 * th);
-          cp_async4(dst + 12, a.cross + 2 * th + 1);
-        }
+        cp_async16(dst, a.scalars + 4 * th);
       } else {
+        cp_async4(dst, a.s0 + th);
         cp_async4(dst + 4, a.s1 + th);
       }
     }
@@ -652,9 +616,10 @@ __global__ void __launch_bounds__(COLS / CPT * 8) delta_scan_kernel(const mdb_sc
       float* orow = a.out + (static_cast<int64_t>(t0 + t) * a.heads + w.head) * a.vdim + mycol;
 #pragma unroll
       for (int i = 0; i < CPT; ++i) {
+        // s1, s2 = (k . q, products with the token before, beta)
         const float v1 = st[Stage::OFF_V + t * COLS + cg * CPT + i], v2 = st[Stage::OFF_V + (t + 1) * COLS + cg * CPT + i];
-        const float u1 = s1.x * (v1 - r[4 * i]);
-        const float u2 = s2.x * (v2 - fmaf(s2.z, u1, r[4 * i + 2]));
+        const float u1 = s1.w * (v1 - r[4 * i]);
+        const float u2 = s2.w * (v2 - fmaf(s2.y, u1, r[4 * i + 2]));
         const f32x2 p1 = pack2(u1, u1), p2 = pack2(u2, u2);
         if (KEEP_K) {
 #pragma unroll
@@ -671,8 +636,8 @@ __global__ void __launch_bounds__(COLS / CPT * 8) delta_scan_kernel(const mdb_sc
           }
         }
         if (mycol + i < a.vdim) {
-          if (l8 == i) orow[i] = fmaf(s1.y, u1, r[4 * i + 1]);
-          if (l8 == CPT + i && t + 1 < n) orow[static_cast<int64_t>(a.heads) * a.vdim + i] = fmaf(s2.y, u2, fmaf(s2.w, u1, r[4 * i + 3]));
+          if (l8 == i) orow[i] = fmaf(s1.x, u1, r[4 * i + 1]);
+          if (l8 == CPT + i && t + 1 < n) orow[static_cast<int64_t>(a.heads) * a.vdim + i] = fmaf(s2.x, u2, fmaf(s2.z, u1, r[4 * i + 3]));
         }
       }
     }
@@ -854,7 +819,7 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
     if (!fresh) m_old = mstate[0];
   }
   const float s0 = a.s0[t * a.heads + head];
-  const float s1 = MODE == kScanDelta ? a.s1[t * a.kv_heads + kvh] : a.s1[t * a.heads + head];
+  const float s1 = MODE == kScanMlstm ? a.s1[t * a.heads + head] : 0.f;
   float v[CPT];
 #pragma unroll
   for (int i = 0; i < CPT; ++i) v[i] = mycol + i < a.vdim ? a.v[(t * a.heads + head) * a.vdim + mycol + i] : 0.f;
@@ -872,7 +837,7 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
   const float* ka = sh + l8 * 4;
   float out[CPT];
   if (MODE == kScanDelta) {
-    f32x2 A[CPT], B[CPT];
+    f32x2 A[CPT], B[CPT], C = 0ull;
 #pragma unroll
     for (int i = 0; i < CPT; ++i) A[i] = B[i] = 0ull;
 #pragma unroll
@@ -882,7 +847,8 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
       lds2(ka + DP + c * 32, q[0], q[1]);
       lds2(ka + 2 * DP + c * 32, g[0], g[1]);
 #pragma unroll
-      for (int e = 0; e < 2; ++e)
+      for (int e = 0; e < 2; ++e) {
+        C = fma2(k[e], q[e], C);
 #pragma unroll
         for (int i = 0; i < CPT; ++i) {
           const f32x2 s = mul2(S.v[i][2 * c + e], g[e]);
@@ -890,13 +856,16 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
           B[i] = fma2(s, q[e], B[i]);
           S.v[i][2 * c + e] = s;
         }
+      }
     }
+    const float2 cc = unpack2(C);
+    const float kq = sum8(cc.x + cc.y);
     f32x2 u2[CPT];
 #pragma unroll
     for (int i = 0; i < CPT; ++i) {
       const float2 x = unpack2(A[i]), y = unpack2(B[i]);
       const float u = s0 * (v[i] - sum8(x.x + x.y));
-      out[i] = fmaf(s1, u, sum8(y.x + y.y));
+      out[i] = fmaf(kq, u, sum8(y.x + y.y));
       u2[i] = pack2(u, u);
     }
 #pragma unroll
@@ -1053,7 +1022,7 @@ int mdb_delta_prep(const mdb_delta_prep_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(a.channels == 2 * a.kv_heads * a.dim + a.heads * a.vdim, MDB_ERR_ARG);
   MDB_REQUIRE(rows_present(a.q) && rows_present(a.k) && rows_present(a.v) && rows_present(a.b), MDB_ERR_ARG);
   MDB_REQUIRE(a.conv_q && a.conv_k && a.conv_v && (a.conv_state || a.taps == 1) && a.row_seq &&
-                  seqs_ok(a.cu_q, a.start, a.state_slot) && a.q_out && a.k_out && a.v_out && a.beta_out && a.kq_out,
+                  seqs_ok(a.cu_q, a.start, a.state_slot) && a.q_out && a.k_out && a.v_out && a.beta_out,
               MDB_ERR_ARG);
   MDB_REQUIRE(a.copy_cols == 0 || (rows_present(a.copy) && a.copy_out && a.copy_cols % 4 == 0 && a.copy_ld % 4 == 0 && rows_ok(a.copy)),
               MDB_ERR_ARG);
@@ -1066,8 +1035,9 @@ int mdb_delta_prep(const mdb_delta_prep_args* args, mdb_stream_t stream) {
       (a.q.parts != nullptr) == (a.v.parts != nullptr) && (a.copy_cols == 0 || (a.q.parts != nullptr) == (a.copy.parts != nullptr)) &&
       (a.dtype == MDB_BF16 || a.q.parts == nullptr)) {
     const int run = a.m >= 4096 ? 32 : (a.m >= 1024 ? 8 : 1);      // rows a warp walks
-    const int units = a.kv_heads + a.heads * ((a.vdim + 127) / 128) + 1 + (a.copy_cols + 127) / 128;
-    const dim3 grid((a.m + run - 1) / run, (units + kPrepWarps - 1) / kPrepWarps);
+    const int units = 2 * a.kv_heads + a.heads * ((a.vdim + 127) / 128) + 1 + (a.copy_cols + 127) / 128;
+    // the units of a row tile run next to one another, so that whole rows are read together
+    const dim3 grid((units + kPrepWarps - 1) / kPrepWarps, (a.m + run - 1) / run);
     const bool parts = a.q.parts != nullptr;
     const dim3 block(kPrepWarps * 32);
     if (a.dtype == MDB_F32) rc = mdb_launch(delta_prep_rows_kernel<float, false>, grid, block, 0, st, a, run);
@@ -1090,10 +1060,10 @@ int mdb_channel_decay(const mdb_decay_args* args, mdb_stream_t stream) {
   const mdb_decay_args a = *args;
   MDB_REQUIRE(a.m >= 0 && a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.dim_pad >= a.dim, MDB_ERR_ARG);
   if (a.m == 0) return MDB_OK;
-  MDB_REQUIRE(a.x && a.a_log && a.dt_bias && a.q && a.k && a.g && a.cross && a.row_seq && a.cu_q &&
+  MDB_REQUIRE(a.x && a.a_log && a.dt_bias && a.q && a.k && a.g && a.scalars && a.beta && a.row_seq && a.cu_q &&
                   a.ldx >= static_cast<int64_t>(a.heads) * a.dim,
               MDB_ERR_ARG);
-  MDB_REQUIRE(a.dim_pad % 4 == 0 && mdb_aligned16(a.g) && mdb_aligned16(a.q) && mdb_aligned16(a.k), MDB_ERR_ALIGN);
+  MDB_REQUIRE(a.dim_pad % 4 == 0 && mdb_aligned16(a.g) && mdb_aligned16(a.q) && mdb_aligned16(a.k) && mdb_aligned16(a.scalars), MDB_ERR_ALIGN);
   const dim3 grid(a.m, a.m >= 1024 ? 1 : (a.heads + 3) / 4);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (a.dim % 4 == 0 && a.ldx % 4 == 0 && mdb_aligned16(a.x) && mdb_aligned16(a.dt_bias))
@@ -1129,15 +1099,15 @@ int mdb_scan(const mdb_scan_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(a.mode == MDB_SCAN_DELTA || a.mode == MDB_SCAN_MLSTM, MDB_ERR_ARG);
   MDB_REQUIRE(a.bs >= 0 && a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.vdim > 0, MDB_ERR_ARG);
   if (a.bs == 0) return MDB_OK;
-  MDB_REQUIRE(a.q && a.k && a.v && a.s0 && a.s1 && a.state && seqs_ok(a.cu_q, a.start, a.state_slot), MDB_ERR_ARG);
+  MDB_REQUIRE(a.q && a.k && a.v && a.state && (a.mode == MDB_SCAN_DELTA ? a.fused == 0 || a.s0 : a.s0 && a.s1) && seqs_ok(a.cu_q, a.start, a.state_slot), MDB_ERR_ARG);
   MDB_REQUIRE(a.mode != MDB_SCAN_MLSTM || (a.mstate && a.kv_heads == a.heads), MDB_ERR_ARG);
   if (a.fused) {
     MDB_REQUIRE(rows_present(a.gate) && a.norm && a.y, MDB_ERR_ARG);
     MDB_REQUIRE(a.mode != MDB_SCAN_DELTA || (rows_present(a.raw_decay) && a.a_log && a.dt_bias), MDB_ERR_ARG);
   } else {
-    MDB_REQUIRE(a.out != nullptr && (a.mode == MDB_SCAN_DELTA ? a.g && a.cross : a.den != nullptr), MDB_ERR_ARG);
+    MDB_REQUIRE(a.out != nullptr && (a.mode == MDB_SCAN_DELTA ? a.g && a.scalars : a.den != nullptr), MDB_ERR_ARG);
   }
-  MDB_REQUIRE(mdb_aligned16(a.q) && mdb_aligned16(a.k) && mdb_aligned16(a.g) && mdb_aligned16(a.state) &&
+  MDB_REQUIRE(mdb_aligned16(a.q) && mdb_aligned16(a.k) && mdb_aligned16(a.g) && mdb_aligned16(a.state) && mdb_aligned16(a.scalars) &&
                   a.state_slot_stride % 4 == 0,
               MDB_ERR_ALIGN);
   MDB_REQUIRE(a.heads <= 65535 && a.bs <= 65535, MDB_ERR_UNSUPPORTED);

@@ -380,25 +380,24 @@ class HybridEngine:
         x = self._linear("mix_in", h, lw["in"])
         low = self.buf("delta_low", m, q0) if x.parts is not None else x.x[:, :q0]     # a1 | g1 columns as GEMM input
         outs = (self.buf("scan_q", m, kvh, dp, dtype=f32), self.buf("scan_k", m, kvh, dp, dtype=f32),
-                self.buf("scan_v", m, heads, vdim, dtype=f32), self.buf("scan_s0", m, heads, dtype=f32),
-                self.buf("scan_s1", m, kvh, dtype=f32))
+                self.buf("scan_v", m, heads, vdim, dtype=f32), self.buf("scan_s0", m, heads, dtype=f32))
         ops.delta_prep(self.dtype, m, b.bs, heads, kvh, dim, vdim, x.cols(q0), x.cols(k0), x.cols(v0), x.cols(b0),
                        (lw["conv_q"], lw["conv_k"], lw["conv_v"]), st["conv"], self._portions(b), outs, b.max_q == 1,
                        copy=x if x.parts is not None else None, copy_out=low if x.parts is not None else None)
-        q, k, v, beta, kq = outs
+        q, k, v, beta = outs
         raw = ops.gemm(low[:, a0:g0], lw["a2"], self.buf("delta_raw", m, lw["a2"].shape[0], dtype=f32))
         gate = self._linear("delta_gate", low[:, g0:q0], lw["g2"], parts=fused)
         y = self.buf(f"mix_o_{heads * vdim}", m, lw["o"].shape[1])
-        common = (ops.SCAN_DELTA, self.dtype, b.bs, heads, kvh, dim, vdim, q, k, v, beta, kq, st["s"], self._portions(b))
+        common = (ops.SCAN_DELTA, self.dtype, b.bs, heads, kvh, dim, vdim, q, k, v, beta, None, st["s"], self._portions(b))
         if fused:
             ops.scan(*common, eps=eps, raw_decay=ops.Rows(raw), a_log=lw["a_log"], dt_bias=lw["dt_bias"], gate=gate,
                      norm=lw["norm"], y=y)
         else:
             g = self.buf("scan_g", m, heads, dp, dtype=f32)
-            cross = self.buf("scan_cross", m, heads, 2, dtype=f32)
-            ops.channel_decay(raw, lw["a_log"], lw["dt_bias"], q, k, self._portions(b), g, cross, dim)
+            scalars = self.buf("scan_scalars", m, heads, 4, dtype=f32)
+            ops.channel_decay(raw, lw["a_log"], lw["dt_bias"], q, k, beta, self._portions(b), g, scalars, dim)
             o = self.buf("scan_o", m, heads, vdim, dtype=f32)
-            ops.scan(*common, g=g, cross=cross, out=o)
+            ops.scan(*common, g=g, scalars=scalars, out=o)
             ops.gated_norm(o, gate, lw["norm"], False, eps, y)
         return self._linear("mix_out", y, lw["o"])
 

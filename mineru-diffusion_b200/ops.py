@@ -669,9 +669,8 @@ def delta_prep(dtype: torch.dtype, m: int, bs: int, heads: int, kv_heads: int, d
                b: Rows, conv: tuple, conv_state: torch.Tensor, portions: tuple, outs: tuple, shift_state: bool,
                copy: Rows | None = None, copy_out: torch.Tensor | None = None) -> None:
     """``conv`` = fp32 [channels, taps] weights of q, k, v; ``conv_state`` [slots, taps - 1, channels]; ``portions`` =
-    (row_seq, cu_q, start, state_slot); ``outs`` = fp32 (q, k [m, kv_heads, dim_pad], v [m, heads, vdim], beta [m, heads],
-    k.q [m, kv_heads])."""
-    qo, ko, vo, bo, kqo = outs
+    (row_seq, cu_q, start, state_slot); ``outs`` = fp32 (q, k [m, kv_heads, dim_pad], v [m, heads, vdim], beta [m, heads])."""
+    qo, ko, vo, bo = outs
     row_seq, cu_q, start, slot = portions
     a = _lib.DeltaPrepArgs(
         dtype=_DTYPES[dtype], m=m, bs=bs, heads=heads, kv_heads=kv_heads, dim=dim, dim_pad=qo.shape[-1], vdim=vdim,
@@ -681,18 +680,19 @@ def delta_prep(dtype: torch.dtype, m: int, bs: int, heads: int, kv_heads: int, d
         conv_k=conv[1].data_ptr(), conv_v=conv[2].data_ptr(), conv_state=conv_state.data_ptr() or None,
         conv_slot_stride=conv_state.stride(0), num_slots=conv_state.shape[0], row_seq=row_seq.data_ptr(),
         cu_q=cu_q.data_ptr(), start=start.data_ptr(), state_slot=slot.data_ptr(), q_out=qo.data_ptr(), k_out=ko.data_ptr(),
-        v_out=vo.data_ptr(), beta_out=bo.data_ptr(), kq_out=kqo.data_ptr())
+        v_out=vo.data_ptr(), beta_out=bo.data_ptr())
     _lib.check(_lib.lib().mdb_delta_prep(a, _stream()), "mdb_delta_prep")
 
 
 def channel_decay(x: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, q: torch.Tensor, k: torch.Tensor,
-                  portions: tuple, out: torch.Tensor, cross: torch.Tensor, dim: int) -> None:
-    """out [m, heads, dim_pad] = exp(-exp(a_log) softplus(x + dt_bias)); x fp32 [m, >= heads * dim]; cross [m, heads, 2]: the
-    products of a portion's odd tokens with the token before (q, k of ``delta_prep``)."""
+                  beta: torch.Tensor, portions: tuple, out: torch.Tensor, scalars: torch.Tensor, dim: int) -> None:
+    """out [m, heads, dim_pad] = exp(-exp(a_log) softplus(x + dt_bias)); x fp32 [m, >= heads * dim]; scalars [m, heads, 4] =
+    (k.q, for a portion's odd tokens the products with the token before, beta); q, k, beta of ``delta_prep``."""
     m, heads, dp = out.shape
     row_seq, cu_q, _, _ = portions
     a = _lib.DecayArgs(m, heads, q.shape[1], dim, dp, x.data_ptr(), _rows(x, "x"), a_log.data_ptr(), dt_bias.data_ptr(),
-                       q.data_ptr(), k.data_ptr(), out.data_ptr(), cross.data_ptr(), row_seq.data_ptr(), cu_q.data_ptr())
+                       q.data_ptr(), k.data_ptr(), beta.data_ptr(), out.data_ptr(), scalars.data_ptr(), row_seq.data_ptr(),
+                       cu_q.data_ptr())
     _lib.check(_lib.lib().mdb_channel_decay(a, _stream()), "mdb_channel_decay")
 
 
@@ -709,7 +709,7 @@ SCAN_DELTA, SCAN_MLSTM = 0, 1
 
 
 def scan(mode: int, dtype: torch.dtype, bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q, k, v, s0, s1, state,
-         portions: tuple, eps: float = 0.0, g=None, cross=None, mstate=None, den=None, out=None, raw_decay: Rows | None = None,
+         portions: tuple, eps: float = 0.0, g=None, scalars=None, mstate=None, den=None, out=None, raw_decay: Rows | None = None,
          a_log=None, dt_bias=None, gate: Rows | None = None, norm=None, per_head_norm: bool = False, y=None) -> None:
     """The recurrence over every sequence's portion; ``state`` [slots, heads, vdim (mLSTM: + 1), dim_pad] fp32.  With ``y``
     the fused one-token form runs (decay from ``raw_decay``, gated norm into ``y``), else ``out`` [m, heads, vdim] fp32
@@ -717,9 +717,9 @@ def scan(mode: int, dtype: torch.dtype, bs: int, heads: int, kv_heads: int, dim:
     _, cu_q, start, slot = portions
     a = _lib.ScanArgs(
         mode=mode, dtype=_DTYPES[dtype], fused=int(y is not None), bs=bs, heads=heads, kv_heads=kv_heads, dim=dim,
-        dim_pad=q.shape[-1], vdim=vdim, eps=eps, q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), g=_ptr(g), s0=s0.data_ptr(),
-        s1=s1.data_ptr(), state=state.data_ptr(), state_slot_stride=state.stride(0), num_slots=state.shape[0],
-        mstate=_ptr(mstate), cross=_ptr(cross), den=_ptr(den), cu_q=cu_q.data_ptr(), start=start.data_ptr(), state_slot=slot.data_ptr(),
+        dim_pad=q.shape[-1], vdim=vdim, eps=eps, q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), g=_ptr(g), s0=_ptr(s0),
+        s1=_ptr(s1), state=state.data_ptr(), state_slot_stride=state.stride(0), num_slots=state.shape[0],
+        mstate=_ptr(mstate), scalars=_ptr(scalars), den=_ptr(den), cu_q=cu_q.data_ptr(), start=start.data_ptr(), state_slot=slot.data_ptr(),
         out=_ptr(out), raw_decay=_rows_c(raw_decay), a_log=_ptr(a_log), dt_bias=_ptr(dt_bias), gate=_rows_c(gate),
         norm=_ptr(norm), norm_head_stride=vdim if per_head_norm else 0, y=_ptr(y), ldy=0 if y is None else _rows(y, "y"))
     _lib.check(_lib.lib().mdb_scan(a, _stream()), "mdb_scan")

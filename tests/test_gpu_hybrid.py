@@ -138,10 +138,10 @@ def _delta_run(case, H, KH, D, DV, counts, dtype, fused=False):
         p = portions_of([n], [at], [1])
         rows = {k: ops.Rows(torch.nn.functional.pad(v[at:at + n], (0, -v.shape[1] % 4)).to(dtype).to(DEV)) for k, v in x.items()}
         q, k = (torch.full((n, KH, dp), 9.0, device=DEV) for _ in range(2))
-        v, beta, kq = (torch.zeros(n, H, DV, device=DEV), torch.zeros(n, H, device=DEV), torch.zeros(n, KH, device=DEV))
-        ops.delta_prep(dtype, n, 1, H, KH, D, DV, rows["q"], rows["k"], rows["v"], rows["b"], cw, cstate, p, (q, k, v, beta, kq), n == 1)
+        v, beta = torch.zeros(n, H, DV, device=DEV), torch.zeros(n, H, device=DEV)
+        ops.delta_prep(dtype, n, 1, H, KH, D, DV, rows["q"], rows["k"], rows["v"], rows["b"], cw, cstate, p, (q, k, v, beta), n == 1)
         r = raw[at:at + n].contiguous().to(DEV)
-        common = (ops.SCAN_DELTA, dtype, 1, H, KH, D, DV, q, k, v, beta, kq, state, p)
+        common = (ops.SCAN_DELTA, dtype, 1, H, KH, D, DV, q, k, v, beta, None, state, p)
         if fused and n == 1:
             y = torch.zeros(1, H * DV, dtype=dtype, device=DEV)
             gate = torch.full((1, (H * DV + 3) // 4 * 4), 100.0, dtype=dtype, device=DEV)      # sigmoid = 1
@@ -149,9 +149,9 @@ def _delta_run(case, H, KH, D, DV, counts, dtype, fused=False):
                      norm=torch.ones(DV, device=DEV), y=y)
             outs.append(y.float().view(1, H, DV))
         else:
-            g, o, cross = torch.zeros(n, H, dp, device=DEV), torch.zeros(n, H, DV, device=DEV), torch.full((n, H, 2), 9.0, device=DEV)
-            ops.channel_decay(r, a_log.to(DEV), dt.to(DEV), q, k, p, g, cross, D)
-            ops.scan(*common, g=g, cross=cross, out=o)
+            g, o, sc = torch.zeros(n, H, dp, device=DEV), torch.zeros(n, H, DV, device=DEV), torch.full((n, H, 4), 9.0, device=DEV)
+            ops.channel_decay(r, a_log.to(DEV), dt.to(DEV), q, k, beta, p, g, sc, D)
+            ops.scan(*common, g=g, scalars=sc, out=o)
             outs.append(orc.rms(o, 1e-5) if fused else o)
         at += n
     torch.cuda.synchronize()
@@ -176,6 +176,14 @@ def test_delta_scan_fused_token(H, KH, D, DV, taps):
     assert rel(_delta_run(case, H, KH, D, DV, [30] + [1] * 10, F32, fused=True), ref) < 2e-5
 
 
+def delta_scalars(q, k, g, beta):
+    """The per-token scalars of the prompt scan: k.q, the products with the token before, beta."""
+    s = torch.zeros(*beta.shape, 4)
+    s[..., 0], s[..., 3] = (k * q).sum(-1), beta
+    s[1:, :, 1], s[1:, :, 2] = (g[1:] * k[:-1] * k[1:]).sum(-1), (g[1:] * k[:-1] * q[1:]).sum(-1)
+    return s
+
+
 def test_delta_remembers_a_far_key():
     """A value written under one key long ago, no decay and orthogonal writes since, comes back whole."""
     ops, T, D, DV = pkg.ops, 400, 64, 16
@@ -185,12 +193,10 @@ def test_delta_remembers_a_far_key():
     q = torch.zeros(T, 1, D)
     q[:, 0, 0] = 1.0
     v = torch.randn(T, 1, DV, generator=gen(1))
-    one, z = torch.ones(T, 1), (k * q).sum(-1)
+    sc = delta_scalars(q, k, torch.ones_like(k), torch.ones(T, 1))
     state, o = torch.zeros(1, 1, DV, D, device=DEV), torch.zeros(T, 1, DV, device=DEV)
-    cross = torch.zeros(T, 1, 2)
-    cross[1:, :, 0], cross[1:, :, 1] = (k[:-1] * k[1:]).sum(-1), (k[:-1] * q[1:]).sum(-1)
-    ops.scan(ops.SCAN_DELTA, F32, 1, 1, 1, D, DV, q.to(DEV), k.to(DEV), v.to(DEV), one.to(DEV), z.to(DEV), state,
-             portions_of([T], slots=[0]), g=torch.ones(T, 1, D, device=DEV), cross=cross.to(DEV), out=o)
+    ops.scan(ops.SCAN_DELTA, F32, 1, 1, 1, D, DV, q.to(DEV), k.to(DEV), v.to(DEV), None, None, state,
+             portions_of([T], slots=[0]), g=torch.ones(T, 1, D, device=DEV), scalars=sc.to(DEV), out=o)
     o = o.cpu()
     assert float(o[:3].abs().max()) == 0 and float((o[3:, 0] - v[3, 0]).abs().max()) < 1e-5
 
@@ -242,12 +248,10 @@ def test_scans_of_unequal_portions_in_one_batch():
     T = sum(counts)
     q, k, g = (torch.randn(T, H, D, generator=gen(i)) for i in range(3))
     g, k = torch.sigmoid(g + 2), torch.nn.functional.normalize(k, dim=-1)
-    v, beta, kq = torch.randn(T, H, DV, generator=gen(4)), torch.rand(T, H, generator=gen(5)), (q * k).sum(-1)
+    v, beta = torch.randn(T, H, DV, generator=gen(4)), torch.rand(T, H, generator=gen(5))
     state, o = torch.zeros(3, H, DV, D, device=DEV), torch.full((T, H, DV), 4.0, device=DEV)
-    cross = torch.zeros(T, H, 2)
-    cross[1:, :, 0], cross[1:, :, 1] = (g[1:] * k[:-1] * k[1:]).sum(-1), (g[1:] * k[:-1] * q[1:]).sum(-1)
-    ops.scan(ops.SCAN_DELTA, F32, 4, H, H, D, DV, *(t.to(DEV) for t in (q, k, v, beta, kq)), state, portions_of(counts, slots=slots),
-             g=g.to(DEV), cross=cross.to(DEV), out=o)
+    ops.scan(ops.SCAN_DELTA, F32, 4, H, H, D, DV, *(t.to(DEV) for t in (q, k, v)), None, None, state, portions_of(counts, slots=slots),
+             g=g.to(DEV), scalars=delta_scalars(q, k, g, beta).to(DEV), out=o)
     at = 0
     for n, s in zip(counts, slots):
         r = slice(at, at + n)
