@@ -227,7 +227,7 @@ __device__ __forceinline__ float dot4(float4 a, float4 b) { return a.x * b.x + a
 __device__ __forceinline__ float4 scale4(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
 
 template <typename T, bool PARTS>
-__global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_rows_kernel(const mdb_delta_prep_args a, const int run) {
+__global__ void __launch_bounds__(kPrepWarps * 32, 7) delta_prep_rows_kernel(const mdb_delta_prep_args a, const int run) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31, c = lane * 4;
@@ -1034,7 +1034,7 @@ int mdb_delta_prep(const mdb_delta_prep_args* args, mdb_stream_t stream) {
       mdb_aligned16(a.conv_v) && (a.q.parts != nullptr) == (a.k.parts != nullptr) &&
       (a.q.parts != nullptr) == (a.v.parts != nullptr) && (a.copy_cols == 0 || (a.q.parts != nullptr) == (a.copy.parts != nullptr)) &&
       (a.dtype == MDB_BF16 || a.q.parts == nullptr)) {
-    const int run = a.m >= 4096 ? 32 : (a.m >= 1024 ? 8 : 1);      // rows a warp walks
+    const int run = a.m >= 4096 ? 16 : (a.m >= 1024 ? 8 : 1);      // rows a warp walks
     const int units = 2 * a.kv_heads + a.heads * ((a.vdim + 127) / 128) + 1 + (a.copy_cols + 127) / 128;
     // the units of a row tile run next to one another, so that whole rows are read together
     const dim3 grid((units + kPrepWarps - 1) / kPrepWarps, (a.m + run - 1) / run);
