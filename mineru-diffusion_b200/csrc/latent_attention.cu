@@ -55,17 +55,19 @@ __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], 
 
 constexpr int kLatKeys = 32, kLatHeads = 16, kLatThreads = 256;
 constexpr int kLatPStride = kLatKeys + 8;
+constexpr int kLatSStride = kLatKeys + 8;
 
 template <int WIDTH>
 struct LatPlan {
   static constexpr int kStride = WIDTH + 8;                    // bf16 elements; the pad spreads rows over the banks
   static constexpr int kTile = kLatKeys * kStride * 2;
   static constexpr int kStages = WIDTH > 256 ? 2 : 3;          // two CTAs per SM at every width
-  static constexpr int kOffQ = 0;
-  static constexpr int kOffTiles = kOffQ + kLatHeads * kStride * 2;
-  static constexpr int kOffS = kOffTiles + kStages * kTile;            // [2][16][32] fp32
-  static constexpr int kOffP = kOffS + 2 * kLatHeads * kLatKeys * 4;      // [2][16][40] bf16: high and low parts
-  static constexpr int kOffF = kOffP + 2 * kLatHeads * kLatPStride * 2;   // [16] fp32
+  static constexpr int kOffTiles = 0;
+  static constexpr int kOffS = kOffTiles + kStages * kTile;                        // [8 warps][16][40] fp32 partial scores;
+  static constexpr int kQBytes = kLatHeads * kStride * 2;                          // q passes through it on its way to registers
+  static constexpr int kSBytes = 8 * kLatHeads * kLatSStride * 4;
+  static constexpr int kOffP = kOffS + (kQBytes > kSBytes ? kQBytes : kSBytes);    // [2][16][40] bf16: high and low parts
+  static constexpr int kOffF = kOffP + 2 * kLatHeads * kLatPStride * 2;            // [16] fp32
   static constexpr int kBytes = kOffF + 64;
 };
 
@@ -91,7 +93,7 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_mma_kernel(const Late
     return;
   }
   const uint32_t base = smem_u32(lat_smem);
-  bf16* qs = reinterpret_cast<bf16*>(lat_smem + P::kOffQ);
+  bf16* qs = reinterpret_cast<bf16*>(lat_smem + P::kOffS);
   {
     const bf16* q = static_cast<const bf16*>(a.q) + (static_cast<int64_t>(row) * a.heads + head0) * WIDTH;
     for (int i = threadIdx.x; i < kLatHeads * (WIDTH / 8); i += kLatThreads) {
@@ -120,6 +122,14 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_mma_kernel(const Late
   };
 #pragma unroll
   for (int t = 0; t < P::kStages - 1; ++t) load_tile(t);
+  // warp w owns columns [w, w + 1) * WIDTH / 8 of q (in registers), of the scores' sum and of the output
+  constexpr int KS = WIDTH / 128;          // k steps of 16 of a warp's share
+  const int c_first = warp * (WIDTH / 8);
+  uint32_t qf[KS][4];
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < KS; ++k) ldsm4(base + P::kOffS + ((lane & 15) * P::kStride + c_first + 16 * k + (lane >> 4) * 8) * 2, qf[k]);
+  __syncthreads();                         // the scores' buffer is free
   float acc[NT][4];
 #pragma unroll
   for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
@@ -135,31 +145,36 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_mma_kernel(const Late
     load_tile(t + P::kStages - 1);
     const uint32_t tile = base + P::kOffTiles + (t % P::kStages) * P::kTile;
     {
-      // scores: warp w has keys 8 (w & 3) .. + 8 and half of the width
-      const int j = warp & 3, kh = warp >> 2;
-      float s[4] = {0.f, 0.f, 0.f, 0.f};
-      const uint32_t qa = base + P::kOffQ + ((lane & 15) * P::kStride + kh * (WIDTH / 2) + (lane >> 4) * 8) * 2;
-      const uint32_t ka = tile + ((8 * j + (lane & 7)) * P::kStride + kh * (WIDTH / 2) + (lane >> 3) * 8) * 2;
+      // scores of all 32 keys over this warp's columns: four independent products
+      float sc[4][4];
 #pragma unroll
-      for (int k = 0; k < WIDTH / 2; k += 32) {
-        uint32_t q0[4], q1[4], kb[4];
-        ldsm4(qa + k * 2, q0);
-        ldsm4(qa + (k + 16) * 2, q1);
-        ldsm4(ka + k * 2, kb);
-        mma16816(s, q0, kb[0], kb[1]);
-        mma16816(s, q1, kb[2], kb[3]);
+      for (int n = 0; n < 4; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+#pragma unroll
+      for (int k = 0; k < KS; ++k) {
+        uint32_t b0[4], b1[4];             // first and second eight columns of the step, keys 0..31
+        const uint32_t ka = tile + (lane * P::kStride + c_first + 16 * k) * 2;
+        ldsm4(ka, b0);
+        ldsm4(ka + 16, b1);
+#pragma unroll
+        for (int n = 0; n < 4; ++n) mma16816(sc[n], qf[k], b0[n], b1[n]);
       }
-      float* so = ss + (kh * kLatHeads + g) * kLatKeys + 8 * j + 2 * (lane & 3);
-      *reinterpret_cast<float2*>(so) = make_float2(s[0], s[1]);
-      *reinterpret_cast<float2*>(so + 8 * kLatKeys) = make_float2(s[2], s[3]);
+      float* so = ss + (warp * kLatHeads + g) * kLatSStride + 2 * (lane & 3);
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        *reinterpret_cast<float2*>(so + 8 * n) = make_float2(sc[n][0], sc[n][1]);
+        *reinterpret_cast<float2*>(so + 8 * kLatSStride + 8 * n) = make_float2(sc[n][2], sc[n][3]);
+      }
     }
     __syncthreads();
     {
-      const float2 s0 = *reinterpret_cast<const float2*>(ss + srow * kLatKeys + 2 * sj);
-      const float2 s1 = *reinterpret_cast<const float2*>(ss + (kLatHeads + srow) * kLatKeys + 2 * sj);
+      float2 sv[8];
+#pragma unroll
+      for (int w = 0; w < 8; ++w) sv[w] = *reinterpret_cast<const float2*>(ss + (w * kLatHeads + srow) * kLatSStride + 2 * sj);
+      const float x0 = ((sv[0].x + sv[1].x) + (sv[2].x + sv[3].x)) + ((sv[4].x + sv[5].x) + (sv[6].x + sv[7].x));
+      const float x1 = ((sv[0].y + sv[1].y) + (sv[2].y + sv[3].y)) + ((sv[4].y + sv[5].y) + (sv[6].y + sv[7].y));
       const int key = k_begin + t * kLatKeys + 2 * sj;
-      const float a0 = key < k_end ? (s0.x + s1.x) * a.scale_log2 : -INFINITY;
-      const float a1 = key + 1 < k_end ? (s0.y + s1.y) * a.scale_log2 : -INFINITY;
+      const float a0 = key < k_end ? x0 * a.scale_log2 : -INFINITY;
+      const float a1 = key + 1 < k_end ? x1 * a.scale_log2 : -INFINITY;
       float mx = fmaxf(a0, a1);
 #pragma unroll
       for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -184,11 +199,10 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_mma_kernel(const Late
         ldsm4(pa, ph[ks]);
         ldsm4(pa + kLatHeads * kLatPStride * 2, pl[ks]);
       }
-      const int c0 = warp * (WIDTH / 8);
 #pragma unroll
       for (int i = 0; i < NT; ++i) {
         uint32_t v[4];                     // keys 0..31 of eight columns
-        ldsm4_t(tile + (lane * P::kStride + c0 + 8 * i) * 2, v);
+        ldsm4_t(tile + (lane * P::kStride + c_first + 8 * i) * 2, v);
         mma16816(acc[i], ph[0], v[0], v[1]);
         mma16816(acc[i], pl[0], v[0], v[1]);
         mma16816(acc[i], ph[1], v[2], v[3]);
@@ -202,7 +216,7 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_mma_kernel(const Late
   __syncthreads();
   if (sj == 0) fs[srow] = 1.0f / l_run;
   __syncthreads();
-  const int c0 = warp * (WIDTH / 8) + 2 * (lane & 3);
+  const int c0 = c_first + 2 * (lane & 3);
   if (a.nsplit == 1) {
     bf16* out = static_cast<bf16*>(a.out) + (static_cast<int64_t>(row) * a.heads + head0) * WIDTH;
     const float f0 = fs[g], f1 = fs[g + 8];
