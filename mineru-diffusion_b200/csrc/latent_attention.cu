@@ -4,10 +4,9 @@
 //
 //   latent_attn_mma_kernel   bf16: a CTA takes 16 heads of one token and a range of its keys (split over CTAs, merged by
 //                            latent_combine_kernel).  Latent tiles of 32 keys come through a cp.async ring;
-//                            scores and outputs are m16n8k16 products, the 16 heads being the 16 rows.  The work is
-//                            bound by the latent stream (a key feeds 16 heads x 4 x width flop), which is why the
-//                            narrow warp-level product suffices here.  Softmax in fp32; the weights enter the second
-//                            product as the sum of two bf16 numbers, so they keep 16 significant bits.
+//                            scores and outputs are m16n8k16 products, the 16 heads being the 16 rows: a 128-row
+//                            tile of the tensor-memory kind would be seven-eighths empty.  Softmax in fp32; the weights
+//                            enter the second product as the sum of two bf16 numbers, so they keep 16 significant bits.
 //   latent_attn_rows_kernel  fp32, and widths the first kernel does not take: one CTA per (token, head), a warp per key.
 #include "mdb_common.cuh"
 

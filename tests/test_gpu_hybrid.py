@@ -616,3 +616,21 @@ def test_trace_replay_writes_wanted_logits(tmp_path):
     for step, places in ((1, [120, 122]), (2, [1, 123]), (3, [49])):
         got = torch.frombuffer(bytearray((out / f"{step}.f32").read_bytes()), dtype=torch.float32).view(len(places), raw["vocab"])
         _close(got, ref[places], "float32")
+
+
+def test_generate_command_line_runs_a_model_folder(tmp_path, capsys):
+    import json
+    from importlib import import_module
+    from safetensors.torch import save_file
+    t = hc.tensors(WIDE, seed=6)
+    save_file(t, str(tmp_path / "model.safetensors"))
+    (tmp_path / "config.json").write_text(json.dumps(WIDE))
+    gen = import_module("mineru-diffusion_b200.generate")
+    args = ["--model", str(tmp_path), "--prompt", "5,6,7", "--prompt", "9", "--greedy", "--dtype", "float32", "--max-new-tokens", "8",
+            "--max-num-seqs", "2", "--max-model-len", "512"]
+    assert gen.main(args) == 0
+    lines = [json.loads(x) for x in capsys.readouterr().out.splitlines() if x.startswith("{")]
+    assert [x["prompt"] for x in lines] == [[5, 6, 7], [9]]
+    for x in lines:
+        assert x["tokens"] == _greedy(WIDE, t, x["prompt"], 8)
+    assert gen.main(args + ["--max-new-tokens", "600"]) == 2

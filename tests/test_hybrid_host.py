@@ -211,3 +211,12 @@ def test_oracle_mlstm_matches_unscaled_sums():
         # the floor exp(-m) is in the running maximum's units: 1 in unscaled ones
         ref = (s[:, None] * v[:t + 1, 0]).sum(0) / torch.maximum(s.sum().abs(), torch.tensor(1.0, dtype=torch.float64))
         assert torch.allclose(o[t, 0], ref, atol=1e-4)
+
+
+def test_generate_command_line():
+    from importlib import import_module
+    gen = import_module("mineru-diffusion_b200.generate")
+    a = gen.parse(["--model", "m", "--prompt", "1,2 3", "--prompt", "7", "--greedy", "--stop", "4", "--stop", "5"])
+    assert a.prompt == [[1, 2, 3], [7]] and a.greedy and a.stop == [4, 5] and a.dtype == "bfloat16"
+    with pytest.raises(SystemExit):
+        gen.parse(["--model", "m", "--prompt", ","])
