@@ -352,8 +352,9 @@ typedef struct {
 } mdb_rows;
 
 enum { MDB_GEMM_PLAIN = 0, MDB_GEMM_HEADS = 1, MDB_GEMM_EXPERTS = 2 };
-enum { MDB_ACT_NONE = 0, MDB_ACT_RELU2 = 1 };
-/* y = act(x W^T).  PLAIN: x [m, k], w [n, k], y [m, n].  HEADS: head h takes columns [h k, (h + 1) k) of x, rows
+enum { MDB_ACT_NONE = 0, MDB_ACT_RELU2 = 1, MDB_ACT_RELU_GLU = 2 };
+/* y = act(x W^T).  PLAIN: x [m, k], w [n, k], y [m, n]; with RELU_GLU w is [2 n, k], gate rows first, and y =
+ * relu(gate) * up (activation type, n % 128 == 0).  HEADS: head h takes columns [h k, (h + 1) k) of x, rows
  * [h n, (h + 1) n) of w and writes columns [h n, (h + 1) n) of y.  EXPERTS: rows of x and y are laid out by expert
  * in tiles of 128 (mdb_moe_plan); tile t uses rows [e n, (e + 1) n) of w, e = tile_expert[t], for t < *num_tiles;
  * m = rows of the buffers; max_rows_per_expert (0: unknown) bounds the rows in use in a tile.  y is of the
@@ -371,9 +372,10 @@ typedef struct {
 } mdb_gemm_args;
 int mdb_gemm(const mdb_gemm_args* args, mdb_stream_t stream);
 
-/* residual [m][width_pad] fp32: with ids, = embed[id] * embed_scale, else += ; plus the rows of up to two
- * projections, plus sum_k moe_weight[row][k] * moe_rows[moe_slot[row][k]].  y (may be NULL) = residual / sqrt(mean
- * of its first `width` columns squared + eps) * weight. */
+/* residual [m][width_pad] fp32: with ids, = embed[id] * embed_scale, else *= res_scale; plus the rows of up to two
+ * projections, plus sum_k moe_weight[row][k] * moe_rows[moe_slot[row][k]].  y (may be NULL) = norm(residual) * weight,
+ * norm(x) = x / sqrt(mean of its first `width` columns squared + eps); weight NULL: y = residual.  With `post` the residual
+ * itself becomes norm(residual) * weight, and y = residual or, with weight2, norm(residual) * weight2. */
 typedef struct {
   int32_t dtype, m, width, width_pad;
   float* residual;
@@ -390,6 +392,9 @@ typedef struct {
   int64_t ldy;
   float embed_scale, eps;
   int32_t moe_top;
+  int32_t post;
+  const float* weight2;
+  float res_scale;
 } mdb_residual_norm_args;
 int mdb_residual_norm(const mdb_residual_norm_args* args, mdb_stream_t stream);
 
@@ -421,6 +426,19 @@ typedef struct {
   float eps;
 } mdb_gated_norm_args;
 int mdb_gated_norm(const mdb_gated_norm_args* args, mdb_stream_t stream);
+
+/* y[row][c] for n columns in `parts` equal parts, each normalised by its own root mean square:
+ * gate_first: norm(o * silu(gate)) * weight, else norm(o) * weight * sigmoid(gate); times out_scale.  o fp32 [m][n]. */
+typedef struct {
+  int32_t dtype, m, n, parts, gate_first;
+  float out_scale, eps;
+  const float* o;
+  mdb_rows gate;
+  const float* weight;
+  void* y;
+  int64_t ldy;
+} mdb_part_norm_args;
+int mdb_part_norm(const mdb_part_norm_args* args, mdb_stream_t stream);
 
 /* Key channels of a recurrent head as the state stores them (a multiple of 64; 0: not supported), and the number of
  * copies of the mLSTM maximum a head keeps. */
@@ -490,14 +508,41 @@ typedef struct {
 } mdb_mlstm_prep_args;
 int mdb_mlstm_prep(const mdb_mlstm_prep_args* args, mdb_stream_t stream);
 
+/* Inputs of the decay scan (a linear recurrence with one decay per head): v [m][heads][vdim], k, q [m][kv_heads][dim_pad]
+ * = silu of the projections or, with taps > 0, silu of a causal short convolution with bias over time (channels ordered
+ * v | k | q; conv fp32 [channels][taps], the last tap is the current token's; conv_state as in mdb_delta_prep).  With dt:
+ * step = softplus(dt + dt_bias), decay = exp(-exp(a_log) * step); else step = 1, decay = decay_const[h]. */
+typedef struct {
+  int32_t dtype, m, bs, heads, kv_heads, dim, dim_pad, vdim, taps, channels, shift_state;
+  mdb_rows q, k, v, dt;
+  const float* conv;
+  const float* conv_bias;
+  void* conv_state;
+  int64_t conv_slot_stride, num_slots;
+  const int32_t* row_seq;
+  const int32_t* cu_q;
+  const int32_t* start;
+  const int32_t* state_slot;
+  const float* a_log;
+  const float* dt_bias;
+  const float* decay_const;
+  float* q_out;
+  float* k_out;
+  float* v_out;
+  float* decay_out; /* [m][heads] */
+  float* step_out;
+} mdb_decay_prep_args;
+int mdb_decay_prep(const mdb_decay_prep_args* args, mdb_stream_t stream);
+
 /* The recurrences over every sequence's portion; state [slot][heads][vdim][dim_pad] fp32 is read and written.
  * DELTA: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q; beta comes
  * with the scalars of mdb_channel_decay, in the fused form as s0.  MLSTM: m' = max(f + m, i);
  * S, n <- exp(f + m - m') (.) + exp(i - m') k (v^T, 1); o = S^T q, den [m][heads] = max(|n . q|, exp(-m')) + 1e-6;
  * s0 = i, s1 = f; its state has one more column per head (vdim + 1), which is n; mstate [slot][heads][mdb_scan_blocks].
+ * DECAY: S <- s0 S + s1 k v^T; o = S^T q + skip[h] v (skip may be NULL); with `fused` only the form changes, out is written.
  * out [m][heads][vdim] fp32; with `fused` (every portion is one token) the decay comes from raw_decay + dt_bias and
  * a_log, and y = the gated norm of o / den (as mdb_gated_norm) is written instead. */
-enum { MDB_SCAN_DELTA = 0, MDB_SCAN_MLSTM = 1 };
+enum { MDB_SCAN_DELTA = 0, MDB_SCAN_MLSTM = 1, MDB_SCAN_DECAY = 2 };
 typedef struct {
   int32_t mode, dtype, fused, bs, heads, kv_heads, dim, dim_pad, vdim;
   float eps;
@@ -524,6 +569,7 @@ typedef struct {
   int64_t norm_head_stride;
   void* y;
   int64_t ldy;
+  const float* skip; /* DECAY */
 } mdb_scan_args;
 int mdb_scan(const mdb_scan_args* args, mdb_stream_t stream);
 
@@ -568,6 +614,51 @@ int mdb_gather_latents(int dtype, const void* cache, const int32_t* block_table,
 int mdb_attn_causal_varlen(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride,
                            void* out, int64_t out_stride, const int32_t* cu_q, const int32_t* cu_k, int nseq, int max_q,
                            int64_t total_q, int64_t total_k, int hq, int hkv, float scale, mdb_stream_t stream);
+
+/* Queries and keys of rotary attention: per head RMSNorm (weight fp32 [dim]) and rotation of channel pairs (2 i, 2 i + 1),
+ * i < rot_dims / 2, by row_pos * inv_freq[i].  q_out [m][heads][dim_pad]; k and the values v as they come go to row
+ * slots[row] (-1: skipped) of the caches [slots][kv_heads][dim_pad]. */
+typedef struct {
+  int32_t dtype, m, heads, kv_heads, dim, dim_pad, rot_dims;
+  float eps;
+  mdb_rows q, k, v;
+  const float* q_norm;
+  const float* k_norm;
+  const double* inv_freq;
+  const int32_t* row_pos;
+  const int32_t* slots;
+  int64_t num_slots;
+  void* q_out;
+  void* k_cache;
+  void* v_cache;
+} mdb_rotary_commit_args;
+int mdb_rotary_commit(const mdb_rotary_commit_args* args, mdb_stream_t stream);
+
+/* Causal grouped-query attention over the paged caches of mdb_rotary_commit: the row at position p of its sequence sees
+ * keys max(0, p - window + 1) .. p (window 0: all).  sink: one more term exp(0) in the softmax's denominator.  Head h's
+ * output is multiplied by out_scale and, with a gate, by sigmoid(gate[row][h]); out [m] rows of ld_out elements, head h at
+ * column h * dim.  max_q = longest portion, max_ctx = longest context of the step (bounds); portions of many tokens take
+ * the tensor-memory kernel (bf16, dim_pad 128), which needs cu_q and start. */
+typedef struct {
+  int32_t dtype, m, bs, heads, kv_heads, dim, dim_pad, window, sink, max_q, nsplit;
+  float scale, out_scale;
+  const void* q;
+  const void* k_cache;
+  const void* v_cache;
+  const int32_t* block_table;
+  const int32_t* row_seq;
+  const int32_t* row_pos;
+  const int32_t* cu_q;
+  const int32_t* start;
+  int32_t table_stride, num_pages;
+  mdb_rows gate;
+  void* out;
+  int64_t ld_out;
+  void* workspace;
+  int64_t workspace_bytes;
+} mdb_window_attn_args;
+int64_t mdb_window_attn_workspace_bytes(int m, int heads, int dim_pad, int nsplit);
+int mdb_window_attn(const mdb_window_attn_args* args, mdb_stream_t stream);
 
 /* token = argmax of logits / temperature + Gumbel noise (seed, *step_dev, row), or of the logits where the row's
  * temperature is 0; status_out (may be NULL) receives and clears the device status word. */

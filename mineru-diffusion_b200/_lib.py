@@ -30,13 +30,30 @@ GemmArgs = _struct("GemmArgs", [
 ResidualNormArgs = _struct("ResidualNormArgs", [
     ("dtype", _i), ("m", _i), ("width", _i), ("width_pad", _i), ("residual", _p), ("ids", _p), ("embed", _p), ("vocab", _i64),
     ("add", Rows * 2), ("moe_rows", _p), ("moe_ld", _i64), ("moe_slot", _p), ("moe_weight", _p), ("weight", _p), ("y", _p),
-    ("ldy", _i64), ("embed_scale", _f), ("eps", _f), ("moe_top", _i)])
+    ("ldy", _i64), ("embed_scale", _f), ("eps", _f), ("moe_top", _i), ("post", _i), ("weight2", _p), ("res_scale", _f)])
 RmsSegment = _struct("RmsSegment", [
     ("src", Rows), ("weight", _p), ("out", _p), ("ld_out", _i64), ("slots", _p), ("num_slots", _i64), ("n", _i),
     ("n_pad", _i), ("eps", _f)])
 GatedNormArgs = _struct("GatedNormArgs", [
     ("dtype", _i), ("m", _i), ("heads", _i), ("vdim", _i), ("o", _p), ("den", _p), ("gate", Rows), ("weight", _p), ("y", _p),
     ("ldy", _i64), ("weight_head_stride", _i), ("eps", _f)])
+PartNormArgs = _struct("PartNormArgs", [(n, _i) for n in ("dtype", "m", "n", "parts", "gate_first")] + [
+    ("out_scale", _f), ("eps", _f), ("o", _p), ("gate", Rows), ("weight", _p), ("y", _p), ("ldy", _i64)])
+DecayPrepArgs = _struct("DecayPrepArgs", [(n, _i) for n in (
+    "dtype", "m", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim", "taps", "channels", "shift_state")] + [
+    ("q", Rows), ("k", Rows), ("v", Rows), ("dt", Rows), ("conv", _p), ("conv_bias", _p), ("conv_state", _p),
+    ("conv_slot_stride", _i64), ("num_slots", _i64), ("row_seq", _p), ("cu_q", _p), ("start", _p), ("state_slot", _p),
+    ("a_log", _p), ("dt_bias", _p), ("decay_const", _p), ("q_out", _p), ("k_out", _p), ("v_out", _p), ("decay_out", _p),
+    ("step_out", _p)])
+RotaryCommitArgs = _struct("RotaryCommitArgs", [(n, _i) for n in (
+    "dtype", "m", "heads", "kv_heads", "dim", "dim_pad", "rot_dims")] + [
+    ("eps", _f), ("q", Rows), ("k", Rows), ("v", Rows), ("q_norm", _p), ("k_norm", _p), ("inv_freq", _p), ("row_pos", _p),
+    ("slots", _p), ("num_slots", _i64), ("q_out", _p), ("k_cache", _p), ("v_cache", _p)])
+WindowAttnArgs = _struct("WindowAttnArgs", [(n, _i) for n in (
+    "dtype", "m", "bs", "heads", "kv_heads", "dim", "dim_pad", "window", "sink", "max_q", "nsplit")] + [
+    ("scale", _f), ("out_scale", _f), ("q", _p), ("k_cache", _p), ("v_cache", _p), ("block_table", _p), ("row_seq", _p),
+    ("row_pos", _p), ("cu_q", _p), ("start", _p), ("table_stride", _i), ("num_pages", _i), ("gate", Rows), ("out", _p),
+    ("ld_out", _i64), ("workspace", _p), ("workspace_bytes", _i64)])
 DeltaPrepArgs = _struct("DeltaPrepArgs", [(n, _i) for n in (
     "dtype", "m", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim", "taps", "channels", "shift_state", "copy_cols")] + [
     ("q", Rows), ("k", Rows), ("v", Rows), ("b", Rows), ("copy", Rows), ("copy_out", _p), ("copy_ld", _i64), ("conv_q", _p),
@@ -55,7 +72,7 @@ ScanArgs = _struct("ScanArgs", [(n, _i) for n in (
     ("state_slot_stride", _i64), ("num_slots", _i64), ("mstate", _p), ("scalars", _p),
     ("den", _p), ("cu_q", _p), ("start", _p),
     ("state_slot", _p), ("out", _p), ("raw_decay", Rows), ("a_log", _p), ("dt_bias", _p), ("gate", Rows), ("norm", _p),
-    ("norm_head_stride", _i64), ("y", _p), ("ldy", _i64)])
+    ("norm_head_stride", _i64), ("y", _p), ("ldy", _i64), ("skip", _p)])
 MoeRouteArgs = _struct("MoeRouteArgs", [(n, _i) for n in ("m", "experts", "top", "groups", "keep")] + [
     ("logits", Rows), ("row_slot", _p), ("ids", _p), ("weights", _p)])
 MoePlanArgs = _struct("MoePlanArgs", [(n, _i) for n in ("m", "top", "experts", "max_tiles")] + [
@@ -110,6 +127,11 @@ SIGNATURES = {
     "mdb_residual_norm": (_i, [C.POINTER(ResidualNormArgs), _p]),
     "mdb_rms_rows": (_i, [_i, C.POINTER(RmsSegment), _i, _i, _p]),
     "mdb_gated_norm": (_i, [C.POINTER(GatedNormArgs), _p]),
+    "mdb_part_norm": (_i, [C.POINTER(PartNormArgs), _p]),
+    "mdb_decay_prep": (_i, [C.POINTER(DecayPrepArgs), _p]),
+    "mdb_rotary_commit": (_i, [C.POINTER(RotaryCommitArgs), _p]),
+    "mdb_window_attn_workspace_bytes": (_i64, [_i, _i, _i, _i]),
+    "mdb_window_attn": (_i, [C.POINTER(WindowAttnArgs), _p]),
     "mdb_scan_dim_pad": (_i, [_i]),
     "mdb_scan_blocks": (_i, [_i]),
     "mdb_scan_fusable": (_i, [_i, _i]),

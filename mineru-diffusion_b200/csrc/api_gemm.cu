@@ -9,6 +9,25 @@ namespace {
 int gemm_plain_bf16(const mdb_gemm_args& a, cudaStream_t st) {
   const bf16* x = static_cast<const bf16*>(a.x);
   const bf16* w = static_cast<const bf16*>(a.w);
+  if (a.act == MDB_ACT_RELU_GLU) {
+    MDB_REQUIRE(!a.y_f32, MDB_ERR_UNSUPPORTED);
+    if (ws_supported(kWsSwiglu, a.m, 2 * a.n, a.k, a.ldx)) {
+      WsArgs s = {};
+      s.m = a.m; s.n = 2 * a.n; s.k = a.k; s.ksplit = 1;
+      s.inter = a.n;
+      s.glu_relu = 1;
+      s.y = static_cast<bf16*>(a.y);
+      s.ldy = a.ldy;
+      return launch_ws<kWsSwiglu>(x, a.ldx, w, s, st);
+    }
+    MDB_REQUIRE(tc_supported(kTcSwiglu, a.m, a.n, a.k, a.ldx, a.ldy), MDB_ERR_UNSUPPORTED);
+    TcArgs t = {};
+    t.m = a.m; t.n = a.n; t.k = a.k; t.inter = a.n;
+    t.act = a.act;
+    t.y = static_cast<bf16*>(a.y);
+    t.ldy = a.ldy;
+    return launch_tc<kTcSwiglu>(x, a.ldx, w, 2 * a.n, t, st);
+  }
   if (a.act == MDB_ACT_NONE && a.y_f32 && a.ldy == a.n && ws_supported(kWsPartial, a.m, a.n, a.k, a.ldx)) {
     // fp32 rows of a short step: one split-k slice of the streaming kernel
     WsArgs s = {};
@@ -64,7 +83,8 @@ int mdb_gemm(const mdb_gemm_args* args, mdb_stream_t stream) {
   const mdb_gemm_args a = *args;
   MDB_REQUIRE(a.m >= 0 && a.n > 0 && a.k > 0, MDB_ERR_ARG);
   if (a.m == 0) return MDB_OK;
-  MDB_REQUIRE(a.form >= MDB_GEMM_PLAIN && a.form <= MDB_GEMM_EXPERTS && (a.act == MDB_ACT_NONE || a.act == MDB_ACT_RELU2), MDB_ERR_ARG);
+  MDB_REQUIRE(a.form >= MDB_GEMM_PLAIN && a.form <= MDB_GEMM_EXPERTS && a.act >= MDB_ACT_NONE && a.act <= MDB_ACT_RELU_GLU, MDB_ERR_ARG);
+  MDB_REQUIRE(a.act != MDB_ACT_RELU_GLU || a.form == MDB_GEMM_PLAIN, MDB_ERR_UNSUPPORTED);
   MDB_REQUIRE(a.x && a.w && a.y, MDB_ERR_ARG);
   const int64_t groups = a.form == MDB_GEMM_HEADS ? a.heads : 1;
   MDB_REQUIRE(groups >= 1 && a.ldx >= groups * a.k && a.ldy >= groups * a.n, MDB_ERR_ARG);

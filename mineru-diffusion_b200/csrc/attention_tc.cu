@@ -1,11 +1,15 @@
-// Attention on the 5th-generation tensor cores, in two forms that share one
+// Attention on the 5th-generation tensor cores, in three forms that share one
 // warp-specialised pipeline:
 //   * block attention over the paged KV cache (decode: the masked block of
 //     every request against its committed prefix, every key visible;
 //     flash_attn_with_kvcache as nanovllm/layers/sdar_attention.py:50-55 calls it);
 //   * staircase attention over packed sequences (prefill: a query row sees the
 //     keys up to the right edge of its right-aligned block;
-//     nanovllm/kernels/triton/attention/block_prefill_attention_v2.py:17-166).
+//     nanovllm/kernels/triton/attention/block_prefill_attention_v2.py:17-166);
+//   * window attention of prompt portions over the paged KV cache (WIN, a kind of
+//     staircase with stairs of one token: a query row sees the last `window` keys
+//     up to its own), with an optional sink in the softmax's denominator, one output
+//     gate per head, and heads of 64 or 128 stored channels.
 //
 // One work unit = the query rows of `tokens x group` (tokens of one request or
 // sequence times the query heads that share a KV head; row = token * group +
@@ -106,6 +110,12 @@ struct AtArgs {
   int64_t out_stride;
   int nseq, max_qtiles, log2_stairs;
   float q_scale;            // applied to q and rounded to bf16: log2(e) / sqrt(D) as the reference kernel does, or 1
+  // window form (with the page table above and cu_seqlens_q)
+  const int32_t* start;     // position of every sequence's first query
+  int window, sink;         // window 0: every key up to the query
+  int dim, halves;          // channels of a head in the output; stored channels / 64
+  float out_scale;
+  mdb_rows gate;            // [rows][hq] before the sigmoid, or absent
 };
 
 __device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int c0, int c1, int c2, uint32_t bar) {
@@ -181,7 +191,7 @@ struct AtUnit {
   int q_start, q_off, m0, Tq;  // ... first packed query row, tokens in front of it, first query of the unit, number of queries
 };
 
-template <bool STAIR>
+template <bool STAIR, bool WIN = false>
 __device__ __forceinline__ AtUnit at_unit(const AtArgs& a, const uint16_t* order, int units, int wave,
                                           int max_ranked = kAtMaxRanked) {
   AtUnit w = {};
@@ -194,22 +204,29 @@ __device__ __forceinline__ AtUnit at_unit(const AtArgs& a, const uint16_t* order
     const int rest = p % per_tile;
     const int seq = rest / a.hkv;
     w.kvh = rest % a.hkv;
-    w.seq_start = a.cu_seqlens[seq];
-    w.T = a.cu_seqlens[seq + 1] - w.seq_start;
     w.m0 = qt * a.tokens_per_unit;
     const int32_t* cu_q = a.cu_seqlens_q != nullptr ? a.cu_seqlens_q : a.cu_seqlens;
     w.q_start = cu_q[seq];
     w.Tq = cu_q[seq + 1] - w.q_start;
-    w.q_off = w.T - w.Tq;
+    if (WIN) {
+      w.req = seq;
+      w.q_off = a.start[seq];
+      w.T = w.q_off + w.Tq;
+    } else {
+      w.seq_start = a.cu_seqlens[seq];
+      w.T = a.cu_seqlens[seq + 1] - w.seq_start;
+      w.q_off = w.T - w.Tq;
+    }
     if (w.m0 >= w.Tq) return w;
     w.valid = true;
     w.q_tok0 = w.q_start + w.m0;
     const int S = 1 << a.log2_stairs;
     const int pad = ((w.T + S - 1) >> a.log2_stairs << a.log2_stairs) - w.T;
     const int last = w.q_off + min(w.m0 + a.tokens_per_unit, w.Tq) - 1;
-    w.kbeg = 0;
+    // window form: from the tile that holds the first query's first key
+    w.kbeg = WIN && a.window > 0 ? max(0, w.q_off + w.m0 - a.window + 1) / kAtKeys * kAtKeys : 0;
     w.kend = min(w.T, ((((last + pad) >> a.log2_stairs) + 1) << a.log2_stairs) - pad);
-    w.ntiles = (w.kend + kAtKeys - 1) / kAtKeys;
+    w.ntiles = (w.kend - w.kbeg + kAtKeys - 1) / kAtKeys;
     return w;
   }
   const int p = wave * G + ((wave & 1) ? G - 1 - c : c);
@@ -267,12 +284,14 @@ __device__ __forceinline__ bool at_swap(volatile unsigned long long* xch, int la
   }
 }
 
-template <int ROWS, bool STAIR, bool DUP = false>
+template <int ROWS, bool STAIR, bool DUP = false, bool WIN = false>
 __global__ void __launch_bounds__(AtPlan<ROWS, DUP, STAIR>::kThreads, 1)
 attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                const __grid_constant__ CUtensorMap map_v, const AtArgs a, const int units) {
   using P = AtPlan<ROWS, DUP, STAIR>;
   static_assert(!(DUP && STAIR), "row duplication is a paged-form layout");
+  static_assert(!WIN || STAIR, "the window form is a staircase with paged keys");
+  const int halves = WIN ? a.halves : 2;      // 64-channel halves of a stored head
   extern __shared__ __align__(1024) unsigned char at_smem_raw[];
   const uint32_t raw = smem_u32(at_smem_raw);
   const uint32_t base = (raw + 1023u) & ~1023u;
@@ -347,25 +366,25 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         if (!mbar_wait(bar(empty0 + r.stage), r.phase ^ 1)) return false;
         const uint32_t full = bar(full0 + r.stage);
         const uint32_t dst = tiles0 + r.stage * kAtTileBytes;
-        mbar_arrive_expect_tx(full, kAtTileBytes);
-        tma_load_2d(dst, map, kvh * kHeadDim, token_row, full);
-        tma_load_2d(dst + kAtHalfBytes, map, kvh * kHeadDim + 64, token_row, full);
+        mbar_arrive_expect_tx(full, halves * kAtHalfBytes);
+        tma_load_2d(dst, map, kvh * 64 * halves, token_row, full);
+        if (halves > 1) tma_load_2d(dst + kAtHalfBytes, map, kvh * kHeadDim + 64, token_row, full);
         pend |= 1u << r.stage;
         par = (par & ~(1u << r.stage)) | (r.phase << r.stage);
         r.advance(stages);
         return true;
       };
       for (int wave = 0; wave < waves && ok; ++wave) {
-        const AtUnit w = at_unit<STAIR>(a, order, units, wave, P::kMaxRanked);
+        const AtUnit w = at_unit<STAIR, WIN>(a, order, units, wave, P::kMaxRanked);
         if (w.ctx_clamped) report_status(MDB_STATUS_BAD_PAGE);
         if (w.ntiles == 0) continue;
         if (!mbar_wait(bar(kAtBarQEmpty + qr.stage), qr.phase ^ 1)) { ok = false; break; }
         {
           const uint32_t full = bar(kAtBarQFull + qr.stage);
           const uint32_t dst = base + P::kOffQ + qr.stage * P::kQBytes;
-          mbar_arrive_expect_tx(full, static_cast<uint32_t>(rows_used) * (DUP ? 512u : 256u));
+          mbar_arrive_expect_tx(full, static_cast<uint32_t>(rows_used) * (DUP ? 512u : 128u * halves));
           tma_load_3d(dst, &map_q, 0, w.kvh * group, w.q_tok0, full);
-          tma_load_3d(dst + P::kQRows * 128, &map_q, 64, w.kvh * group, w.q_tok0, full);
+          if (halves > 1) tma_load_3d(dst + P::kQRows * 128, &map_q, 64, w.kvh * group, w.q_tok0, full);
           if (DUP) {      // the same rows once more as operand rows 64..
             tma_load_3d(dst + 64 * 128, &map_q, 0, w.kvh * group, w.q_tok0, full);
             tma_load_3d(dst + P::kQRows * 128 + 64 * 128, &map_q, 64, w.kvh * group, w.q_tok0, full);
@@ -376,8 +395,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         }
         auto token_row = [&](int tile) {
           const int key0 = w.kbeg + tile * kAtKeys;
-          if (STAIR) return w.seq_start + key0;
-          int page = a.block_table[static_cast<int64_t>(w.req) * a.table_stride + key0 / kPage];
+          if (STAIR && !WIN) return w.seq_start + key0;
+          int page = !WIN || key0 / kPage < a.table_stride ? a.block_table[static_cast<int64_t>(w.req) * a.table_stride + key0 / kPage] : -1;
           if (page < 0 || page >= a.num_pages) {
             report_status(MDB_STATUS_BAD_PAGE);
             page = 0;
@@ -412,15 +431,15 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
       const uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(kAtKeys >> 3) << 17) |
                                (static_cast<uint32_t>(128 >> 4) << 24);
       const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) |
-                               (static_cast<uint32_t>(kHeadDim >> 3) << 17) | (static_cast<uint32_t>(128 >> 4) << 24);
+                               (static_cast<uint32_t>(halves * 8) << 17) | (static_cast<uint32_t>(128 >> 4) << 24);
       AtRing kr, vr, qr, sr, pr;        // sr: S buffer the next S = Q K^T goes to; pr: P buffer of the next P V
       uint32_t o_phase = 0;             // parity of the o_empty phase to wait for
       bool ok = true;
       for (int wave = 0; wave < waves && ok; ++wave) {
-        const AtUnit w = at_unit<STAIR>(a, order, units, wave, P::kMaxRanked);
+        const AtUnit w = at_unit<STAIR, WIN>(a, order, units, wave, P::kMaxRanked);
         if (w.ntiles == 0) continue;
         // staircase form: the softmax warps scale q in place first
-        if (!mbar_wait_w(bar((STAIR ? kAtBarQReady : kAtBarQFull) + qr.stage), qr.phase)) { ok = false; break; }
+        if (!mbar_wait_w(bar((STAIR && !WIN ? kAtBarQReady : kAtBarQFull) + qr.stage), qr.phase)) { ok = false; break; }
         const uint32_t q_tile = base + P::kOffQ + qr.stage * P::kQBytes;
         auto issue_s = [&](int j) {
           if (!mbar_wait_w(bar(kAtBarKFull + kr.stage), kr.phase)) return false;
@@ -430,6 +449,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
           const uint32_t d_tmem = tmem_base + sr.stage * kAtKeys;
 #pragma unroll
           for (int kk = 0; kk < 8; ++kk) {
+            if (WIN && kk >= 4 * halves) break;
             const uint64_t adesc = umma_desc_sw128(q_tile + (kk >> 2) * (P::kQRows * 128)) + 2 * (kk & 3);
             const uint64_t bdesc = umma_desc_sw128(k_tile + (kk >> 2) * kAtHalfBytes) + 2 * (kk & 3);
             umma_bf16_w(d_tmem, adesc, bdesc, idesc_s, kk > 0 ? 1u : 0u);
@@ -487,11 +507,11 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
     uint32_t o_phase = 0;
     bool ok = true;
     for (int wave = 0; wave < waves && ok; ++wave) {
-      const AtUnit w = at_unit<STAIR>(a, order, units, wave, P::kMaxRanked);
+      const AtUnit w = at_unit<STAIR, WIN>(a, order, units, wave, P::kMaxRanked);
       if (!w.valid) continue;
       const int head = w.kvh * group + head_in_group;
       bool row_valid = row < rows_used;
-      int limit = 0;                 // staircase form: last key this row sees
+      int limit = 0, first = 0;      // staircase form: last (window form: and first) key this row sees
       bf16* out_row;
       int64_t prow = 0;
       if (STAIR) {
@@ -500,7 +520,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         const int S = 1 << a.log2_stairs;
         const int pad = ((w.T + S - 1) >> a.log2_stairs << a.log2_stairs) - w.T;
         limit = row_valid ? min(w.T - 1, ((((i + pad) >> a.log2_stairs) + 1) << a.log2_stairs) - 1 - pad) : -1;
-        out_row = a.out + static_cast<int64_t>(w.q_start + (row_valid ? qi : 0)) * a.out_stride + head * kHeadDim;
+        if (WIN && a.window > 0) first = i - a.window + 1;
+        out_row = a.out + static_cast<int64_t>(w.q_start + (row_valid ? qi : 0)) * a.out_stride + head * (WIN ? a.dim : kHeadDim);
       } else {
         const int tok = w.tok0 + tok_local;
         row_valid = row_valid && tok < a.block;
@@ -522,7 +543,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         }
         continue;
       }
-      if (STAIR) {
+      if (STAIR && !WIN) {
         // q * log2(e)/sqrt(D) rounded to bf16, in place (elementwise, so the swizzle does not matter)
         ok = mbar_wait(bar(kAtBarQFull + qr.stage), qr.phase);
         if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
@@ -567,6 +588,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         if (nv < NC) {
 #pragma unroll
           for (int i = 0; i < NC; ++i) if (i >= nv) s[i] = -INFINITY;   // also replaces NaN from stale rows
+        }
+        if (WIN && first > key0) {
+#pragma unroll
+          for (int i = 0; i < NC; ++i) if (i < first - key0) s[i] = -INFINITY;
         }
         // eight independent chains: the warp is alone on its sub-partition, nothing else hides the ALU latency
         float mxv[8];
@@ -639,12 +664,13 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                        "r"(pk[4 * q]), "r"(pk[4 * q + 1]), "r"(pk[4 * q + 2]), "r"(pk[4 * q + 3])
                        : "memory");
         }
-        if (!STAIR && nvalid < kAtKeys) {
+        const int held = WIN ? w.kend - key0 : nvalid;      // keys of the tile that belong to the context
+        if ((!STAIR || WIN) && held < kAtKeys) {
           // stale cache rows past the context end must not reach O through 0 * (Inf or NaN): clear them in V
           ok = mbar_wait(bar(kAtBarVFull + vr.stage), vr.phase);
           if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
           const uint32_t v_tile = base + P::kOffV + vr.stage * kAtTileBytes;
-          for (int r = nvalid + lane_row; r < kAtKeys; r += 32 * P::kSoftmaxWarps) {
+          for (int r = held + lane_row; r < kAtKeys; r += 32 * P::kSoftmaxWarps) {
 #pragma unroll
             for (int h = 0; h < 2; ++h)
 #pragma unroll
@@ -678,13 +704,27 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
       if (half != 0) {
         // DUP: lanes 64..127 of O belong to operand rows nobody wrote; the rows' outputs leave from lanes 0..63
       } else if (STAIR || a.nsplit == 1) {
-        const float inv = l > 0.f ? 1.0f / l : 0.f;
+        float inv;
+        if (WIN) {
+          // the sink's term exp(0) in the units of the running reference
+          const float den = a.sink ? l + ex2_approx(-m_ref) : l;
+          float z = a.out_scale;
+          if (row_valid && rows_present(a.gate)) z *= sigmoid_f(rows_at<bf16>(a.gate, w.q_start + w.m0 + tok_local, head));
+          inv = den > 0.f ? z / den : 0.f;
+        } else {
+          inv = l > 0.f ? 1.0f / l : 0.f;
+        }
+        const bool ragged = WIN && a.dim != 64 * halves;      // fewer channels leave than are stored
 #pragma unroll 1
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < 2 * halves; ++c) {
           float o[32];
           tmem_ld32(tmem_o + lane_field + 32 * c, o);
           tmem_ld_wait();
-          if (row_valid) {
+          if (row_valid && ragged) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (32 * c + i < a.dim) out_row[32 * c + i] = __float2bfloat16_rn(o[i] * inv);
+          } else if (row_valid) {
 #pragma unroll
             for (int q4 = 0; q4 < 4; ++q4)
               reinterpret_cast<uint4*>(out_row + 32 * c)[q4] =
@@ -725,27 +765,27 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
 struct QMapKey {
   const void* ptr;
   int64_t tokens, row_stride;
-  int hq, group, box_tokens;
+  int hq, group, box_tokens, head_dim;
   bool operator==(const QMapKey& o) const {
     return ptr == o.ptr && tokens == o.tokens && row_stride == o.row_stride && hq == o.hq && group == o.group &&
-           box_tokens == o.box_tokens;
+           box_tokens == o.box_tokens && head_dim == o.head_dim;
   }
 };
 struct QMapKeyHash {
   size_t operator()(const QMapKey& k) const {
     return reinterpret_cast<size_t>(k.ptr) ^ static_cast<size_t>(k.tokens) * 0x9e3779b97f4a7c15ull ^
            static_cast<size_t>(k.row_stride) * 0xc2b2ae3d27d4eb4full ^
-           static_cast<size_t>(k.hq * 131 + k.group * 17 + k.box_tokens);
+           static_cast<size_t>((k.hq * 131 + k.group * 17 + k.box_tokens) * 257 + k.head_dim);
   }
 };
 
-// Tensor map of q [tokens, hq, 128] bf16 (token stride row_stride elements) read in boxes of
+// Tensor map of q [tokens, hq, head_dim] bf16 (token stride row_stride elements) read in boxes of
 // 64 channels x group heads x box_tokens tokens.
 static bool get_q_tensor_map(const void* ptr, int64_t tokens, int64_t row_stride, int hq, int group, int box_tokens,
-                             CUtensorMap* out) {
+                             CUtensorMap* out, int head_dim = kHeadDim) {
   static std::mutex mu;
   static std::unordered_map<QMapKey, CUtensorMap, QMapKeyHash> cache;
-  const QMapKey key{ptr, tokens, row_stride, hq, group, box_tokens};
+  const QMapKey key{ptr, tokens, row_stride, hq, group, box_tokens, head_dim};
   std::lock_guard<std::mutex> lock(mu);
   auto it = cache.find(key);
   if (it != cache.end()) {
@@ -755,8 +795,8 @@ static bool get_q_tensor_map(const void* ptr, int64_t tokens, int64_t row_stride
   EncodeTiledFn enc = encode_tiled_fn();
   if (enc == nullptr) return false;
   CUtensorMap m;
-  const cuuint64_t dims[3] = {static_cast<cuuint64_t>(kHeadDim), static_cast<cuuint64_t>(hq), static_cast<cuuint64_t>(tokens)};
-  const cuuint64_t strides[2] = {static_cast<cuuint64_t>(kHeadDim) * 2, static_cast<cuuint64_t>(row_stride) * 2};
+  const cuuint64_t dims[3] = {static_cast<cuuint64_t>(head_dim), static_cast<cuuint64_t>(hq), static_cast<cuuint64_t>(tokens)};
+  const cuuint64_t strides[2] = {static_cast<cuuint64_t>(head_dim) * 2, static_cast<cuuint64_t>(row_stride) * 2};
   const cuuint32_t box[3] = {64u, static_cast<cuuint32_t>(group), static_cast<cuuint32_t>(box_tokens)};
   const cuuint32_t estr[3] = {1, 1, 1};
   if (enc(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr,
@@ -780,7 +820,7 @@ static int at_sm_count() {
   return sm_count;
 }
 
-template <int ROWS, bool STAIR, bool DUP = false>
+template <int ROWS, bool STAIR, bool DUP = false, bool WIN = false>
 static int at_launch(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v, const AtArgs& a,
                      int64_t units, cudaStream_t st) {
   using P = AtPlan<ROWS, DUP, STAIR>;
@@ -788,7 +828,7 @@ static int at_launch(const CUtensorMap& map_q, const CUtensorMap& map_k, const C
   const int dev = attr_once.slot();
   if (dev < 0) return MDB_ERR_CUDA;
   if (!attr_once.done[dev]) {
-    if (cudaFuncSetAttribute(attn_tc_kernel<ROWS, STAIR, DUP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(attn_tc_kernel<ROWS, STAIR, DUP, WIN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              P::kSmemBytes) != cudaSuccess)
       return MDB_ERR_CUDA;
     attr_once.done[dev] = true;
@@ -796,7 +836,7 @@ static int at_launch(const CUtensorMap& map_q, const CUtensorMap& map_k, const C
   if (units > (1 << 30)) return MDB_ERR_UNSUPPORTED;
   const int sms = at_sm_count();
   const int grid = units < sms ? static_cast<int>(units) : sms;
-  return mdb_launch(attn_tc_kernel<ROWS, STAIR, DUP>, dim3(grid), dim3(P::kThreads), P::kSmemBytes, st, map_q, map_k,
+  return mdb_launch(attn_tc_kernel<ROWS, STAIR, DUP, WIN>, dim3(grid), dim3(P::kThreads), P::kSmemBytes, st, map_q, map_k,
                     map_v, a, static_cast<int>(units));
 }
 
@@ -865,6 +905,41 @@ static int attn_stair_tc_launch(const AttnStairArgs& sa, int nseq, int max_seqle
   if (!get_tensor_map(sa.v, total_tokens, sa.hkv * kHeadDim, sa.v_stride, kAtKeys, &map_v)) return MDB_ERR_CUDA;
   const int64_t units = static_cast<int64_t>(a.max_qtiles) * nseq * sa.hkv;
   return at_launch<128, true>(map_q, map_k, map_v, a, units, st);
+}
+
+// ---- window form ----
+static bool attn_win_tc_supported(const mdb_window_attn_args& w) {
+  return w.dtype == MDB_BF16 && (w.dim_pad == 64 || w.dim_pad == 128) && w.heads / w.kv_heads <= 128 && w.scale > 0.f && w.cu_q && w.start;
+}
+
+static int attn_win_tc_launch(const mdb_window_attn_args& w, cudaStream_t st) {
+  AtArgs a = {};
+  a.q = static_cast<const bf16*>(w.q);
+  a.out = static_cast<bf16*>(w.out);
+  a.hq = w.heads; a.hkv = w.kv_heads; a.group = w.heads / w.kv_heads;
+  a.scale_log2 = w.scale * 1.4426950408889634f;
+  a.q_scale = 1.0f;
+  a.cu_seqlens_q = w.cu_q;
+  a.start = w.start;
+  a.block_table = w.block_table;
+  a.table_stride = w.table_stride;
+  a.num_pages = w.num_pages;
+  a.out_stride = w.ld_out;
+  a.nseq = w.bs;
+  a.tokens_per_unit = 128 / a.group;
+  a.max_qtiles = (w.max_q + a.tokens_per_unit - 1) / a.tokens_per_unit;
+  a.nsplit = 1;
+  a.window = w.window; a.sink = w.sink;
+  a.dim = w.dim; a.halves = w.dim_pad / 64;
+  a.out_scale = w.out_scale;
+  a.gate = w.gate;
+  CUtensorMap map_q, map_k, map_v;
+  const int64_t cache_rows = static_cast<int64_t>(w.num_pages) * kPage;
+  const int cols = w.kv_heads * w.dim_pad;
+  if (!get_q_tensor_map(w.q, w.m, static_cast<int64_t>(w.heads) * w.dim_pad, w.heads, a.group, a.tokens_per_unit, &map_q, w.dim_pad)) return MDB_ERR_CUDA;
+  if (!get_tensor_map(w.k_cache, cache_rows, cols, cols, kAtKeys, &map_k)) return MDB_ERR_CUDA;
+  if (!get_tensor_map(w.v_cache, cache_rows, cols, cols, kAtKeys, &map_v)) return MDB_ERR_CUDA;
+  return at_launch<128, true, false, true>(map_q, map_k, map_v, a, static_cast<int64_t>(a.max_qtiles) * w.bs * w.kv_heads, st);
 }
 
 }  // namespace mdb

@@ -542,6 +542,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
               float r[2];
 #pragma unroll
               for (int e = 0; e < 2; ++e) {
+                if (a.act == MDB_ACT_RELU_GLU) {
+                  r[e] = fmaxf(g[2 * i + e], 0.f) * u[2 * i + e];
+                  continue;
+                }
                 const float gt = bf16_round(g[2 * i + e]);
                 const float up = bf16_round(u[2 * i + e]);
                 const float sl = gt * rcp_approx(1.0f + __expf(-gt));   // fp32 SiLU, rounded to bf16 below

@@ -52,6 +52,7 @@ struct WsArgs {
   int chunks_total;    // k / 64
   int stages;
   int inter;           // swiglu: rows of the gate half
+  int glu_relu;        // swiglu form: relu(gate) * up in place of the SiLU
   float* partials;     // [ksplit][m][n]
   bf16* y;             // bf16 / swiglu output
   int64_t ldy;
@@ -446,6 +447,10 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             const int tt = 16 * tg + i;
             const int r = 32 * half + tt;
             if (r < a.m) {
+              if (a.glu_relu) {
+                a.y[r * a.ldy + col] = __float2bfloat16_rn(fmaxf(epi[c * 33 + tt], 0.f) * epi[(64 + c) * 33 + tt]);
+                continue;
+              }
               const float gt = bf16_round(epi[c * 33 + tt]);
               const float up = bf16_round(epi[(64 + c) * 33 + tt]);
               const float s = gt * __frcp_rn(1.0f + __expf(-gt));

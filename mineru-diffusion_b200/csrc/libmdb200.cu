@@ -2,16 +2,17 @@
 // word and a few launch helpers, so the parts are included here in order
 // rather than linked as relocatable device code.
 #include "elementwise.cu"
+#include "rows32.cu"
 #include "attention.cu"
 #include "sampler.cu"
 #include "gemm_ws.cu"
 #include "gemm_tc.cu"
 #include "attention_tc.cu"
 #include "api_linear.cu"
-#include "rows32.cu"
 #include "moe.cu"
 #include "gemm_f32.cu"
 #include "api_gemm.cu"
 #include "recurrent.cu"
 #include "latent_attention.cu"
+#include "window_attention.cu"
 #include "tp_p2p.cu"

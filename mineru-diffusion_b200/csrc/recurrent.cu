@@ -1,5 +1,5 @@
-// Recurrent mixers with a matrix state per head: the gated delta rule with one decay per key channel, and the mLSTM
-// matrix memory.  A scan kernel each for prompts and their portions, one for single tokens; the state lives in fp32 in a slot
+// Recurrent mixers with a matrix state per head: the gated delta rule with one decay per key channel, the mLSTM matrix
+// memory, and plain linear recurrences with one decay per head, fixed or per token (lightning attention, Mamba-2).  A scan kernel each for prompts and their portions, one for single tokens; the state lives in fp32 in a slot
 // per sequence and every product of the recurrence is an fp32 FMA (packed two at a time, fma.rn.f32x2).
 //
 // State layout: [slot][head][value column][key channel padded to a multiple of 64], so a value column is contiguous.
@@ -14,6 +14,8 @@
 //   a2 = S'^T k2 + ((g2 k1) . k2) u1,  b2 = S'^T q2 + ((g2 k1) . q2) u1,  S <- S' + (g2 k1) u1^T + k2 u2^T,
 // the same number of FMAs per token with half the dependent shuffle reductions; these products of keys and queries are
 // computed beforehand, with the decays.
+//
+// The linear recurrence S <- a S + b k v^T, o = S^T q + skip v is the mLSTM's scan with its gates given and no normaliser.
 //
 // mLSTM: the normaliser n is one more column of the state (its value is 1 for every token); the division by
 // max(|n . q|, exp(-m)) + 1e-6 happens where the read-out is normalised.
@@ -72,11 +74,12 @@ __device__ __forceinline__ float sum8(float v) {
 constexpr int kPrepWarps = 4;
 constexpr int kMaxTaps = 16;
 
-template <typename T>
+template <typename T, typename Args>
 struct ConvCtx {
-  const mdb_delta_prep_args* a;
+  const Args* a;
   int64_t row;
   int tloc, slot;      // token index inside this step's portion; state slot (-1: starts from zeros)
+  int state_slot;      // the sequence's slot, whether or not its state counts
   // input of channel `col` of projection `src`, `back` tokens ago
   __device__ __forceinline__ float at(const mdb_rows& src, int col, int channel, int back) const {
     if (back <= tloc) return rows_at<T>(src, row - back, col);
@@ -84,10 +87,20 @@ struct ConvCtx {
     if (slot < 0 || idx < 0) return 0.f;
     return act_to_f(static_cast<const T*>(a->conv_state)[slot * a->conv_slot_stride + static_cast<int64_t>(idx) * a->channels + channel]);
   }
-  __device__ __forceinline__ float conv_silu(const mdb_rows& src, const float* w, int col, int channel) const {
-    float acc = 0.f;
+  __device__ __forceinline__ float conv_silu(const mdb_rows& src, const float* w, int col, int channel, float bias = 0.f) const {
+    float acc = bias;
     for (int j = 0; j < a->taps; ++j) acc = fmaf(w[static_cast<int64_t>(col) * a->taps + j], at(src, col, channel, a->taps - 1 - j), acc);
     return acc / (1.0f + expf(-acc));
+  }
+  // one-token portions move the convolution state along: the caller owns the channel
+  __device__ __forceinline__ void shift(const mdb_rows& src, int col, int channel) const {
+    if (!a->shift_state || a->taps < 2) return;
+    T* st = static_cast<T*>(a->conv_state) + state_slot * a->conv_slot_stride + channel;
+    float keep[kMaxTaps];
+#pragma unroll 1
+    for (int j = 0; j < a->taps - 1; ++j) keep[j] = at(src, col, channel, a->taps - 2 - j);
+#pragma unroll 1
+    for (int j = 0; j < a->taps - 1; ++j) st[static_cast<int64_t>(j) * a->channels] = act_from_f<T>(keep[j]);
   }
 };
 
@@ -105,17 +118,7 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const mdb_d
     if (lane == 0) report_status(MDB_STATUS_BAD_SLOT);
     return;
   }
-  ConvCtx<T> cx = {&a, row, static_cast<int>(row) - a.cu_q[seq], a.start[seq] == 0 ? -1 : slot};
-  // one-token portions move the convolution state along right here: the warp owns its channels
-  auto shift = [&](const mdb_rows& src, int col, int channel) {
-    if (!a.shift_state || a.taps < 2) return;
-    T* st = static_cast<T*>(a.conv_state) + slot * a.conv_slot_stride + channel;
-    float keep[kMaxTaps];
-#pragma unroll 1
-    for (int j = 0; j < a.taps - 1; ++j) keep[j] = cx.at(src, col, channel, a.taps - 2 - j);
-#pragma unroll 1
-    for (int j = 0; j < a.taps - 1; ++j) st[static_cast<int64_t>(j) * a.channels] = act_from_f<T>(keep[j]);
-  };
+  const ConvCtx<T, mdb_delta_prep_args> cx = {&a, row, static_cast<int>(row) - a.cu_q[seq], a.start[seq] == 0 ? -1 : slot, slot};
   if (unit < a.kv_heads) {
     float* qo = a.q_out + (row * a.kv_heads + unit) * a.dim_pad;
     float* ko = a.k_out + (row * a.kv_heads + unit) * a.dim_pad;
@@ -127,8 +130,8 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const mdb_d
         const int col = unit * a.dim + d;
         q = cx.conv_silu(a.q, a.conv_q, col, col);
         k = cx.conv_silu(a.k, a.conv_k, col, kq_channels + col);
-        shift(a.q, col, col);
-        shift(a.k, col, kq_channels + col);
+        cx.shift(a.q, col, col);
+        cx.shift(a.k, col, kq_channels + col);
       }
       qo[d] = q;
       ko[d] = k;
@@ -149,7 +152,7 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const mdb_d
     for (int d = lane; d < a.vdim; d += 32) {
       const int col = vu * a.vdim + d, channel = 2 * a.kv_heads * a.dim + col;
       const float v = cx.conv_silu(a.v, a.conv_v, col, channel);
-      shift(a.v, col, channel);
+      cx.shift(a.v, col, channel);
       vo[d] = v;
     }
     return;
@@ -164,6 +167,11 @@ __global__ void __launch_bounds__(kPrepWarps * 32) delta_prep_kernel(const mdb_d
     if (c < a.copy_cols) act_store4(static_cast<T*>(a.copy_out) + row * a.copy_ld + c, rows_at4<T>(a.copy, row, c));
   }
 }
+
+// silu; the approximate division and exponential are good to a few units in the last place of fp32, and a large negative
+// argument (whose exponential leaves the range of the fast division) gives 0
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-fmaxf(z, -80.f))); }
+__device__ __forceinline__ float4 silu4(float4 z) { return make_float4(silu_fast(z.x), silu_fast(z.y), silu_fast(z.z), silu_fast(z.w)); }
 
 // The same work for heads of at most 128 channels and up to four taps, sizes in multiples of four: a lane owns four
 // channels and walks `run` consecutive rows with the last inputs in registers, so every input is read once.
@@ -188,8 +196,8 @@ struct ConvWindow {
       w[j] = make_float4(e[0], e[1], e[2], e[3]);
     }
   }
-  __device__ __forceinline__ void refill(const mdb_delta_prep_args& a, const mdb_rows& src, int64_t row, int tloc, int slot, int col,
-                                         int channel) {
+  template <typename Args>
+  __device__ __forceinline__ void refill(const Args& a, const mdb_rows& src, int64_t row, int tloc, int slot, int col, int channel) {
 #pragma unroll
     for (int back = 1; back <= 3; ++back) {
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -202,20 +210,18 @@ struct ConvWindow {
       x[3 - back] = v;
     }
   }
-  __device__ __forceinline__ float4 step(float4 now) {
+  __device__ __forceinline__ float4 step(float4 now, float4 bias = make_float4(0.f, 0.f, 0.f, 0.f)) {
     float4 y;
-    y.x = fmaf(w[3].x, now.x, fmaf(w[2].x, x[2].x, fmaf(w[1].x, x[1].x, w[0].x * x[0].x)));
-    y.y = fmaf(w[3].y, now.y, fmaf(w[2].y, x[2].y, fmaf(w[1].y, x[1].y, w[0].y * x[0].y)));
-    y.z = fmaf(w[3].z, now.z, fmaf(w[2].z, x[2].z, fmaf(w[1].z, x[1].z, w[0].z * x[0].z)));
-    y.w = fmaf(w[3].w, now.w, fmaf(w[2].w, x[2].w, fmaf(w[1].w, x[1].w, w[0].w * x[0].w)));
+    y.x = fmaf(w[3].x, now.x, fmaf(w[2].x, x[2].x, fmaf(w[1].x, x[1].x, fmaf(w[0].x, x[0].x, bias.x))));
+    y.y = fmaf(w[3].y, now.y, fmaf(w[2].y, x[2].y, fmaf(w[1].y, x[1].y, fmaf(w[0].y, x[0].y, bias.y))));
+    y.z = fmaf(w[3].z, now.z, fmaf(w[2].z, x[2].z, fmaf(w[1].z, x[1].z, fmaf(w[0].z, x[0].z, bias.z))));
+    y.w = fmaf(w[3].w, now.w, fmaf(w[2].w, x[2].w, fmaf(w[1].w, x[1].w, fmaf(w[0].w, x[0].w, bias.w))));
     x[0] = x[1]; x[1] = x[2]; x[2] = now;
-    // silu; the approximate division and exponential are good to a few units in the last place of fp32
-    y.x = __fdividef(y.x, 1.0f + __expf(-y.x)); y.y = __fdividef(y.y, 1.0f + __expf(-y.y));
-    y.z = __fdividef(y.z, 1.0f + __expf(-y.z)); y.w = __fdividef(y.w, 1.0f + __expf(-y.w));
-    return y;
+    return silu4(y);
   }
   // one-token portions: the last taps - 1 inputs back into the slot
-  __device__ __forceinline__ void save(const mdb_delta_prep_args& a, int slot, int channel) const {
+  template <typename Args>
+  __device__ __forceinline__ void save(const Args& a, int slot, int channel) const {
     T* st = static_cast<T*>(a.conv_state) + slot * a.conv_slot_stride + channel;
     for (int j = 0; j < a.taps - 1; ++j) {
       const int i = 3 - (a.taps - 1) + j;          // oldest first
@@ -294,9 +300,27 @@ __global__ void __launch_bounds__(kPrepWarps * 32, 7) delta_prep_rows_kernel(con
       act_store4(static_cast<T*>(a.copy_out) + row * a.copy_ld + cc, rows_at4_of<T, PARTS>(a.copy, row, cc));
 }
 
+// Where a convolution channel's input comes from: the projection, and `channel` turned into a column of it.
+__device__ __forceinline__ const mdb_rows& conv_source(const mdb_delta_prep_args& a, int& channel) {
+  const int kc = a.kv_heads * a.dim;
+  if (channel < kc) return a.q;
+  channel -= kc;
+  if (channel < kc) return a.k;
+  channel -= kc;
+  return a.v;
+}
+__device__ __forceinline__ const mdb_rows& conv_source(const mdb_decay_prep_args& a, int& channel) {
+  const int kc = a.kv_heads * a.dim, vc = a.heads * a.vdim;
+  if (channel < vc) return a.v;
+  channel -= vc;
+  if (channel < kc) return a.k;
+  channel -= kc;
+  return a.q;
+}
+
 // The last taps - 1 inputs of every channel after a step of arbitrary portions: one thread per (sequence, channel).
-template <typename T>
-__global__ void __launch_bounds__(256) conv_state_kernel(const mdb_delta_prep_args a) {
+template <typename T, typename Args>
+__global__ void __launch_bounds__(256) conv_state_kernel(const Args a) {
   pdl_launch_dependents();
   pdl_wait();
   const int seq = blockIdx.y;
@@ -305,10 +329,9 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const mdb_delta_prep_ar
   if (slot < 0 || slot >= a.num_slots || channel >= a.channels) return;
   const int t0 = a.cu_q[seq], n = a.cu_q[seq + 1] - t0;
   if (n <= 0) return;
-  const int kc = a.kv_heads * a.dim;
-  const mdb_rows& src = channel < kc ? a.q : (channel < 2 * kc ? a.k : a.v);
-  const int col = channel < kc ? channel : (channel < 2 * kc ? channel - kc : channel - 2 * kc);
-  ConvCtx<T> cx = {&a, t0 + n - 1, n - 1, a.start[seq] == 0 ? -1 : slot};
+  int col = channel;
+  const mdb_rows& src = conv_source(a, col);
+  const ConvCtx<T, Args> cx = {&a, t0 + n - 1, n - 1, a.start[seq] == 0 ? -1 : slot, slot};
   float keep[kMaxTaps];
 #pragma unroll 1
   for (int j = 0; j < a.taps - 1; ++j) keep[j] = cx.at(src, col, channel, a.taps - 2 - j);
@@ -419,9 +442,130 @@ __global__ void __launch_bounds__(256) mlstm_prep_kernel(const mdb_mlstm_prep_ar
 }
 
 // ---------------------------------------------------------------------------
+// Before the decay scan: silu or short convolution + silu of v, k and q, and the two scalars of a head.  Work items of a row:
+// channels of v, of k, of q (padding channels: zeros), then one per head for the scalars.
+// ---------------------------------------------------------------------------
+template <typename T>
+__device__ __forceinline__ void decay_prep_scalars(const mdb_decay_prep_args& a, int64_t row, int head) {
+  float decay, step = 1.0f;
+  if (rows_present(a.dt)) {
+    step = softplus_f(rows_at<T>(a.dt, row, head) + a.dt_bias[head]);
+    decay = expf(-expf(a.a_log[head]) * step);
+  } else {
+    decay = a.decay_const[head];
+  }
+  a.decay_out[row * a.heads + head] = decay;
+  a.step_out[row * a.heads + head] = step;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) decay_prep_kernel(const mdb_decay_prep_args a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t row = blockIdx.x;
+  const int seq = a.row_seq[row];
+  const int slot = a.state_slot[seq];
+  if (slot < 0) return;
+  if (slot >= a.num_slots) {
+    if (threadIdx.x == 0) report_status(MDB_STATUS_BAD_SLOT);
+    return;
+  }
+  int i = blockIdx.y * 256 + threadIdx.x;
+  const int nv = a.heads * a.vdim, nk = a.kv_heads * a.dim_pad, kc = a.kv_heads * a.dim;
+  if (i >= nv + 2 * nk) {
+    if (i - nv - 2 * nk < a.heads) decay_prep_scalars<T>(a, row, i - nv - 2 * nk);
+    return;
+  }
+  const int stream = i < nv ? 0 : (i < nv + nk ? 1 : 2);
+  i -= stream == 0 ? 0 : (stream == 1 ? nv : nv + nk);
+  const mdb_rows& src = stream == 0 ? a.v : (stream == 1 ? a.k : a.q);
+  float* out = stream == 0 ? a.v_out + row * nv + i : (stream == 1 ? a.k_out : a.q_out) + row * nk + i;
+  int col = i;
+  if (stream > 0) {
+    const int d = i % a.dim_pad;
+    if (d >= a.dim) {
+      *out = 0.f;
+      return;
+    }
+    col = i / a.dim_pad * a.dim + d;
+  }
+  if (a.taps == 0) {
+    const float x = rows_at<T>(src, row, col);
+    *out = x / (1.0f + expf(-x));
+    return;
+  }
+  const ConvCtx<T, mdb_decay_prep_args> cx = {&a, row, static_cast<int>(row) - a.cu_q[seq], a.start[seq] == 0 ? -1 : slot, slot};
+  const int channel = col + (stream == 0 ? 0 : (stream == 1 ? nv : nv + kc));
+  const float* w = a.conv + static_cast<int64_t>(channel - col) * a.taps;
+  *out = cx.conv_silu(src, w, col, channel, a.conv_bias[channel]);
+  cx.shift(src, col, channel);
+}
+
+// Sizes in multiples of four and up to four taps: a thread owns four channels and walks `run` consecutive rows with the last
+// inputs in registers.
+constexpr int kDecayPrepThreads = 128;
+template <typename T, bool PARTS>
+__global__ void __launch_bounds__(kDecayPrepThreads) decay_prep_rows_kernel(const mdb_decay_prep_args a, const int run) {
+  pdl_launch_dependents();
+  pdl_wait();
+  int i = blockIdx.x * kDecayPrepThreads + threadIdx.x;
+  const int64_t row0 = static_cast<int64_t>(blockIdx.y) * run, row1 = min(row0 + run, static_cast<int64_t>(a.m));
+  const int nv = a.heads * a.vdim, nk = a.kv_heads * a.dim_pad, kc = a.kv_heads * a.dim;
+  const int iv = nv / 4, ik = nk / 4;
+  if (i >= iv + 2 * ik) {
+    i -= iv + 2 * ik;
+    if (i < a.heads)
+      for (int64_t row = row0; row < row1; ++row) decay_prep_scalars<T>(a, row, i);
+    return;
+  }
+  const int stream = i < iv ? 0 : (i < iv + ik ? 1 : 2);
+  i -= stream == 0 ? 0 : (stream == 1 ? iv : iv + ik);
+  mdb_rows src = a.v;
+  if (stream == 1) src = a.k;
+  if (stream == 2) src = a.q;
+  const int64_t out_ld = stream == 0 ? nv : nk;
+  float* out = (stream == 0 ? a.v_out : (stream == 1 ? a.k_out : a.q_out)) + i * 4;
+  int col = i * 4;
+  if (stream > 0) {
+    const int d = i * 4 % a.dim_pad;
+    if (d >= a.dim) {
+      for (int64_t row = row0; row < row1; ++row) *reinterpret_cast<float4*>(out + row * out_ld) = make_float4(0.f, 0.f, 0.f, 0.f);
+      return;
+    }
+    col = i * 4 / a.dim_pad * a.dim + d;
+  }
+  if (a.taps == 0) {
+#pragma unroll 4
+    for (int64_t row = row0; row < row1; ++row) *reinterpret_cast<float4*>(out + row * out_ld) = silu4(rows_at4_of<T, PARTS>(src, row, col));
+    return;
+  }
+  const int channel = col + (stream == 0 ? 0 : (stream == 1 ? nv : nv + kc));
+  ConvWindow<T, PARTS> win;
+  win.load_taps(a.conv, channel, a.taps);
+  const float4 bias = *reinterpret_cast<const float4*>(a.conv_bias + channel);
+  int seq = -1, slot = -1;
+  for (int64_t row = row0; row < row1; ++row) {
+    const int s = a.row_seq[row];
+    const float4 in = rows_at4_of<T, PARTS>(src, row, col);
+    if (s != seq) {
+      seq = s;
+      slot = a.state_slot[s];
+      if (slot >= a.num_slots) {
+        report_status(MDB_STATUS_BAD_SLOT);
+        slot = -1;
+      }
+      if (slot >= 0) win.refill(a, src, row, static_cast<int>(row) - a.cu_q[s], a.start[s] == 0 ? -1 : slot, col, channel);
+    }
+    if (slot < 0) continue;
+    *reinterpret_cast<float4*>(out + row * out_ld) = win.step(in, bias);
+    if (a.shift_state && a.taps > 1) win.save(a, slot, channel);
+  }
+}
+
+// ---------------------------------------------------------------------------
 // The scan
 // ---------------------------------------------------------------------------
-enum { kScanDelta = MDB_SCAN_DELTA, kScanMlstm = MDB_SCAN_MLSTM };
+enum { kScanDelta = MDB_SCAN_DELTA, kScanMlstm = MDB_SCAN_MLSTM, kScanDecay = MDB_SCAN_DECAY };
 constexpr int kScanFusedThreads = 512, kScanFusedMaxDim = 256;
 constexpr int kScanBlockCols = 16;       // granularity of the copies of the mLSTM maximum; narrowest block of a prompt CTA
 constexpr int kScanTokens = 16;          // tokens of a stage of the prompt form (even)
@@ -529,7 +673,7 @@ struct ScanStage {
         if (MODE == kScanDelta) st[(2 * TB + n) * DP + i] = 1.f;
       }
       for (int i = threadIdx.x; i < COLS; i += step) st[OFF_V + n * COLS + i] = 0.f;
-      if (threadIdx.x < 4) st[OFF_S + 4 * n + threadIdx.x] = 0.f;
+      if (threadIdx.x < 4) st[OFF_S + 4 * n + threadIdx.x] = MODE == kScanDecay && threadIdx.x == 0 ? 1.f : 0.f;
     }
     cp_async_commit();
   }
@@ -667,20 +811,21 @@ __device__ __forceinline__ float reduce_scatter16(float (&r)[V], int l16) {
   return r[0];
 }
 
-// mLSTM, prompt form: sixteen lanes per CPT columns (a shared-memory read costs the same whatever the lanes do with it, so
-// a lane's channels serve four columns), sums handed out one per lane.
-template <int DP, int CPT, int COLS>
-__global__ void __launch_bounds__(COLS / CPT * 16) mlstm_scan_kernel(const mdb_scan_args a) {
+// mLSTM and decay scan, prompt form: sixteen lanes per CPT columns (a shared-memory read costs the same whatever the lanes
+// do with it, so a lane's channels serve four columns), sums handed out one per lane.
+template <int MODE, int DP, int CPT, int COLS>
+__global__ void __launch_bounds__(COLS / CPT * 16) gated_scan_kernel(const mdb_scan_args a) {
   constexpr int NR = DP / 64;            // float4 per lane and column
-  using Stage = ScanStage<kScanMlstm, DP, COLS>;
+  using Stage = ScanStage<MODE, DP, COLS>;
   constexpr int TB = Stage::TB, OFF_V = Stage::OFF_V, OFF_S = Stage::OFF_S;
   constexpr int VALS = 2 * CPT, PER = 16 / VALS;      // sums of a pair of tokens; lanes per sum
   extern __shared__ __align__(16) float scan_smem[];
   __shared__ float4 sh_gate[TB];         // forget factor, input factor, exp(-m) per token of the stage
   pdl_launch_dependents();
   pdl_wait();
-  const ScanJob w = scan_job<kScanMlstm, DP, COLS>(a);
+  const ScanJob w = scan_job<MODE, DP, COLS>(a);
   if (!w.live) return;
+  const float skip = MODE == kScanDecay && a.skip != nullptr ? a.skip[w.head] : 0.f;
   const int l16 = threadIdx.x & 15, cg = threadIdx.x >> 4, mycol = w.col0 + cg * CPT;
   f32x2 S[CPT][2 * NR];
 #pragma unroll
@@ -695,8 +840,8 @@ __global__ void __launch_bounds__(COLS / CPT * 16) mlstm_scan_kernel(const mdb_s
     }
   // every block of columns keeps a copy of the running maximum, so that no CTA reads what another writes
   const int blocks = (w.columns + kScanBlockCols - 1) / kScanBlockCols, block0 = w.col0 / kScanBlockCols;
-  float* mstate = a.mstate + (static_cast<int64_t>(w.slot) * a.heads + w.head) * blocks;
-  float run_max = w.fresh ? 0.f : mstate[block0];
+  float* mstate = MODE == kScanMlstm ? a.mstate + (static_cast<int64_t>(w.slot) * a.heads + w.head) * blocks : nullptr;
+  float run_max = w.fresh || MODE != kScanMlstm ? 0.f : mstate[block0];
   Stage::fill(a, w, w.t_begin, scan_smem);
   int buf = 0;
   for (int t0 = w.t_begin; t0 < w.t_end; t0 += TB, buf ^= 1) {
@@ -704,7 +849,7 @@ __global__ void __launch_bounds__(COLS / CPT * 16) mlstm_scan_kernel(const mdb_s
     Stage::turn(a, w, t0, scan_smem, buf);
     const float* st = scan_smem + buf * Stage::FLOATS;
     // m_t = max(f_t + m_(t-1), i_t) over the stage as a scan of the maps x -> max(x + F, I)
-    if (threadIdx.x < 32) {
+    if (MODE == kScanMlstm && threadIdx.x < 32) {
       const int l = threadIdx.x;
       const float li = l < n ? st[OFF_S + 4 * l] : -INFINITY, lf = l < n ? st[OFF_S + 4 * l + 1] : 0.f;
       float F = lf, I = li;
@@ -720,11 +865,13 @@ __global__ void __launch_bounds__(COLS / CPT * 16) mlstm_scan_kernel(const mdb_s
       else if (l < TB) sh_gate[l] = make_float4(1.f, 0.f, 0.f, 0.f);
       run_max = __shfl_sync(0xffffffffu, m, n - 1);
     }
-    __syncthreads();
+    if (MODE == kScanMlstm) __syncthreads();
     for (int t = 0; t < n; t += 2) {
       const float* k1p = st + t * DP + l16 * 4;
       const float* k2p = k1p + DP;
-      const float4 ga = sh_gate[t], gb = sh_gate[t + 1];
+      // (forget factor, input factor, ...) of the two tokens; the decay scan is handed them
+      const float4* gates = MODE == kScanMlstm ? sh_gate : reinterpret_cast<const float4*>(st + OFF_S);
+      const float4 ga = gates[t], gb = gates[t + 1];
       const f32x2 f1 = pack2(ga.x, ga.x), f2 = pack2(gb.x, gb.x);
       f32x2 v1[CPT], v2[CPT], acc[CPT][2];
 #pragma unroll
@@ -762,8 +909,9 @@ __global__ void __launch_bounds__(COLS / CPT * 16) mlstm_scan_kernel(const mdb_s
       const int mine = l16 / PER, col = mine >> 1, kind = mine & 1;      // kind: first or second token of the pair
       if (l16 % PER == 0 && t + kind < n) {
         const int64_t th = static_cast<int64_t>(t0 + t + kind) * a.heads + w.head;
-        if (mycol + col < a.vdim) a.out[th * a.vdim + mycol + col] = sum;
-        else if (mycol + col == a.vdim) a.den[th] = fmaxf(fabsf(sum), kind ? gb.z : ga.z) + 1e-6f;      // the normaliser's column
+        if (mycol + col < a.vdim)
+          a.out[th * a.vdim + mycol + col] = MODE == kScanDecay ? fmaf(skip, st[OFF_V + (t + kind) * COLS + cg * CPT + col], sum) : sum;
+        else if (MODE == kScanMlstm && mycol + col == a.vdim) a.den[th] = fmaxf(fabsf(sum), kind ? gb.z : ga.z) + 1e-6f;      // the normaliser's column
       }
     }
     __syncthreads();       // the stage may be refilled
@@ -777,12 +925,13 @@ __global__ void __launch_bounds__(COLS / CPT * 16) mlstm_scan_kernel(const mdb_s
         *reinterpret_cast<float4*>(w.state + static_cast<int64_t>(mycol + i) * DP + c * 64 + l16 * 4) = make_float4(lo.x, lo.y, hi.x, hi.y);
       }
     }
-  if (threadIdx.x == 0)
+  if (MODE == kScanMlstm && threadIdx.x == 0)
     for (int b = block0; b < blocks && b * kScanBlockCols < w.col0 + COLS; ++b) mstate[b] = run_max;
 }
 
-// One-token form: every sequence brings one token and a CTA owns all columns of a head.  The decay is computed from the
-// raw projection, and the head's output is normalised, gated and stored as the next projection's input.  The state is
+// One-token form: every sequence brings one token and a CTA owns all columns of a head.  The delta rule's decay is computed
+// from the raw projection; delta rule and mLSTM normalise and gate the head's output and store it as the next projection's
+// input, the decay scan (whose norms span heads) leaves it in fp32.  The state is
 // fetched into L2 before the wait for the preceding kernel (a prefetch reads nothing that could be stale).
 template <typename T, int MODE, int NCH, int CPT>
 __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb_scan_args a) {
@@ -819,7 +968,7 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
     if (!fresh) m_old = mstate[0];
   }
   const float s0 = a.s0[t * a.heads + head];
-  const float s1 = MODE == kScanMlstm ? a.s1[t * a.heads + head] : 0.f;
+  const float s1 = MODE != kScanDelta ? a.s1[t * a.heads + head] : 0.f;
   float v[CPT];
 #pragma unroll
   for (int i = 0; i < CPT; ++i) v[i] = mycol + i < a.vdim ? a.v[(t * a.heads + head) * a.vdim + mycol + i] : 0.f;
@@ -879,7 +1028,8 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
     }
   } else {
     const float m_new = fmaxf(s1 + m_old, s0);
-    const float fa = expf(s1 + m_old - m_new), ib = expf(s0 - m_new), em = expf(-m_new);
+    const float fa = MODE == kScanDecay ? s0 : expf(s1 + m_old - m_new), ib = MODE == kScanDecay ? s1 : expf(s0 - m_new);
+    const float em = expf(-m_new);
     const f32x2 f2 = pack2(fa, fa), i2 = pack2(ib, ib);
     f32x2 B[CPT], vb[CPT], D = 0ull;
 #pragma unroll
@@ -906,7 +1056,7 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
       }
     }
     const float2 dd = unpack2(D);
-    const float inv = 1.0f / (fmaxf(fabsf(sum8(dd.x + dd.y)), em) + 1e-6f);
+    const float inv = MODE == kScanDecay ? 1.0f : 1.0f / (fmaxf(fabsf(sum8(dd.x + dd.y)), em) + 1e-6f);
 #pragma unroll
     for (int i = 0; i < CPT; ++i) {
       const float2 y = unpack2(B[i]);
@@ -919,6 +1069,13 @@ __global__ void __launch_bounds__(kScanFusedThreads) scan_token_kernel(const mdb
     }
   }
   S.store(state, mycol, a.vdim, l8);
+  if constexpr (MODE == kScanDecay) {
+    const float skip = a.skip != nullptr ? a.skip[head] : 0.f;
+#pragma unroll
+    for (int i = 0; i < CPT; ++i)
+      if (l8 == i && mycol + i < a.vdim) a.out[(t * a.heads + head) * a.vdim + mycol + i] = fmaf(skip, v[i], out[i]);
+    return;
+  }
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < CPT; ++i)
@@ -962,7 +1119,7 @@ int launch_scan_prompt(const mdb_scan_args& a, cudaStream_t st) {
   constexpr int threads = MODE == kScanDelta ? COLS / DELTA_CPT * 8 : COLS / MLSTM_CPT * 16;
   void (*kernel)(mdb_scan_args);
   if constexpr (MODE == kScanDelta) kernel = delta_scan_kernel<DP / 32, DELTA_CPT, COLS>;
-  else kernel = mlstm_scan_kernel<DP, MLSTM_CPT, COLS>;
+  else kernel = gated_scan_kernel<MODE, DP, MLSTM_CPT, COLS>;
   static PerDeviceOnce attr_once;
   const int dev = attr_once.slot();
   if (dev < 0) return MDB_ERR_CUDA;
@@ -1051,8 +1208,45 @@ int mdb_delta_prep(const mdb_delta_prep_args* args, mdb_stream_t stream) {
   }
   if (rc != MDB_OK || a.shift_state || a.taps < 2) return rc;
   const dim3 cgrid((a.channels + 255) / 256, a.bs);
-  return a.dtype == MDB_F32 ? mdb_launch(conv_state_kernel<float>, cgrid, dim3(256), 0, st, a)
-                            : mdb_launch(conv_state_kernel<bf16>, cgrid, dim3(256), 0, st, a);
+  return a.dtype == MDB_F32 ? mdb_launch(conv_state_kernel<float, mdb_delta_prep_args>, cgrid, dim3(256), 0, st, a)
+                            : mdb_launch(conv_state_kernel<bf16, mdb_delta_prep_args>, cgrid, dim3(256), 0, st, a);
+}
+
+int mdb_decay_prep(const mdb_decay_prep_args* args, mdb_stream_t stream) {
+  MDB_REQUIRE(args != nullptr, MDB_ERR_ARG);
+  const mdb_decay_prep_args a = *args;
+  MDB_REQUIRE(a.m >= 0 && a.bs >= 0 && a.heads > 0 && a.kv_heads > 0 && a.dim > 0 && a.vdim > 0 && a.taps >= 0, MDB_ERR_ARG);
+  if (a.m == 0) return MDB_OK;
+  MDB_REQUIRE(a.heads % a.kv_heads == 0 && a.dim_pad >= a.dim && a.dim_pad % 4 == 0, MDB_ERR_ARG);
+  MDB_REQUIRE(rows_present(a.q) && rows_present(a.k) && rows_present(a.v), MDB_ERR_ARG);
+  MDB_REQUIRE(a.row_seq && seqs_ok(a.cu_q, a.start, a.state_slot) && a.q_out && a.k_out && a.v_out && a.decay_out && a.step_out, MDB_ERR_ARG);
+  MDB_REQUIRE(rows_present(a.dt) ? a.a_log && a.dt_bias : a.decay_const != nullptr, MDB_ERR_ARG);
+  MDB_REQUIRE(a.taps == 0 || (a.conv && a.conv_bias && (a.conv_state || a.taps == 1)), MDB_ERR_ARG);
+  MDB_REQUIRE(a.taps == 0 || a.channels == 2 * a.kv_heads * a.dim + a.heads * a.vdim, MDB_ERR_ARG);
+  MDB_REQUIRE(a.taps <= kMaxTaps, MDB_ERR_UNSUPPORTED);
+  const bool parts = a.q.parts != nullptr;
+  MDB_REQUIRE((a.k.parts != nullptr) == parts && (a.v.parts != nullptr) == parts && (!parts || a.dtype == MDB_BF16), MDB_ERR_UNSUPPORTED);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  int rc;
+  if (a.dim % 4 == 0 && a.vdim % 4 == 0 && a.taps <= 4 && rows_ok(a.q) && rows_ok(a.k) && rows_ok(a.v) && a.conv_slot_stride % 4 == 0 &&
+      mdb_aligned16(a.q_out) && mdb_aligned16(a.k_out) && mdb_aligned16(a.v_out) && mdb_aligned16(a.conv) && mdb_aligned16(a.conv_bias)) {
+    const int run = a.m >= 4096 ? 16 : (a.m >= 1024 ? 8 : 1);      // rows a thread walks
+    const int items = a.heads * a.vdim / 4 + 2 * a.kv_heads * (a.dim_pad / 4) + a.heads;
+    const dim3 grid((items + kDecayPrepThreads - 1) / kDecayPrepThreads, (a.m + run - 1) / run), block(kDecayPrepThreads);
+    MDB_REQUIRE(grid.y <= 65535, MDB_ERR_UNSUPPORTED);
+    if (a.dtype == MDB_F32) rc = mdb_launch(decay_prep_rows_kernel<float, false>, grid, block, 0, st, a, run);
+    else if (parts) rc = mdb_launch(decay_prep_rows_kernel<bf16, true>, grid, block, 0, st, a, run);
+    else rc = mdb_launch(decay_prep_rows_kernel<bf16, false>, grid, block, 0, st, a, run);
+  } else {
+    const int items = a.heads * a.vdim + 2 * a.kv_heads * a.dim_pad + a.heads;
+    const dim3 grid(a.m, (items + 255) / 256);
+    rc = a.dtype == MDB_F32 ? mdb_launch(decay_prep_kernel<float>, grid, dim3(256), 0, st, a)
+                            : mdb_launch(decay_prep_kernel<bf16>, grid, dim3(256), 0, st, a);
+  }
+  if (rc != MDB_OK || a.shift_state || a.taps < 2) return rc;
+  const dim3 cgrid((a.channels + 255) / 256, a.bs);
+  return a.dtype == MDB_F32 ? mdb_launch(conv_state_kernel<float, mdb_decay_prep_args>, cgrid, dim3(256), 0, st, a)
+                            : mdb_launch(conv_state_kernel<bf16, mdb_decay_prep_args>, cgrid, dim3(256), 0, st, a);
 }
 
 int mdb_channel_decay(const mdb_decay_args* args, mdb_stream_t stream) {
@@ -1096,12 +1290,14 @@ int mdb_mlstm_prep(const mdb_mlstm_prep_args* args, mdb_stream_t stream) {
 int mdb_scan(const mdb_scan_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(args != nullptr, MDB_ERR_ARG);
   const mdb_scan_args a = *args;
-  MDB_REQUIRE(a.mode == MDB_SCAN_DELTA || a.mode == MDB_SCAN_MLSTM, MDB_ERR_ARG);
+  MDB_REQUIRE(a.mode >= MDB_SCAN_DELTA && a.mode <= MDB_SCAN_DECAY, MDB_ERR_ARG);
   MDB_REQUIRE(a.bs >= 0 && a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.dim > 0 && a.vdim > 0, MDB_ERR_ARG);
   if (a.bs == 0) return MDB_OK;
   MDB_REQUIRE(a.q && a.k && a.v && a.state && (a.mode == MDB_SCAN_DELTA ? a.fused == 0 || a.s0 : a.s0 && a.s1) && seqs_ok(a.cu_q, a.start, a.state_slot), MDB_ERR_ARG);
   MDB_REQUIRE(a.mode != MDB_SCAN_MLSTM || (a.mstate && a.kv_heads == a.heads), MDB_ERR_ARG);
-  if (a.fused) {
+  if (a.mode == MDB_SCAN_DECAY) {
+    MDB_REQUIRE(a.out != nullptr, MDB_ERR_ARG);
+  } else if (a.fused) {
     MDB_REQUIRE(rows_present(a.gate) && a.norm && a.y, MDB_ERR_ARG);
     MDB_REQUIRE(a.mode != MDB_SCAN_DELTA || (rows_present(a.raw_decay) && a.a_log && a.dt_bias), MDB_ERR_ARG);
   } else {
@@ -1112,6 +1308,7 @@ int mdb_scan(const mdb_scan_args* args, mdb_stream_t stream) {
               MDB_ERR_ALIGN);
   MDB_REQUIRE(a.heads <= 65535 && a.bs <= 65535, MDB_ERR_UNSUPPORTED);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (a.mode == MDB_SCAN_DECAY) return launch_scan<kScanDecay>(a, st);
   return a.mode == MDB_SCAN_DELTA ? launch_scan<kScanDelta>(a, st) : launch_scan<kScanMlstm>(a, st);
 }
 

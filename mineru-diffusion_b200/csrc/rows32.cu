@@ -89,9 +89,10 @@ __device__ __forceinline__ float cta_sum(float v, float* red) {
 
 constexpr int kRes32Threads = 256;
 
-// One CTA per row.  residual (+= or, with ids, = embed[id] * scale) + up to two projections + the weighted sum of
-// the chosen experts' rows; y = residual / rms * weight.  NV float4 chunks of the row per thread.
-template <typename T, int NV>
+// One CTA per row.  residual (scaled or, with ids, = embed[id] * scale) + up to two projections + the weighted sum of
+// the chosen experts' rows; y = residual / rms * weight.  POST: the norm replaces the residual, and y is the new residual or
+// its norm with a second weight.  NV float4 chunks of the row per thread.
+template <typename T, int NV, bool POST>
 __global__ void __launch_bounds__(kRes32Threads) residual_norm_kernel(const mdb_residual_norm_args a) {
   pdl_launch_dependents();
   pdl_wait();
@@ -121,6 +122,7 @@ __global__ void __launch_bounds__(kRes32Threads) residual_norm_kernel(const mdb_
       }
     } else {
       x = *reinterpret_cast<const float4*>(res + c);
+      if (POST) { x.x *= a.res_scale; x.y *= a.res_scale; x.z *= a.res_scale; x.w *= a.res_scale; }
     }
 #pragma unroll
     for (int s = 0; s < 2; ++s) {
@@ -139,18 +141,42 @@ __global__ void __launch_bounds__(kRes32Threads) residual_norm_kernel(const mdb_
       }
       x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
     }
-    *reinterpret_cast<float4*>(res + c) = x;
+    if (!POST) *reinterpret_cast<float4*>(res + c) = x;
     v[i] = x;
     ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;      // columns past width hold zeros
   }
-  if (a.y == nullptr) return;
-  const float rstd = 1.0f / sqrtf(cta_sum(ss, red) / static_cast<float>(a.width) + a.eps);
+  if (!POST && a.y == nullptr) return;
   T* y = static_cast<T*>(a.y) + row * a.ldy;
+  if (!POST && a.weight == nullptr) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * kRes32Threads) * 4;
+      if (c < a.width_pad) act_store4(y + c, v[i]);
+    }
+    return;
+  }
+  float rstd = 1.0f / sqrtf(cta_sum(ss, red) / static_cast<float>(a.width) + a.eps);
+  if (POST) {
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * kRes32Threads) * 4;
+      if (c >= a.width_pad) continue;
+      const float4 w = *reinterpret_cast<const float4*>(a.weight + c);
+      v[i] = make_float4(v[i].x * rstd * w.x, v[i].y * rstd * w.y, v[i].z * rstd * w.z, v[i].w * rstd * w.w);
+      *reinterpret_cast<float4*>(res + c) = v[i];
+      if (a.y != nullptr && a.weight2 == nullptr) act_store4(y + c, v[i]);
+      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    if (a.y == nullptr || a.weight2 == nullptr) return;
+    rstd = 1.0f / sqrtf(cta_sum(ss, red) / static_cast<float>(a.width) + a.eps);
+  }
+  const float* weight = POST ? a.weight2 : a.weight;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int c = (threadIdx.x + i * kRes32Threads) * 4;
     if (c >= a.width_pad) continue;
-    const float4 w = *reinterpret_cast<const float4*>(a.weight + c);
+    const float4 w = *reinterpret_cast<const float4*>(weight + c);
     act_store4(y + c, make_float4(v[i].x * rstd * w.x, v[i].y * rstd * w.y, v[i].z * rstd * w.z, v[i].w * rstd * w.w));
   }
 }
@@ -261,6 +287,76 @@ __global__ void __launch_bounds__(128) gated_norm_kernel(const mdb_gated_norm_ar
   }
 }
 
+// A CTA per (row, part): one root mean square over the part's columns of a row, gate before the norm (silu) or after the weight
+// (sigmoid).  The first kKeep pieces stay in registers between the two passes.
+constexpr int kPartNormThreads = 256;
+template <typename T, bool VEC, bool PARTS>
+__global__ void __launch_bounds__(kPartNormThreads) part_norm_kernel(const mdb_part_norm_args a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[kPartNormThreads / 32];
+  const int64_t row = blockIdx.x;
+  const int n = a.n / a.parts, col0 = blockIdx.y * n;
+  const float* o = a.o + row * a.n + col0;
+  const float* w = a.weight + col0;
+  T* y = static_cast<T*>(a.y) + row * a.ldy + col0;
+  if (VEC) {
+    constexpr int kKeep = 4;
+    const int step = blockDim.x * 4;
+    float4 v[kKeep], g[kKeep];
+    auto gated = [&](float4 x, float4 z) {
+      return a.gate_first ? make_float4(x.x * z.x * sigmoid_f(z.x), x.y * z.y * sigmoid_f(z.y), x.z * z.z * sigmoid_f(z.z), x.w * z.w * sigmoid_f(z.w)) : x;
+    };
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      const int c = threadIdx.x * 4 + i * step;
+      v[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < n) {
+        v[i] = *reinterpret_cast<const float4*>(o + c);
+        g[i] = rows_at4_of<T, PARTS>(a.gate, row, col0 + c);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      v[i] = gated(v[i], g[i]);
+      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    for (int c = threadIdx.x * 4 + kKeep * step; c < n; c += step) {
+      const float4 x = gated(*reinterpret_cast<const float4*>(o + c), rows_at4_of<T, PARTS>(a.gate, row, col0 + c));
+      ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+    }
+    const float rstd = a.out_scale / sqrtf(cta_sum(ss, red) / static_cast<float>(n) + a.eps);
+    auto put = [&](int c, float4 x, float4 z) {
+      const float4 wv = *reinterpret_cast<const float4*>(w + c);
+      x = make_float4(x.x * rstd * wv.x, x.y * rstd * wv.y, x.z * rstd * wv.z, x.w * rstd * wv.w);
+      if (!a.gate_first) x = make_float4(x.x * sigmoid_f(z.x), x.y * sigmoid_f(z.y), x.z * sigmoid_f(z.z), x.w * sigmoid_f(z.w));
+      act_store4(y + c, x);
+    };
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      const int c = threadIdx.x * 4 + i * step;
+      if (c < n) put(c, v[i], g[i]);
+    }
+    for (int c = threadIdx.x * 4 + kKeep * step; c < n; c += step) {
+      const float4 z = rows_at4_of<T, PARTS>(a.gate, row, col0 + c);
+      put(c, gated(*reinterpret_cast<const float4*>(o + c), z), z);
+    }
+  } else {
+    auto value = [&](int c, float z) { return a.gate_first ? o[c] * z * sigmoid_f(z) : o[c]; };
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < n; c += blockDim.x) {
+      const float x = value(c, rows_at<T>(a.gate, row, col0 + c));
+      ss += x * x;
+    }
+    const float rstd = a.out_scale / sqrtf(cta_sum(ss, red) / static_cast<float>(n) + a.eps);
+    for (int c = threadIdx.x; c < n; c += blockDim.x) {
+      const float z = rows_at<T>(a.gate, row, col0 + c);
+      y[c] = act_from_f<T>(value(c, z) * rstd * w[c] * (a.gate_first ? 1.0f : sigmoid_f(z)));
+    }
+  }
+}
+
 // Row r of the output = the latent of token r - cu[seq] of its sequence, read through the page table.
 template <typename T>
 __global__ void __launch_bounds__(64) gather_latents_kernel(const T* cache, const int32_t* table,
@@ -335,13 +431,13 @@ bool rows_ok(const mdb_rows& s) {
                               (s.parts == nullptr || (s.nparts >= 1 && s.part_stride % 4 == 0)));
 }
 
-template <typename T>
+template <typename T, bool POST>
 int launch_residual_norm(const mdb_residual_norm_args& a, cudaStream_t st) {
   const int chunks = (a.width_pad / 4 + kRes32Threads - 1) / kRes32Threads;
-  if (chunks <= 1) return mdb_launch(residual_norm_kernel<T, 1>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
-  if (chunks <= 2) return mdb_launch(residual_norm_kernel<T, 2>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
-  if (chunks <= 4) return mdb_launch(residual_norm_kernel<T, 4>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
-  if (chunks <= 8) return mdb_launch(residual_norm_kernel<T, 8>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  if (chunks <= 1) return mdb_launch(residual_norm_kernel<T, 1, POST>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  if (chunks <= 2) return mdb_launch(residual_norm_kernel<T, 2, POST>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  if (chunks <= 4) return mdb_launch(residual_norm_kernel<T, 4, POST>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  if (chunks <= 8) return mdb_launch(residual_norm_kernel<T, 8, POST>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
   return MDB_ERR_UNSUPPORTED;
 }
 }  // namespace
@@ -354,13 +450,16 @@ int mdb_residual_norm(const mdb_residual_norm_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(a.m >= 0 && a.width > 0 && a.width_pad >= a.width, MDB_ERR_ARG);
   if (a.m == 0) return MDB_OK;
   MDB_REQUIRE(a.residual && (a.ids == nullptr || (a.embed && a.vocab > 0)), MDB_ERR_ARG);
-  MDB_REQUIRE(a.y == nullptr || (a.weight && a.ldy >= a.width_pad && a.ldy % 4 == 0), MDB_ERR_ARG);
+  MDB_REQUIRE(a.y == nullptr || (a.ldy >= a.width_pad && a.ldy % 4 == 0), MDB_ERR_ARG);
+  MDB_REQUIRE(a.post ? a.weight != nullptr && a.ids == nullptr : a.weight2 == nullptr && a.res_scale == 1.0f, MDB_ERR_ARG);
   MDB_REQUIRE(a.moe_rows == nullptr || (a.moe_slot && a.moe_weight && a.moe_top > 0 && a.moe_ld % 4 == 0), MDB_ERR_ARG);
   MDB_REQUIRE(a.width_pad % 4 == 0 && rows_ok(a.add[0]) && rows_ok(a.add[1]) && mdb_aligned16(a.residual) &&
-                  mdb_aligned16(a.embed) && mdb_aligned16(a.weight) && mdb_aligned16(a.y) && mdb_aligned16(a.moe_rows),
+                  mdb_aligned16(a.embed) && mdb_aligned16(a.weight) && mdb_aligned16(a.weight2) && mdb_aligned16(a.y) &&
+                  mdb_aligned16(a.moe_rows),
               MDB_ERR_ALIGN);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return a.dtype == MDB_F32 ? launch_residual_norm<float>(a, st) : launch_residual_norm<bf16>(a, st);
+  if (a.post) return a.dtype == MDB_F32 ? launch_residual_norm<float, true>(a, st) : launch_residual_norm<bf16, true>(a, st);
+  return a.dtype == MDB_F32 ? launch_residual_norm<float, false>(a, st) : launch_residual_norm<bf16, false>(a, st);
 }
 
 int mdb_rms_rows(int dtype, const mdb_rms_segment* segments, int nseg, int m, mdb_stream_t stream) {
@@ -401,6 +500,26 @@ int mdb_gated_norm(const mdb_gated_norm_args* args, mdb_stream_t stream) {
   if (!vec) return mdb_launch(gated_norm_kernel<bf16, false, true>, grid, dim3(128), 0, st, a);
   return parts ? mdb_launch(gated_norm_kernel<bf16, true, true>, grid, dim3(128), 0, st, a)
                : mdb_launch(gated_norm_kernel<bf16, true, false>, grid, dim3(128), 0, st, a);
+}
+
+int mdb_part_norm(const mdb_part_norm_args* args, mdb_stream_t stream) {
+  MDB_REQUIRE(args != nullptr, MDB_ERR_ARG);
+  const mdb_part_norm_args a = *args;
+  MDB_REQUIRE(a.m >= 0 && a.n > 0 && a.parts > 0 && a.n % a.parts == 0, MDB_ERR_ARG);
+  if (a.m == 0) return MDB_OK;
+  MDB_REQUIRE(a.o && a.weight && a.y && rows_present(a.gate) && a.ldy >= a.n, MDB_ERR_ARG);
+  MDB_REQUIRE(a.parts <= 65535, MDB_ERR_UNSUPPORTED);
+  const int n = a.n / a.parts;
+  const bool vec = n % 4 == 0 && rows_ok(a.gate) && a.ldy % 4 == 0 && mdb_aligned16(a.o) && mdb_aligned16(a.y) && mdb_aligned16(a.weight);
+  const bool parts = a.gate.parts != nullptr;
+  const dim3 grid(a.m, a.parts), block(n <= 128 ? 32 : (n <= 512 ? 64 : (n <= 2048 ? 128 : kPartNormThreads)));
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (a.dtype == MDB_F32)
+    return vec && !parts ? mdb_launch(part_norm_kernel<float, true, false>, grid, block, 0, st, a)
+                         : mdb_launch(part_norm_kernel<float, false, true>, grid, block, 0, st, a);
+  if (!vec) return mdb_launch(part_norm_kernel<bf16, false, true>, grid, block, 0, st, a);
+  return parts ? mdb_launch(part_norm_kernel<bf16, true, true>, grid, block, 0, st, a)
+               : mdb_launch(part_norm_kernel<bf16, true, false>, grid, block, 0, st, a);
 }
 
 int mdb_gather_latents(int dtype, const void* cache, const int32_t* block_table, int table_stride, int num_pages,

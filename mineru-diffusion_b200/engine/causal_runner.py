@@ -124,13 +124,13 @@ class CausalModelRunner:
         self.graphs.clear()
 
     def _size_cache(self):
-        """Latent pages and state slots: as configured, else a slot per request in flight and what memory is left."""
+        """Cache pages and state slots: as configured, else a slot per request in flight and what memory is left."""
         config = self.config
         if config.num_state_slots <= 0:
             config.num_state_slots = config.max_num_seqs
         page = bytes_per_page(self.cfg, self.dtype)
         if config.num_kvcache_blocks <= 0:
-            if page == 0:                       # no latent attention: pages only bound the lengths
+            if page == 0:                       # no attention: pages only bound the lengths
                 config.num_kvcache_blocks = self.max_pages * config.max_num_seqs
                 return
             free, total = torch.cuda.mem_get_info(self.device)
@@ -140,20 +140,13 @@ class CausalModelRunner:
             wanted = self.max_pages * config.max_num_seqs
             config.num_kvcache_blocks = min(wanted, (budget - reserve) // page)
         if config.num_kvcache_blocks <= 0:
-            raise AssertionError("no memory left for the latent cache")
+            raise AssertionError("no memory left for the paged cache")
 
     # ------------------------------------------------------------------ the step function
-    def _batch(self, inp: _StepInputs, m: int, bs: int, max_q: int, total_k: int, nsplit: int) -> StepBatch:
+    def _batch(self, inp: _StepInputs, m: int, bs: int, max_q: int, total_k: int, max_ctx: int) -> StepBatch:
         d = inp.d
         return StepBatch(m, bs, d["ids"][:m], d["pos"][:m], d["row_seq"][:m], d["slots"][:m], d["cu_q"][:bs + 1],
-                         d["cu_k"][:bs + 1], d["start"][:bs], d["slot"][:bs], d["table"][:bs], max_q, total_k, nsplit)
-
-    def attn_nsplit(self, rows: int, max_ctx: int) -> int:
-        """Key-range parts of the latent-space attention: about two CTAs per SM, parts of at least 128 keys."""
-        heads = max((l.mixer.heads for l in self.cfg.layers if l.type == "latent_attention"), default=0)
-        if heads == 0:
-            return 1
-        return max(1, min(296 // max(1, rows * -(-heads // 16)), max_ctx // 128, 64))
+                         d["cu_k"][:bs + 1], d["start"][:bs], d["slot"][:bs], d["table"][:bs], max_q, total_k, max_ctx)
 
     def _check_counts(self, seqs, counts):
         if len(seqs) > self.max_bs:
@@ -165,10 +158,10 @@ class CausalModelRunner:
             if seq.state_slot < 0:
                 raise AssertionError("a sequence holds no state slot")
 
-    def _one_token_body(self, bs: int, nsplit: int):
+    def _one_token_body(self, bs: int):
         """All of a one-token step that depends only on device buffers, for a bucket of ``bs`` requests."""
         eng, d = self.engine, self.inputs.d
-        h = eng.forward(self._batch(self.inputs, bs, bs, 1, 0, nsplit))
+        h = eng.forward(self._batch(self.inputs, bs, bs, 1, 0, self.config.max_model_len))
         eng.logits(h, self.logits_dev[:bs])
         status = self.res_dev[bs:bs + 1].view(torch.int32)
         ops.pick_token(self.logits_dev[:bs], self.cfg.vocab_size, d["temp"][:bs], self.noise_seed, d["step"], self.res_dev[:bs],
@@ -206,8 +199,8 @@ class CausalModelRunner:
         self._mark(0)
         inp.send()
         eng = self.engine
-        nsplit = self.attn_nsplit(m, max(s.num_cached_tokens + n for s, n in zip(seqs, counts)))
-        hidden = eng.forward(self._batch(inp, m, bs, max_q, total_k, nsplit))
+        max_ctx = max(s.num_cached_tokens + n for s, n in zip(seqs, counts))
+        hidden = eng.forward(self._batch(inp, m, bs, max_q, total_k, max_ctx))
         logits, tokens = [], []
         for lo in range(0, nw, self.max_want) or [0]:
             n = min(self.max_want, nw - lo)
@@ -266,13 +259,12 @@ class CausalModelRunner:
             self.inputs.fill([], [], pad_to=bs)
             self.inputs.h["temp"].fill(0.0)
             self.inputs.send()
-            nsplit = self.attn_nsplit(bs, self.config.max_model_len)
-            self._one_token_body(bs, nsplit)        # sets kernel attributes and allocates buffers outside the capture
+            self._one_token_body(bs)        # sets kernel attributes and allocates buffers outside the capture
             torch.cuda.synchronize()
             graph = torch.cuda.CUDAGraph()
             with torch.cuda.graph(graph, pool):
                 self.inputs.send()
-                self._one_token_body(bs, nsplit)
+                self._one_token_body(bs)
                 self.res_host[:bs + 1].copy_(self.res_dev[:bs + 1], non_blocking=True)
             if pool is None:
                 pool = graph.pool()

@@ -9,7 +9,7 @@ from dataclasses import dataclass
 from importlib import import_module
 from typing import Callable
 
-from .hybrid_config import HybridConfig
+from .hybrid_config import DESIGNS, HybridConfig
 
 
 @dataclass(frozen=True)
@@ -69,5 +69,6 @@ def causal_request(token_ids, params, config):
 
 register(Architecture("sdar", object, _read_sdar, ".model_runner:ModelRunner", ".scheduler:Scheduler",
                       ".registry:sdar_request"))
-register(Architecture("Zikunex", HybridConfig, HybridConfig.from_json, ".causal_runner:CausalModelRunner",
-                      ".causal_scheduler:CausalScheduler", ".registry:causal_request"))
+for _name in DESIGNS:
+    register(Architecture(_name, HybridConfig, HybridConfig.from_json, ".causal_runner:CausalModelRunner",
+                          ".causal_scheduler:CausalScheduler", ".registry:causal_request"))

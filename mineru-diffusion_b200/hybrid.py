@@ -1,4 +1,4 @@
-"""Layer stack of decoders whose layers mix recurrences, latent attention and experts (``HybridConfig``).
+"""Layer stack of decoders whose layers mix recurrences, attention and experts (``HybridConfig``).
 
 ``HybridWeights`` holds the checkpoint's tensors in the layout the kernels read: every projection of a mixer that
 takes the layer's normed input is stacked into one matrix, rows and columns are padded with zeros to multiples of
@@ -8,10 +8,14 @@ the stack over a step's rows:
     residual += previous output, RMSNorm -> one GEMM for all inputs of the mixer -> mixer -> output projection
     residual += ..., RMSNorm -> feed-forward (dense, or router -> plan -> gather -> grouped GEMMs)
 
+In designs with the norm behind the sum the same row kernel leaves norm(scale * residual + output) as the new residual.  Two
+mixers side by side share the input GEMM and the output GEMM: each leaves its scaled output in its own columns of one
+buffer, and the product with the joined output matrices is their sum.
+
 The residual is fp32; activations are bf16 or, in the fp32 mode, fp32 throughout.  A step is ragged: it brings any
 number of tokens of any number of sequences.  Steps of at most 64 rows leave their projections as fp32 split-k slices
 that the next kernel sums; steps that bring one token per sequence take the fused one-token form of the recurrences.
-Recurrent and convolution state lives in a slot per sequence, latents in the paged cache.
+Recurrent and convolution state lives in a slot per sequence, latents, keys and values in paged caches.
 """
 from __future__ import annotations
 
@@ -20,7 +24,8 @@ from dataclasses import dataclass, field
 import torch
 
 from . import ops
-from .engine.hybrid_config import (ChannelDeltaSpec, DenseSpec, HybridConfig, LatentAttentionSpec, MlstmSpec, MoeSpec)
+from .engine.hybrid_config import (ChannelDeltaSpec, DecayScanSpec, DenseSpec, HybridConfig, LatentAttentionSpec, MlstmSpec,
+                                   MoeSpec, ParallelSpec, WindowAttentionSpec, parts_of)
 
 PAGE = 256
 SKINNY_MAX_ROWS = 64
@@ -31,6 +36,17 @@ EXPAND_MIN_TOKENS = 32
 
 def pad128(n: int) -> int:
     return (n + 127) // 128 * 128
+
+
+def pad_head(dim: int) -> int:
+    """Channels of an attention head as the paged K and V caches store them."""
+    return (dim + 63) // 64 * 64
+
+
+def key_parts(ctas: int, keys: int) -> int:
+    """Key-range parts of an attention of ``ctas`` CTAs over up to ``keys`` keys each: about two CTAs per SM, parts of at least
+    128 keys."""
+    return max(1, min(296 // max(1, ctas), keys // 128, 64))
 
 
 class MissingTensors(KeyError):
@@ -62,14 +78,15 @@ class _Source:
 @dataclass
 class HybridWeights:
     dtype: torch.dtype
-    embed: torch.Tensor                 # [vocab, Wp]
+    embed: torch.Tensor                 # [vocab, Wp]; [pad128(vocab), Wp] where it is the output matrix too
     head: torch.Tensor                  # [pad128(vocab), Wp]
     final_norm: torch.Tensor            # fp32 [Wp]
     layers: list[dict] = field(default_factory=list)
 
     def nbytes(self) -> int:
-        tensors = [self.embed, self.head, self.final_norm]
-        tensors += [t for lw in self.layers for t in lw.values() if isinstance(t, torch.Tensor)]
+        tensors = [self.embed, self.final_norm] + ([] if self.head is self.embed else [self.head])
+        tensors += [t for lw in self.layers for d in (lw, *lw.get("parts", ())) if d is not None for t in d.values()
+                    if isinstance(t, torch.Tensor)]
         return sum(t.numel() * t.element_size() for t in tensors)
 
     @classmethod
@@ -113,11 +130,62 @@ class HybridWeights:
         def four(n: int) -> int:
             return (n + 3) // 4 * 4
 
+        def residual_norm(name: str) -> torch.Tensor:
+            return vec(src(name, w).float() + cfg.design.norm_offset, wp)
+
+        def window_attention(mx: WindowAttentionSpec, m: str) -> tuple[list, dict, torch.Tensor]:
+            """(input projections, parameters, output projection) of a mixer whose tensors start with ``m``."""
+            parts = [(src(m + "q", mx.heads * mx.dim, w), four(mx.heads * mx.dim)),
+                     (src(m + "k", mx.kv_heads * mx.dim, w), four(mx.kv_heads * mx.dim)), (src(m + "g", mx.heads, w), four(mx.heads))]
+            pairs = torch.arange(mx.rot_dims // 2, dtype=torch.float64)
+            inv_freq = (mx.rot_base ** (-2.0 * pairs / max(1, mx.rot_dims))).to(device)
+            params = {"q_norm": vec(src(m + "q.norm", mx.dim), four(mx.dim)), "k_norm": vec(src(m + "k.norm", mx.dim), four(mx.dim)),
+                      "inv_freq": inv_freq}
+            return parts, params, src(m + "o", w, mx.heads * mx.dim)
+
+        def decay_scan(mx: DecayScanSpec, m: str) -> tuple[list, dict, torch.Tensor]:
+            nv, nk = mx.heads * mx.vdim, mx.kv_heads * mx.dim
+            params = {"norm": vec(src(m + "norm", nv), four(nv))}
+            if mx.decay is not None:
+                # in the order of the other form's inputs: gate, values, keys, queries
+                parts = [(src(m + "g", nv, w), four(nv)), (src(m + "v", nv, w), four(nv)), (src(m + "k", nk, w), four(nk)),
+                         (src(m + "q", nk, w), four(nk))]
+                params["decay"] = torch.tensor(mx.decay, dtype=torch.float32, device=device)
+            else:
+                z, x, b, c, dt = src(m + "in", 2 * nv + 2 * nk + mx.heads, w).split([nv, nv, nk, nk, mx.heads])
+                parts = [(z, four(nv)), (x, four(nv)), (b, four(nk)), (c, four(nk)), (dt, four(mx.heads))]
+                params["conv"] = src(m + "conv", nv + 2 * nk, mx.conv).to(device=device, dtype=torch.float32).contiguous()
+                params["conv_bias"] = vec(src(m + "conv.b", nv + 2 * nk), four(nv + 2 * nk))
+                for key, name in (("dt_bias", "dt_bias"), ("a_log", "A_log"), ("skip", "D")):
+                    params[key] = vec(src(m + name, mx.heads), mx.heads)
+            return parts, params, src(m + "o", w, nv)
+
+        def joined(mixers: list) -> dict:
+            """Weights of mixers that read one input and whose outputs are summed: both GEMMs are shared."""
+            stacked, starts = stack([p for parts, _, _ in mixers for p in parts])
+            offsets, at = [], 0
+            for _, _, o in mixers:
+                offsets.append(at)
+                at += (o.shape[1] + 7) // 8 * 8
+            out = torch.zeros(wp, pad128(at), dtype=dtype, device=device)
+            subs = []
+            for (parts, params, o), off in zip(mixers, offsets):
+                out[:w, off:off + o.shape[1]].copy_(o)
+                subs.append({**params, "starts": starts[:len(parts)], "out": off})
+                starts = starts[len(parts):]
+            return {"in": stacked, "o": out, "parts": subs}
+
         layers = []
         for i, layer in enumerate(cfg.layers):
             p, mx, lw = f"l{i}.", layer.mixer, {}
-            lw["norm1"] = vec(src(p + "norm1", w), wp)
-            if isinstance(mx, ChannelDeltaSpec):
+            lw["norm1"] = residual_norm(p + "norm1")
+            if isinstance(mx, ParallelSpec):
+                lw.update(joined([window_attention(mx.left, p + "mix.left."), decay_scan(mx.right, p + "mix.right.")]))
+            elif isinstance(mx, WindowAttentionSpec):
+                lw.update(joined([window_attention(mx, p + "mix.")]))
+            elif isinstance(mx, DecayScanSpec):
+                lw.update(joined([decay_scan(mx, p + "mix.")]))
+            elif isinstance(mx, ChannelDeltaSpec):
                 nq, nv = mx.kv_heads * mx.dim, mx.heads * mx.vdim
                 a1, g1 = src(p + "mix.a1", None, w), src(p + "mix.g1", None, w)
                 ra, rg = a1.shape[0], g1.shape[0]
@@ -162,10 +230,12 @@ class HybridWeights:
                 lw["o"] = heads_cols(src(p + "mix.o", w, mx.heads * mx.vdim), mx.heads, mx.vdim, vp)
             mlp = layer.mlp
             if mlp is not None:
-                lw["norm2"] = vec(src(p + "norm2", w), wp)
+                lw["norm2"] = residual_norm(p + "norm2")
             if isinstance(mlp, DenseSpec):
                 fp = pad128(mlp.ff)
                 lw["up"], lw["down"] = mat(src(p + "mlp.up", mlp.ff, w), fp, wp), mat(src(p + "mlp.down", w, mlp.ff), wp, fp)
+                if mlp.act == "relu_glu":
+                    lw["up"] = torch.cat([mat(src(p + "mlp.gate", mlp.ff, w), fp, wp), lw["up"]])
             elif isinstance(mlp, MoeSpec):
                 fp = pad128(mlp.expert_ff)
                 lw["router"] = mat(src(p + "mlp.router", mlp.experts, w), pad128(mlp.experts), wp)
@@ -180,8 +250,10 @@ class HybridWeights:
                     lw["s_up"] = mat(src(p + "mlp.shared.up", mlp.shared_ff, w), sp, wp)
                     lw["s_down"] = mat(src(p + "mlp.shared.down", w, mlp.shared_ff), wp, sp)
             layers.append(lw)
-        out = cls(dtype, mat(src("embed", cfg.vocab_size, w), cfg.vocab_size, wp),
-                  mat(src("head", cfg.vocab_size, w), pad128(cfg.vocab_size), wp), vec(src("final.norm", w), wp), layers)
+        tied = cfg.design.tied_head
+        embed = mat(src("embed", cfg.vocab_size, w), pad128(cfg.vocab_size) if tied else cfg.vocab_size, wp)
+        head = embed if tied else mat(src("head", cfg.vocab_size, w), pad128(cfg.vocab_size), wp)
+        out = cls(dtype, embed, head, residual_norm("final.norm"), layers)
         src.check_all_taken()
         return out
 
@@ -199,7 +271,23 @@ def tensor_shapes(cfg: HybridConfig, rank: int = 128) -> dict[str, tuple]:
         p, mx, mlp = f"l{i}.", layer.mixer, layer.mlp
         shapes[p + "norm1"] = (w,)
         m = p + "mix."
-        if isinstance(mx, ChannelDeltaSpec):
+        if isinstance(mx, (ParallelSpec, WindowAttentionSpec, DecayScanSpec)):
+            subs = parts_of(mx)
+            for sub, pre in zip(subs, (m + "left.", m + "right.") if len(subs) > 1 else (m,)):
+                if isinstance(sub, WindowAttentionSpec):
+                    nq, nk = sub.heads * sub.dim, sub.kv_heads * sub.dim
+                    shapes.update({pre + "q": (nq, w), pre + "k": (nk, w), pre + "q.norm": (sub.dim,), pre + "k.norm": (sub.dim,),
+                                   pre + "g": (sub.heads, w), pre + "o": (w, nq)})
+                    continue
+                nv, nk = sub.heads * sub.vdim, sub.kv_heads * sub.dim
+                shapes.update({pre + "norm": (nv,), pre + "o": (w, nv)})
+                if sub.decay is not None:
+                    shapes.update({pre + "q": (nk, w), pre + "k": (nk, w), pre + "v": (nv, w), pre + "g": (nv, w)})
+                else:
+                    shapes.update({pre + "in": (2 * nv + 2 * nk + sub.heads, w), pre + "conv": (nv + 2 * nk, sub.conv),
+                                   pre + "conv.b": (nv + 2 * nk,), pre + "dt_bias": (sub.heads,), pre + "A_log": (sub.heads,),
+                                   pre + "D": (sub.heads,)})
+        elif isinstance(mx, ChannelDeltaSpec):
             nq, nv = mx.kv_heads * mx.dim, mx.heads * mx.vdim
             for name, n in (("q", nq), ("k", nq), ("v", nv)):
                 shapes[m + name], shapes[m + name + ".conv"] = (n, w), (n, mx.conv)
@@ -222,13 +310,17 @@ def tensor_shapes(cfg: HybridConfig, rank: int = 128) -> dict[str, tuple]:
             shapes[p + "norm2"] = (w,)
         if isinstance(mlp, DenseSpec):
             shapes.update({m + "up": (mlp.ff, w), m + "down": (w, mlp.ff)})
+            if mlp.act == "relu_glu":
+                shapes[m + "gate"] = (mlp.ff, w)
         elif isinstance(mlp, MoeSpec):
             for e in range(mlp.experts):
                 shapes.update({m + f"e{e}.up": (mlp.expert_ff, w), m + f"e{e}.down": (w, mlp.expert_ff)})
             shapes[m + "router"] = (mlp.experts, w)
             if mlp.shared_ff is not None:
                 shapes.update({m + "shared.up": (mlp.shared_ff, w), m + "shared.down": (w, mlp.shared_ff)})
-    shapes["final.norm"], shapes["head"] = (w,), (cfg.vocab_size, w)
+    shapes["final.norm"] = (w,)
+    if not cfg.design.tied_head:
+        shapes["head"] = (cfg.vocab_size, w)
     return shapes
 
 
@@ -238,13 +330,15 @@ def random_tensors(cfg: HybridConfig, seed: int, device, rank: int = 128, std: f
     out = {}
     for name, shape in tensor_shapes(cfg, rank).items():
         t = torch.randn(shape, generator=g, device=device, dtype=torch.float32)
-        if name.endswith("norm") or ".norm" in name:
+        if name.endswith(("norm1", "norm2", "final.norm")):
+            t = 1.0 - cfg.design.norm_offset + 0.1 * t
+        elif name.endswith("norm") or ".norm" in name:
             t = 1.0 + 0.1 * t
         elif name.endswith("A_log"):
             t = t - 2.0
         elif name.endswith("f.b"):
             t = t + 3.0
-        elif name.endswith((".b", ".dt_bias")) and len(shape) == 1:
+        elif name.endswith((".b", ".dt_bias", ".D")) and len(shape) == 1:
             pass
         elif name.endswith(".conv"):
             t = t * (0.5 / shape[1] ** 0.5) + 0.25
@@ -270,7 +364,7 @@ class StepBatch:
     table: torch.Tensor          # [bs, pages]
     max_q: int                   # longest portion
     total_k: int                 # cu_k[-1]; 0 in steps of one token per sequence
-    nsplit: int = 1              # key-range parts of the latent-space attention
+    max_ctx: int = 1             # longest context after the step (a bound)
 
 
 class HybridEngine:
@@ -286,15 +380,18 @@ class HybridEngine:
         self._one_token = False                  # the step in progress brings one token per sequence
         self.collect: list | None = None         # tests: receives the residual after every layer
         self.latents: dict[int, torch.Tensor] = {}
+        self.kv: dict[int, tuple] = {}
         self.state: dict[int, dict] = {}
         for i, layer in enumerate(cfg.layers):
-            mx = layer.mixer
-            if isinstance(mx, LatentAttentionSpec):
-                if mx.kv_from is None:
-                    self.latents[i] = torch.zeros(num_pages * PAGE, pad128(mx.kv_rank), dtype=self.dtype, device=device)
-            else:
-                self.state[i] = {k: torch.zeros(num_slots, *shape, dtype=dt, device=device)
-                                 for k, (shape, dt) in state_shapes(mx, self.dtype).items()}
+            for mx in parts_of(layer.mixer):
+                caches = [torch.zeros(num_pages * PAGE, *shape, dtype=self.dtype, device=device) for shape in cache_shapes(mx)]
+                if isinstance(mx, WindowAttentionSpec):
+                    self.kv[i] = tuple(caches)
+                elif caches:
+                    self.latents[i] = caches[0]
+                if state_shapes(mx, self.dtype):
+                    self.state[i] = {k: torch.zeros(num_slots, *shape, dtype=dt, device=device)
+                                     for k, (shape, dt) in state_shapes(mx, self.dtype).items()}
         self.residual = torch.zeros(max_tokens, self.width_pad, dtype=torch.float32, device=device)
 
     # ------------------------------------------------------------------ buffers
@@ -340,25 +437,40 @@ class HybridEngine:
         h = self.buf("h", m, self.width_pad)
         res = self.residual[:m]
 
+        post = cfg.design.post_norm
+
         def norm(weight, **kw):
             ops.residual_norm(res, cfg.hidden_size, cfg.rms_norm_eps, self.dtype, weight=weight, out=h, **kw)
 
-        norm(self.w.layers[0]["norm1"] if cfg.layers else self.w.final_norm, ids=b.ids, embed=self.w.embed,
-             embed_scale=cfg.embed_scale)
+        first = self.w.final_norm if not cfg.layers else (None if post else self.w.layers[0]["norm1"])
+        norm(first, ids=b.ids, embed=self.w.embed[:cfg.vocab_size], embed_scale=cfg.embed_scale)
         for i, (layer, lw) in enumerate(zip(cfg.layers, self.w.layers)):
-            mx = layer.mixer
-            if isinstance(mx, ChannelDeltaSpec):
+            mx, last = layer.mixer, i + 1 == len(cfg.layers)
+            if "parts" in lw:
+                y = self._joined(i, mx, lw, h, b)
+            elif isinstance(mx, ChannelDeltaSpec):
                 y = self._channel_delta(i, mx, lw, h, b)
             elif isinstance(mx, MlstmSpec):
                 y = self._mlstm(i, mx, lw, h, b)
             else:
                 y = self._latent_attention(i, mx, lw, h, b)
             after = {"add": (y,)}
-            if layer.mlp is not None:
-                norm(lw["norm2"], **after)
-                after = self._dense(layer.mlp, lw, h) if isinstance(layer.mlp, DenseSpec) else self._moe(layer.mlp, lw, h, b)
-            last = i + 1 == len(cfg.layers)
-            norm(self.w.final_norm if last else self.w.layers[i + 1]["norm1"], **after)
+
+            def feed_forward():
+                return self._dense(layer.mlp, lw, h) if isinstance(layer.mlp, DenseSpec) else self._moe(layer.mlp, lw, h, b)
+
+            if post:
+                # every sum is normalised into the residual; the last one also meets the final norm
+                behind = dict(post=True, res_scale=cfg.residual_scale)
+                final = self.w.final_norm if last else None
+                norm(lw["norm1"], weight2=final if layer.mlp is None else None, **behind, **after)
+                if layer.mlp is not None:
+                    norm(lw["norm2"], weight2=final, **behind, **feed_forward())
+            else:
+                if layer.mlp is not None:
+                    norm(lw["norm2"], **after)
+                    after = feed_forward()
+                norm(self.w.final_norm if last else self.w.layers[i + 1]["norm1"], **after)
             if self.collect is not None:
                 self.collect.append(res[:, :cfg.hidden_size].clone())
         return h
@@ -370,6 +482,48 @@ class HybridEngine:
     # ------------------------------------------------------------------ mixers
     def _portions(self, b: StepBatch):
         return b.row_seq, b.cu_q, b.start, b.state_slot
+
+    def _joined(self, li: int, mx, lw: dict, h: torch.Tensor, b: StepBatch) -> ops.Rows:
+        """One mixer, or several side by side, on one input product; their outputs meet in one output product."""
+        scales = (mx.left_scale, mx.right_scale) if isinstance(mx, ParallelSpec) else (1.0,)
+        x = self._linear("mix_in", h, lw["in"])
+        widths = tuple(part.heads * (part.dim if isinstance(part, WindowAttentionSpec) else part.vdim) for part in parts_of(mx))
+        y = self.buf("joined_o_" + "_".join(map(str, widths)), b.m, lw["o"].shape[1])
+        for part, pw, n, scale in zip(parts_of(mx), lw["parts"], widths, scales):
+            run = self._window_attention if isinstance(part, WindowAttentionSpec) else self._decay_scan
+            run(li, part, pw, x, y[:, pw["out"]:pw["out"] + n], scale, b)
+        return self._linear("mix_out", y, lw["o"])
+
+    def _window_attention(self, li: int, mx: WindowAttentionSpec, pw: dict, x: ops.Rows, y: torch.Tensor, scale: float, b: StepBatch):
+        m, (k_cache, v_cache) = b.m, self.kv[li]
+        q0, k0, g0 = pw["starts"]
+        q = self.buf(f"window_q_{mx.dim}", m, mx.heads, k_cache.shape[2])
+        ops.rotary_commit(x.cols(q0), x.cols(k0), x.cols(k0), mx.heads, mx.kv_heads, mx.dim, pw["q_norm"], pw["k_norm"],
+                          self.cfg.rms_norm_eps, pw["inv_freq"], b.row_pos, b.slots, q, k_cache, v_cache)
+        keys = min(b.max_ctx, mx.window) if mx.window else b.max_ctx
+        nsplit = key_parts(m * mx.kv_heads * -(-mx.heads // mx.kv_heads // 16), keys)
+        ws = self.scratch("window_ws", max(16, ops.window_attn_workspace_bytes(m, mx.heads, q.shape[2], nsplit)), torch.uint8)
+        ops.window_attn(q, k_cache, v_cache, b.table, self._portions(b), b.row_pos, b.max_q, mx.dim, mx.window, mx.sink, mx.scale, y,
+                        gate=x.cols(g0), out_scale=scale, nsplit=nsplit, workspace=ws)
+
+    def _decay_scan(self, li: int, mx: DecayScanSpec, pw: dict, x: ops.Rows, y: torch.Tensor, scale: float, b: StepBatch):
+        m, st, f32 = b.m, self.state[li], torch.float32
+        heads, kvh, dim, vdim = mx.heads, mx.kv_heads, mx.dim, mx.vdim
+        dp, one_token = ops.scan_dim_pad(dim), b.max_q == 1
+        z0, v0, k0, q0, *dt0 = pw["starts"]
+        outs = (self.buf("scan_q", m, kvh, dp, dtype=f32), self.buf("scan_k", m, kvh, dp, dtype=f32),
+                self.buf("scan_v", m, heads, vdim, dtype=f32), self.buf("scan_s0", m, heads, dtype=f32),
+                self.buf("scan_s1", m, heads, dtype=f32))
+        scalars = dict(decay=pw["decay"]) if mx.decay is not None else dict(
+            dt=x.cols(dt0[0]), a_log=pw["a_log"], dt_bias=pw["dt_bias"], conv=pw["conv"], conv_bias=pw["conv_bias"],
+            conv_state=st["conv"], shift_state=one_token)
+        ops.decay_prep(self.dtype, m, b.bs, heads, kvh, dim, vdim, x.cols(q0), x.cols(k0), x.cols(v0), self._portions(b), outs, **scalars)
+        o = self.buf("scan_o", m, heads, vdim, dtype=f32)
+        ops.scan(ops.SCAN_DECAY, self.dtype, b.bs, heads, kvh, dim, vdim, *outs, st["s"], self._portions(b), out=o, skip=pw.get("skip"),
+                 one_token=one_token and ops.scan_fusable(dp, vdim))
+        # lightning attention gates behind its norm, Mamba-2 in front of it
+        ops.part_norm(o.view(m, heads * vdim), x.cols(z0), pw["norm"], mx.norm_groups, mx.decay is None, self.cfg.rms_norm_eps, y,
+                      out_scale=scale)
 
     def _channel_delta(self, li: int, mx: ChannelDeltaSpec, lw: dict, h: torch.Tensor, b: StepBatch) -> ops.Rows:
         m, st, f32 = b.m, self.state[li], torch.float32
@@ -448,14 +602,16 @@ class HybridEngine:
         else:
             ql = ops.gemm_heads(q, lw["uk_t"], self.buf("latent_qk", m, heads * kr))
             ol = self.buf("latent_o", m, heads * kr)
-            ws = self.scratch("latent_ws", max(16, ops.latent_attn_workspace_bytes(m, heads, kr, b.nsplit)), torch.uint8)
-            ops.latent_attn(ql, cache, b.table, b.row_seq, b.row_pos, heads, mx.scale, ol, b.nsplit, ws)
+            nsplit = key_parts(m * -(-heads // 16), b.max_ctx)
+            ws = self.scratch("latent_ws", max(16, ops.latent_attn_workspace_bytes(m, heads, kr, nsplit)), torch.uint8)
+            ops.latent_attn(ql, cache, b.table, b.row_seq, b.row_pos, heads, mx.scale, ol, nsplit, ws)
             ops.gemm_heads(ol, lw["uv"], o)
         return self._linear("mix_out", o, lw["o"])
 
     # ------------------------------------------------------------------ feed-forward
     def _dense(self, mlp: DenseSpec, lw: dict, h: torch.Tensor) -> dict:
-        act = ops.gemm(h, lw["up"], self.buf("ff_act", h.shape[0], lw["up"].shape[0]), act=ops.ACT_RELU2)
+        act = ops.gemm(h, lw["up"], self.buf("ff_act", h.shape[0], lw["down"].shape[1]),
+                       act=ops.ACT_RELU_GLU if mlp.act == "relu_glu" else ops.ACT_RELU2)
         return {"add": (self._linear("ff_out", act, lw["down"]),)}
 
     def _moe(self, mlp: MoeSpec, lw: dict, h: torch.Tensor, b: StepBatch) -> dict:
@@ -484,29 +640,42 @@ class HybridEngine:
         return out
 
 
+def cache_shapes(mx) -> list[tuple]:
+    """What a mixer keeps per token in paged caches."""
+    if isinstance(mx, WindowAttentionSpec):
+        return [(mx.kv_heads, pad_head(mx.dim))] * 2
+    if isinstance(mx, LatentAttentionSpec) and mx.kv_from is None:
+        return [(pad128(mx.kv_rank),)]
+    return []
+
+
 def state_shapes(mx, dtype: torch.dtype) -> dict[str, tuple]:
     """Per-slot state of a recurrent mixer: name -> (shape, dtype)."""
+    if isinstance(mx, (LatentAttentionSpec, WindowAttentionSpec)):
+        return {}
     dp = ops.scan_dim_pad(mx.dim)
     if isinstance(mx, ChannelDeltaSpec):
         channels = 2 * mx.kv_heads * mx.dim + mx.heads * mx.vdim
         return {"s": ((mx.heads, mx.vdim, dp), torch.float32), "conv": ((mx.conv - 1, channels), dtype)}
+    if isinstance(mx, DecayScanSpec):
+        shapes = {"s": ((mx.heads, mx.vdim, dp), torch.float32)}
+        if mx.conv:
+            shapes["conv"] = ((mx.conv - 1, 2 * mx.kv_heads * mx.dim + mx.heads * mx.vdim), dtype)
+        return shapes
     blocks = ops.scan_blocks(mx.vdim)
     return {"s": ((mx.heads, mx.vdim + 1, dp), torch.float32), "m": ((mx.heads, blocks), torch.float32)}
 
 
+def _bytes(shape, dtype: torch.dtype) -> int:
+    n = torch.empty(0, dtype=dtype).element_size()
+    for s in shape:
+        n *= s
+    return n
+
+
 def bytes_per_page(cfg: HybridConfig, dtype: torch.dtype) -> int:
-    e = 2 if dtype == torch.bfloat16 else 4
-    return sum(PAGE * pad128(l.mixer.kv_rank) * e for l in cfg.layers
-               if isinstance(l.mixer, LatentAttentionSpec) and l.mixer.kv_from is None)
+    return sum(PAGE * _bytes(shape, dtype) for l in cfg.layers for mx in parts_of(l.mixer) for shape in cache_shapes(mx))
 
 
 def bytes_per_slot(cfg: HybridConfig, dtype: torch.dtype) -> int:
-    total = 0
-    for l in cfg.layers:
-        if not isinstance(l.mixer, LatentAttentionSpec):
-            for shape, dt in state_shapes(l.mixer, dtype).values():
-                n = 1
-                for s in shape:
-                    n *= s
-                total += n * torch.empty(0, dtype=dt).element_size()
-    return total
+    return sum(_bytes(shape, dt) for l in cfg.layers for mx in parts_of(l.mixer) for shape, dt in state_shapes(mx, dtype).values())

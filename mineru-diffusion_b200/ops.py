@@ -543,7 +543,7 @@ def lm_head_sample_tp(hidden: torch.Tensor, weight: torch.Tensor, temperatures: 
 # Decoders with an fp32 residual: recurrent mixers, latent attention, experts.  Activations are bf16 or fp32 tensors.
 
 _DTYPES = {torch.bfloat16: 0, torch.float32: 1}
-ACT_NONE, ACT_RELU2 = 0, 1
+ACT_NONE, ACT_RELU2, ACT_RELU_GLU = 0, 1, 2
 
 
 class Rows:
@@ -580,9 +580,10 @@ def _act_dtype(t: torch.Tensor, name: str) -> int:
 
 
 def gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: int = ACT_NONE) -> torch.Tensor:
-    """out = act(x w^T); x [m, k] (row stride free), w [n, k]; out of the activation type, or fp32."""
+    """out = act(x w^T); x [m, k] (row stride free), w [n, k]; out of the activation type, or fp32.  ACT_RELU_GLU: w is
+    [2 n, k], gate rows first, and out = relu(gate) * up."""
     m, k = x.shape
-    n = w.shape[0]
+    n = w.shape[0] // 2 if act == ACT_RELU_GLU else w.shape[0]
     a = _lib.GemmArgs(_act_dtype(x, "x"), 0, act, int(out.dtype == torch.float32), x.data_ptr(), w.data_ptr(),
                       out.data_ptr(), _rows(x, "x"), _rows(out, "out"), m, n, k, 0, 0, 0, None, None)
     _lib.check(_lib.lib().mdb_gemm(a, _stream()), "mdb_gemm")
@@ -611,12 +612,16 @@ def gemm_experts(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_exper
 
 def residual_norm(residual: torch.Tensor, width: int, eps: float, dtype: torch.dtype, weight: torch.Tensor | None = None,
                   out: torch.Tensor | None = None, add: tuple = (), ids: torch.Tensor | None = None,
-                  embed: torch.Tensor | None = None, embed_scale: float = 1.0, moe: tuple | None = None) -> None:
+                  embed: torch.Tensor | None = None, embed_scale: float = 1.0, moe: tuple | None = None, post: bool = False,
+                  res_scale: float = 1.0, weight2: torch.Tensor | None = None) -> None:
     """Folds projections (``add``), chosen experts' rows (``moe`` = rows, slots [m, top], weights [m, top]) or the scaled
-    embedding (``ids``) into the fp32 residual and writes its RMSNorm to ``out``."""
+    embedding (``ids``) into the fp32 residual and writes its RMSNorm to ``out`` (without ``weight``: the residual itself).
+    ``post``: the residual, scaled by ``res_scale`` before the sum, becomes its own norm, and ``out`` receives it or its norm
+    with ``weight2``."""
     m, wp = residual.shape
     a = _lib.ResidualNormArgs(dtype=_DTYPES[dtype], m=m, width=width, width_pad=wp, residual=residual.data_ptr(), eps=eps,
-                              weight=_ptr(weight), y=_ptr(out), ldy=0 if out is None else _rows(out, "out"))
+                              weight=_ptr(weight), y=_ptr(out), ldy=0 if out is None else _rows(out, "out"), post=int(post),
+                              weight2=_ptr(weight2), res_scale=res_scale)
     if ids is not None:
         _need(ids, torch.int64, "ids")
         a.ids, a.embed, a.vocab, a.embed_scale = ids.data_ptr(), embed.data_ptr(), embed.shape[0], embed_scale
@@ -648,6 +653,16 @@ def gated_norm(o: torch.Tensor, gate: Rows, weight: torch.Tensor, per_head_weigh
     a = _lib.GatedNormArgs(_act_dtype(out, "out"), m, heads, vdim, o.data_ptr(), _ptr(den), gate.c(), weight.data_ptr(),
                            out.data_ptr(), _rows(out, "out"), vdim if per_head_weight else 0, eps)
     _lib.check(_lib.lib().mdb_gated_norm(a, _stream()), "mdb_gated_norm")
+
+
+def part_norm(o: torch.Tensor, gate: Rows, weight: torch.Tensor, parts: int, gate_first: bool, eps: float, out: torch.Tensor,
+              out_scale: float = 1.0) -> None:
+    """o [m, n] fp32 in ``parts`` equal parts, each by its own root mean square: norm(o * silu(gate)) * weight with
+    ``gate_first``, else norm(o) * weight * sigmoid(gate); times out_scale into the first n columns of ``out``."""
+    m, n = o.shape
+    a = _lib.PartNormArgs(_act_dtype(out, "out"), m, n, parts, int(gate_first), out_scale, eps, o.data_ptr(), gate.c(),
+                          weight.data_ptr(), out.data_ptr(), _rows(out, "out"))
+    _lib.check(_lib.lib().mdb_part_norm(a, _stream()), "mdb_part_norm")
 
 
 def scan_dim_pad(dim: int) -> int:
@@ -705,23 +720,47 @@ def mlstm_prep(dtype: torch.dtype, m: int, heads: int, dim: int, vdim: int, q: R
     _lib.check(_lib.lib().mdb_mlstm_prep(a, _stream()), "mdb_mlstm_prep")
 
 
-SCAN_DELTA, SCAN_MLSTM = 0, 1
+def decay_prep(dtype: torch.dtype, m: int, bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q: Rows, k: Rows, v: Rows,
+               portions: tuple, outs: tuple, dt: Rows | None = None, a_log: torch.Tensor | None = None,
+               dt_bias: torch.Tensor | None = None, decay: torch.Tensor | None = None, conv: torch.Tensor | None = None,
+               conv_bias: torch.Tensor | None = None, conv_state: torch.Tensor | None = None, shift_state: bool = False) -> None:
+    """Inputs of the decay scan: ``outs`` = fp32 (q, k [m, kv_heads, dim_pad], v [m, heads, vdim], decay, step [m, heads]).
+    ``conv`` fp32 [channels, taps] (v | k | q) with ``conv_bias`` and ``conv_state`` [slots, taps - 1, channels], or None: silu
+    alone.  Scalars from ``dt`` with ``a_log`` and ``dt_bias``, or the fixed ``decay`` [heads] and step 1."""
+    qo, ko, vo, do, so = outs
+    row_seq, cu_q, start, slot = portions
+    taps = 0 if conv is None else conv.shape[1]
+    a = _lib.DecayPrepArgs(
+        dtype=_DTYPES[dtype], m=m, bs=bs, heads=heads, kv_heads=kv_heads, dim=dim, dim_pad=qo.shape[-1], vdim=vdim, taps=taps,
+        channels=0 if conv is None else conv.shape[0], shift_state=int(shift_state), q=q.c(), k=k.c(), v=v.c(), dt=_rows_c(dt),
+        conv=_ptr(conv), conv_bias=_ptr(conv_bias), conv_state=(_ptr(conv_state) or None) if taps > 1 else None,
+        conv_slot_stride=conv_state.stride(0) if taps > 1 else 0, num_slots=conv_state.shape[0] if taps > 1 else 1 << 30,
+        row_seq=row_seq.data_ptr(), cu_q=cu_q.data_ptr(), start=start.data_ptr(), state_slot=slot.data_ptr(), a_log=_ptr(a_log),
+        dt_bias=_ptr(dt_bias), decay_const=_ptr(decay), q_out=qo.data_ptr(), k_out=ko.data_ptr(), v_out=vo.data_ptr(),
+        decay_out=do.data_ptr(), step_out=so.data_ptr())
+    _lib.check(_lib.lib().mdb_decay_prep(a, _stream()), "mdb_decay_prep")
+
+
+SCAN_DELTA, SCAN_MLSTM, SCAN_DECAY = 0, 1, 2
 
 
 def scan(mode: int, dtype: torch.dtype, bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q, k, v, s0, s1, state,
          portions: tuple, eps: float = 0.0, g=None, scalars=None, mstate=None, den=None, out=None, raw_decay: Rows | None = None,
-         a_log=None, dt_bias=None, gate: Rows | None = None, norm=None, per_head_norm: bool = False, y=None) -> None:
+         a_log=None, dt_bias=None, gate: Rows | None = None, norm=None, per_head_norm: bool = False, y=None, skip=None,
+         one_token: bool = False) -> None:
     """The recurrence over every sequence's portion; ``state`` [slots, heads, vdim (mLSTM: + 1), dim_pad] fp32.  With ``y``
     the fused one-token form runs (decay from ``raw_decay``, gated norm into ``y``), else ``out`` [m, heads, vdim] fp32
-    (mLSTM: and ``den`` [m, heads]) is written."""
+    (mLSTM: and ``den`` [m, heads]) is written.  Decay scan: s0 = decay, s1 = step, ``skip`` [heads] times v is added to the
+    read-out; ``one_token`` picks its one-token form."""
     _, cu_q, start, slot = portions
     a = _lib.ScanArgs(
-        mode=mode, dtype=_DTYPES[dtype], fused=int(y is not None), bs=bs, heads=heads, kv_heads=kv_heads, dim=dim,
+        mode=mode, dtype=_DTYPES[dtype], fused=int(y is not None or one_token), bs=bs, heads=heads, kv_heads=kv_heads, dim=dim,
         dim_pad=q.shape[-1], vdim=vdim, eps=eps, q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), g=_ptr(g), s0=_ptr(s0),
         s1=_ptr(s1), state=state.data_ptr(), state_slot_stride=state.stride(0), num_slots=state.shape[0],
         mstate=_ptr(mstate), scalars=_ptr(scalars), den=_ptr(den), cu_q=cu_q.data_ptr(), start=start.data_ptr(), state_slot=slot.data_ptr(),
         out=_ptr(out), raw_decay=_rows_c(raw_decay), a_log=_ptr(a_log), dt_bias=_ptr(dt_bias), gate=_rows_c(gate),
-        norm=_ptr(norm), norm_head_stride=vdim if per_head_norm else 0, y=_ptr(y), ldy=0 if y is None else _rows(y, "y"))
+        norm=_ptr(norm), norm_head_stride=vdim if per_head_norm else 0, y=_ptr(y), ldy=0 if y is None else _rows(y, "y"),
+        skip=_ptr(skip))
     _lib.check(_lib.lib().mdb_scan(a, _stream()), "mdb_scan")
 
 
@@ -782,6 +821,41 @@ def causal_attn_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_q: 
         q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), out.data_ptr(), out.stride(0),
         cu_q.data_ptr(), cu_k.data_ptr(), nseq, max_q, q.shape[0], k.shape[0], q.shape[1], k.shape[1], scale, _stream()),
         "mdb_attn_causal_varlen")
+
+
+def rotary_commit(q: Rows, k: Rows, v: Rows, heads: int, kv_heads: int, dim: int, q_norm: torch.Tensor, k_norm: torch.Tensor,
+                  eps: float, inv_freq: torch.Tensor, row_pos: torch.Tensor, slots: torch.Tensor, q_out: torch.Tensor,
+                  k_cache: torch.Tensor, v_cache: torch.Tensor) -> None:
+    """Per-head norms and interleaved rotation (of 2 * len(inv_freq) channels) of q and k; q_out [m, heads, dim_pad], caches
+    [slots, kv_heads, dim_pad]; v goes to its cache as it comes."""
+    m, _, dp = q_out.shape
+    _need(inv_freq, torch.float64, "inv_freq")
+    a = _lib.RotaryCommitArgs(_act_dtype(q_out, "q_out"), m, heads, kv_heads, dim, dp, 2 * inv_freq.numel(), eps, q.c(), k.c(), v.c(),
+                              q_norm.data_ptr(), k_norm.data_ptr(), inv_freq.data_ptr() or None, row_pos.data_ptr(), slots.data_ptr(),
+                              k_cache.shape[0], q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr())
+    _lib.check(_lib.lib().mdb_rotary_commit(a, _stream()), "mdb_rotary_commit")
+
+
+def window_attn_workspace_bytes(m: int, heads: int, dim_pad: int, nsplit: int) -> int:
+    return int(_lib.lib().mdb_window_attn_workspace_bytes(m, heads, dim_pad, nsplit))
+
+
+def window_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, portions: tuple,
+                row_pos: torch.Tensor, max_q: int, dim: int, window: int, sink: bool, scale: float, out: torch.Tensor,
+                gate: Rows | None = None, out_scale: float = 1.0, nsplit: int = 1, workspace: torch.Tensor | None = None) -> None:
+    """q [m, heads, dim_pad]; caches [pages * 256, kv_heads, dim_pad]; head h of a row goes to columns [h * dim, (h + 1) * dim)
+    of ``out``.  ``portions`` = (row_seq, cu_q, start, state_slot)."""
+    m, heads, dp = q.shape
+    row_seq, cu_q, start, _ = portions
+    _need(block_table, torch.int32, "block_table")
+    a = _lib.WindowAttnArgs(
+        dtype=_act_dtype(q, "q"), m=m, bs=start.numel(), heads=heads, kv_heads=k_cache.shape[1], dim=dim, dim_pad=dp, window=window,
+        sink=int(sink), max_q=max_q, nsplit=nsplit, scale=scale, out_scale=out_scale, q=q.data_ptr(), k_cache=k_cache.data_ptr(),
+        v_cache=v_cache.data_ptr(), block_table=block_table.data_ptr(), row_seq=row_seq.data_ptr(), row_pos=row_pos.data_ptr(),
+        cu_q=cu_q.data_ptr(), start=start.data_ptr(), table_stride=block_table.stride(0), num_pages=k_cache.shape[0] // 256,
+        gate=_rows_c(gate), out=out.data_ptr(), ld_out=_rows(out, "out"), workspace=_ptr(workspace),
+        workspace_bytes=0 if workspace is None else workspace.numel() * workspace.element_size())
+    _lib.check(_lib.lib().mdb_window_attn(a, _stream()), "mdb_window_attn")
 
 
 def pick_token(logits: torch.Tensor, vocab: int, temperatures: torch.Tensor, seed: int, step_dev: torch.Tensor | None,
