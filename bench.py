@@ -1,7 +1,7 @@
 """Benchmark of the block-diffusion decode path.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference]
-    python bench.py --design hybrid [--size 2k|4k]        (see bench_hybrid.py)
+    python bench.py --design hybrid|nipadra [--size 2k|4k]        (see bench_hybrid.py)
 
 Workload at N=1 ("config2"): the full decoder at the reference's configuration
 defaults (28 layers, hidden 2048, 16 query / 8 KV heads, vocabulary 151936,
@@ -688,14 +688,15 @@ def main():
     ap.add_argument("--requests", type=int, default=0,
                     help="requests in flight per GPU instead of the workload's own count (config3 / config5: the "
                          "batch sizes between one request and 64)")
-    ap.add_argument("--design", default="block-diffusion", choices=["block-diffusion", "hybrid"],
+    ap.add_argument("--design", default="block-diffusion", choices=["block-diffusion", "hybrid", "nipadra"],
                     help="hybrid: prefill and decode of the hybrid decoder design (one GPU) beside the block-diffusion "
                          "decoder at equal size, with a roofline per operation, instead of the workloads above")
     ap.add_argument("--size", default="2k", choices=["2k", "4k"], help="width of the --design hybrid models")
     args = ap.parse_args()
-    if args.design == "hybrid":
+    if args.design != "block-diffusion":
         import bench_hybrid
-        print(json.dumps(bench_hybrid.main(importlib.import_module("mineru-diffusion_b200"), args.size, load_peaks(), ClockSampler(0))))
+        print(json.dumps(bench_hybrid.main(importlib.import_module("mineru-diffusion_b200"), args.size, load_peaks(), ClockSampler(0),
+                                           args.design)))
         return
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))

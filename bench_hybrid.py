@@ -1,6 +1,8 @@
-"""Speed of the hybrid decoder design beside the block-diffusion decoder at equal width, layers and vocabulary.
+"""Speed of the causal decoder designs beside the framework's closest other models at equal width, layers and vocabulary.
 
-``python bench.py --design hybrid [--size 2k|4k]`` prints one JSON line: prefill and decode throughput of both (random
+``python bench.py --design hybrid [--size 2k|4k]`` sets the hybrid design (Zikunex) beside the block-diffusion decoder,
+``--design nipadra`` the Nipadra design beside the hybrid one with dense feed-forwards and the block-diffusion decoder.
+One JSON line: prefill and decode throughput of all (random
 weights, synthetic tokens), and for every kernel-launching operation of a prompt and of a decode step the time of one
 call and its fraction of the roofline.  Times are CUDA events on the launching stream, the median of several calls
 with an L2 flush (a 256 MB write) before each.  Roofline of an operation: the slowest of its bytes at the copy rate,
@@ -40,6 +42,31 @@ def design_config(pkg, s: dict):
         "layers": [dict(l, mlp=m) for l, m in layers]})
 
 
+def dense_hybrid_config(pkg, s: dict):
+    """The hybrid design without experts: eight layers of mLSTM, latent attention and delta rule, dense feed-forwards."""
+    heads, dense = s["heads"], {"kind": "dense", "ff": s["ff"]}
+    delta = {"type": "channel_delta", "mixer": dict(heads=heads, kv_heads=heads, dim=128, vdim=128, conv=4)}
+    mlstm = {"type": "mlstm", "mixer": dict(heads=heads // 2, dim=128, vdim=256, gate_cap=15.0)}
+    latent = {"type": "latent_attention", "mixer": dict(heads=heads, dim=128, vdim=128, q_rank=s["q_rank"], kv_rank=s["kv_rank"],
+                                                        scale=128 ** -0.5)}
+    return pkg.HybridConfig.from_json({
+        "architecture": "Zikunex", "vocab": s["vocab"], "width": s["width"], "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5},
+        "layers": [dict(l, mlp=dense) for l in (mlstm, latent, mlstm, delta) * 2]})
+
+
+def nipadra_config(pkg, s: dict):
+    """Eight layers, lightning attention and the parallel mixer in turn: 128 channels a head, eight key heads, a window of
+    1024, a Mamba-2 branch of twice the width; every second lightning layer without a feed-forward."""
+    heads, dense = s["heads"], {"kind": "dense", "ff": s["ff"]}
+    light = {"type": "lightning", "mixer": dict(heads=heads, dim=128, vdim=128, decay=[1 - 2.0 ** (-1 - 8 * h / heads) for h in range(heads)])}
+    left = dict(heads=heads, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, mask={"size": 1024}, rot={"base": 1e4, "dims": 128})
+    right = dict(heads=2 * s["width"] // 64, vdim=64, state=128, groups=8, conv=4, norm_groups=8)
+    par = {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.9, "right_scale": 1.1}}
+    return pkg.HybridConfig.from_json({
+        "architecture": "Nipadra", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "postln_alpha": 2.0,
+        "layers": [dict(light, mlp=dense), dict(par, mlp=dense), dict(light, mlp=None), dict(par, mlp=dense)] * 2})
+
+
 def closest_config(pkg, s: dict):
     return pkg.DecoderConfig(vocab_size=s["vocab"], hidden_size=s["width"], intermediate_size=s["ff"], num_hidden_layers=8,
                              num_attention_heads=s["heads"], num_key_value_heads=8, max_position_embeddings=16384)
@@ -50,7 +77,7 @@ class Recorder:
     """Swaps the functions of ``ops`` for ones that note every call."""
     NAMES = ("gemm", "gemm_heads", "gemm_experts", "gemm_splitk_partials", "linear", "gateup_swiglu", "residual_norm", "rms_rows",
              "add_rms_norm", "gated_norm", "delta_prep", "channel_decay", "mlstm_prep", "scan", "moe_route", "moe_plan", "moe_gather",
-             "latent_attn", "gather_latents", "causal_attn_varlen", "sparse_attn_varlen", "block_attn_with_kvcache",
+             "part_norm", "decay_prep", "chunk_scan", "rotary_commit", "window_attn", "latent_attn", "gather_latents", "causal_attn_varlen", "sparse_attn_varlen", "block_attn_with_kvcache",
              "qkv_proj_rope_commit", "qknorm_rope_commit", "pick_token", "lm_head_sample", "gather_rows")
 
     def __init__(self, ops):
@@ -90,7 +117,8 @@ def work_of(name: str, a: tuple, k: dict, ctx: dict):
     if name in ("gemm", "linear", "gemm_splitk_partials"):
         x, w = a[0], a[1]
         m, kk, n = x.shape[0], w.shape[1], w.shape[0]
-        return f"{name} {m}x{n}x{kk}", (m * kk + n * kk + m * n) * e, 2 * m * n * kk, 0
+        glu = k.get("act") == 2
+        return f"{name} {m}x{n}x{kk}" + (" glu" if glu else ""), (m * kk + n * kk + m * (n // 2 if glu else n)) * e, 2 * m * n * kk, 0
     if name == "gateup_swiglu":
         m, kk, n = a[0].shape[0], a[1].shape[1], a[1].shape[0]
         return f"gateup {m}x{n}x{kk}", (m * kk + n * kk + m * n // 2) * e, 2 * m * n * kk, 0
@@ -126,7 +154,7 @@ def work_of(name: str, a: tuple, k: dict, ctx: dict):
         mode, bs, heads, kvh, dim, vdim, rows = a[0], a[2], a[3], a[4], a[5], a[6], a[7].shape[0]
         per = dim * vdim
         io = rows * heads * (vdim * 8 + dim * (8 * kvh / heads + (4 if mode == 0 else 0))) + 2 * bs * heads * per * 4
-        return ("delta scan" if mode == 0 else "mlstm scan"), io, 0, rows * heads * per * (8 if mode == 0 else 6)
+        return ("delta scan", "mlstm scan", f"decay scan {heads}x{dim}x{vdim}")[mode], io, 0, rows * heads * per * (8 if mode == 0 else 6)
     if name == "residual_norm":
         m, wp = a[0].shape
         n = sum(e for _ in k.get("add", ())) + (ctx["top"] * e if k.get("moe") else 0) + e
@@ -138,6 +166,28 @@ def work_of(name: str, a: tuple, k: dict, ctx: dict):
         m, heads, kvh, dim, vdim = a[1], a[3], a[4], a[5], a[6]
         c = 2 * kvh * dim + heads * vdim
         return "delta inputs", m * c * (e + 4), 0, 0
+    if name == "window_attn":
+        q, kc, starts, cu, window = a[0], a[1], a[4][2].tolist(), a[4][1].tolist(), a[8]
+        m, h, d, keys, reads = q.shape[0], q.shape[1], a[7], 0, 0
+        for i, s0 in enumerate(starts):
+            n = cu[i + 1] - cu[i]
+            keys += sum(min(window or p + 1, p + 1) for p in range(s0, s0 + n))       # (query, key) pairs
+            reads += min(s0 + n, (window or s0 + n) + n - 1)                            # keys anyone sees
+        return "window attention", (2 * reads * kc.shape[1] + 2 * m * h) * d * e, 4 * d * h * keys, 0
+    if name == "chunk_scan":
+        heads, kvh, vdim, rows, dim = a[1], a[2], a[3], a[4].shape[0], a[4].shape[2]
+        io = rows * (heads * vdim * (e + 4) + 2 * kvh * dim * e) + 2 * a[0] * heads * dim * vdim * 4
+        # products of a 64-token chunk: scores (lower half), weighted scores and values (lower half, two terms), state read-out
+        # and state update (two terms each)
+        return f"chunk scan {heads}x{dim}x{vdim}", io, rows * heads * (64 * dim + 2 * 64 * vdim + 8 * dim * vdim), 0
+    if name == "rotary_commit":
+        h, g, d, m = a[3], a[4], a[5], a[12].shape[0]
+        return "rotation + cache rows", m * (2 * h + 3 * g) * d * e, 0, 0
+    if name == "decay_prep":
+        m, heads, kvh, dim, vdim = a[1], a[3], a[4], a[5], a[6]
+        return f"decay inputs {heads}x{dim}x{vdim}", m * (2 * kvh * dim + heads * vdim) * (e + 4), 0, 0
+    if name == "part_norm":
+        return f"gated norm in {a[3]} parts", a[0].numel() * (4 + 2 * e), 0, 0
     if name == "mlstm_prep":
         m, heads, dim, vdim = a[1:5]
         return "mlstm inputs", m * heads * (2 * dim + vdim) * (e + 4), 0, 0
@@ -193,8 +243,7 @@ def timed(fn, reps: int = 5, warmup: int = 3) -> float:
 
 
 # ----------------------------------------------------------------------------- the two models
-def measure_design(pkg, s: dict, peaks: dict, prompts, batches, context: int, tables: bool) -> dict:
-    cfg = design_config(pkg, s)
+def measure_design(pkg, cfg, s: dict, peaks: dict, prompts, batches, context: int, tables: int) -> dict:
     max_seqs, max_len = max(batches), context + 512
     max_tokens = max(n * l for n, l in prompts)
     max_len = max(max_len, max(l for _, l in prompts))
@@ -231,8 +280,8 @@ def measure_design(pkg, s: dict, peaks: dict, prompts, batches, context: int, ta
                 with Recorder(pkg.ops) as rec:
                     runner.execute(batch, counts)
                 runner.graphs = graphs
-                ids = next(a[0] for nm, _, a, _ in reversed(rec.calls) if nm == "moe_plan")
-                ctx = dict(rows=sum(counts), top=s["top"], touched=int(torch.unique(ids).numel()))
+                ids = [a[0] for nm, _, a, _ in rec.calls if nm == "moe_plan"]
+                ctx = dict(rows=sum(counts), top=s["top"], touched=int(torch.unique(ids[-1]).numel()) if ids else 0)
                 res[label] = op_table(rec, peaks, ctx)
     assert pkg._lib.device_status(clear=True) == 0
     runner.exit()
@@ -289,22 +338,27 @@ def measure_closest(pkg, s: dict, peaks: dict, prompts, requests, context: int, 
     return res
 
 
-def main(pkg, size: str, peaks: dict, sampler) -> dict:
+def main(pkg, size: str, peaks: dict, sampler, which: str = "hybrid") -> dict:
     s = SIZES[size]
     peaks = {"hbm_gbs": float(peaks.get("hbm_gbs", HBM_GBS)), "bf16_tflops": float(peaks.get("bf16_tflops", BF16_TFLOPS)),
              "source": "measured" if peaks else "fallback", "fp32_tflops": round(FP32_TFLOPS, 1)}
     prompts, context = [(1, 1024), (1, 4096), (4, 2048)], 2048
     sampler.start()
-    design = measure_design(pkg, s, peaks, prompts, [1, 32, 128], context, tables=32)
+    cfg = {"hybrid": design_config, "nipadra": nipadra_config}[which](pkg, s)
+    design = measure_design(pkg, cfg, s, peaks, prompts, [1, 32, 128], context, tables=32)
     torch.cuda.empty_cache()
+    hybrid = {}
+    if which == "nipadra":
+        hybrid["closest_causal"] = measure_design(pkg, dense_hybrid_config(pkg, s), s, peaks, prompts, [1, 32, 128], context, tables=32)
+        torch.cuda.empty_cache()
     closest = measure_closest(pkg, s, peaks, prompts, [1, 4], context, tables=True)
     clocks = sampler.stop()
-    return {"metric": "hybrid decoder design: decoded tokens/s, 32 requests", "unit": "tokens/s",
+    return {"metric": f"{which} decoder design: decoded tokens/s, 32 requests", "unit": "tokens/s",
             "value": design["decode"][f"32 requests at {context}"]["tokens_per_s"], "higher_is_better": True, "dtype": "bf16",
             "data": "synthetic tokens, random weights", "n_gpus": 1, "peaks": peaks, "clocks": clocks,
-            "config": {"model": f"8 hybrid layers beside 8 block-diffusion layers, size {size}", **s,
+            "config": {"model": f"8 {which} layers beside 8 block-diffusion layers, size {size}", **s,
                        "l2_policy": "operations: 256 MB written before each call; steps: weights exceed L2"},
-            "design": design, "closest": closest}
+            "design": design, **hybrid, "closest": closest}
 
 
 if __name__ == "__main__":

@@ -511,9 +511,10 @@ int mdb_mlstm_prep(const mdb_mlstm_prep_args* args, mdb_stream_t stream);
 /* Inputs of the decay scan (a linear recurrence with one decay per head): v [m][heads][vdim], k, q [m][kv_heads][dim_pad]
  * = silu of the projections or, with taps > 0, silu of a causal short convolution with bias over time (channels ordered
  * v | k | q; conv fp32 [channels][taps], the last tap is the current token's; conv_state as in mdb_delta_prep).  With dt:
- * step = softplus(dt + dt_bias), decay = exp(-exp(a_log) * step); else step = 1, decay = decay_const[h]. */
+ * step = softplus(dt + dt_bias), decay = exp(-exp(a_log) * step); else step = 1, decay = decay_const[h].  for_chunks: q, k, v
+ * leave in bf16 and decay_out holds the logarithm, as mdb_chunk_scan takes them. */
 typedef struct {
-  int32_t dtype, m, bs, heads, kv_heads, dim, dim_pad, vdim, taps, channels, shift_state;
+  int32_t dtype, m, bs, heads, kv_heads, dim, dim_pad, vdim, taps, channels, shift_state, for_chunks;
   mdb_rows q, k, v, dt;
   const float* conv;
   const float* conv_bias;
@@ -526,9 +527,9 @@ typedef struct {
   const float* a_log;
   const float* dt_bias;
   const float* decay_const;
-  float* q_out;
-  float* k_out;
-  float* v_out;
+  void* q_out; /* fp32, or bf16 with for_chunks */
+  void* k_out;
+  void* v_out;
   float* decay_out; /* [m][heads] */
   float* step_out;
 } mdb_decay_prep_args;
@@ -572,6 +573,27 @@ typedef struct {
   const float* skip; /* DECAY */
 } mdb_scan_args;
 int mdb_scan(const mdb_scan_args* args, mdb_stream_t stream);
+
+/* The decay scan over prompt portions in chunks of 64 tokens on the tensor cores: q, k bf16 [m][kv_heads][dim_pad], v bf16
+ * [m][heads][vdim], log_decay and step [m][heads]; state and out as in mdb_scan. */
+typedef struct {
+  int32_t bs, heads, kv_heads, dim_pad, vdim;
+  const void* q;
+  const void* k;
+  const void* v;
+  const float* log_decay;
+  const float* step;
+  const float* skip; /* [heads], may be NULL */
+  float* state;
+  int64_t state_slot_stride, num_slots;
+  const int32_t* cu_q;
+  const int32_t* start;
+  const int32_t* state_slot;
+  float* out;
+} mdb_chunk_scan_args;
+/* 1 when mdb_chunk_scan takes this head shape */
+int mdb_chunk_scan_supported(int dim_pad, int vdim);
+int mdb_chunk_scan(const mdb_chunk_scan_args* args, mdb_stream_t stream);
 
 /* Group-limited top-k routing of fp32 logits [m][experts]: ids and weights [m][top]; rows with row_slot < 0 (may be
  * NULL) get ids -1. */

@@ -40,7 +40,8 @@ GatedNormArgs = _struct("GatedNormArgs", [
 PartNormArgs = _struct("PartNormArgs", [(n, _i) for n in ("dtype", "m", "n", "parts", "gate_first")] + [
     ("out_scale", _f), ("eps", _f), ("o", _p), ("gate", Rows), ("weight", _p), ("y", _p), ("ldy", _i64)])
 DecayPrepArgs = _struct("DecayPrepArgs", [(n, _i) for n in (
-    "dtype", "m", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim", "taps", "channels", "shift_state")] + [
+    "dtype", "m", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim", "taps", "channels", "shift_state",
+    "for_chunks")] + [
     ("q", Rows), ("k", Rows), ("v", Rows), ("dt", Rows), ("conv", _p), ("conv_bias", _p), ("conv_state", _p),
     ("conv_slot_stride", _i64), ("num_slots", _i64), ("row_seq", _p), ("cu_q", _p), ("start", _p), ("state_slot", _p),
     ("a_log", _p), ("dt_bias", _p), ("decay_const", _p), ("q_out", _p), ("k_out", _p), ("v_out", _p), ("decay_out", _p),
@@ -73,6 +74,9 @@ ScanArgs = _struct("ScanArgs", [(n, _i) for n in (
     ("den", _p), ("cu_q", _p), ("start", _p),
     ("state_slot", _p), ("out", _p), ("raw_decay", Rows), ("a_log", _p), ("dt_bias", _p), ("gate", Rows), ("norm", _p),
     ("norm_head_stride", _i64), ("y", _p), ("ldy", _i64), ("skip", _p)])
+ChunkScanArgs = _struct("ChunkScanArgs", [(n, _i) for n in ("bs", "heads", "kv_heads", "dim_pad", "vdim")] + [
+    ("q", _p), ("k", _p), ("v", _p), ("log_decay", _p), ("step", _p), ("skip", _p), ("state", _p), ("state_slot_stride", _i64),
+    ("num_slots", _i64), ("cu_q", _p), ("start", _p), ("state_slot", _p), ("out", _p)])
 MoeRouteArgs = _struct("MoeRouteArgs", [(n, _i) for n in ("m", "experts", "top", "groups", "keep")] + [
     ("logits", Rows), ("row_slot", _p), ("ids", _p), ("weights", _p)])
 MoePlanArgs = _struct("MoePlanArgs", [(n, _i) for n in ("m", "top", "experts", "max_tiles")] + [
@@ -139,6 +143,8 @@ SIGNATURES = {
     "mdb_channel_decay": (_i, [C.POINTER(DecayArgs), _p]),
     "mdb_mlstm_prep": (_i, [C.POINTER(MlstmPrepArgs), _p]),
     "mdb_scan": (_i, [C.POINTER(ScanArgs), _p]),
+    "mdb_chunk_scan_supported": (_i, [_i, _i]),
+    "mdb_chunk_scan": (_i, [C.POINTER(ChunkScanArgs), _p]),
     "mdb_moe_route": (_i, [C.POINTER(MoeRouteArgs), _p]),
     "mdb_moe_plan": (_i, [C.POINTER(MoePlanArgs), _p]),
     "mdb_moe_max_tiles": (_i, [_i, _i, _i]),

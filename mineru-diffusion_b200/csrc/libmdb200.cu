@@ -15,4 +15,5 @@
 #include "recurrent.cu"
 #include "latent_attention.cu"
 #include "window_attention.cu"
+#include "chunk_scan.cu"
 #include "tp_p2p.cu"

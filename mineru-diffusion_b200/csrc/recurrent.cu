@@ -447,18 +447,20 @@ __global__ void __launch_bounds__(256) mlstm_prep_kernel(const mdb_mlstm_prep_ar
 // ---------------------------------------------------------------------------
 template <typename T>
 __device__ __forceinline__ void decay_prep_scalars(const mdb_decay_prep_args& a, int64_t row, int head) {
+  constexpr float kMinLog = -104.0f;         // e^-104 is 0 in fp32; the bound keeps the sums of logs of a chunk small
   float decay, step = 1.0f;
   if (rows_present(a.dt)) {
     step = softplus_f(rows_at<T>(a.dt, row, head) + a.dt_bias[head]);
-    decay = expf(-expf(a.a_log[head]) * step);
+    const float log_decay = -expf(a.a_log[head]) * step;
+    decay = a.for_chunks ? fmaxf(log_decay, kMinLog) : expf(log_decay);
   } else {
-    decay = a.decay_const[head];
+    decay = a.for_chunks ? fmaxf(logf(a.decay_const[head]), kMinLog) : a.decay_const[head];
   }
   a.decay_out[row * a.heads + head] = decay;
   a.step_out[row * a.heads + head] = step;
 }
 
-template <typename T>
+template <typename T, typename O>
 __global__ void __launch_bounds__(256) decay_prep_kernel(const mdb_decay_prep_args a) {
   pdl_launch_dependents();
   pdl_wait();
@@ -479,32 +481,32 @@ __global__ void __launch_bounds__(256) decay_prep_kernel(const mdb_decay_prep_ar
   const int stream = i < nv ? 0 : (i < nv + nk ? 1 : 2);
   i -= stream == 0 ? 0 : (stream == 1 ? nv : nv + nk);
   const mdb_rows& src = stream == 0 ? a.v : (stream == 1 ? a.k : a.q);
-  float* out = stream == 0 ? a.v_out + row * nv + i : (stream == 1 ? a.k_out : a.q_out) + row * nk + i;
+  O* out = static_cast<O*>(stream == 0 ? a.v_out : (stream == 1 ? a.k_out : a.q_out)) + row * (stream == 0 ? nv : nk) + i;
   int col = i;
   if (stream > 0) {
     const int d = i % a.dim_pad;
     if (d >= a.dim) {
-      *out = 0.f;
+      *out = act_from_f<O>(0.f);
       return;
     }
     col = i / a.dim_pad * a.dim + d;
   }
   if (a.taps == 0) {
     const float x = rows_at<T>(src, row, col);
-    *out = x / (1.0f + expf(-x));
+    *out = act_from_f<O>(x / (1.0f + expf(-x)));
     return;
   }
   const ConvCtx<T, mdb_decay_prep_args> cx = {&a, row, static_cast<int>(row) - a.cu_q[seq], a.start[seq] == 0 ? -1 : slot, slot};
   const int channel = col + (stream == 0 ? 0 : (stream == 1 ? nv : nv + kc));
   const float* w = a.conv + static_cast<int64_t>(channel - col) * a.taps;
-  *out = cx.conv_silu(src, w, col, channel, a.conv_bias[channel]);
+  *out = act_from_f<O>(cx.conv_silu(src, w, col, channel, a.conv_bias[channel]));
   cx.shift(src, col, channel);
 }
 
 // Sizes in multiples of four and up to four taps: a thread owns four channels and walks `run` consecutive rows with the last
 // inputs in registers.
 constexpr int kDecayPrepThreads = 128;
-template <typename T, bool PARTS>
+template <typename T, typename O, bool PARTS>
 __global__ void __launch_bounds__(kDecayPrepThreads) decay_prep_rows_kernel(const mdb_decay_prep_args a, const int run) {
   pdl_launch_dependents();
   pdl_wait();
@@ -524,19 +526,19 @@ __global__ void __launch_bounds__(kDecayPrepThreads) decay_prep_rows_kernel(cons
   if (stream == 1) src = a.k;
   if (stream == 2) src = a.q;
   const int64_t out_ld = stream == 0 ? nv : nk;
-  float* out = (stream == 0 ? a.v_out : (stream == 1 ? a.k_out : a.q_out)) + i * 4;
+  O* out = static_cast<O*>(stream == 0 ? a.v_out : (stream == 1 ? a.k_out : a.q_out)) + i * 4;
   int col = i * 4;
   if (stream > 0) {
     const int d = i * 4 % a.dim_pad;
     if (d >= a.dim) {
-      for (int64_t row = row0; row < row1; ++row) *reinterpret_cast<float4*>(out + row * out_ld) = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int64_t row = row0; row < row1; ++row) act_store4(out + row * out_ld, make_float4(0.f, 0.f, 0.f, 0.f));
       return;
     }
     col = i * 4 / a.dim_pad * a.dim + d;
   }
   if (a.taps == 0) {
 #pragma unroll 4
-    for (int64_t row = row0; row < row1; ++row) *reinterpret_cast<float4*>(out + row * out_ld) = silu4(rows_at4_of<T, PARTS>(src, row, col));
+    for (int64_t row = row0; row < row1; ++row) act_store4(out + row * out_ld, silu4(rows_at4_of<T, PARTS>(src, row, col)));
     return;
   }
   const int channel = col + (stream == 0 ? 0 : (stream == 1 ? nv : nv + kc));
@@ -557,7 +559,7 @@ __global__ void __launch_bounds__(kDecayPrepThreads) decay_prep_rows_kernel(cons
       if (slot >= 0) win.refill(a, src, row, static_cast<int>(row) - a.cu_q[s], a.start[s] == 0 ? -1 : slot, col, channel);
     }
     if (slot < 0) continue;
-    *reinterpret_cast<float4*>(out + row * out_ld) = win.step(in, bias);
+    act_store4(out + row * out_ld, win.step(in, bias));
     if (a.shift_state && a.taps > 1) win.save(a, slot, channel);
   }
 }
@@ -1223,7 +1225,7 @@ int mdb_decay_prep(const mdb_decay_prep_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(rows_present(a.dt) ? a.a_log && a.dt_bias : a.decay_const != nullptr, MDB_ERR_ARG);
   MDB_REQUIRE(a.taps == 0 || (a.conv && a.conv_bias && (a.conv_state || a.taps == 1)), MDB_ERR_ARG);
   MDB_REQUIRE(a.taps == 0 || a.channels == 2 * a.kv_heads * a.dim + a.heads * a.vdim, MDB_ERR_ARG);
-  MDB_REQUIRE(a.taps <= kMaxTaps, MDB_ERR_UNSUPPORTED);
+  MDB_REQUIRE(a.taps <= kMaxTaps && (!a.for_chunks || a.dtype == MDB_BF16), MDB_ERR_UNSUPPORTED);
   const bool parts = a.q.parts != nullptr;
   MDB_REQUIRE((a.k.parts != nullptr) == parts && (a.v.parts != nullptr) == parts && (!parts || a.dtype == MDB_BF16), MDB_ERR_UNSUPPORTED);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
@@ -1234,14 +1236,17 @@ int mdb_decay_prep(const mdb_decay_prep_args* args, mdb_stream_t stream) {
     const int items = a.heads * a.vdim / 4 + 2 * a.kv_heads * (a.dim_pad / 4) + a.heads;
     const dim3 grid((items + kDecayPrepThreads - 1) / kDecayPrepThreads, (a.m + run - 1) / run), block(kDecayPrepThreads);
     MDB_REQUIRE(grid.y <= 65535, MDB_ERR_UNSUPPORTED);
-    if (a.dtype == MDB_F32) rc = mdb_launch(decay_prep_rows_kernel<float, false>, grid, block, 0, st, a, run);
-    else if (parts) rc = mdb_launch(decay_prep_rows_kernel<bf16, true>, grid, block, 0, st, a, run);
-    else rc = mdb_launch(decay_prep_rows_kernel<bf16, false>, grid, block, 0, st, a, run);
+    if (a.dtype == MDB_F32) rc = mdb_launch(decay_prep_rows_kernel<float, float, false>, grid, block, 0, st, a, run);
+    else if (a.for_chunks && parts) rc = mdb_launch(decay_prep_rows_kernel<bf16, bf16, true>, grid, block, 0, st, a, run);
+    else if (a.for_chunks) rc = mdb_launch(decay_prep_rows_kernel<bf16, bf16, false>, grid, block, 0, st, a, run);
+    else if (parts) rc = mdb_launch(decay_prep_rows_kernel<bf16, float, true>, grid, block, 0, st, a, run);
+    else rc = mdb_launch(decay_prep_rows_kernel<bf16, float, false>, grid, block, 0, st, a, run);
   } else {
     const int items = a.heads * a.vdim + 2 * a.kv_heads * a.dim_pad + a.heads;
     const dim3 grid(a.m, (items + 255) / 256);
-    rc = a.dtype == MDB_F32 ? mdb_launch(decay_prep_kernel<float>, grid, dim3(256), 0, st, a)
-                            : mdb_launch(decay_prep_kernel<bf16>, grid, dim3(256), 0, st, a);
+    if (a.dtype == MDB_F32) rc = mdb_launch(decay_prep_kernel<float, float>, grid, dim3(256), 0, st, a);
+    else if (a.for_chunks) rc = mdb_launch(decay_prep_kernel<bf16, bf16>, grid, dim3(256), 0, st, a);
+    else rc = mdb_launch(decay_prep_kernel<bf16, float>, grid, dim3(256), 0, st, a);
   }
   if (rc != MDB_OK || a.shift_state || a.taps < 2) return rc;
   const dim3 cgrid((a.channels + 255) / 256, a.bs);

@@ -32,6 +32,8 @@ SKINNY_MAX_ROWS = 64
 # Prompt portions of at least this many tokens per sequence expand keys and values per head (tcgen05 attention);
 # shorter ones, like decoding, attend in the latent space.
 EXPAND_MIN_TOKENS = 32
+# Steps with a portion of at least this many tokens run their decay scans in chunks on the tensor cores.
+CHUNK_MIN_TOKENS = 8
 
 
 def pad128(n: int) -> int:
@@ -510,17 +512,22 @@ class HybridEngine:
         m, st, f32 = b.m, self.state[li], torch.float32
         heads, kvh, dim, vdim = mx.heads, mx.kv_heads, mx.dim, mx.vdim
         dp, one_token = ops.scan_dim_pad(dim), b.max_q == 1
+        chunks = self.dtype == torch.bfloat16 and b.max_q >= CHUNK_MIN_TOKENS and ops.chunk_scan_supported(dp, vdim)
+        act = self.dtype if chunks else f32
         z0, v0, k0, q0, *dt0 = pw["starts"]
-        outs = (self.buf("scan_q", m, kvh, dp, dtype=f32), self.buf("scan_k", m, kvh, dp, dtype=f32),
-                self.buf("scan_v", m, heads, vdim, dtype=f32), self.buf("scan_s0", m, heads, dtype=f32),
+        outs = (self.buf("scan_q", m, kvh, dp, dtype=act), self.buf("scan_k", m, kvh, dp, dtype=act),
+                self.buf("scan_v", m, heads, vdim, dtype=act), self.buf("scan_s0", m, heads, dtype=f32),
                 self.buf("scan_s1", m, heads, dtype=f32))
         scalars = dict(decay=pw["decay"]) if mx.decay is not None else dict(
             dt=x.cols(dt0[0]), a_log=pw["a_log"], dt_bias=pw["dt_bias"], conv=pw["conv"], conv_bias=pw["conv_bias"],
             conv_state=st["conv"], shift_state=one_token)
         ops.decay_prep(self.dtype, m, b.bs, heads, kvh, dim, vdim, x.cols(q0), x.cols(k0), x.cols(v0), self._portions(b), outs, **scalars)
         o = self.buf("scan_o", m, heads, vdim, dtype=f32)
-        ops.scan(ops.SCAN_DECAY, self.dtype, b.bs, heads, kvh, dim, vdim, *outs, st["s"], self._portions(b), out=o, skip=pw.get("skip"),
-                 one_token=one_token and ops.scan_fusable(dp, vdim))
+        if chunks:
+            ops.chunk_scan(b.bs, heads, kvh, vdim, *outs, st["s"], self._portions(b), o, skip=pw.get("skip"))
+        else:
+            ops.scan(ops.SCAN_DECAY, self.dtype, b.bs, heads, kvh, dim, vdim, *outs, st["s"], self._portions(b), out=o,
+                     skip=pw.get("skip"), one_token=one_token and ops.scan_fusable(dp, vdim))
         # lightning attention gates behind its norm, Mamba-2 in front of it
         ops.part_norm(o.view(m, heads * vdim), x.cols(z0), pw["norm"], mx.norm_groups, mx.decay is None, self.cfg.rms_norm_eps, y,
                       out_scale=scale)

@@ -724,7 +724,8 @@ def decay_prep(dtype: torch.dtype, m: int, bs: int, heads: int, kv_heads: int, d
                portions: tuple, outs: tuple, dt: Rows | None = None, a_log: torch.Tensor | None = None,
                dt_bias: torch.Tensor | None = None, decay: torch.Tensor | None = None, conv: torch.Tensor | None = None,
                conv_bias: torch.Tensor | None = None, conv_state: torch.Tensor | None = None, shift_state: bool = False) -> None:
-    """Inputs of the decay scan: ``outs`` = fp32 (q, k [m, kv_heads, dim_pad], v [m, heads, vdim], decay, step [m, heads]).
+    """Inputs of the decay scan: ``outs`` = fp32 (q, k [m, kv_heads, dim_pad], v [m, heads, vdim], decay, step [m, heads]); with
+    q, k, v in bf16 the inputs of the chunk form, whose decay is the logarithm.
     ``conv`` fp32 [channels, taps] (v | k | q) with ``conv_bias`` and ``conv_state`` [slots, taps - 1, channels], or None: silu
     alone.  Scalars from ``dt`` with ``a_log`` and ``dt_bias``, or the fixed ``decay`` [heads] and step 1."""
     qo, ko, vo, do, so = outs
@@ -732,7 +733,8 @@ def decay_prep(dtype: torch.dtype, m: int, bs: int, heads: int, kv_heads: int, d
     taps = 0 if conv is None else conv.shape[1]
     a = _lib.DecayPrepArgs(
         dtype=_DTYPES[dtype], m=m, bs=bs, heads=heads, kv_heads=kv_heads, dim=dim, dim_pad=qo.shape[-1], vdim=vdim, taps=taps,
-        channels=0 if conv is None else conv.shape[0], shift_state=int(shift_state), q=q.c(), k=k.c(), v=v.c(), dt=_rows_c(dt),
+        channels=0 if conv is None else conv.shape[0], shift_state=int(shift_state),
+        for_chunks=int(qo.dtype == _BF16), q=q.c(), k=k.c(), v=v.c(), dt=_rows_c(dt),
         conv=_ptr(conv), conv_bias=_ptr(conv_bias), conv_state=(_ptr(conv_state) or None) if taps > 1 else None,
         conv_slot_stride=conv_state.stride(0) if taps > 1 else 0, num_slots=conv_state.shape[0] if taps > 1 else 1 << 30,
         row_seq=row_seq.data_ptr(), cu_q=cu_q.data_ptr(), start=start.data_ptr(), state_slot=slot.data_ptr(), a_log=_ptr(a_log),
@@ -762,6 +764,22 @@ def scan(mode: int, dtype: torch.dtype, bs: int, heads: int, kv_heads: int, dim:
         norm=_ptr(norm), norm_head_stride=vdim if per_head_norm else 0, y=_ptr(y), ldy=0 if y is None else _rows(y, "y"),
         skip=_ptr(skip))
     _lib.check(_lib.lib().mdb_scan(a, _stream()), "mdb_scan")
+
+
+def chunk_scan_supported(dim_pad: int, vdim: int) -> bool:
+    return bool(_lib.lib().mdb_chunk_scan_supported(dim_pad, vdim))
+
+
+def chunk_scan(bs: int, heads: int, kv_heads: int, vdim: int, q, k, v, log_decay, step, state, portions: tuple, out, skip=None) -> None:
+    """The decay scan over prompt portions on the tensor cores: q, k, v bf16 and log decays of ``decay_prep``; ``state`` and
+    ``out`` as in ``scan``."""
+    _, cu_q, start, slot = portions
+    for t, nm in ((q, "q"), (k, "k"), (v, "v")):
+        _need(t, _BF16, nm)
+    a = _lib.ChunkScanArgs(bs, heads, kv_heads, q.shape[-1], vdim, q.data_ptr(), k.data_ptr(), v.data_ptr(), log_decay.data_ptr(),
+                           step.data_ptr(), _ptr(skip), state.data_ptr(), state.stride(0), state.shape[0], cu_q.data_ptr(),
+                           start.data_ptr(), slot.data_ptr(), out.data_ptr())
+    _lib.check(_lib.lib().mdb_chunk_scan(a, _stream()), "mdb_chunk_scan")
 
 
 def moe_route(logits: Rows, m: int, experts: int, top: int, groups: int, keep: int, ids: torch.Tensor, weights: torch.Tensor,

@@ -309,8 +309,8 @@ def _scan_ref(case, H, G, D, DV, taps):
     return orc.linear_scan(q, k, v, decay, torch.ones_like(decay))
 
 
-def _scan_run(case, H, G, D, DV, taps, counts, dtype, as_parts=False):
-    """One sequence in portions of ``counts`` tokens through the kernels, in slot 1 of 3."""
+def _scan_run(case, H, G, D, DV, taps, counts, dtype, as_parts=False, chunks=False):
+    """One sequence in portions of ``counts`` tokens through the kernels, in slot 1 of 3; ``chunks``: the tensor-core form."""
     ops = pkg.ops
     x, par = case
     dp, c = ops.scan_dim_pad(D), par["conv"].shape[0]
@@ -323,13 +323,17 @@ def _scan_run(case, H, G, D, DV, taps, counts, dtype, as_parts=False):
     for n in counts:
         p = portions_of([n], [at], [1])
         r = {k: rows(v[at:at + n], dtype, as_parts) for k, v in x.items()}
-        outs = (torch.full((n, G, dp), 9.0, device=DEV), torch.full((n, G, dp), 9.0, device=DEV), torch.zeros(n, H, DV, device=DEV),
-                torch.zeros(n, H, device=DEV), torch.zeros(n, H, device=DEV))
+        act = BF if chunks else F32
+        outs = (torch.full((n, G, dp), 9.0, device=DEV, dtype=act), torch.full((n, G, dp), 9.0, device=DEV, dtype=act),
+                torch.zeros(n, H, DV, device=DEV, dtype=act), torch.zeros(n, H, device=DEV), torch.zeros(n, H, device=DEV))
         ops.decay_prep(dtype, n, 1, H, G, D, DV, r["q"], r["k"], r["v"], p, outs, **extra,
                        **(dict(dt=r["dt"], shift_state=n == 1) if taps else {}))
         o = torch.zeros(n, H, DV, device=DEV)
-        ops.scan(ops.SCAN_DECAY, dtype, 1, H, G, D, DV, *outs, state, p, out=o, skip=dev["skip"] if taps else None,
-                 one_token=n == 1 and ops.scan_fusable(dp, DV))
+        if chunks:
+            ops.chunk_scan(1, H, G, DV, *outs, state, p, o, skip=dev["skip"] if taps else None)
+        else:
+            ops.scan(ops.SCAN_DECAY, dtype, 1, H, G, D, DV, *outs, state, p, out=o, skip=dev["skip"] if taps else None,
+                     one_token=n == 1 and ops.scan_fusable(dp, DV))
         out.append(o)
         at += n
     assert float((state[0] - 3).abs().max()) == 0 and float((state[2] - 3).abs().max()) == 0
@@ -349,6 +353,64 @@ def test_decay_scan_in_portions(dtype, H, G, D, DV, taps):
         assert rel(_scan_run(case, H, G, D, DV, taps, counts, dtype), ref) < (2e-5 if dtype is F32 else 4e-3 if taps else 2e-5), counts
     if dtype is BF:
         assert rel(_scan_run(case, H, G, D, DV, taps, [30] + [1] * 45, dtype, as_parts=True), ref) < 4e-3
+        if ops_take_chunks(D, DV):
+            for counts in ([T], [2, 33, 1, 1, 2, 36], [64, 11]):
+                assert rel(_scan_run(case, H, G, D, DV, taps, counts, dtype, chunks=True), ref) < 1e-2, counts
+            assert rel(_scan_run(case, H, G, D, DV, taps, [T], dtype, as_parts=True, chunks=True), ref) < 1e-2
+
+
+def ops_take_chunks(dim, vdim):
+    return pkg.ops.chunk_scan_supported(pkg.ops.scan_dim_pad(dim), vdim)
+
+
+@pytest.mark.parametrize("counts", [[200], [64, 128, 8], [1, 63, 65, 71], [2] * 10 + [180], [130, 1, 1, 68]])
+@pytest.mark.parametrize("H,G,D,DV", [(4, 2, 64, 24), (2, 1, 128, 64), (3, 3, 192, 136), (1, 1, 256, 96), (96, 4, 128, 128)])
+def test_chunk_scan_is_the_recurrence(H, G, D, DV, counts):
+    """Operands that bf16 holds exactly: what is left is the state's and the scores' 16 significant bits.  Decays from none to a
+    state that is wiped out between two tokens; other sequences in the batch; a padding entry."""
+    ops, T = pkg.ops, sum(counts)
+    if H == 96 and len(counts) > 3:
+        pytest.skip("enough heads for wide column blocks: the plain cuts are enough")
+    q, k, v = rand(T, G, D, seed=1, scale=D ** -0.5), rand(T, G, D, seed=2), rand(T, H, DV, seed=3)
+    log = -torch.rand(T, H, generator=gen(4)) * torch.logspace(-4, 0.5, H)
+    log[T // 2, 0], log[T // 3, H - 1] = -104.0, 0.0
+    step, skip = torch.rand(T, H, generator=gen(5)) + 0.1, rand(H, seed=6)
+    rep = lambda t: t.double().repeat_interleave(H // G, 1)
+    ref = orc.linear_scan(rep(q), rep(k), v.double(), torch.exp(log.double()), step.double()) + skip.double()[:, None] * v.double()
+    state = torch.full((4, H, DV, D), 3.0, device=DEV)
+    at, outs = 0, []
+    for n in counts:
+        p = portions_of([5, n, 3], [7, at, 0], [0, 2, -1])
+        pad = lambda t: torch.cat([t[:5], t[at:at + n], t[:3]]).to(DEV)
+        o = torch.full((n + 8, H, DV), 4.0, device=DEV)
+        ops.chunk_scan(3, H, G, DV, *(pad(t).to(BF) for t in (q, k, v)), pad(log), pad(step), state, p, o, skip=skip.to(DEV))
+        assert float((o[5 + n:] - 4).abs().max()) == 0 and float((o[:5] - 4).abs().min()) > 0
+        outs.append(o[5:5 + n])
+        at += n
+    got = torch.cat(outs)
+    assert rel(got, ref) < 3e-5
+    row = (got.double().cpu() - ref).pow(2).mean((1, 2)).sqrt() / ref.pow(2).mean().sqrt()
+    assert float(row.max()) < 2e-4, int(row.argmax())
+    assert float((state[1] - 3).abs().max()) == 0 and float((state[3] - 3).abs().max()) == 0
+
+
+@pytest.mark.parametrize("far", [1, 62, 63, 64, 65, 300])
+def test_chunk_scan_remembers_a_far_key(far):
+    """One key written and asked for ``far`` tokens later, over chunk borders, orthogonal writes in between."""
+    ops, T, D, DV, decay = pkg.ops, 400, 64, 16, 0.998
+    for at in (0, 3, 63, 64):
+        k = torch.zeros(T, 1, D)
+        k[:, 0, 1:] = rand(T, D - 1, seed=0)
+        k[at, 0], k[at, 0, 0] = 0.0, 1.0
+        q = torch.zeros(T, 1, D)
+        q[at + far, 0, 0] = 1.0
+        v = rand(T, 1, DV, seed=1)
+        state, o = torch.zeros(1, 1, DV, D, device=DEV), torch.zeros(T, 1, DV, device=DEV)
+        ops.chunk_scan(1, 1, 1, DV, *(t.to(BF).to(DEV) for t in (q, k, v)), torch.full((T, 1), decay, device=DEV).log(),
+                       torch.full((T, 1), 0.5, device=DEV), state, portions_of([T], slots=[0]), o)
+        want = torch.zeros(T, DV)
+        want[at + far] = 0.5 * v[at, 0] * decay ** far
+        assert float((o[:, 0].cpu() - want).abs().max()) < 1e-4
 
 
 def test_decay_scan_remembers_a_far_key():
