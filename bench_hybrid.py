@@ -117,8 +117,8 @@ def work_of(name: str, a: tuple, k: dict, ctx: dict):
     if name in ("gemm", "linear", "gemm_splitk_partials"):
         x, w = a[0], a[1]
         m, kk, n = x.shape[0], w.shape[1], w.shape[0]
-        glu = k.get("act") == 2
-        return f"{name} {m}x{n}x{kk}" + (" glu" if glu else ""), (m * kk + n * kk + m * (n // 2 if glu else n)) * e, 2 * m * n * kk, 0
+        glu, silu = k.get("act") == 2, k.get("act") == 3
+        return f"{name} {m}x{n}x{kk}" + (" glu" if glu else " silu" if silu else ""), (m * kk + n * kk + m * (n // 2 if glu else n)) * e, 2 * m * n * kk, 0
     if name == "gateup_swiglu":
         m, kk, n = a[0].shape[0], a[1].shape[1], a[1].shape[0]
         return f"gateup {m}x{n}x{kk}", (m * kk + n * kk + m * n // 2) * e, 2 * m * n * kk, 0
@@ -175,7 +175,7 @@ def work_of(name: str, a: tuple, k: dict, ctx: dict):
             reads += min(s0 + n, (window or s0 + n) + n - 1)                            # keys anyone sees
         return "window attention", (2 * reads * kc.shape[1] + 2 * m * h) * d * e, 4 * d * h * keys, 0
     if name == "chunk_scan":
-        heads, kvh, vdim, rows, dim = a[1], a[2], a[3], a[4].shape[0], a[4].shape[2]
+        heads, kvh, dim, vdim, rows = a[1], a[2], a[3], a[4], a[5].shape[0]
         io = rows * (heads * vdim * (e + 4) + 2 * kvh * dim * e) + 2 * a[0] * heads * dim * vdim * 4
         # products of a 64-token chunk: scores (lower half), weighted scores and values (lower half, two terms), state read-out
         # and state update (two terms each)
@@ -185,7 +185,7 @@ def work_of(name: str, a: tuple, k: dict, ctx: dict):
         return "rotation + cache rows", m * (2 * h + 3 * g) * d * e, 0, 0
     if name == "decay_prep":
         m, heads, kvh, dim, vdim = a[1], a[3], a[4], a[5], a[6]
-        return f"decay inputs {heads}x{dim}x{vdim}", m * (2 * kvh * dim + heads * vdim) * (e + 4), 0, 0
+        return f"decay inputs {heads}x{dim}x{vdim}", m * (2 * kvh * dim + heads * vdim) * (e + a[11][0].element_size()), 0, 0
     if name == "part_norm":
         return f"gated norm in {a[3]} parts", a[0].numel() * (4 + 2 * e), 0, 0
     if name == "mlstm_prep":

@@ -352,9 +352,10 @@ typedef struct {
 } mdb_rows;
 
 enum { MDB_GEMM_PLAIN = 0, MDB_GEMM_HEADS = 1, MDB_GEMM_EXPERTS = 2 };
-enum { MDB_ACT_NONE = 0, MDB_ACT_RELU2 = 1, MDB_ACT_RELU_GLU = 2 };
+enum { MDB_ACT_NONE = 0, MDB_ACT_RELU2 = 1, MDB_ACT_RELU_GLU = 2, MDB_ACT_SILU = 3 };
 /* y = act(x W^T).  PLAIN: x [m, k], w [n, k], y [m, n]; with RELU_GLU w is [2 n, k], gate rows first, and y =
- * relu(gate) * up (activation type, n % 128 == 0).  HEADS: head h takes columns [h k, (h + 1) k) of x, rows
+ * relu(gate) * up (activation type, n % 128 == 0); with SILU only columns from act_from (a multiple of 4) on are
+ * activated.  HEADS: head h takes columns [h k, (h + 1) k) of x, rows
  * [h n, (h + 1) n) of w and writes columns [h n, (h + 1) n) of y.  EXPERTS: rows of x and y are laid out by expert
  * in tiles of 128 (mdb_moe_plan); tile t uses rows [e n, (e + 1) n) of w, e = tile_expert[t], for t < *num_tiles;
  * m = rows of the buffers; max_rows_per_expert (0: unknown) bounds the rows in use in a tile.  y is of the
@@ -369,6 +370,7 @@ typedef struct {
   int32_t heads, experts, max_rows_per_expert;
   const int32_t* tile_expert;
   const int32_t* num_tiles;
+  int32_t act_from;
 } mdb_gemm_args;
 int mdb_gemm(const mdb_gemm_args* args, mdb_stream_t stream);
 
@@ -574,13 +576,16 @@ typedef struct {
 } mdb_scan_args;
 int mdb_scan(const mdb_scan_args* args, mdb_stream_t stream);
 
-/* The decay scan over prompt portions in chunks of 64 tokens on the tensor cores: q, k bf16 [m][kv_heads][dim_pad], v bf16
- * [m][heads][vdim], log_decay and step [m][heads]; state and out as in mdb_scan. */
+/* The decay scan over prompt portions in chunks of 64 tokens on the tensor cores: bf16 rows of ldq / ldk elements with head
+ * g of q and k at column g * dim (dim a multiple of 8, missing channels up to dim_pad count as zeros) and rows of ldv elements
+ * with head h of v at column h * vdim; log_decay (at least -104) and step are rows of heads, ld_scalars elements apart
+ * (0: the same for every token); state and out as in mdb_scan. */
 typedef struct {
-  int32_t bs, heads, kv_heads, dim_pad, vdim;
+  int32_t bs, heads, kv_heads, dim, dim_pad, vdim;
   const void* q;
   const void* k;
   const void* v;
+  int64_t ldq, ldk, ldv, ld_scalars;
   const float* log_decay;
   const float* step;
   const float* skip; /* [heads], may be NULL */

@@ -26,7 +26,7 @@ Rows = _struct("Rows", [("x", _p), ("parts", _p), ("ld", _i64), ("part_stride", 
 GemmArgs = _struct("GemmArgs", [
     ("dtype", _i), ("form", _i), ("act", _i), ("y_f32", _i), ("x", _p), ("w", _p), ("y", _p), ("ldx", _i64), ("ldy", _i64),
     ("m", _i), ("n", _i), ("k", _i), ("heads", _i), ("experts", _i), ("max_rows_per_expert", _i), ("tile_expert", _p),
-    ("num_tiles", _p)])
+    ("num_tiles", _p), ("act_from", _i)])
 ResidualNormArgs = _struct("ResidualNormArgs", [
     ("dtype", _i), ("m", _i), ("width", _i), ("width_pad", _i), ("residual", _p), ("ids", _p), ("embed", _p), ("vocab", _i64),
     ("add", Rows * 2), ("moe_rows", _p), ("moe_ld", _i64), ("moe_slot", _p), ("moe_weight", _p), ("weight", _p), ("y", _p),
@@ -74,8 +74,8 @@ ScanArgs = _struct("ScanArgs", [(n, _i) for n in (
     ("den", _p), ("cu_q", _p), ("start", _p),
     ("state_slot", _p), ("out", _p), ("raw_decay", Rows), ("a_log", _p), ("dt_bias", _p), ("gate", Rows), ("norm", _p),
     ("norm_head_stride", _i64), ("y", _p), ("ldy", _i64), ("skip", _p)])
-ChunkScanArgs = _struct("ChunkScanArgs", [(n, _i) for n in ("bs", "heads", "kv_heads", "dim_pad", "vdim")] + [
-    ("q", _p), ("k", _p), ("v", _p), ("log_decay", _p), ("step", _p), ("skip", _p), ("state", _p), ("state_slot_stride", _i64),
+ChunkScanArgs = _struct("ChunkScanArgs", [(n, _i) for n in ("bs", "heads", "kv_heads", "dim", "dim_pad", "vdim")] + [
+    ("q", _p), ("k", _p), ("v", _p), ("ldq", _i64), ("ldk", _i64), ("ldv", _i64), ("ld_scalars", _i64), ("log_decay", _p), ("step", _p), ("skip", _p), ("state", _p), ("state_slot_stride", _i64),
     ("num_slots", _i64), ("cu_q", _p), ("start", _p), ("state_slot", _p), ("out", _p)])
 MoeRouteArgs = _struct("MoeRouteArgs", [(n, _i) for n in ("m", "experts", "top", "groups", "keep")] + [
     ("logits", Rows), ("row_slot", _p), ("ids", _p), ("weights", _p)])

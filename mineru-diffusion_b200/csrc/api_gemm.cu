@@ -46,6 +46,7 @@ int gemm_plain_bf16(const mdb_gemm_args& a, cudaStream_t st) {
   TcArgs t = {};
   t.m = a.m; t.n = a.n; t.k = a.k;
   t.act = a.act;
+  t.act_from = a.act_from;
   t.ldy = a.ldy;
   if (a.y_f32) t.y32 = static_cast<float*>(a.y);
   else t.y = static_cast<bf16*>(a.y);
@@ -83,8 +84,9 @@ int mdb_gemm(const mdb_gemm_args* args, mdb_stream_t stream) {
   const mdb_gemm_args a = *args;
   MDB_REQUIRE(a.m >= 0 && a.n > 0 && a.k > 0, MDB_ERR_ARG);
   if (a.m == 0) return MDB_OK;
-  MDB_REQUIRE(a.form >= MDB_GEMM_PLAIN && a.form <= MDB_GEMM_EXPERTS && a.act >= MDB_ACT_NONE && a.act <= MDB_ACT_RELU_GLU, MDB_ERR_ARG);
-  MDB_REQUIRE(a.act != MDB_ACT_RELU_GLU || a.form == MDB_GEMM_PLAIN, MDB_ERR_UNSUPPORTED);
+  MDB_REQUIRE(a.form >= MDB_GEMM_PLAIN && a.form <= MDB_GEMM_EXPERTS && a.act >= MDB_ACT_NONE && a.act <= MDB_ACT_SILU, MDB_ERR_ARG);
+  MDB_REQUIRE(a.act < MDB_ACT_RELU_GLU || a.form == MDB_GEMM_PLAIN, MDB_ERR_UNSUPPORTED);
+  MDB_REQUIRE(a.act_from >= 0 && a.act_from % 4 == 0 && (a.act == MDB_ACT_SILU || a.act_from == 0), MDB_ERR_ARG);
   MDB_REQUIRE(a.x && a.w && a.y, MDB_ERR_ARG);
   const int64_t groups = a.form == MDB_GEMM_HEADS ? a.heads : 1;
   MDB_REQUIRE(groups >= 1 && a.ldx >= groups * a.k && a.ldy >= groups * a.n, MDB_ERR_ARG);

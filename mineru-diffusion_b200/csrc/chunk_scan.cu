@@ -24,15 +24,14 @@ struct ChunkPlan {
   static constexpr int kOffV = kOffK + 2 * kTileK;                      // two buffers
   static constexpr int kOffS = kOffV + 2 * kTileV;                      // high and low parts of the state, [DP][kVS]
   static constexpr int kOffRaw = kOffS + 2 * kTileS;                    // two buffers of log decays and steps
-  static constexpr int kOffCum = kOffRaw + 2 * 2 * kChunk * 4;          // c_i in log2 units, then the state's weights
-  static constexpr int kBytes = kOffCum + 2 * kChunk * 4 + kChunk * 4;  // ... and the steps
+  static constexpr int kOffCum = kOffRaw + 2 * 2 * kChunk * 4;          // c_j - log b_j in log2 units, the state's weights, c_i
+  static constexpr int kBytes = kOffCum + 3 * kChunk * 4;
 };
 
 // high and low bf16 parts of two numbers
 __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  const float hx = bf16_round(x), hy = bf16_round(y);
-  hi = pack_bf16x2(hx, hy);
-  lo = pack_bf16x2(x - hx, y - hy);
+  hi = pack_bf16x2(x, y);
+  lo = pack_bf16x2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
 }
 
 template <int DP, int PB>
@@ -60,10 +59,10 @@ __global__ void __launch_bounds__(kChunkThreads, DP <= 128 ? 2 : 1) chunk_scan_k
   const uint32_t base = smem_u32(chunk_smem);
   float* cum = reinterpret_cast<float*>(chunk_smem + P::kOffCum);
   float* wgt = cum + kChunk;
-  float* stp = wgt + kChunk;
+  float* crow = wgt + kChunk;
 
-  const bf16* q = static_cast<const bf16*>(a.q) + static_cast<int64_t>(kvh) * DP;
-  const bf16* k = static_cast<const bf16*>(a.k) + static_cast<int64_t>(kvh) * DP;
+  const bf16* q = static_cast<const bf16*>(a.q) + static_cast<int64_t>(kvh) * a.dim;
+  const bf16* k = static_cast<const bf16*>(a.k) + static_cast<int64_t>(kvh) * a.dim;
   const bf16* v = static_cast<const bf16*>(a.v) + static_cast<int64_t>(head) * a.vdim + col0;
   auto copy16 = [&](uint32_t dst, const bf16* src, bool live) {       // size 0 reads nothing and writes zeros
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(live ? 16 : 0) : "memory");
@@ -73,22 +72,22 @@ __global__ void __launch_bounds__(kChunkThreads, DP <= 128 ? 2 : 1) chunk_scan_k
     if (n > 0) {
       for (int i = threadIdx.x; i < kChunk * (DP / 8); i += kChunkThreads) {
         const int t = i / (DP / 8), c = i % (DP / 8) * 8;
-        const bool live = t < n;
-        const int64_t off = live ? static_cast<int64_t>(t0 + t) * a.kv_heads * DP + c : 0;
-        copy16(base + P::kOffQ + (t * P::kQS + c) * 2, q + off, live);
-        copy16(base + P::kOffK + buf * P::kTileK + (t * P::kQS + c) * 2, k + off, live);
+        const bool live = t < n && c < a.dim;
+        const int64_t row = live ? t0 + t : t_begin;
+        copy16(base + P::kOffQ + (t * P::kQS + c) * 2, q + row * a.ldq + (live ? c : 0), live);
+        copy16(base + P::kOffK + buf * P::kTileK + (t * P::kQS + c) * 2, k + row * a.ldk + (live ? c : 0), live);
       }
       for (int i = threadIdx.x; i < kChunk * (PB / 8); i += kChunkThreads) {
         const int t = i / (PB / 8), c = i % (PB / 8) * 8;
         const bool live = t < n && col0 + c < a.vdim;
-        copy16(base + P::kOffV + buf * P::kTileV + (t * P::kVS + c) * 2, v + (live ? static_cast<int64_t>(t0 + t) * a.heads * a.vdim + c : 0), live);
+        copy16(base + P::kOffV + buf * P::kTileV + (t * P::kVS + c) * 2, v + (live ? (t0 + t) * a.ldv + c : 0), live);
       }
       if (threadIdx.x < 2 * kChunk) {              // tokens past the end: no decay, no input
         const int t = threadIdx.x & (kChunk - 1);
         const float* src = threadIdx.x < kChunk ? a.log_decay : a.step;
         const bool live = t < n;
         asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(base + P::kOffRaw + (buf * 2 * kChunk + threadIdx.x) * 4),
-                     "l"(src + (live ? static_cast<int64_t>(t0 + t) * a.heads + head : 0)), "r"(live ? 4 : 0) : "memory");
+                     "l"(src + (live ? (t0 + t) * a.ld_scalars + head : 0)), "r"(live ? 4 : 0) : "memory");
       }
     }
     cp_async_commit();
@@ -148,8 +147,8 @@ __global__ void __launch_bounds__(kChunkThreads, DP <= 128 ? 2 : 1) chunk_scan_k
       }
       const float total = __shfl_sync(0xffffffffu, s, 31), b0 = raw[kChunk + 2 * lane], b1 = raw[kChunk + 2 * lane + 1];
       const float c0 = s - x1, c1 = s;
-      *reinterpret_cast<float2*>(cum + 2 * lane) = make_float2(c0, c1);
-      *reinterpret_cast<float2*>(stp + 2 * lane) = make_float2(b0, b1);
+      *reinterpret_cast<float2*>(crow + 2 * lane) = make_float2(c0, c1);
+      *reinterpret_cast<float2*>(cum + 2 * lane) = make_float2(c0 - log2f(b0), c1 - log2f(b1));      // (step 0: +inf, weight 0)
       *reinterpret_cast<float2*>(wgt + 2 * lane) = make_float2(b0 * exp2f(total - c0), b1 * exp2f(total - c1));
     }
     const uint32_t qt = base + P::kOffQ + 16 * rg * P::kQS * 2, kt = base + P::kOffK + buf * P::kTileK, vt = base + P::kOffV + buf * P::kTileV;
@@ -186,7 +185,7 @@ __global__ void __launch_bounds__(kChunkThreads, DP <= 128 ? 2 : 1) chunk_scan_k
     __syncthreads();                               // q and the state's parts have been read; sums and weights are written
     request(t0 + kChunk, buf ^ 1);
     const int r0 = 16 * rg + g;
-    const float c0 = cum[r0], c1 = cum[r0 + 8];
+    const float c0 = crow[r0], c1 = crow[r0 + 8];
     {
       const float e0 = exp2f(c0), e1 = exp2f(c1);
 #pragma unroll
@@ -199,10 +198,16 @@ __global__ void __launch_bounds__(kChunkThreads, DP <= 128 ? 2 : 1) chunk_scan_k
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
         const int t = 16 * j + 8 * n + j2;
-        const float2 cj = *reinterpret_cast<const float2*>(cum + t), bj = *reinterpret_cast<const float2*>(stp + t);
+        const float2 cj = *reinterpret_cast<const float2*>(cum + t);
         const float (&x)[4] = G[2 * j + n];
-        const float m0 = t <= r0 ? x[0] * bj.x * exp2f(c0 - cj.x) : 0.f, m1 = t + 1 <= r0 ? x[1] * bj.y * exp2f(c0 - cj.y) : 0.f;
-        const float m2 = t <= r0 + 8 ? x[2] * bj.x * exp2f(c1 - cj.x) : 0.f, m3 = t + 1 <= r0 + 8 ? x[3] * bj.y * exp2f(c1 - cj.y) : 0.f;
+        float m0 = x[0] * ex2_approx(c0 - cj.x), m1 = x[1] * ex2_approx(c0 - cj.y);
+        float m2 = x[2] * ex2_approx(c1 - cj.x), m3 = x[3] * ex2_approx(c1 - cj.y);
+        if (j == rg) {                             // the diagonal tile: tokens up to the row's own
+          m0 = t <= r0 ? m0 : 0.f;
+          m1 = t + 1 <= r0 ? m1 : 0.f;
+          m2 = t <= r0 + 8 ? m2 : 0.f;
+          m3 = t + 1 <= r0 + 8 ? m3 : 0.f;
+        }
         split2(m0, m1, mh[2 * n], ml[2 * n]);
         split2(m2, m3, mh[2 * n + 1], ml[2 * n + 1]);
       }
@@ -231,7 +236,7 @@ __global__ void __launch_bounds__(kChunkThreads, DP <= 128 ? 2 : 1) chunk_scan_k
       }
     }
     // the state
-    const float total = exp2f(cum[kChunk - 1]);
+    const float total = exp2f(crow[kChunk - 1]);
 #pragma unroll
     for (int i = 0; i < NU; ++i)
 #pragma unroll
@@ -316,7 +321,12 @@ int mdb_chunk_scan(const mdb_chunk_scan_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(a.bs >= 0 && a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.vdim > 0, MDB_ERR_ARG);
   if (a.bs == 0) return MDB_OK;
   MDB_REQUIRE(a.q && a.k && a.v && a.log_decay && a.step && a.state && a.cu_q && a.start && a.state_slot && a.out, MDB_ERR_ARG);
-  MDB_REQUIRE(mdb_aligned16(a.q) && mdb_aligned16(a.k) && mdb_aligned16(a.v) && mdb_aligned16(a.out), MDB_ERR_ALIGN);
+  MDB_REQUIRE(a.dim > 0 && a.dim <= a.dim_pad && a.ldq >= static_cast<int64_t>(a.kv_heads) * a.dim && a.ldk >= static_cast<int64_t>(a.kv_heads) * a.dim &&
+                  a.ldv >= static_cast<int64_t>(a.heads) * a.vdim && a.ld_scalars >= 0,
+              MDB_ERR_ARG);
+  MDB_REQUIRE(a.dim % 8 == 0 && a.ldq % 8 == 0 && a.ldk % 8 == 0 && a.ldv % 8 == 0 && mdb_aligned16(a.q) && mdb_aligned16(a.k) &&
+                  mdb_aligned16(a.v) && mdb_aligned16(a.out),
+              MDB_ERR_ALIGN);
   MDB_REQUIRE(mdb_chunk_scan_supported(a.dim_pad, a.vdim) && a.heads <= 65535 && a.bs <= 65535, MDB_ERR_UNSUPPORTED);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   switch (a.dim_pad) {

@@ -66,6 +66,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const mdb_gemm_args a) {
       if (col >= a.n) continue;
       float v = acc[i][j];
       if (a.act == MDB_ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+      if (a.act == MDB_ACT_SILU && col >= a.act_from) v /= 1.0f + expf(-v);
       if (GLU) v = fmaxf(v, 0.f) * up[i][j];
       y[row * a.ldy + y_col + col] = v;
     }

@@ -103,6 +103,7 @@ struct TcArgs {
   int ksplit;
   // plain and GROUP epilogues: activation applied to the fp32 accumulator, and fp32 rows instead of bf16 (same ldy)
   int act;
+  int act_from;                // SILU: first column that is activated
   float* y32;
   // GROUP form
   int heads;                   // > 0: per-head products; 0: per-expert products
@@ -113,6 +114,7 @@ struct TcArgs {
 
 __device__ __forceinline__ float tc_act(int act, float v) {
   if (act == MDB_ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+  if (act == MDB_ACT_SILU) v *= rcp_approx(1.0f + __expf(-v));
   return v;
 }
 
@@ -454,9 +456,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           tmem_ld16(taddr + 32 * c + 16, v1);
           tmem_ld_wait();
           const int col = tn * kTcBN + 32 * c;
-          if (a.act != MDB_ACT_NONE) {
+          if (a.act != MDB_ACT_NONE && col >= a.act_from) {
 #pragma unroll
             for (int i = 0; i < 16; ++i) { v0[i] = tc_act(a.act, v0[i]); v1[i] = tc_act(a.act, v1[i]); }
+          } else if (a.act != MDB_ACT_NONE && col + 32 > a.act_from) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+              if (col + i >= a.act_from) v0[i] = tc_act(a.act, v0[i]);
+              if (col + 16 + i >= a.act_from) v1[i] = tc_act(a.act, v1[i]);
+            }
           }
           if (a.y32 != nullptr) {
             if (row < a.m) {
@@ -819,8 +827,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           for (int j = 1; j < 8; ++j)
             if (j < ks) { sum.x += v[j].x; sum.y += v[j].y; sum.z += v[j].z; sum.w += v[j].w; }
           const int grow = tm * kTcBM + r, col = tn * kTcBN + 4 * c4;
-          sum.x = tc_act(a.act, sum.x); sum.y = tc_act(a.act, sum.y);
-          sum.z = tc_act(a.act, sum.z); sum.w = tc_act(a.act, sum.w);
+          if (col >= a.act_from) {
+            sum.x = tc_act(a.act, sum.x); sum.y = tc_act(a.act, sum.y);
+            sum.z = tc_act(a.act, sum.z); sum.w = tc_act(a.act, sum.w);
+          }
           if (grow < a.m && a.y32 != nullptr) {
             if (col + 4 <= a.n) *reinterpret_cast<float4*>(a.y32 + static_cast<int64_t>(grow) * a.ldy + col) = sum;
           } else if (grow < a.m) {

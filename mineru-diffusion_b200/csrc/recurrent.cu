@@ -503,11 +503,21 @@ __global__ void __launch_bounds__(256) decay_prep_kernel(const mdb_decay_prep_ar
   cx.shift(src, col, channel);
 }
 
+// Four activations as they lie in memory.
+template <typename T> struct ActRaw;
+template <> struct ActRaw<float> { typedef float4 type; };
+template <> struct ActRaw<bf16> { typedef uint2 type; };
+__device__ __forceinline__ float4 act_raw4(float4 v) { return v; }
+__device__ __forceinline__ float4 act_raw4(uint2 u) {
+  const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
 // Sizes in multiples of four and up to four taps: a thread owns four channels and walks `run` consecutive rows with the last
 // inputs in registers.
 constexpr int kDecayPrepThreads = 128;
 template <typename T, typename O, bool PARTS>
-__global__ void __launch_bounds__(kDecayPrepThreads) decay_prep_rows_kernel(const mdb_decay_prep_args a, const int run) {
+__global__ void __launch_bounds__(kDecayPrepThreads, 8) decay_prep_rows_kernel(const mdb_decay_prep_args a, const int run) {
   pdl_launch_dependents();
   pdl_wait();
   int i = blockIdx.x * kDecayPrepThreads + threadIdx.x;
@@ -546,9 +556,20 @@ __global__ void __launch_bounds__(kDecayPrepThreads) decay_prep_rows_kernel(cons
   win.load_taps(a.conv, channel, a.taps);
   const float4 bias = *reinterpret_cast<const float4*>(a.conv_bias + channel);
   int seq = -1, slot = -1;
-  for (int64_t row = row0; row < row1; ++row) {
+  constexpr int kAhead = PARTS ? 1 : 4;        // rows whose inputs are requested together
+  typedef typename ActRaw<T>::type Raw;
+  for (int64_t row = row0; row < row1;) {
+    if (!PARTS && row + kAhead <= row1 && a.row_seq[row] == seq && a.row_seq[row + kAhead - 1] == seq && slot >= 0 && !a.shift_state) {
+      Raw in[kAhead];
+      const T* x = static_cast<const T*>(src.x) + row * src.ld + src.col + col;
+#pragma unroll
+      for (int r = 0; r < kAhead; ++r) in[r] = *reinterpret_cast<const Raw*>(x + r * src.ld);
+#pragma unroll
+      for (int r = 0; r < kAhead; ++r) act_store4(out + (row + r) * out_ld, win.step(act_raw4(in[r]), bias));
+      row += kAhead;
+      continue;
+    }
     const int s = a.row_seq[row];
-    const float4 in = rows_at4_of<T, PARTS>(src, row, col);
     if (s != seq) {
       seq = s;
       slot = a.state_slot[s];
@@ -558,9 +579,11 @@ __global__ void __launch_bounds__(kDecayPrepThreads) decay_prep_rows_kernel(cons
       }
       if (slot >= 0) win.refill(a, src, row, static_cast<int>(row) - a.cu_q[s], a.start[s] == 0 ? -1 : slot, col, channel);
     }
-    if (slot < 0) continue;
-    act_store4(out + row * out_ld, win.step(in, bias));
-    if (a.shift_state && a.taps > 1) win.save(a, slot, channel);
+    if (slot >= 0) {
+      act_store4(out + row * out_ld, win.step(rows_at4_of<T, PARTS>(src, row, col), bias));
+      if (a.shift_state && a.taps > 1) win.save(a, slot, channel);
+    }
+    ++row;
   }
 }
 
@@ -1232,7 +1255,7 @@ int mdb_decay_prep(const mdb_decay_prep_args* args, mdb_stream_t stream) {
   int rc;
   if (a.dim % 4 == 0 && a.vdim % 4 == 0 && a.taps <= 4 && rows_ok(a.q) && rows_ok(a.k) && rows_ok(a.v) && a.conv_slot_stride % 4 == 0 &&
       mdb_aligned16(a.q_out) && mdb_aligned16(a.k_out) && mdb_aligned16(a.v_out) && mdb_aligned16(a.conv) && mdb_aligned16(a.conv_bias)) {
-    const int run = a.m >= 4096 ? 16 : (a.m >= 1024 ? 8 : 1);      // rows a thread walks
+    const int run = a.m >= 4096 ? 33 : (a.m >= 1024 ? 9 : 1);      // rows a thread walks: one to look the sequence up, then fours
     const int items = a.heads * a.vdim / 4 + 2 * a.kv_heads * (a.dim_pad / 4) + a.heads;
     const dim3 grid((items + kDecayPrepThreads - 1) / kDecayPrepThreads, (a.m + run - 1) / run), block(kDecayPrepThreads);
     MDB_REQUIRE(grid.y <= 65535, MDB_ERR_UNSUPPORTED);

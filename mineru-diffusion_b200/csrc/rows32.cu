@@ -91,8 +91,8 @@ constexpr int kRes32Threads = 256;
 
 // One CTA per row.  residual (scaled or, with ids, = embed[id] * scale) + up to two projections + the weighted sum of
 // the chosen experts' rows; y = residual / rms * weight.  POST: the norm replaces the residual, and y is the new residual or
-// its norm with a second weight.  NV float4 chunks of the row per thread.
-template <typename T, int NV, bool POST>
+// its norm with a second weight.  NV float4 chunks of the row per thread; PARTS: a projection may come as split-k slices.
+template <typename T, int NV, bool POST, bool PARTS>
 __global__ void __launch_bounds__(kRes32Threads) residual_norm_kernel(const mdb_residual_norm_args a) {
   pdl_launch_dependents();
   pdl_wait();
@@ -127,7 +127,7 @@ __global__ void __launch_bounds__(kRes32Threads) residual_norm_kernel(const mdb_
 #pragma unroll
     for (int s = 0; s < 2; ++s) {
       if (!rows_present(a.add[s])) continue;
-      const float4 d = rows_at4<T>(a.add[s], row, c);
+      const float4 d = PARTS ? rows_at4<T>(a.add[s], row, c) : rows_at4_of<T, false>(a.add[s], row, c);
       x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
     }
     if (a.moe_rows != nullptr) {
@@ -357,6 +357,56 @@ __global__ void __launch_bounds__(kPartNormThreads) part_norm_kernel(const mdb_p
   }
 }
 
+// The same for parts of at most 1024 columns: a warp per (row, part), everything in registers, no barrier.
+template <typename T, int NK, bool PARTS>
+__global__ void __launch_bounds__(kPartNormThreads) part_norm_warp_kernel(const mdb_part_norm_args a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t unit = static_cast<int64_t>(blockIdx.x) * (kPartNormThreads / 32) + (threadIdx.x >> 5);
+  const int64_t row = unit / a.parts;
+  if (row >= a.m) return;
+  const int n = a.n / a.parts, col0 = static_cast<int>(unit % a.parts) * n, lane = threadIdx.x & 31;
+  const float* o = a.o + row * a.n + col0;
+  float4 v[NK], g[NK];
+#pragma unroll
+  for (int i = 0; i < NK; ++i) {
+    const int c = lane * 4 + 128 * i;
+    v[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < n) {
+      v[i] = *reinterpret_cast<const float4*>(o + c);
+      g[i] = rows_at4_of<T, PARTS>(a.gate, row, col0 + c);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NK; ++i) {
+    const float4 s = make_float4(sigmoid_f(g[i].x), sigmoid_f(g[i].y), sigmoid_f(g[i].z), sigmoid_f(g[i].w));
+    if (a.gate_first) v[i] = make_float4(v[i].x * g[i].x * s.x, v[i].y * g[i].y * s.y, v[i].z * g[i].z * s.z, v[i].w * g[i].w * s.w);
+    ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    g[i] = a.gate_first ? make_float4(1.f, 1.f, 1.f, 1.f) : s;
+  }
+  const float rstd = a.out_scale / sqrtf(warp_sum(ss) / static_cast<float>(n) + a.eps);
+  T* y = static_cast<T*>(a.y) + row * a.ldy + col0;
+#pragma unroll
+  for (int i = 0; i < NK; ++i) {
+    const int c = lane * 4 + 128 * i;
+    if (c >= n) continue;
+    const float4 w = *reinterpret_cast<const float4*>(a.weight + col0 + c);
+    act_store4(y + c, make_float4(v[i].x * rstd * w.x * g[i].x, v[i].y * rstd * w.y * g[i].y, v[i].z * rstd * w.z * g[i].z, v[i].w * rstd * w.w * g[i].w));
+  }
+}
+
+template <typename T, bool PARTS>
+static int launch_part_norm_warp(const mdb_part_norm_args& a, cudaStream_t st) {
+  const int n = a.n / a.parts;
+  const int64_t units = static_cast<int64_t>(a.m) * a.parts;
+  const dim3 grid(static_cast<unsigned>((units + kPartNormThreads / 32 - 1) / (kPartNormThreads / 32))), block(kPartNormThreads);
+  if (n <= 128) return mdb_launch(part_norm_warp_kernel<T, 1, PARTS>, grid, block, 0, st, a);
+  if (n <= 256) return mdb_launch(part_norm_warp_kernel<T, 2, PARTS>, grid, block, 0, st, a);
+  if (n <= 512) return mdb_launch(part_norm_warp_kernel<T, 4, PARTS>, grid, block, 0, st, a);
+  return mdb_launch(part_norm_warp_kernel<T, 8, PARTS>, grid, block, 0, st, a);
+}
+
 // Row r of the output = the latent of token r - cu[seq] of its sequence, read through the page table.
 template <typename T>
 __global__ void __launch_bounds__(64) gather_latents_kernel(const T* cache, const int32_t* table,
@@ -431,14 +481,19 @@ bool rows_ok(const mdb_rows& s) {
                               (s.parts == nullptr || (s.nparts >= 1 && s.part_stride % 4 == 0)));
 }
 
+template <typename T, bool POST, bool PARTS>
+int launch_residual_norm_of(const mdb_residual_norm_args& a, cudaStream_t st) {
+  const int chunks = (a.width_pad / 4 + kRes32Threads - 1) / kRes32Threads;
+  if (chunks <= 1) return mdb_launch(residual_norm_kernel<T, 1, POST, PARTS>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  if (chunks <= 2) return mdb_launch(residual_norm_kernel<T, 2, POST, PARTS>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  if (chunks <= 4) return mdb_launch(residual_norm_kernel<T, 4, POST, PARTS>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  if (chunks <= 8) return mdb_launch(residual_norm_kernel<T, 8, POST, PARTS>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
+  return MDB_ERR_UNSUPPORTED;
+}
 template <typename T, bool POST>
 int launch_residual_norm(const mdb_residual_norm_args& a, cudaStream_t st) {
-  const int chunks = (a.width_pad / 4 + kRes32Threads - 1) / kRes32Threads;
-  if (chunks <= 1) return mdb_launch(residual_norm_kernel<T, 1, POST>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
-  if (chunks <= 2) return mdb_launch(residual_norm_kernel<T, 2, POST>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
-  if (chunks <= 4) return mdb_launch(residual_norm_kernel<T, 4, POST>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
-  if (chunks <= 8) return mdb_launch(residual_norm_kernel<T, 8, POST>, dim3(a.m), dim3(kRes32Threads), 0, st, a);
-  return MDB_ERR_UNSUPPORTED;
+  return a.add[0].parts != nullptr || a.add[1].parts != nullptr ? launch_residual_norm_of<T, POST, true>(a, st)
+                                                                : launch_residual_norm_of<T, POST, false>(a, st);
 }
 }  // namespace
 
@@ -512,8 +567,12 @@ int mdb_part_norm(const mdb_part_norm_args* args, mdb_stream_t stream) {
   const int n = a.n / a.parts;
   const bool vec = n % 4 == 0 && rows_ok(a.gate) && a.ldy % 4 == 0 && mdb_aligned16(a.o) && mdb_aligned16(a.y) && mdb_aligned16(a.weight);
   const bool parts = a.gate.parts != nullptr;
-  const dim3 grid(a.m, a.parts), block(n <= 128 ? 32 : (n <= 512 ? 64 : (n <= 2048 ? 128 : kPartNormThreads)));
+  const dim3 grid(a.m, a.parts), block(n <= 2048 ? 128 : kPartNormThreads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (vec && n <= 1024 && !(parts && a.dtype == MDB_F32)) {
+    if (a.dtype == MDB_F32) return launch_part_norm_warp<float, false>(a, st);
+    return parts ? launch_part_norm_warp<bf16, true>(a, st) : launch_part_norm_warp<bf16, false>(a, st);
+  }
   if (a.dtype == MDB_F32)
     return vec && !parts ? mdb_launch(part_norm_kernel<float, true, false>, grid, block, 0, st, a)
                          : mdb_launch(part_norm_kernel<float, false, true>, grid, block, 0, st, a);

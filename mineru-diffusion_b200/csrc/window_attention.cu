@@ -19,7 +19,8 @@ namespace mdb {
 // ---------------------------------------------------------------------------
 constexpr int kRotThreads = 256, kRotMaxPairs = 512;
 
-template <typename T, bool VEC, bool PARTS>
+// KEEP > 0: heads of up to 128 KEEP channels in registers, four per lane and step.
+template <typename T, int KEEP, bool PARTS>
 __global__ void __launch_bounds__(kRotThreads) rotary_commit_kernel(const mdb_rotary_commit_args a) {
   pdl_launch_dependents();
   pdl_wait();
@@ -42,16 +43,20 @@ __global__ void __launch_bounds__(kRotThreads) rotary_commit_kernel(const mdb_ro
     slot = -1;
   }
   const int lane = threadIdx.x & 31;
+#pragma unroll 2
   for (int unit = threadIdx.x >> 5; unit < a.heads + 2 * a.kv_heads; unit += kRotThreads / 32) {
     const int kind = unit < a.heads ? 0 : (unit < a.heads + a.kv_heads ? 1 : 2);      // q, k or v
     const int head = unit - (kind == 0 ? 0 : (kind == 1 ? a.heads : a.heads + a.kv_heads));
     if (kind > 0 && slot < 0) continue;
-    const mdb_rows& src = kind == 0 ? a.q : (kind == 1 ? a.k : a.v);
+    // by value: a reference picked at run time would be read through memory at every use
+    mdb_rows src = a.q;
+    if (kind == 1) src = a.k;
+    if (kind == 2) src = a.v;
     T* out = kind == 0 ? static_cast<T*>(a.q_out) + (row * a.heads + head) * a.dim_pad
                        : static_cast<T*>(kind == 1 ? a.k_cache : a.v_cache) + (slot * a.kv_heads + head) * a.dim_pad;
     const float* w = kind == 0 ? a.q_norm : a.k_norm;
-    if (VEC) {
-      constexpr int kKeep = 2;                 // heads of up to 256 channels stay in registers
+    if constexpr (KEEP > 0) {
+      constexpr int kKeep = KEEP;
       float4 x[kKeep];
       float ss = 0.f;
 #pragma unroll
@@ -506,11 +511,14 @@ int mdb_rotary_commit(const mdb_rotary_commit_args* args, mdb_stream_t stream) {
   const dim3 grid(a.m), block(kRotThreads);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (a.dtype == MDB_F32)
-    return vec ? mdb_launch(rotary_commit_kernel<float, true, false>, grid, block, 0, st, a)
-               : mdb_launch(rotary_commit_kernel<float, false, false>, grid, block, 0, st, a);
-  if (!vec) return mdb_launch(rotary_commit_kernel<bf16, false, false>, grid, block, 0, st, a);
-  return parts ? mdb_launch(rotary_commit_kernel<bf16, true, true>, grid, block, 0, st, a)
-               : mdb_launch(rotary_commit_kernel<bf16, true, false>, grid, block, 0, st, a);
+    return vec ? mdb_launch(rotary_commit_kernel<float, 2, false>, grid, block, 0, st, a)
+               : mdb_launch(rotary_commit_kernel<float, 0, false>, grid, block, 0, st, a);
+  if (!vec) return mdb_launch(rotary_commit_kernel<bf16, 0, false>, grid, block, 0, st, a);
+  if (parts)
+    return a.dim <= 128 ? mdb_launch(rotary_commit_kernel<bf16, 1, true>, grid, block, 0, st, a)
+                        : mdb_launch(rotary_commit_kernel<bf16, 2, true>, grid, block, 0, st, a);
+  return a.dim <= 128 ? mdb_launch(rotary_commit_kernel<bf16, 1, false>, grid, block, 0, st, a)
+                      : mdb_launch(rotary_commit_kernel<bf16, 2, false>, grid, block, 0, st, a);
 }
 
 int64_t mdb_window_attn_workspace_bytes(int m, int heads, int dim_pad, int nsplit) {

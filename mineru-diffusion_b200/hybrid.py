@@ -132,6 +132,9 @@ class HybridWeights:
         def four(n: int) -> int:
             return (n + 3) // 4 * 4
 
+        def eight(n: int) -> int:
+            return (n + 7) // 8 * 8
+
         def residual_norm(name: str) -> torch.Tensor:
             return vec(src(name, w).float() + cfg.design.norm_offset, wp)
 
@@ -150,9 +153,11 @@ class HybridWeights:
             params = {"norm": vec(src(m + "norm", nv), four(nv))}
             if mx.decay is not None:
                 # in the order of the other form's inputs: gate, values, keys, queries
-                parts = [(src(m + "g", nv, w), four(nv)), (src(m + "v", nv, w), four(nv)), (src(m + "k", nk, w), four(nk)),
-                         (src(m + "q", nk, w), four(nk))]
+                parts = [(src(m + "g", nv, w), eight(nv)), (src(m + "v", nv, w), eight(nv)), (src(m + "k", nk, w), eight(nk)),
+                         (src(m + "q", nk, w), eight(nk))]
                 params["decay"] = torch.tensor(mx.decay, dtype=torch.float32, device=device)
+                params["log_decay"] = torch.tensor(mx.decay, dtype=torch.float64).log().clamp_min(-104.0).to(device, torch.float32)
+                params["step"] = torch.ones_like(params["decay"])
             else:
                 z, x, b, c, dt = src(m + "in", 2 * nv + 2 * nk + mx.heads, w).split([nv, nv, nk, nk, mx.heads])
                 parts = [(z, four(nv)), (x, four(nv)), (b, four(nk)), (c, four(nk)), (dt, four(mx.heads))]
@@ -340,7 +345,9 @@ def random_tensors(cfg: HybridConfig, seed: int, device, rank: int = 128, std: f
             t = t - 2.0
         elif name.endswith("f.b"):
             t = t + 3.0
-        elif name.endswith((".b", ".dt_bias", ".D")) and len(shape) == 1:
+        elif name.endswith(".D"):
+            t = 1.0 + 0.3 * t
+        elif name.endswith((".b", ".dt_bias")) and len(shape) == 1:
             pass
         elif name.endswith(".conv"):
             t = t * (0.5 / shape[1] ** 0.5) + 0.25
@@ -418,8 +425,9 @@ class HybridEngine:
             t = self._bufs[key] = torch.empty(n, dtype=dtype, device=self.device)
         return t[:n]
 
-    def _linear(self, name: str, x: torch.Tensor, w: torch.Tensor, parts: bool = True, f32: bool = False) -> ops.Rows:
-        """x w^T as its consumer takes it: split-k slices for a short bf16 step, else rows."""
+    def _linear(self, name: str, x: torch.Tensor, w: torch.Tensor, parts: bool = True, f32: bool = False, silu_from: int | None = None) -> ops.Rows:
+        """x w^T as its consumer takes it: split-k slices for a short bf16 step, else rows, whose columns from ``silu_from`` on
+        are activated."""
         m, n = x.shape[0], w.shape[0]
         if parts and m <= SKINNY_MAX_ROWS and self.dtype == torch.bfloat16:
             ks = ops.pick_ksplit(m, n, w.shape[1])
@@ -427,7 +435,7 @@ class HybridEngine:
             ops.gemm_splitk_partials(x, w, ks, out)
             return ops.Rows(parts=out)
         out = self.buf("rows_" + name, m, n, dtype=torch.float32 if f32 else None)
-        return ops.Rows(ops.gemm(x, w, out))
+        return ops.Rows(ops.gemm(x, w, out) if silu_from is None else ops.gemm(x, w, out, act=ops.ACT_SILU, act_from=silu_from))
 
     # ------------------------------------------------------------------ forward
     def forward(self, b: StepBatch) -> torch.Tensor:
@@ -488,12 +496,16 @@ class HybridEngine:
     def _joined(self, li: int, mx, lw: dict, h: torch.Tensor, b: StepBatch) -> ops.Rows:
         """One mixer, or several side by side, on one input product; their outputs meet in one output product."""
         scales = (mx.left_scale, mx.right_scale) if isinstance(mx, ParallelSpec) else (1.0,)
-        x = self._linear("mix_in", h, lw["in"])
+        # plain projections of a chunked scan take their silu in the product's epilogue and go into the scan as they are
+        silu_from = None
+        if isinstance(mx, DecayScanSpec) and mx.decay is not None and mx.dim % 8 == 0 and self._chunks(mx, b) and b.m > SKINNY_MAX_ROWS:
+            silu_from = lw["parts"][0]["starts"][1]
+        x = self._linear("mix_in", h, lw["in"], silu_from=silu_from)
         widths = tuple(part.heads * (part.dim if isinstance(part, WindowAttentionSpec) else part.vdim) for part in parts_of(mx))
         y = self.buf("joined_o_" + "_".join(map(str, widths)), b.m, lw["o"].shape[1])
         for part, pw, n, scale in zip(parts_of(mx), lw["parts"], widths, scales):
             run = self._window_attention if isinstance(part, WindowAttentionSpec) else self._decay_scan
-            run(li, part, pw, x, y[:, pw["out"]:pw["out"] + n], scale, b)
+            run(li, part, pw, x, y[:, pw["out"]:pw["out"] + n], scale, b, **({} if silu_from is None else {"activated": True}))
         return self._linear("mix_out", y, lw["o"])
 
     def _window_attention(self, li: int, mx: WindowAttentionSpec, pw: dict, x: ops.Rows, y: torch.Tensor, scale: float, b: StepBatch):
@@ -508,13 +520,29 @@ class HybridEngine:
         ops.window_attn(q, k_cache, v_cache, b.table, self._portions(b), b.row_pos, b.max_q, mx.dim, mx.window, mx.sink, mx.scale, y,
                         gate=x.cols(g0), out_scale=scale, nsplit=nsplit, workspace=ws)
 
-    def _decay_scan(self, li: int, mx: DecayScanSpec, pw: dict, x: ops.Rows, y: torch.Tensor, scale: float, b: StepBatch):
+    def _chunks(self, mx: DecayScanSpec, b: StepBatch) -> bool:
+        return self.dtype == torch.bfloat16 and b.max_q >= CHUNK_MIN_TOKENS and ops.chunk_scan_supported(ops.scan_dim_pad(mx.dim), mx.vdim)
+
+    def _decay_scan(self, li: int, mx: DecayScanSpec, pw: dict, x: ops.Rows, y: torch.Tensor, scale: float, b: StepBatch,
+                    activated: bool = False):
         m, st, f32 = b.m, self.state[li], torch.float32
         heads, kvh, dim, vdim = mx.heads, mx.kv_heads, mx.dim, mx.vdim
         dp, one_token = ops.scan_dim_pad(dim), b.max_q == 1
-        chunks = self.dtype == torch.bfloat16 and b.max_q >= CHUNK_MIN_TOKENS and ops.chunk_scan_supported(dp, vdim)
+        chunks = self._chunks(mx, b)
         act = self.dtype if chunks else f32
         z0, v0, k0, q0, *dt0 = pw["starts"]
+        o = self.buf("scan_o", m, heads, vdim, dtype=f32)
+
+        def leave():
+            # lightning attention gates behind its norm, Mamba-2 in front of it
+            ops.part_norm(o.view(m, heads * vdim), x.cols(z0), pw["norm"], mx.norm_groups, mx.decay is None, self.cfg.rms_norm_eps, y,
+                          out_scale=scale)
+
+        if activated:
+            rows = x.x
+            ops.chunk_scan(b.bs, heads, kvh, dim, vdim, rows[:, q0:], rows[:, k0:], rows[:, v0:], pw["log_decay"], pw["step"], st["s"],
+                           self._portions(b), o)
+            return leave()
         outs = (self.buf("scan_q", m, kvh, dp, dtype=act), self.buf("scan_k", m, kvh, dp, dtype=act),
                 self.buf("scan_v", m, heads, vdim, dtype=act), self.buf("scan_s0", m, heads, dtype=f32),
                 self.buf("scan_s1", m, heads, dtype=f32))
@@ -522,15 +550,14 @@ class HybridEngine:
             dt=x.cols(dt0[0]), a_log=pw["a_log"], dt_bias=pw["dt_bias"], conv=pw["conv"], conv_bias=pw["conv_bias"],
             conv_state=st["conv"], shift_state=one_token)
         ops.decay_prep(self.dtype, m, b.bs, heads, kvh, dim, vdim, x.cols(q0), x.cols(k0), x.cols(v0), self._portions(b), outs, **scalars)
-        o = self.buf("scan_o", m, heads, vdim, dtype=f32)
         if chunks:
-            ops.chunk_scan(b.bs, heads, kvh, vdim, *outs, st["s"], self._portions(b), o, skip=pw.get("skip"))
+            q, k, v, *scalars = outs
+            ops.chunk_scan(b.bs, heads, kvh, dp, vdim, q.view(m, -1), k.view(m, -1), v.view(m, -1), *scalars, st["s"], self._portions(b), o,
+                           skip=pw.get("skip"))
         else:
             ops.scan(ops.SCAN_DECAY, self.dtype, b.bs, heads, kvh, dim, vdim, *outs, st["s"], self._portions(b), out=o,
                      skip=pw.get("skip"), one_token=one_token and ops.scan_fusable(dp, vdim))
-        # lightning attention gates behind its norm, Mamba-2 in front of it
-        ops.part_norm(o.view(m, heads * vdim), x.cols(z0), pw["norm"], mx.norm_groups, mx.decay is None, self.cfg.rms_norm_eps, y,
-                      out_scale=scale)
+        leave()
 
     def _channel_delta(self, li: int, mx: ChannelDeltaSpec, lw: dict, h: torch.Tensor, b: StepBatch) -> ops.Rows:
         m, st, f32 = b.m, self.state[li], torch.float32

@@ -543,7 +543,7 @@ def lm_head_sample_tp(hidden: torch.Tensor, weight: torch.Tensor, temperatures: 
 # Decoders with an fp32 residual: recurrent mixers, latent attention, experts.  Activations are bf16 or fp32 tensors.
 
 _DTYPES = {torch.bfloat16: 0, torch.float32: 1}
-ACT_NONE, ACT_RELU2, ACT_RELU_GLU = 0, 1, 2
+ACT_NONE, ACT_RELU2, ACT_RELU_GLU, ACT_SILU = 0, 1, 2, 3
 
 
 class Rows:
@@ -579,13 +579,13 @@ def _act_dtype(t: torch.Tensor, name: str) -> int:
     return _DTYPES[t.dtype]
 
 
-def gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: int = ACT_NONE) -> torch.Tensor:
+def gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: int = ACT_NONE, act_from: int = 0) -> torch.Tensor:
     """out = act(x w^T); x [m, k] (row stride free), w [n, k]; out of the activation type, or fp32.  ACT_RELU_GLU: w is
-    [2 n, k], gate rows first, and out = relu(gate) * up."""
+    [2 n, k], gate rows first, and out = relu(gate) * up.  ACT_SILU activates the columns from act_from on."""
     m, k = x.shape
     n = w.shape[0] // 2 if act == ACT_RELU_GLU else w.shape[0]
     a = _lib.GemmArgs(_act_dtype(x, "x"), 0, act, int(out.dtype == torch.float32), x.data_ptr(), w.data_ptr(),
-                      out.data_ptr(), _rows(x, "x"), _rows(out, "out"), m, n, k, 0, 0, 0, None, None)
+                      out.data_ptr(), _rows(x, "x"), _rows(out, "out"), m, n, k, 0, 0, 0, None, None, act_from)
     _lib.check(_lib.lib().mdb_gemm(a, _stream()), "mdb_gemm")
     return out
 
@@ -770,13 +770,16 @@ def chunk_scan_supported(dim_pad: int, vdim: int) -> bool:
     return bool(_lib.lib().mdb_chunk_scan_supported(dim_pad, vdim))
 
 
-def chunk_scan(bs: int, heads: int, kv_heads: int, vdim: int, q, k, v, log_decay, step, state, portions: tuple, out, skip=None) -> None:
-    """The decay scan over prompt portions on the tensor cores: q, k, v bf16 and log decays of ``decay_prep``; ``state`` and
+def chunk_scan(bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q, k, v, log_decay, step, state, portions: tuple, out,
+               skip=None) -> None:
+    """The decay scan over prompt portions on the tensor cores: bf16 q, k [m, >= kv_heads * dim] and v [m, >= heads * vdim] (row
+    strides free), logarithms of the decays (at least -104) and steps [m, heads], or [heads] for all tokens; ``state`` and
     ``out`` as in ``scan``."""
     _, cu_q, start, slot = portions
     for t, nm in ((q, "q"), (k, "k"), (v, "v")):
         _need(t, _BF16, nm)
-    a = _lib.ChunkScanArgs(bs, heads, kv_heads, q.shape[-1], vdim, q.data_ptr(), k.data_ptr(), v.data_ptr(), log_decay.data_ptr(),
+    a = _lib.ChunkScanArgs(bs, heads, kv_heads, dim, state.shape[-1], vdim, q.data_ptr(), k.data_ptr(), v.data_ptr(), _rows(q, "q"),
+                           _rows(k, "k"), _rows(v, "v"), heads if log_decay.dim() > 1 else 0, log_decay.data_ptr(),
                            step.data_ptr(), _ptr(skip), state.data_ptr(), state.stride(0), state.shape[0], cu_q.data_ptr(),
                            start.data_ptr(), slot.data_ptr(), out.data_ptr())
     _lib.check(_lib.lib().mdb_chunk_scan(a, _stream()), "mdb_chunk_scan")

@@ -105,6 +105,31 @@ def test_gated_product(dtype, m, n, k):
     assert rel(y, torch.relu(z[:, :n]) * z[:, n:]) < (2e-6 if dtype is F32 else 4e-3)
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("m,n,k,from_", [(65, 256, 2048, 72), (300, 384, 128, 0), (2100, 512, 256, 260), (130, 640, 1024, 128)])
+def test_product_activated_from_a_column_on(dtype, m, n, k, from_):
+    x, w = rand(m, k, seed=1), rand(n, k, seed=2, scale=k ** -0.5)
+    y = torch.zeros(m, n, dtype=dtype, device=DEV)
+    pkg.ops.gemm(x.to(dtype).to(DEV), w.to(dtype).to(DEV), y, act=pkg.ops.ACT_SILU, act_from=from_)
+    ref = x.double() @ w.double().T
+    ref[:, from_:] = orc.silu(ref[:, from_:])
+    assert rel(y, ref) < (2e-6 if dtype is F32 else 4e-3)
+
+
+def test_chunk_scan_reads_columns_of_a_projection():
+    """Heads of 40 channels in rows of another matrix: missing channels of the stored state count as zeros."""
+    ops, T, H, D, DV = pkg.ops, 150, 3, 40, 24
+    x = rand(T, 8 + 2 * H * D + H * DV + 16, seed=1, scale=0.5)
+    q, k, v = x[:, 8:8 + H * D], x[:, 128:128 + H * D], x[:, 248:248 + H * DV]
+    log = torch.tensor([-0.5, -0.01, -3.0])
+    decay = torch.exp(log.double()).expand(T, H)
+    ref = orc.linear_scan(q.double().view(T, H, D), k.double().view(T, H, D), v.double().view(T, H, DV), decay, torch.ones_like(decay))
+    xd = x.to(BF).to(DEV)
+    state, o = torch.full((1, H, DV, 64), 5.0, device=DEV), torch.zeros(T, H, DV, device=DEV)
+    ops.chunk_scan(1, H, H, D, DV, xd[:, 8:], xd[:, 128:], xd[:, 248:], log.to(DEV), torch.ones(H, device=DEV), state, portions_of([T], slots=[0]), o)
+    assert rel(o, ref) < 3e-5 and float(state[..., D:].abs().max()) == 0
+
+
 # --------------------------------------------------------------------------- rotation and caches
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("as_parts", [False, True])
@@ -330,7 +355,8 @@ def _scan_run(case, H, G, D, DV, taps, counts, dtype, as_parts=False, chunks=Fal
                        **(dict(dt=r["dt"], shift_state=n == 1) if taps else {}))
         o = torch.zeros(n, H, DV, device=DEV)
         if chunks:
-            ops.chunk_scan(1, H, G, DV, *outs, state, p, o, skip=dev["skip"] if taps else None)
+            q, k, v, *sc = outs
+            ops.chunk_scan(1, H, G, dp, DV, q.view(n, -1), k.view(n, -1), v.view(n, -1), *sc, state, p, o, skip=dev["skip"] if taps else None)
         else:
             ops.scan(ops.SCAN_DECAY, dtype, 1, H, G, D, DV, *outs, state, p, out=o, skip=dev["skip"] if taps else None,
                      one_token=n == 1 and ops.scan_fusable(dp, DV))
@@ -383,7 +409,7 @@ def test_chunk_scan_is_the_recurrence(H, G, D, DV, counts):
         p = portions_of([5, n, 3], [7, at, 0], [0, 2, -1])
         pad = lambda t: torch.cat([t[:5], t[at:at + n], t[:3]]).to(DEV)
         o = torch.full((n + 8, H, DV), 4.0, device=DEV)
-        ops.chunk_scan(3, H, G, DV, *(pad(t).to(BF) for t in (q, k, v)), pad(log), pad(step), state, p, o, skip=skip.to(DEV))
+        ops.chunk_scan(3, H, G, D, DV, *(pad(t).to(BF).flatten(1) for t in (q, k, v)), pad(log), pad(step), state, p, o, skip=skip.to(DEV))
         assert float((o[5 + n:] - 4).abs().max()) == 0 and float((o[:5] - 4).abs().min()) > 0
         outs.append(o[5:5 + n])
         at += n
@@ -406,8 +432,8 @@ def test_chunk_scan_remembers_a_far_key(far):
         q[at + far, 0, 0] = 1.0
         v = rand(T, 1, DV, seed=1)
         state, o = torch.zeros(1, 1, DV, D, device=DEV), torch.zeros(T, 1, DV, device=DEV)
-        ops.chunk_scan(1, 1, 1, DV, *(t.to(BF).to(DEV) for t in (q, k, v)), torch.full((T, 1), decay, device=DEV).log(),
-                       torch.full((T, 1), 0.5, device=DEV), state, portions_of([T], slots=[0]), o)
+        ops.chunk_scan(1, 1, 1, D, DV, *(t.to(BF).to(DEV).flatten(1) for t in (q, k, v)), torch.full((1,), decay, device=DEV).log(),
+                       torch.full((1,), 0.5, device=DEV), state, portions_of([T], slots=[0]), o)
         want = torch.zeros(T, DV)
         want[at + far] = 0.5 * v[at, 0] * decay ** far
         assert float((o[:, 0].cpu() - want).abs().max()) < 1e-4
