@@ -305,6 +305,9 @@ static int launch_chunk_scan_cols(const mdb_chunk_scan_args& a, cudaStream_t st)
   return a.vdim <= 32 || wide < 148 ? launch_chunk_scan<DP, 32>(a, st) : launch_chunk_scan<DP, 64>(a, st);
 }
 
+// the form for portions of more than one chunk (defined with the tensor-memory kernels' helpers in scope)
+template <int NH> static int launch_chunk_scan_tc(const mdb_chunk_scan_args& a, cudaStream_t st);
+
 }  // namespace mdb
 
 using namespace mdb;
@@ -330,8 +333,8 @@ int mdb_chunk_scan(const mdb_chunk_scan_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(mdb_chunk_scan_supported(a.dim_pad, a.vdim) && a.heads <= 65535 && a.bs <= 65535, MDB_ERR_UNSUPPORTED);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   switch (a.dim_pad) {
-    case 64: return launch_chunk_scan_cols<64>(a, st);
-    case 128: return launch_chunk_scan_cols<128>(a, st);
+    case 64: return a.max_q > kChunk ? launch_chunk_scan_tc<1>(a, st) : launch_chunk_scan_cols<64>(a, st);
+    case 128: return a.max_q > kChunk ? launch_chunk_scan_tc<2>(a, st) : launch_chunk_scan_cols<128>(a, st);
     case 192: return launch_chunk_scan_cols<192>(a, st);
     default: return launch_chunk_scan_cols<256>(a, st);
   }

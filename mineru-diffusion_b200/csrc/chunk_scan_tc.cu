@@ -1,0 +1,368 @@
+// The decay scan of chunk_scan.cu with chunks of 128 tokens on the 5th-generation tensor cores, for stored heads of 64 or 128
+// key channels.  A CTA owns 64 value columns of one head of one sequence and walks its chunks:
+//
+//   G  = Q K^T                              128 tokens x 128 tokens
+//   Y1 = Q S          (S in two bf16 parts)  what the state gives, times e^(c_i) per row
+//   D  = K^T (w V)    (w V in two parts)     what the chunk adds to the state, w_j = e^(c_last - c_j) b_j
+//   Y2 = M V          (M in two parts)       M = G e^(c_i - c_j) b_j below the diagonal
+//
+// with the accumulators in tensor memory.  One warp issues the products; eight warps do the rest, a pair of warps per 32
+// rows, half of the columns each: w V (shared memory to shared memory), M (tensor memory to tensor memory, where it is
+// the left operand of its product), the outputs, and the state, which stays in their registers in fp32 (a thread holds one
+// key channel of 32 columns).  D does not wait for M and runs under it.  The next chunk's k and v are requested at the
+// start of a chunk, q once Y1 is complete.
+#include "mdb_common.cuh"
+
+namespace mdb {
+
+constexpr int kCtL = 128, kCtCols = 64, kCtWarps = 8, kCtThreads = (kCtWarps + 1) * 32;
+constexpr int kCtHalf = kCtL * 128;          // [128 rows][64 bf16]: one swizzled tile
+
+enum { kCtBarOps = 0, kCtBarW, kCtBarM, kCtBarG, kCtBarY, kCtBarO, kCtBars };
+
+struct CtPlan {
+  static constexpr int kOffQ = 0;                              // two halves of 64 channels
+  static constexpr int kOffK = kOffQ + 2 * kCtHalf;            // two buffers
+  static constexpr int kOffV = kOffK + 4 * kCtHalf;            // two buffers
+  static constexpr int kOffW = kOffV + 2 * kCtHalf;            // high and low parts of w V
+  static constexpr int kOffS = kOffW + 2 * kCtHalf;            // high and low parts of the state [channel][64 columns]
+  static constexpr int kOffRaw = kOffS + 2 * kCtHalf;          // two buffers of log decays and steps
+  static constexpr int kOffSums = kOffRaw + 2 * 2 * kCtL * 4;  // per warp: c_j - log b_j, w_j, c_i (all in log2 units but w)
+  static constexpr int kOffBars = kOffSums + kCtWarps * 3 * kCtL * 4;
+  static constexpr int kBytes = 1024 + kOffBars + 8 * kCtBars + 16;
+};
+static_assert(CtPlan::kBytes <= 227 * 1024, "shared memory of the chunk scan");
+
+// tensor memory columns
+constexpr uint32_t kCtG = 0, kCtMh = 128, kCtMl = 192, kCtY1 = 256, kCtY2 = 320, kCtD = 384;
+
+// left operand in tensor memory: bf16 pairs, one row per lane
+__device__ __forceinline__ void umma_bf16_ts_w(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t"
+      "elect.sync _|q, 0xffffffff;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+      ::"r"(d_tmem), "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+
+// 16-byte piece c of row r of a tile with 128-byte swizzle
+__device__ __forceinline__ int ct_at(int r, int c) { return r * 128 + ((c ^ (r & 7)) << 4); }
+
+template <int NH>
+__global__ void __launch_bounds__(kCtThreads, 1) chunk_scan_tc_kernel(const mdb_chunk_scan_args a) {
+  using P = CtPlan;
+  constexpr int DP = 64 * NH;
+  extern __shared__ __align__(1024) unsigned char ct_smem_raw[];
+  const uint32_t raw_base = smem_u32(ct_smem_raw);
+  const uint32_t base = (raw_base + 1023u) & ~1023u;
+  unsigned char* mem = ct_smem_raw + (base - raw_base);
+  const uint32_t bars = base + P::kOffBars;
+  volatile uint32_t* misc = reinterpret_cast<volatile uint32_t*>(mem + P::kOffBars + 8 * kCtBars);      // tensor memory base, abort flag
+  pdl_launch_dependents();
+  pdl_wait();
+  const int seq = blockIdx.z, head = blockIdx.y, col0 = blockIdx.x * kCtCols;
+  const int slot = a.state_slot[seq];
+  if (slot < 0) return;
+  if (slot >= a.num_slots) {
+    if (threadIdx.x == 0) report_status(MDB_STATUS_BAD_SLOT);
+    return;
+  }
+  const int t_begin = a.cu_q[seq], t_end = a.cu_q[seq + 1];
+  if (t_begin >= t_end) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < kCtBars; ++s) mbar_init(bars + 8 * s, s < kCtBarG ? kCtWarps : 1);
+    misc[1] = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (warp == kCtWarps) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(const_cast<uint32_t*>(&misc[0]))), "r"(512u)
+                 : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = misc[0];
+  // A wait that runs out raises the abort flag; the roles then walk to the end without waiting again.
+  auto wait = [&](int s, uint32_t parity) {
+    if (misc[1] != 0) return;
+    if (!mbar_wait(bars + 8 * s, parity)) {
+      misc[1] = 1;
+      report_status(MDB_STATUS_WAIT_TIMEOUT);
+    }
+  };
+  uint32_t parity = 0;
+
+  if (warp == kCtWarps) {
+    // ---------------------------------------------------------------- products
+    const uint32_t kF32 = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(128 >> 4) << 24);      // bf16 x bf16 -> fp32, M = 128
+    const uint32_t id_g = kF32 | (static_cast<uint32_t>(kCtL >> 3) << 17);
+    const uint32_t id_y = kF32 | (1u << 16) | (static_cast<uint32_t>(kCtCols >> 3) << 17);                     // right operand stored K first
+    const uint32_t id_d = id_y | (1u << 15);                                                                   // ... and the left one
+    int buf = 0;
+    for (int t0 = t_begin; t0 < t_end; t0 += kCtL, buf ^= 1, parity ^= 1) {
+      const uint32_t qt = base + P::kOffQ, kt = base + P::kOffK + buf * 2 * kCtHalf, vt = base + P::kOffV + buf * kCtHalf;
+      const uint32_t wt = base + P::kOffW, st = base + P::kOffS;
+      wait(kCtBarOps, parity);
+      __syncwarp();
+      tc_fence_after();
+#pragma unroll
+      for (int k = 0; k < 4 * NH; ++k)
+        umma_bf16_w(tmem + kCtG, umma_desc_sw128(qt + (k >> 2) * kCtHalf) + 2 * (k & 3), umma_desc_sw128(kt + (k >> 2) * kCtHalf) + 2 * (k & 3), id_g,
+                    k > 0 ? 1u : 0u);
+      umma_commit_w(bars + 8 * kCtBarG);
+#pragma unroll
+      for (int p = 0; p < 2; ++p)
+#pragma unroll
+        for (int k = 0; k < 4 * NH; ++k)
+          umma_bf16_w(tmem + kCtY1, umma_desc_sw128(qt + (k >> 2) * kCtHalf) + 2 * (k & 3), umma_desc_sw128_mn(st + p * kCtHalf + k * 2048), id_y,
+                      p + k > 0 ? 1u : 0u);
+      umma_commit_w(bars + 8 * kCtBarY);
+      wait(kCtBarW, parity);
+      __syncwarp();
+      tc_fence_after();
+#pragma unroll
+      for (int p = 0; p < 2; ++p)
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          umma_bf16_w(tmem + kCtD, umma_desc_sw128_mn(kt + k * 2048), umma_desc_sw128_mn(wt + p * kCtHalf + k * 2048), id_d, p + k > 0 ? 1u : 0u);
+      wait(kCtBarM, parity);
+      __syncwarp();
+      tc_fence_after();
+#pragma unroll
+      for (int p = 0; p < 2; ++p)
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          umma_bf16_ts_w(tmem + kCtY2, tmem + (p ? kCtMl : kCtMh) + 8 * k, umma_desc_sw128_mn(vt + k * 2048), id_y, p + k > 0 ? 1u : 0u);
+      umma_commit_w(bars + 8 * kCtBarO);
+    }
+  } else {
+    // ------------------------------------------------------------ everything else
+    const int quad = warp & 3, hf = warp >> 2;
+    const int r = 32 * quad + lane;                  // this thread's token of the chunk, and its key channel of the state
+    const uint32_t lanes = static_cast<uint32_t>(32 * quad) << 16;
+    const bool fresh = a.start[seq] == 0;
+    const int kvh = head / (a.heads / a.kv_heads);
+    const float skip = a.skip != nullptr ? a.skip[head] : 0.f;
+    const bf16* q = static_cast<const bf16*>(a.q) + static_cast<int64_t>(kvh) * a.dim;
+    const bf16* k = static_cast<const bf16*>(a.k) + static_cast<int64_t>(kvh) * a.dim;
+    const bf16* v = static_cast<const bf16*>(a.v) + static_cast<int64_t>(head) * a.vdim + col0;
+    auto copy16 = [&](uint32_t dst, const bf16* src, bool live) {       // size 0 reads nothing and writes zeros
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(live ? 16 : 0) : "memory");
+    };
+    auto request_channels = [&](const bf16* src, int64_t ld, int t0, uint32_t dst) {
+      for (int i = threadIdx.x; i < kCtL * 8 * NH; i += kCtWarps * 32) {
+        const int t = i / (8 * NH), c = i % (8 * NH);
+        const bool live = t0 + t < t_end && 8 * c < a.dim;
+        copy16(dst + (c >> 3) * kCtHalf + ct_at(t, c & 7), src + (live ? (t0 + t) * ld + 8 * c : 0), live);
+      }
+    };
+    auto request_rest = [&](int t0, int buf) {
+      request_channels(k, a.ldk, t0, base + P::kOffK + buf * 2 * kCtHalf);
+      for (int i = threadIdx.x; i < kCtL * 8; i += kCtWarps * 32) {
+        const int t = i >> 3, c = i & 7;
+        const bool live = t0 + t < t_end && col0 + 8 * c < a.vdim;
+        copy16(base + P::kOffV + buf * kCtHalf + ct_at(t, c), v + (live ? (t0 + t) * a.ldv + 8 * c : 0), live);
+      }
+      {                                              // tokens past the end: no decay, no input
+        const int t = threadIdx.x & (kCtL - 1);
+        const float* src = threadIdx.x < kCtL ? a.log_decay : a.step;
+        const bool live = t0 + t < t_end;
+        asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(base + P::kOffRaw + (buf * 2 * kCtL + threadIdx.x) * 4),
+                     "l"(src + (live ? (t0 + t) * a.ld_scalars + head : 0)), "r"(live ? 4 : 0) : "memory");
+      }
+    };
+    request_channels(q, a.ldq, t_begin, base + P::kOffQ);
+    request_rest(t_begin, 0);
+    cp_async_commit();
+
+    float* state = a.state + slot * a.state_slot_stride + static_cast<int64_t>(head) * a.vdim * DP;
+    const int sc0 = col0 + 32 * hf;                  // first of this thread's 32 columns
+    const bool has_state = r < DP;
+    float S[32];
+#pragma unroll
+    for (int i = 0; i < 32; ++i) S[i] = has_state && !fresh && sc0 + i < a.vdim ? state[static_cast<int64_t>(sc0 + i) * DP + r] : 0.f;
+    auto publish = [&]() {                           // the state's two parts for the next read-out
+      if (!has_state) return;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) split2(S[8 * c + 2 * e], S[8 * c + 2 * e + 1], hi[e], lo[e]);
+        unsigned char* at = mem + P::kOffS + ct_at(r, 4 * hf + c);
+        *reinterpret_cast<uint4*>(at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(at + kCtHalf) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      }
+    };
+    publish();
+    float* cum = reinterpret_cast<float*>(mem + P::kOffSums) + warp * 3 * kCtL;
+    float* wgt = cum + kCtL;
+    float* crow = wgt + kCtL;
+    int buf = 0;
+    for (int t0 = t_begin; t0 < t_end; t0 += kCtL, buf ^= 1, parity ^= 1) {
+      const bool more = t0 + kCtL < t_end;
+      cp_async_wait<0>();
+      fence_async_smem();
+      tc_fence_before();                             // (this thread's reads of the last chunk's accumulators)
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bars + 8 * kCtBarOps);
+      asm volatile("bar.sync 1, 256;" ::: "memory"); // the whole chunk has landed, the other buffers are free
+      if (more) request_rest(t0 + kCtL, buf ^ 1);
+      cp_async_commit();
+      {
+        // inclusive sums over 128 tokens, four per lane; every warp for itself
+        const float* raw = reinterpret_cast<const float*>(mem + P::kOffRaw) + buf * 2 * kCtL;
+        const float4 x = *reinterpret_cast<const float4*>(raw + 4 * lane), b = *reinterpret_cast<const float4*>(raw + kCtL + 4 * lane);
+        constexpr float kLog2e = 1.4426950408889634f;
+        float4 c = make_float4(x.x * kLog2e, x.y * kLog2e, x.z * kLog2e, x.w * kLog2e);
+        c.y += c.x; c.z += c.y; c.w += c.z;
+        float s = c.w;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          const float p = __shfl_up_sync(0xffffffffu, s, o);
+          if (lane >= o) s += p;
+        }
+        const float before = s - c.w, total = __shfl_sync(0xffffffffu, s, 31);
+        c.x += before; c.y += before; c.z += before; c.w = s;
+        *reinterpret_cast<float4*>(crow + 4 * lane) = c;
+        *reinterpret_cast<float4*>(wgt + 4 * lane) = make_float4(b.x * exp2f(total - c.x), b.y * exp2f(total - c.y), b.z * exp2f(total - c.z), b.w * exp2f(total - c.w));
+        // (step 0: +inf, weight 0)
+        *reinterpret_cast<float4*>(cum + 4 * lane) = make_float4(c.x - log2f(b.x), c.y - log2f(b.y), c.z - log2f(b.z), c.w - log2f(b.w));
+        __syncwarp();
+      }
+      const unsigned char* vt = mem + P::kOffV + buf * kCtHalf;
+      {
+        // w V of 16 tokens per warp: a lane takes half a row
+        const int t = 16 * warp + (lane >> 1);
+        const float w = wgt[t];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int at = ct_at(t, 4 * (lane & 1) + i);
+          const uint4 x = *reinterpret_cast<const uint4*>(vt + at);
+          const uint32_t in[4] = {x.x, x.y, x.z, x.w};
+          uint32_t hi[4], lo[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float2 f = unpack_bf16x2(in[e]);
+            split2(f.x * w, f.y * w, hi[e], lo[e]);
+          }
+          *reinterpret_cast<uint4*>(mem + P::kOffW + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          *reinterpret_cast<uint4*>(mem + P::kOffW + kCtHalf + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        }
+        fence_async_smem();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(bars + 8 * kCtBarW);
+      }
+      const float ci = crow[r];
+      wait(kCtBarG, parity);
+      __syncwarp();
+      tc_fence_after();
+      {
+        uint32_t mh[32], ml[32];
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int j0 = 64 * hf + 32 * half;        // 32 tokens; the warp's rows start at 32 quad
+          if (j0 > 32 * quad) {                      // behind all of them
+#pragma unroll
+            for (int i = 0; i < 16; ++i) mh[16 * half + i] = ml[16 * half + i] = 0u;
+            continue;
+          }
+          float g[32];
+          tmem_ld32(tmem + kCtG + lanes + j0, g);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            const float4 cj = *reinterpret_cast<const float4*>(cum + j0 + 4 * i);
+            g[4 * i] *= ex2_approx(ci - cj.x);
+            g[4 * i + 1] *= ex2_approx(ci - cj.y);
+            g[4 * i + 2] *= ex2_approx(ci - cj.z);
+            g[4 * i + 3] *= ex2_approx(ci - cj.w);
+          }
+          if (j0 == 32 * quad) {                     // the diagonal: tokens up to the row's own
+#pragma unroll
+            for (int i = 0; i < 32; ++i) g[i] = i <= lane ? g[i] : 0.f;
+          }
+#pragma unroll
+          for (int i = 0; i < 16; ++i) split2(g[2 * i], g[2 * i + 1], mh[16 * half + i], ml[16 * half + i]);
+        }
+        tmem_st32(tmem + kCtMh + lanes + 32 * hf, reinterpret_cast<const float (&)[32]>(mh));
+        tmem_st32(tmem + kCtMl + lanes + 32 * hf, reinterpret_cast<const float (&)[32]>(ml));
+        tmem_st_wait();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(bars + 8 * kCtBarM);
+      }
+      wait(kCtBarY, parity);
+      __syncwarp();
+      tc_fence_after();
+      if (more) request_channels(q, a.ldq, t0 + kCtL, base + P::kOffQ);
+      cp_async_commit();
+      float y[32];
+      tmem_ld32(tmem + kCtY1 + lanes + 32 * hf, y);
+      tmem_ld_wait();
+      {
+        const float e = exp2f(ci);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const uint4 x = *reinterpret_cast<const uint4*>(vt + ct_at(r, 4 * hf + c));
+          const uint32_t in[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const float2 f = unpack_bf16x2(in[i]);
+            y[8 * c + 2 * i] = fmaf(y[8 * c + 2 * i], e, skip * f.x);
+            y[8 * c + 2 * i + 1] = fmaf(y[8 * c + 2 * i + 1], e, skip * f.y);
+          }
+        }
+      }
+      const float keep = exp2f(crow[kCtL - 1]);
+      wait(kCtBarO, parity);
+      __syncwarp();
+      tc_fence_after();
+      {
+        float d[32];
+        tmem_ld32(tmem + kCtD + lanes + 32 * hf, d);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) S[i] = fmaf(S[i], keep, d[i]);
+        if (more) publish();
+        tmem_ld32(tmem + kCtY2 + lanes + 32 * hf, d);
+        tmem_ld_wait();
+        if (t0 + r < t_end) {
+          float* out = a.out + (static_cast<int64_t>(t0 + r) * a.heads + head) * a.vdim + sc0;
+#pragma unroll
+          for (int i = 0; i < 32; i += 4)
+            if (sc0 + i < a.vdim) *reinterpret_cast<float4*>(out + i) = make_float4(y[i] + d[i], y[i + 1] + d[i + 1], y[i + 2] + d[i + 2], y[i + 3] + d[i + 3]);
+        }
+      }
+    }
+    cp_async_wait<0>();
+    if (has_state) {
+#pragma unroll
+      for (int i = 0; i < 32; ++i)
+        if (sc0 + i < a.vdim) state[static_cast<int64_t>(sc0 + i) * DP + r] = S[i];
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == kCtWarps) {
+    tc_fence_after();
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
+  }
+}
+
+template <int NH>
+static int launch_chunk_scan_tc(const mdb_chunk_scan_args& a, cudaStream_t st) {
+  static PerDeviceOnce attr_once;
+  const int dev = attr_once.slot();
+  if (dev < 0) return MDB_ERR_CUDA;
+  if (!attr_once.done[dev]) {
+    if (cudaFuncSetAttribute(chunk_scan_tc_kernel<NH>, cudaFuncAttributeMaxDynamicSharedMemorySize, CtPlan::kBytes) != cudaSuccess) return MDB_ERR_CUDA;
+    attr_once.done[dev] = true;
+  }
+  return mdb_launch(chunk_scan_tc_kernel<NH>, dim3((a.vdim + kCtCols - 1) / kCtCols, a.heads, a.bs), dim3(kCtThreads), CtPlan::kBytes, st, a);
+}
+
+}  // namespace mdb

@@ -541,7 +541,7 @@ class HybridEngine:
         if activated:
             rows = x.x
             ops.chunk_scan(b.bs, heads, kvh, dim, vdim, rows[:, q0:], rows[:, k0:], rows[:, v0:], pw["log_decay"], pw["step"], st["s"],
-                           self._portions(b), o)
+                           self._portions(b), b.max_q, o)
             return leave()
         outs = (self.buf("scan_q", m, kvh, dp, dtype=act), self.buf("scan_k", m, kvh, dp, dtype=act),
                 self.buf("scan_v", m, heads, vdim, dtype=act), self.buf("scan_s0", m, heads, dtype=f32),
@@ -552,8 +552,8 @@ class HybridEngine:
         ops.decay_prep(self.dtype, m, b.bs, heads, kvh, dim, vdim, x.cols(q0), x.cols(k0), x.cols(v0), self._portions(b), outs, **scalars)
         if chunks:
             q, k, v, *scalars = outs
-            ops.chunk_scan(b.bs, heads, kvh, dp, vdim, q.view(m, -1), k.view(m, -1), v.view(m, -1), *scalars, st["s"], self._portions(b), o,
-                           skip=pw.get("skip"))
+            ops.chunk_scan(b.bs, heads, kvh, dp, vdim, q.view(m, -1), k.view(m, -1), v.view(m, -1), *scalars, st["s"], self._portions(b),
+                           b.max_q, o, skip=pw.get("skip"))
         else:
             ops.scan(ops.SCAN_DECAY, self.dtype, b.bs, heads, kvh, dim, vdim, *outs, st["s"], self._portions(b), out=o,
                      skip=pw.get("skip"), one_token=one_token and ops.scan_fusable(dp, vdim))

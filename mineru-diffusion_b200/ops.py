@@ -770,7 +770,7 @@ def chunk_scan_supported(dim_pad: int, vdim: int) -> bool:
     return bool(_lib.lib().mdb_chunk_scan_supported(dim_pad, vdim))
 
 
-def chunk_scan(bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q, k, v, log_decay, step, state, portions: tuple, out,
+def chunk_scan(bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q, k, v, log_decay, step, state, portions: tuple, max_q: int, out,
                skip=None) -> None:
     """The decay scan over prompt portions on the tensor cores: bf16 q, k [m, >= kv_heads * dim] and v [m, >= heads * vdim] (row
     strides free), logarithms of the decays (at least -104) and steps [m, heads], or [heads] for all tokens; ``state`` and
@@ -778,7 +778,7 @@ def chunk_scan(bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q, k, v,
     _, cu_q, start, slot = portions
     for t, nm in ((q, "q"), (k, "k"), (v, "v")):
         _need(t, _BF16, nm)
-    a = _lib.ChunkScanArgs(bs, heads, kv_heads, dim, state.shape[-1], vdim, q.data_ptr(), k.data_ptr(), v.data_ptr(), _rows(q, "q"),
+    a = _lib.ChunkScanArgs(bs, heads, kv_heads, dim, state.shape[-1], vdim, max_q, q.data_ptr(), k.data_ptr(), v.data_ptr(), _rows(q, "q"),
                            _rows(k, "k"), _rows(v, "v"), heads if log_decay.dim() > 1 else 0, log_decay.data_ptr(),
                            step.data_ptr(), _ptr(skip), state.data_ptr(), state.stride(0), state.shape[0], cu_q.data_ptr(),
                            start.data_ptr(), slot.data_ptr(), out.data_ptr())

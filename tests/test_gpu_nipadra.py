@@ -116,7 +116,8 @@ def test_product_activated_from_a_column_on(dtype, m, n, k, from_):
     assert rel(y, ref) < (2e-6 if dtype is F32 else 4e-3)
 
 
-def test_chunk_scan_reads_columns_of_a_projection():
+@pytest.mark.parametrize("mq", [64, 150])
+def test_chunk_scan_reads_columns_of_a_projection(mq):
     """Heads of 40 channels in rows of another matrix: missing channels of the stored state count as zeros."""
     ops, T, H, D, DV = pkg.ops, 150, 3, 40, 24
     x = rand(T, 8 + 2 * H * D + H * DV + 16, seed=1, scale=0.5)
@@ -126,7 +127,7 @@ def test_chunk_scan_reads_columns_of_a_projection():
     ref = orc.linear_scan(q.double().view(T, H, D), k.double().view(T, H, D), v.double().view(T, H, DV), decay, torch.ones_like(decay))
     xd = x.to(BF).to(DEV)
     state, o = torch.full((1, H, DV, 64), 5.0, device=DEV), torch.zeros(T, H, DV, device=DEV)
-    ops.chunk_scan(1, H, H, D, DV, xd[:, 8:], xd[:, 128:], xd[:, 248:], log.to(DEV), torch.ones(H, device=DEV), state, portions_of([T], slots=[0]), o)
+    ops.chunk_scan(1, H, H, D, DV, xd[:, 8:], xd[:, 128:], xd[:, 248:], log.to(DEV), torch.ones(H, device=DEV), state, portions_of([T], slots=[0]), mq, o)
     assert rel(o, ref) < 3e-5 and float(state[..., D:].abs().max()) == 0
 
 
@@ -356,7 +357,7 @@ def _scan_run(case, H, G, D, DV, taps, counts, dtype, as_parts=False, chunks=Fal
         o = torch.zeros(n, H, DV, device=DEV)
         if chunks:
             q, k, v, *sc = outs
-            ops.chunk_scan(1, H, G, dp, DV, q.view(n, -1), k.view(n, -1), v.view(n, -1), *sc, state, p, o, skip=dev["skip"] if taps else None)
+            ops.chunk_scan(1, H, G, dp, DV, q.view(n, -1), k.view(n, -1), v.view(n, -1), *sc, state, p, n, o, skip=dev["skip"] if taps else None)
         else:
             ops.scan(ops.SCAN_DECAY, dtype, 1, H, G, D, DV, *outs, state, p, out=o, skip=dev["skip"] if taps else None,
                      one_token=n == 1 and ops.scan_fusable(dp, DV))
@@ -409,7 +410,7 @@ def test_chunk_scan_is_the_recurrence(H, G, D, DV, counts):
         p = portions_of([5, n, 3], [7, at, 0], [0, 2, -1])
         pad = lambda t: torch.cat([t[:5], t[at:at + n], t[:3]]).to(DEV)
         o = torch.full((n + 8, H, DV), 4.0, device=DEV)
-        ops.chunk_scan(3, H, G, D, DV, *(pad(t).to(BF).flatten(1) for t in (q, k, v)), pad(log), pad(step), state, p, o, skip=skip.to(DEV))
+        ops.chunk_scan(3, H, G, D, DV, *(pad(t).to(BF).flatten(1) for t in (q, k, v)), pad(log), pad(step), state, p, n, o, skip=skip.to(DEV))
         assert float((o[5 + n:] - 4).abs().max()) == 0 and float((o[:5] - 4).abs().min()) > 0
         outs.append(o[5:5 + n])
         at += n
@@ -420,11 +421,12 @@ def test_chunk_scan_is_the_recurrence(H, G, D, DV, counts):
     assert float((state[1] - 3).abs().max()) == 0 and float((state[3] - 3).abs().max()) == 0
 
 
-@pytest.mark.parametrize("far", [1, 62, 63, 64, 65, 300])
-def test_chunk_scan_remembers_a_far_key(far):
+@pytest.mark.parametrize("mq", [64, 400])
+@pytest.mark.parametrize("far", [1, 62, 63, 64, 65, 127, 128, 129, 270])
+def test_chunk_scan_remembers_a_far_key(far, mq):
     """One key written and asked for ``far`` tokens later, over chunk borders, orthogonal writes in between."""
     ops, T, D, DV, decay = pkg.ops, 400, 64, 16, 0.998
-    for at in (0, 3, 63, 64):
+    for at in (0, 3, 63, 64, 127):
         k = torch.zeros(T, 1, D)
         k[:, 0, 1:] = rand(T, D - 1, seed=0)
         k[at, 0], k[at, 0, 0] = 0.0, 1.0
@@ -433,7 +435,7 @@ def test_chunk_scan_remembers_a_far_key(far):
         v = rand(T, 1, DV, seed=1)
         state, o = torch.zeros(1, 1, DV, D, device=DEV), torch.zeros(T, 1, DV, device=DEV)
         ops.chunk_scan(1, 1, 1, D, DV, *(t.to(BF).to(DEV).flatten(1) for t in (q, k, v)), torch.full((1,), decay, device=DEV).log(),
-                       torch.full((1,), 0.5, device=DEV), state, portions_of([T], slots=[0]), o)
+                       torch.full((1,), 0.5, device=DEV), state, portions_of([T], slots=[0]), mq, o)
         want = torch.zeros(T, DV)
         want[at + far] = 0.5 * v[at, 0] * decay ** far
         assert float((o[:, 0].cpu() - want).abs().max()) < 1e-4
