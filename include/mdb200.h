@@ -579,10 +579,10 @@ int mdb_scan(const mdb_scan_args* args, mdb_stream_t stream);
 /* The decay scan over prompt portions in chunks of 64 tokens on the tensor cores: bf16 rows of ldq / ldk elements with head
  * g of q and k at column g * dim (dim a multiple of 8, missing channels up to dim_pad count as zeros) and rows of ldv elements
  * with head h of v at column h * vdim; log_decay (at least -104) and step are rows of heads, ld_scalars elements apart
- * (0: the same for every token); state and out as in mdb_scan; max_q = longest portion.  Key heads of up to 128 channels take
- * chunks of 128 tokens where a portion is longer than 64. */
+ * (0: the same for every token); state and out as in mdb_scan; max_q = longest portion, m = rows.  Key heads of exactly 64 or
+ * 128 channels take chunks of 128 tokens where a portion is longer than 64. */
 typedef struct {
-  int32_t bs, heads, kv_heads, dim, dim_pad, vdim, max_q;
+  int32_t m, bs, heads, kv_heads, dim, dim_pad, vdim, max_q;
   const void* q;
   const void* k;
   const void* v;

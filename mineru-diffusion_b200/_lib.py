@@ -74,7 +74,7 @@ ScanArgs = _struct("ScanArgs", [(n, _i) for n in (
     ("den", _p), ("cu_q", _p), ("start", _p),
     ("state_slot", _p), ("out", _p), ("raw_decay", Rows), ("a_log", _p), ("dt_bias", _p), ("gate", Rows), ("norm", _p),
     ("norm_head_stride", _i64), ("y", _p), ("ldy", _i64), ("skip", _p)])
-ChunkScanArgs = _struct("ChunkScanArgs", [(n, _i) for n in ("bs", "heads", "kv_heads", "dim", "dim_pad", "vdim", "max_q")] + [
+ChunkScanArgs = _struct("ChunkScanArgs", [(n, _i) for n in ("m", "bs", "heads", "kv_heads", "dim", "dim_pad", "vdim", "max_q")] + [
     ("q", _p), ("k", _p), ("v", _p), ("ldq", _i64), ("ldk", _i64), ("ldv", _i64), ("ld_scalars", _i64), ("log_decay", _p), ("step", _p), ("skip", _p), ("state", _p), ("state_slot_stride", _i64),
     ("num_slots", _i64), ("cu_q", _p), ("start", _p), ("state_slot", _p), ("out", _p)])
 MoeRouteArgs = _struct("MoeRouteArgs", [(n, _i) for n in ("m", "experts", "top", "groups", "keep")] + [

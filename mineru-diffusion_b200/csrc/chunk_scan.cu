@@ -324,7 +324,7 @@ int mdb_chunk_scan(const mdb_chunk_scan_args* args, mdb_stream_t stream) {
   MDB_REQUIRE(a.bs >= 0 && a.heads > 0 && a.kv_heads > 0 && a.heads % a.kv_heads == 0 && a.vdim > 0, MDB_ERR_ARG);
   if (a.bs == 0) return MDB_OK;
   MDB_REQUIRE(a.q && a.k && a.v && a.log_decay && a.step && a.state && a.cu_q && a.start && a.state_slot && a.out, MDB_ERR_ARG);
-  MDB_REQUIRE(a.dim > 0 && a.dim <= a.dim_pad && a.ldq >= static_cast<int64_t>(a.kv_heads) * a.dim && a.ldk >= static_cast<int64_t>(a.kv_heads) * a.dim &&
+  MDB_REQUIRE(a.m > 0 && a.dim > 0 && a.dim <= a.dim_pad && a.ldq >= static_cast<int64_t>(a.kv_heads) * a.dim && a.ldk >= static_cast<int64_t>(a.kv_heads) * a.dim &&
                   a.ldv >= static_cast<int64_t>(a.heads) * a.vdim && a.ld_scalars >= 0,
               MDB_ERR_ARG);
   MDB_REQUIRE(a.dim % 8 == 0 && a.ldq % 8 == 0 && a.ldk % 8 == 0 && a.ldv % 8 == 0 && mdb_aligned16(a.q) && mdb_aligned16(a.k) &&
@@ -332,9 +332,10 @@ int mdb_chunk_scan(const mdb_chunk_scan_args* args, mdb_stream_t stream) {
               MDB_ERR_ALIGN);
   MDB_REQUIRE(mdb_chunk_scan_supported(a.dim_pad, a.vdim) && a.heads <= 65535 && a.bs <= 65535, MDB_ERR_UNSUPPORTED);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool long_chunks = a.max_q > kChunk && a.dim == a.dim_pad;
   switch (a.dim_pad) {
-    case 64: return a.max_q > kChunk ? launch_chunk_scan_tc<1>(a, st) : launch_chunk_scan_cols<64>(a, st);
-    case 128: return a.max_q > kChunk ? launch_chunk_scan_tc<2>(a, st) : launch_chunk_scan_cols<128>(a, st);
+    case 64: return long_chunks ? launch_chunk_scan_tc<1>(a, st) : launch_chunk_scan_cols<64>(a, st);
+    case 128: return long_chunks ? launch_chunk_scan_tc<2>(a, st) : launch_chunk_scan_cols<128>(a, st);
     case 192: return launch_chunk_scan_cols<192>(a, st);
     default: return launch_chunk_scan_cols<256>(a, st);
   }

@@ -6,11 +6,13 @@
 //   D  = K^T (w V)    (w V in two parts)     what the chunk adds to the state, w_j = e^(c_last - c_j) b_j
 //   Y2 = M V          (M in two parts)       M = G e^(c_i - c_j) b_j below the diagonal
 //
-// with the accumulators in tensor memory.  One warp issues the products; eight warps do the rest, a pair of warps per 32
-// rows, half of the columns each: w V (shared memory to shared memory), M (tensor memory to tensor memory, where it is
-// the left operand of its product), the outputs, and the state, which stays in their registers in fp32 (a thread holds one
-// key channel of 32 columns).  D does not wait for M and runs under it.  The next chunk's k and v are requested at the
-// start of a chunk, q once Y1 is complete.
+// with the accumulators in tensor memory.  One warp issues the products and the loads (TMA: the next chunk's k and v at the
+// start of a chunk, q once Y1 is complete) and, while it waits for M, sums the next chunk's log decays.  Eight warps do
+// the rest, a pair of warps per 32 rows, half of the columns each: w V (shared memory to shared memory), M (tensor memory
+// to tensor memory, where it is the left operand of its product), the outputs, and the state, which stays in their
+// registers in fp32 (a thread holds one key channel of 32 columns).  D does not wait for M and runs under it; the next
+// chunk's first products run under the outputs.  Rows of a tile past the end of a portion belong to another sequence: they
+// are cleared before they meet a product whose result is kept.
 #include "mdb_common.cuh"
 
 namespace mdb {
@@ -18,23 +20,23 @@ namespace mdb {
 constexpr int kCtL = 128, kCtCols = 64, kCtWarps = 8, kCtThreads = (kCtWarps + 1) * 32;
 constexpr int kCtHalf = kCtL * 128;          // [128 rows][64 bf16]: one swizzled tile
 
-enum { kCtBarOps = 0, kCtBarW, kCtBarM, kCtBarG, kCtBarY, kCtBarO, kCtBars };
+// arrivals by every working warp: operands of a chunk, w V, M; by commits: G, Y1, everything; by TMA: q, k and v; sums
+enum { kCtBarOps = 0, kCtBarW, kCtBarM, kCtBarG, kCtBarY, kCtBarO, kCtBarQ, kCtBarKV, kCtBarSum, kCtBars };
 
 struct CtPlan {
   static constexpr int kOffQ = 0;                              // two halves of 64 channels
   static constexpr int kOffK = kOffQ + 2 * kCtHalf;            // two buffers
   static constexpr int kOffV = kOffK + 4 * kCtHalf;            // two buffers
-  static constexpr int kOffW = kOffV + 2 * kCtHalf;            // high and low parts of w V
+  static constexpr int kOffW = kOffV + 2 * kCtHalf;            // high and low parts of w V; later outputs on their way out
   static constexpr int kOffS = kOffW + 2 * kCtHalf;            // high and low parts of the state [channel][64 columns]
-  static constexpr int kOffRaw = kOffS + 2 * kCtHalf;          // two buffers of log decays and steps
-  static constexpr int kOffSums = kOffRaw + 2 * 2 * kCtL * 4;  // per warp: c_j - log b_j, w_j, c_i (all in log2 units but w)
-  static constexpr int kOffBars = kOffSums + kCtWarps * 3 * kCtL * 4;
+  static constexpr int kOffSums = kOffS + 2 * kCtHalf;         // two buffers: c_j - log b_j, w_j, c_i (in log2 units but w)
+  static constexpr int kOffBars = kOffSums + 2 * 3 * kCtL * 4;
   static constexpr int kBytes = 1024 + kOffBars + 8 * kCtBars + 16;
 };
 static_assert(CtPlan::kBytes <= 227 * 1024, "shared memory of the chunk scan");
 
 // tensor memory columns
-constexpr uint32_t kCtG = 0, kCtMh = 128, kCtMl = 192, kCtY1 = 256, kCtY2 = 320, kCtD = 384;
+constexpr uint32_t kCtG = 0, kCtMh = 128, kCtMl = 192, kCtY1 = 256 /* high | low part of S */, kCtY2 = 384, kCtD = 448;
 
 // left operand in tensor memory: bf16 pairs, one row per lane
 __device__ __forceinline__ void umma_bf16_ts_w(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
@@ -51,7 +53,8 @@ __device__ __forceinline__ void umma_bf16_ts_w(uint32_t d_tmem, uint32_t a_tmem,
 __device__ __forceinline__ int ct_at(int r, int c) { return r * 128 + ((c ^ (r & 7)) << 4); }
 
 template <int NH>
-__global__ void __launch_bounds__(kCtThreads, 1) chunk_scan_tc_kernel(const mdb_chunk_scan_args a) {
+__global__ void __launch_bounds__(kCtThreads, 1) chunk_scan_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+                     const __grid_constant__ CUtensorMap map_v, const mdb_chunk_scan_args a) {
   using P = CtPlan;
   constexpr int DP = 64 * NH;
   extern __shared__ __align__(1024) unsigned char ct_smem_raw[];
@@ -95,17 +98,77 @@ __global__ void __launch_bounds__(kCtThreads, 1) chunk_scan_tc_kernel(const mdb_
     }
   };
   uint32_t parity = 0;
+  const int kvh = head / (a.heads / a.kv_heads);
+  float* sums = reinterpret_cast<float*>(mem + P::kOffSums);
 
   if (warp == kCtWarps) {
     // ---------------------------------------------------------------- products
     const uint32_t kF32 = (1u << 4) | (1u << 7) | (1u << 10) | (static_cast<uint32_t>(128 >> 4) << 24);      // bf16 x bf16 -> fp32, M = 128
     const uint32_t id_g = kF32 | (static_cast<uint32_t>(kCtL >> 3) << 17);
     const uint32_t id_y = kF32 | (1u << 16) | (static_cast<uint32_t>(kCtCols >> 3) << 17);                     // right operand stored K first
+    const uint32_t id_y1 = kF32 | (1u << 16) | (static_cast<uint32_t>(2 * kCtCols >> 3) << 17);                // both parts of S side by side
     const uint32_t id_d = id_y | (1u << 15);                                                                   // ... and the left one
+    int q_loads = 0, kv_loads = 0;
+    auto load_q = [&](int t0) {
+      ++q_loads;
+      mbar_arrive_expect_tx_w(bars + 8 * kCtBarQ, NH * kCtHalf);
+#pragma unroll
+      for (int h = 0; h < NH; ++h) tma_load_2d_w(base + P::kOffQ + h * kCtHalf, &map_q, kvh * DP + 64 * h, t0, bars + 8 * kCtBarQ);
+    };
+    auto load_kv = [&](int t0, int buf) {
+      ++kv_loads;
+      mbar_arrive_expect_tx_w(bars + 8 * kCtBarKV, (NH + 1) * kCtHalf);
+#pragma unroll
+      for (int h = 0; h < NH; ++h)
+        tma_load_2d_w(base + P::kOffK + (2 * buf + h) * kCtHalf, &map_k, kvh * DP + 64 * h, t0, bars + 8 * kCtBarKV);
+      tma_load_2d_w(base + P::kOffV + buf * kCtHalf, &map_v, head * a.vdim + col0, t0, bars + 8 * kCtBarKV);
+    };
+    // log decays and steps of four tokens per lane (past the end: no decay, no input), and their sums over the chunk
+    float x[4], b[4];
+    auto load_scalars = [&](int t0) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int t = t0 + 4 * lane + i;
+        x[i] = t < t_end ? a.log_decay[t * a.ld_scalars + head] : 0.f;
+        b[i] = t < t_end ? a.step[t * a.ld_scalars + head] : 0.f;
+      }
+    };
+    auto sum_scalars = [&](int buf) {
+      constexpr float kLog2e = 1.4426950408889634f;
+      float c[4] = {x[0] * kLog2e, x[1] * kLog2e, x[2] * kLog2e, x[3] * kLog2e};
+      c[1] += c[0]; c[2] += c[1]; c[3] += c[2];
+      float s = c[3];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float p = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= o) s += p;
+      }
+      const float before = s - c[3], total = __shfl_sync(0xffffffffu, s, 31);
+      c[0] += before; c[1] += before; c[2] += before; c[3] = s;
+      float* at = sums + buf * 3 * kCtL + 4 * lane;
+      float w[4], m[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        w[i] = b[i] * exp2f(total - c[i]);
+        m[i] = c[i] - log2f(b[i]);                   // (step 0: +inf, weight 0)
+      }
+      *reinterpret_cast<float4*>(at) = make_float4(m[0], m[1], m[2], m[3]);
+      *reinterpret_cast<float4*>(at + kCtL) = make_float4(w[0], w[1], w[2], w[3]);
+      *reinterpret_cast<float4*>(at + 2 * kCtL) = make_float4(c[0], c[1], c[2], c[3]);
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bars + 8 * kCtBarSum);
+    };
+    load_q(t_begin);
+    load_kv(t_begin, 0);
+    load_scalars(t_begin);
+    sum_scalars(0);
     int buf = 0;
     for (int t0 = t_begin; t0 < t_end; t0 += kCtL, buf ^= 1, parity ^= 1) {
+      const bool more = t0 + kCtL < t_end;
       const uint32_t qt = base + P::kOffQ, kt = base + P::kOffK + buf * 2 * kCtHalf, vt = base + P::kOffV + buf * kCtHalf;
       const uint32_t wt = base + P::kOffW, st = base + P::kOffS;
+      wait(kCtBarQ, parity);
+      wait(kCtBarKV, parity);
       wait(kCtBarOps, parity);
       __syncwarp();
       tc_fence_after();
@@ -115,20 +178,29 @@ __global__ void __launch_bounds__(kCtThreads, 1) chunk_scan_tc_kernel(const mdb_
                     k > 0 ? 1u : 0u);
       umma_commit_w(bars + 8 * kCtBarG);
 #pragma unroll
-      for (int p = 0; p < 2; ++p)
-#pragma unroll
-        for (int k = 0; k < 4 * NH; ++k)
-          umma_bf16_w(tmem + kCtY1, umma_desc_sw128(qt + (k >> 2) * kCtHalf) + 2 * (k & 3), umma_desc_sw128_mn(st + p * kCtHalf + k * 2048), id_y,
-                      p + k > 0 ? 1u : 0u);
+      for (int k = 0; k < 4 * NH; ++k)
+        umma_bf16_w(tmem + kCtY1, umma_desc_sw128(qt + (k >> 2) * kCtHalf) + 2 * (k & 3), umma_desc_sw128_mn(st + k * 2048), id_y1, k > 0 ? 1u : 0u);
       umma_commit_w(bars + 8 * kCtBarY);
       wait(kCtBarW, parity);
       __syncwarp();
       tc_fence_after();
+      if (misc[1] != 0) break;
+      // every working warp has seen this chunk's k and v arrive, and the other buffers were last read in the chunk before
+      if (more) {
+        load_kv(t0 + kCtL, buf ^ 1);
+        load_scalars(t0 + kCtL);
+      }
 #pragma unroll
       for (int p = 0; p < 2; ++p)
 #pragma unroll
         for (int k = 0; k < 8; ++k)
           umma_bf16_w(tmem + kCtD, umma_desc_sw128_mn(kt + k * 2048), umma_desc_sw128_mn(wt + p * kCtHalf + k * 2048), id_d, p + k > 0 ? 1u : 0u);
+      if (more) {
+        wait(kCtBarY, parity);
+        __syncwarp();
+        load_q(t0 + kCtL);
+        sum_scalars(buf ^ 1);
+      }
       wait(kCtBarM, parity);
       __syncwarp();
       tc_fence_after();
@@ -139,46 +211,17 @@ __global__ void __launch_bounds__(kCtThreads, 1) chunk_scan_tc_kernel(const mdb_
           umma_bf16_ts_w(tmem + kCtY2, tmem + (p ? kCtMl : kCtMh) + 8 * k, umma_desc_sw128_mn(vt + k * 2048), id_y, p + k > 0 ? 1u : 0u);
       umma_commit_w(bars + 8 * kCtBarO);
     }
+    if (misc[1] != 0) {                              // given up: let the copies already issued land
+      mbar_wait(bars + 8 * kCtBarQ, (q_loads - 1) & 1);
+      mbar_wait(bars + 8 * kCtBarKV, (kv_loads - 1) & 1);
+    }
   } else {
     // ------------------------------------------------------------ everything else
     const int quad = warp & 3, hf = warp >> 2;
     const int r = 32 * quad + lane;                  // this thread's token of the chunk, and its key channel of the state
     const uint32_t lanes = static_cast<uint32_t>(32 * quad) << 16;
     const bool fresh = a.start[seq] == 0;
-    const int kvh = head / (a.heads / a.kv_heads);
     const float skip = a.skip != nullptr ? a.skip[head] : 0.f;
-    const bf16* q = static_cast<const bf16*>(a.q) + static_cast<int64_t>(kvh) * a.dim;
-    const bf16* k = static_cast<const bf16*>(a.k) + static_cast<int64_t>(kvh) * a.dim;
-    const bf16* v = static_cast<const bf16*>(a.v) + static_cast<int64_t>(head) * a.vdim + col0;
-    auto copy16 = [&](uint32_t dst, const bf16* src, bool live) {       // size 0 reads nothing and writes zeros
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(live ? 16 : 0) : "memory");
-    };
-    auto request_channels = [&](const bf16* src, int64_t ld, int t0, uint32_t dst) {
-      for (int i = threadIdx.x; i < kCtL * 8 * NH; i += kCtWarps * 32) {
-        const int t = i / (8 * NH), c = i % (8 * NH);
-        const bool live = t0 + t < t_end && 8 * c < a.dim;
-        copy16(dst + (c >> 3) * kCtHalf + ct_at(t, c & 7), src + (live ? (t0 + t) * ld + 8 * c : 0), live);
-      }
-    };
-    auto request_rest = [&](int t0, int buf) {
-      request_channels(k, a.ldk, t0, base + P::kOffK + buf * 2 * kCtHalf);
-      for (int i = threadIdx.x; i < kCtL * 8; i += kCtWarps * 32) {
-        const int t = i >> 3, c = i & 7;
-        const bool live = t0 + t < t_end && col0 + 8 * c < a.vdim;
-        copy16(base + P::kOffV + buf * kCtHalf + ct_at(t, c), v + (live ? (t0 + t) * a.ldv + 8 * c : 0), live);
-      }
-      {                                              // tokens past the end: no decay, no input
-        const int t = threadIdx.x & (kCtL - 1);
-        const float* src = threadIdx.x < kCtL ? a.log_decay : a.step;
-        const bool live = t0 + t < t_end;
-        asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(base + P::kOffRaw + (buf * 2 * kCtL + threadIdx.x) * 4),
-                     "l"(src + (live ? (t0 + t) * a.ld_scalars + head : 0)), "r"(live ? 4 : 0) : "memory");
-      }
-    };
-    request_channels(q, a.ldq, t_begin, base + P::kOffQ);
-    request_rest(t_begin, 0);
-    cp_async_commit();
-
     float* state = a.state + slot * a.state_slot_stride + static_cast<int64_t>(head) * a.vdim * DP;
     const int sc0 = col0 + 32 * hf;                  // first of this thread's 32 columns
     const bool has_state = r < DP;
@@ -198,49 +241,38 @@ __global__ void __launch_bounds__(kCtThreads, 1) chunk_scan_tc_kernel(const mdb_
       }
     };
     publish();
-    float* cum = reinterpret_cast<float*>(mem + P::kOffSums) + warp * 3 * kCtL;
-    float* wgt = cum + kCtL;
-    float* crow = wgt + kCtL;
+    auto hand_over = [&]() {                         // state and accumulators of the last chunk are done with
+      fence_async_smem();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bars + 8 * kCtBarOps);
+    };
+    hand_over();
     int buf = 0;
     for (int t0 = t_begin; t0 < t_end; t0 += kCtL, buf ^= 1, parity ^= 1) {
       const bool more = t0 + kCtL < t_end;
-      cp_async_wait<0>();
-      fence_async_smem();
-      tc_fence_before();                             // (this thread's reads of the last chunk's accumulators)
+      const float* cum = sums + buf * 3 * kCtL;
+      const float* wgt = cum + kCtL;
+      const float* crow = wgt + kCtL;
+      asm volatile("bar.sync 1, 256;" ::: "memory"); // the outputs that passed through w V's place are out
+      wait(kCtBarSum, parity);
+      wait(kCtBarKV, parity);
       __syncwarp();
-      if (lane == 0) mbar_arrive(bars + 8 * kCtBarOps);
-      asm volatile("bar.sync 1, 256;" ::: "memory"); // the whole chunk has landed, the other buffers are free
-      if (more) request_rest(t0 + kCtL, buf ^ 1);
-      cp_async_commit();
-      {
-        // inclusive sums over 128 tokens, four per lane; every warp for itself
-        const float* raw = reinterpret_cast<const float*>(mem + P::kOffRaw) + buf * 2 * kCtL;
-        const float4 x = *reinterpret_cast<const float4*>(raw + 4 * lane), b = *reinterpret_cast<const float4*>(raw + kCtL + 4 * lane);
-        constexpr float kLog2e = 1.4426950408889634f;
-        float4 c = make_float4(x.x * kLog2e, x.y * kLog2e, x.z * kLog2e, x.w * kLog2e);
-        c.y += c.x; c.z += c.y; c.w += c.z;
-        float s = c.w;
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-          const float p = __shfl_up_sync(0xffffffffu, s, o);
-          if (lane >= o) s += p;
-        }
-        const float before = s - c.w, total = __shfl_sync(0xffffffffu, s, 31);
-        c.x += before; c.y += before; c.z += before; c.w = s;
-        *reinterpret_cast<float4*>(crow + 4 * lane) = c;
-        *reinterpret_cast<float4*>(wgt + 4 * lane) = make_float4(b.x * exp2f(total - c.x), b.y * exp2f(total - c.y), b.z * exp2f(total - c.z), b.w * exp2f(total - c.w));
-        // (step 0: +inf, weight 0)
-        *reinterpret_cast<float4*>(cum + 4 * lane) = make_float4(c.x - log2f(b.x), c.y - log2f(b.y), c.z - log2f(b.z), c.w - log2f(b.w));
-        __syncwarp();
-      }
-      const unsigned char* vt = mem + P::kOffV + buf * kCtHalf;
+      unsigned char* vt = mem + P::kOffV + buf * kCtHalf;
       {
         // w V of 16 tokens per warp: a lane takes half a row
         const int t = 16 * warp + (lane >> 1);
         const float w = wgt[t];
+        const bool past = t0 + t >= t_end;
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const int at = ct_at(t, 4 * (lane & 1) + i);
+          if (past) {
+            const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+            *reinterpret_cast<uint4*>(vt + at) = zero;
+            *reinterpret_cast<uint4*>(mem + P::kOffK + 2 * buf * kCtHalf + at) = zero;
+            if (NH > 1) *reinterpret_cast<uint4*>(mem + P::kOffK + (2 * buf + 1) * kCtHalf + at) = zero;
+          }
           const uint4 x = *reinterpret_cast<const uint4*>(vt + at);
           const uint32_t in[4] = {x.x, x.y, x.z, x.w};
           uint32_t hi[4], lo[4];
@@ -298,12 +330,14 @@ __global__ void __launch_bounds__(kCtThreads, 1) chunk_scan_tc_kernel(const mdb_
       wait(kCtBarY, parity);
       __syncwarp();
       tc_fence_after();
-      if (more) request_channels(q, a.ldq, t0 + kCtL, base + P::kOffQ);
-      cp_async_commit();
       float y[32];
-      tmem_ld32(tmem + kCtY1 + lanes + 32 * hf, y);
-      tmem_ld_wait();
       {
+        float y_lo[32];
+        tmem_ld32(tmem + kCtY1 + lanes + 32 * hf, y);
+        tmem_ld32(tmem + kCtY1 + lanes + kCtCols + 32 * hf, y_lo);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) y[i] += y_lo[i];
         const float e = exp2f(ci);
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
@@ -327,18 +361,28 @@ __global__ void __launch_bounds__(kCtThreads, 1) chunk_scan_tc_kernel(const mdb_
         tmem_ld_wait();
 #pragma unroll
         for (int i = 0; i < 32; ++i) S[i] = fmaf(S[i], keep, d[i]);
-        if (more) publish();
+        if (more) {
+          publish();
+          hand_over();
+        }
         tmem_ld32(tmem + kCtY2 + lanes + 32 * hf, d);
         tmem_ld_wait();
-        if (t0 + r < t_end) {
-          float* out = a.out + (static_cast<int64_t>(t0 + r) * a.heads + head) * a.vdim + sc0;
+        // 32 rows x 128 bytes turned around in shared memory, so that whole rows leave together
+        unsigned char* stage = mem + P::kOffW + warp * 4096;
 #pragma unroll
-          for (int i = 0; i < 32; i += 4)
-            if (sc0 + i < a.vdim) *reinterpret_cast<float4*>(out + i) = make_float4(y[i] + d[i], y[i + 1] + d[i + 1], y[i + 2] + d[i + 2], y[i + 3] + d[i + 3]);
+        for (int i = 0; i < 8; ++i)
+          *reinterpret_cast<float4*>(stage + ct_at(lane, i)) =
+              make_float4(y[4 * i] + d[4 * i], y[4 * i + 1] + d[4 * i + 1], y[4 * i + 2] + d[4 * i + 2], y[4 * i + 3] + d[4 * i + 3]);
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int row = 4 * i + (lane >> 3), c = lane & 7, t = t0 + 32 * quad + row;
+          const float4 v = *reinterpret_cast<const float4*>(stage + ct_at(row, c));
+          if (t < t_end && sc0 + 4 * c < a.vdim)
+            *reinterpret_cast<float4*>(a.out + (static_cast<int64_t>(t) * a.heads + head) * a.vdim + sc0 + 4 * c) = v;
         }
       }
     }
-    cp_async_wait<0>();
     if (has_state) {
 #pragma unroll
       for (int i = 0; i < 32; ++i)
@@ -355,6 +399,10 @@ __global__ void __launch_bounds__(kCtThreads, 1) chunk_scan_tc_kernel(const mdb_
 
 template <int NH>
 static int launch_chunk_scan_tc(const mdb_chunk_scan_args& a, cudaStream_t st) {
+  CUtensorMap map_q, map_k, map_v;
+  if (!get_tensor_map(a.q, a.m, a.kv_heads * a.dim, a.ldq, kCtL, &map_q) || !get_tensor_map(a.k, a.m, a.kv_heads * a.dim, a.ldk, kCtL, &map_k) ||
+      !get_tensor_map(a.v, a.m, a.heads * a.vdim, a.ldv, kCtL, &map_v))
+    return MDB_ERR_CUDA;
   static PerDeviceOnce attr_once;
   const int dev = attr_once.slot();
   if (dev < 0) return MDB_ERR_CUDA;
@@ -362,7 +410,8 @@ static int launch_chunk_scan_tc(const mdb_chunk_scan_args& a, cudaStream_t st) {
     if (cudaFuncSetAttribute(chunk_scan_tc_kernel<NH>, cudaFuncAttributeMaxDynamicSharedMemorySize, CtPlan::kBytes) != cudaSuccess) return MDB_ERR_CUDA;
     attr_once.done[dev] = true;
   }
-  return mdb_launch(chunk_scan_tc_kernel<NH>, dim3((a.vdim + kCtCols - 1) / kCtCols, a.heads, a.bs), dim3(kCtThreads), CtPlan::kBytes, st, a);
+  return mdb_launch(chunk_scan_tc_kernel<NH>, dim3((a.vdim + kCtCols - 1) / kCtCols, a.heads, a.bs), dim3(kCtThreads), CtPlan::kBytes, st, map_q, map_k,
+                    map_v, a);
 }
 
 }  // namespace mdb

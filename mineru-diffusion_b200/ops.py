@@ -778,7 +778,7 @@ def chunk_scan(bs: int, heads: int, kv_heads: int, dim: int, vdim: int, q, k, v,
     _, cu_q, start, slot = portions
     for t, nm in ((q, "q"), (k, "k"), (v, "v")):
         _need(t, _BF16, nm)
-    a = _lib.ChunkScanArgs(bs, heads, kv_heads, dim, state.shape[-1], vdim, max_q, q.data_ptr(), k.data_ptr(), v.data_ptr(), _rows(q, "q"),
+    a = _lib.ChunkScanArgs(q.shape[0], bs, heads, kv_heads, dim, state.shape[-1], vdim, max_q, q.data_ptr(), k.data_ptr(), v.data_ptr(), _rows(q, "q"),
                            _rows(k, "k"), _rows(v, "v"), heads if log_decay.dim() > 1 else 0, log_decay.data_ptr(),
                            step.data_ptr(), _ptr(skip), state.data_ptr(), state.stride(0), state.shape[0], cu_q.data_ptr(),
                            start.data_ptr(), slot.data_ptr(), out.data_ptr())
